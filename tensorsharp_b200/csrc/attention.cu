@@ -313,7 +313,7 @@ __global__ void attn_combine_kernel(AttnArgs a) {
             o += pv[i] * c;
         }
     }
-    const bf16 ob = f2bf(ll > 0.f ? o / ll : 0.f);
+    const bf16 ob = f2bf(ll > 0.f ? o / ll * attn_gate(a, b, h) : 0.f);
     if (d < a.Dh) a.out[((long)b * a.Hq + h) * a.Dh + d] = ob;
     if (a.out_q != nullptr) {
         // a warp holds 32 consecutive dims = one group (Dh is a multiple of 32); same arithmetic as quantize_q8_kernel
@@ -405,6 +405,16 @@ static int attn_decode_impl(const AttnArgs* args, void* stream, bool allow_fused
     if (a.B == 0) return TSB_OK;
     cudaStream_t s = (cudaStream_t)stream;
     int rc;
+    if (a.gate != nullptr) a.ticket = nullptr;          // the in-kernel merges know no gate
+    if ((a.Dv != 0 && a.Dv != a.Dh) || (a.Dh != 64 && a.Dh != 128 && a.Dh != 256 && a.Dh != 512)) {
+        if (a.Dv == 0) a.Dv = a.Dh;
+        rc = tsb_attn_decode_vd_launch(a, s);
+        if (rc != TSB_OK) return rc;
+        a.Dh = a.Dv;                                    // the combine works on output columns
+        TSB_CHECK_CUDA(tsb_launch(attn_combine_kernel, dim3(a.Hq, a.B), dim3((a.Dh + 31) & ~31), 0, s, a));
+        TSB_CHECK_LAUNCH();
+        return TSB_OK;
+    }
     // Head sizes 64 / 128 with up to 16 query heads per KV head: Q K^T and P V on the tensor cores, the query heads of a
     // KV head as the rows of one tile (attention_decode_mma.cu).  Measured on the Qwen3-4B shape: one sequence 2.015 ->
     // 1.750 ms per step, 16 sequences 5.76 -> 4.48 ms.  TSB_ATTN_MMA=0 keeps the CUDA-core kernels for every shape,
@@ -692,6 +702,8 @@ __global__ void __launch_bounds__(128 * DS) attn_prefill_kernel(AttnArgs a) {
             ll = ll * oc + __expf(sk - mn);
         }
         inv[r] = ll > 0.f ? oc / ll : 0.f;
+        const int row = r_lo + 8 * r;
+        if (a.gate != nullptr && row < rows) inv[r] *= attn_gate(a, q0 + m0 + row, h);
     }
     const int ra = warp * 16 + (lane >> 2), rb = ra + 8;
     if (a.lse_out != nullptr && (lane & 3) == 0 && dset == 0) {
@@ -733,6 +745,8 @@ extern "C" int tsb_attn_prefill(const AttnArgs* args, int max_q_len, void* strea
     TSB_CHECK_ARG(a.cu_q != nullptr, "attn_prefill: cu_q is required");
     if (a.B == 0 || max_q_len == 0) return TSB_OK;
     cudaStream_t s = (cudaStream_t)stream;
+    if ((a.Dv != 0 && a.Dv != a.Dh) || (a.Dh != 64 && a.Dh != 128 && a.Dh != 256 && a.Dh != 512))
+        return tsb_attn_prefill_vd_launch(a, max_q_len, s);
     switch (a.Dh) {
     case 64: return launch_prefill<64>(a, max_q_len, s);
     case 128: return launch_prefill<128>(a, max_q_len, s);

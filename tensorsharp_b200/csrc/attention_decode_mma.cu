@@ -377,7 +377,7 @@ bool tsb_attn_decode_mma_supported(const AttnArgs& a) {
 bool tsb_attn_decode_mma_cluster(const AttnArgs& a) {
     const char* e = getenv("TSB_ATTN_CLUSTER");
     const bool on = e != nullptr && atoi(e) != 0;
-    if (!on || (a.splits != 8 && a.splits != 16)) return false;
+    if (!on || a.gate != nullptr || (a.splits != 8 && a.splits != 16)) return false;
     const int cols = (a.Hq / a.Hkv) * a.Dh;
     return cols % (a.splits * 32) == 0;
 }

@@ -30,7 +30,26 @@ struct AttnArgs {
     // Decode: positions per split fixed by the caller (a multiple of 32), so that a CTA's range and its block-table
     // entries do not wait for the sequence length; 0 = derive it from the length (ceil(span / splits), rounded to 32).
     int split_len;
+    // Output gate: head h of query row t is multiplied by sigmoid(gate[t * gate_tok + h]) (t: packed query row; decode:
+    // the sequence).  Null: none.
+    const void* gate;
+    long gate_tok;            // elements between query rows
+    int gate_f32;
+    int Dv;                   // value head size (0 = Dh): v_cache [slots, Hkv, Dv], out [Tq, Hq, Dv]
 };
+
+#ifdef __CUDACC__
+__device__ __forceinline__ float attn_gate(const AttnArgs& a, long t, int h) {
+    if (a.gate == nullptr) return 1.f;
+    const float g = a.gate_f32 ? reinterpret_cast<const float*>(a.gate)[t * a.gate_tok + h]
+                               : bf2f(reinterpret_cast<const bf16*>(a.gate)[t * a.gate_tok + h]);
+    return 1.f / (1.f + __expf(-g));
+}
+#endif
+
+// attention_vd.cu: key and value head sizes of their own (multiples of 16)
+int tsb_attn_prefill_vd_launch(const AttnArgs& a, int max_q, cudaStream_t s);
+int tsb_attn_decode_vd_launch(const AttnArgs& a, cudaStream_t s);         // the caller launches the combine
 
 // attention_decode_mma.cu: the tensor-core split kernel for decode batches (head sizes 64 / 128, up to 16 query heads
 // per KV head); the caller launches the combine unless `*merged` comes back true (splits merged by a thread-block cluster).

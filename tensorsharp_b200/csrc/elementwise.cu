@@ -219,6 +219,10 @@ struct QkvArgs {
     float q_scale;                      // multiplied into q after RoPE (1 = none)
     int T, Hq, Hkv, Dh;
     RopeParams rp;
+    int Dv;                             // value head size; v_cache is [slots, Hkv, Dv]
+    int norm_n;                         // divisor of the per-head norm (Dh unless the head is padded with zeros)
+    float qt_coef, qt_every;            // query factor 1 + coef ln(floor((p + 1) / every) + 1); every 0: none
+    int out_f32;                        // 1: q_out and the caches are float
 };
 
 __device__ __forceinline__ void rope_cs(const RopeParams& rp, const float* ff, int pair, float pos, float& c, float& s) {
@@ -279,7 +283,7 @@ __global__ void __launch_bounds__(128) qkv_rope_kernel(QkvArgs a) {
     const int H = a.Hq + 2 * a.Hkv;
     if (wid >= (long)a.T * H) return;
     const int t = (int)(wid / H), h = (int)(wid % H);
-    const int Dh = a.Dh;
+    const int Dh = h < a.Hq + a.Hkv ? a.Dh : a.Dv;
     const void* src;
     long off;
     int kind;  // 0 q, 1 k, 2 v
@@ -319,27 +323,33 @@ __global__ void __launch_bounds__(128) qkv_rope_kernel(QkvArgs a) {
     }
     if (nw || (kind == 2 && a.v_norm)) {
         ss = warp_sum(ss);
-        const float rs = rsqrtf(ss / (float)Dh + a.eps);
+        const float rs = rsqrtf(ss / (float)(kind == 2 ? Dh : a.norm_n) + a.eps);
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
             const int e = lane + 32 * j;
             if (e < Dh) v[j] *= rs * nwv[j];
         }
     }
-    bf16* dst;
-    if (kind == 0) dst = a.q_out + ((long)t * a.Hq + h) * Dh;
-    else if (kind == 1) dst = a.k_cache + (slot * a.Hkv + (h - a.Hq)) * Dh;
-    else dst = a.v_cache + (slot * a.Hkv + (h - a.Hq - a.Hkv)) * Dh;
+    bf16* base;
+    long doff;
+    if (kind == 0) { base = a.q_out; doff = ((long)t * a.Hq + h) * Dh; }
+    else if (kind == 1) { base = a.k_cache; doff = (slot * a.Hkv + (h - a.Hq)) * Dh; }
+    else { base = a.v_cache; doff = (slot * a.Hkv + (h - a.Hq - a.Hkv)) * Dh; }
+    auto store = [&](int e, float x) {
+        if (a.out_f32) reinterpret_cast<float*>(base)[doff + e] = x;
+        else base[doff + e] = f2bf(x);
+    };
+    float qs = kind == 0 ? a.q_scale : 1.f;
+    if (kind == 0 && a.qt_every > 0.f) qs *= 1.f + a.qt_coef * logf(floorf(((float)a.pos[t] + 1.f) / a.qt_every) + 1.f);
     if (kind == 2 || rot == 0) {
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
             const int e = lane + 32 * j;
-            if (e < Dh) dst[e] = f2bf(kind == 0 ? v[j] * a.q_scale : v[j]);
+            if (e < Dh) store(e, v[j] * qs);
         }
         return;
     }
     const float pos = (float)a.pos[t];
-    const float qs = kind == 0 ? a.q_scale : 1.f;
     if (a.rp.mode == 0) {
         // NeoX: element e pairs with e + rot/2.  The partner lives in another register or lane;
         // stage through shared memory (one row of 512 floats per warp).
@@ -364,7 +374,7 @@ __global__ void __launch_bounds__(128) qkv_rope_kernel(QkvArgs a) {
                 const float x0 = st[pair], x1 = st[pair + half];
                 o = e < half ? x0 * c - x1 * s : x0 * s + x1 * c;
             }
-            dst[e] = f2bf(o * qs);
+            store(e, o * qs);
         }
     } else {
         // adjacent pairs (2i, 2i+1): the partner is in the neighbouring lane
@@ -379,7 +389,7 @@ __global__ void __launch_bounds__(128) qkv_rope_kernel(QkvArgs a) {
                 if (!tab) rope_lookup(a, t, e >> 1, pos, c, s);
                 o = (e & 1) ? other * s + v[j] * c : v[j] * c - other * s;
             }
-            dst[e] = f2bf(o * qs);
+            store(e, o * qs);
         }
     }
 }
@@ -387,14 +397,17 @@ __global__ void __launch_bounds__(128) qkv_rope_kernel(QkvArgs a) {
 extern "C" int tsb_qkv_rope(const QkvArgs* args, void* stream) {
     const QkvArgs& a = *args;
     TSB_CHECK_ARG(a.Dh > 0 && a.Dh <= 512, "qkv_rope: head dim %d out of range (1..512)", a.Dh);
+    TSB_CHECK_ARG(a.Dv > 0 && a.Dv <= 512, "qkv_rope: value head dim %d out of range (1..512)", a.Dv);
+    TSB_CHECK_ARG(a.norm_n > 0 && a.norm_n <= a.Dh, "qkv_rope: norm over %d of %d values", a.norm_n, a.Dh);
+    const int wide = a.Dh > a.Dv ? a.Dh : a.Dv;
     TSB_CHECK_ARG(a.rp.rot_dim <= a.Dh && a.rp.rot_dim % 2 == 0, "qkv_rope: bad rot_dim %d", a.rp.rot_dim);
     const long warps = (long)a.T * (a.Hq + 2 * a.Hkv);
     if (warps == 0) return TSB_OK;
     const dim3 grid((unsigned)((warps + 3) / 4)), block(128);
     cudaStream_t st = (cudaStream_t)stream;
-    if (a.Dh <= 64) TSB_CHECK_CUDA(tsb_launch(qkv_rope_kernel<2>, grid, block, 0, st, a));
-    else if (a.Dh <= 128) TSB_CHECK_CUDA(tsb_launch(qkv_rope_kernel<4>, grid, block, 0, st, a));
-    else if (a.Dh <= 256) TSB_CHECK_CUDA(tsb_launch(qkv_rope_kernel<8>, grid, block, 0, st, a));
+    if (wide <= 64) TSB_CHECK_CUDA(tsb_launch(qkv_rope_kernel<2>, grid, block, 0, st, a));
+    else if (wide <= 128) TSB_CHECK_CUDA(tsb_launch(qkv_rope_kernel<4>, grid, block, 0, st, a));
+    else if (wide <= 256) TSB_CHECK_CUDA(tsb_launch(qkv_rope_kernel<8>, grid, block, 0, st, a));
     else TSB_CHECK_CUDA(tsb_launch(qkv_rope_kernel<16>, grid, block, 0, st, a));
     return TSB_OK;
 }
@@ -419,6 +432,28 @@ __device__ __forceinline__ float glu_apply(int act, float g, float u) {
     case 7: return u / (1.f + __expf(-g));                                // sigmoid(g) * u
     default: return g * u;
     }
+}
+
+// 32-bit in and out (models that run in float32).
+__global__ void glu_f32_kernel(const float* gate, const float* up, long g_stride, long u_stride, int F, int act, float* out, long rows) {
+    pdl_wait();
+    pdl_trigger();
+    const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= rows * F) return;
+    const long t = idx / F;
+    const int f = (int)(idx % F);
+    const float g = gate[t * g_stride + f], u = up ? up[t * u_stride + f] : 0.f;
+    out[idx] = act == 1 ? g / (1.f + expf(-g)) * u : glu_apply(act, g, u);
+}
+
+extern "C" int tsb_glu_f32(const float* gate, const float* up, long g_stride, long u_stride, long rows, int F, int act, float* out,
+                           void* stream) {
+    TSB_CHECK_ARG(gate && out && rows >= 0 && F >= 0, "glu_f32: bad shape rows=%ld F=%d", rows, F);
+    if (rows == 0 || F == 0) return TSB_OK;
+    TSB_CHECK_CUDA(tsb_launch(glu_f32_kernel, dim3((unsigned)((rows * F + 255) / 256)), dim3(256), 0, (cudaStream_t)stream, gate, up,
+                              g_stride, u_stride, F, act, out, rows));
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
 }
 
 template <typename T>

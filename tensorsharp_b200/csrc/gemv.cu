@@ -345,7 +345,7 @@ extern "C" int tsb_gemv_push(const void* p0, const void* p1, const void* p2, con
     TSB_CHECK_ARG(!q8 || (xq && xds), "gemv: quantised weight type %d needs int8 activations", type);
     TSB_CHECK_ARG(q8 || xb, "gemv: float weight type %d needs bf16 activations", type);
     const bool kq = type == TSB_Q4_K || type == TSB_Q5_K || type == TSB_Q6_K;
-    TSB_CHECK_ARG(K % (kq ? 256 : 32) == 0, "gemv: K=%d not a whole number of blocks for type %d", K, type);
+    TSB_CHECK_ARG(K % (kq ? 256 : q8 ? 32 : 8) == 0, "gemv: K=%d not a whole number of blocks for type %d", K, type);
     const bool glu = act >= ACT_SWIGLU && act <= ACT_SWIGLU_OAI;
     TSB_CHECK_ARG(!glu || N % 2 == 0, "gemv: GLU needs an even row count, got %d", N);
     if (M == 0 || (ids && problems == 0)) return TSB_OK;

@@ -23,23 +23,26 @@
 
 #define MOE_TILE_ROWS 8
 #define MOE_MAX_E 1024
-#define MOE_MAX_K 16
+#define MOE_MAX_K 32
 
 // ---------------------------------------------------------------------------------------------
 // Router: one warp per token.
 // mode 0: top-k of the logits, weights = softmax over the selected logits.
 // mode 1: p = sigmoid(logit); select on p + sel_bias; weights = p, optionally / max(sum, 6.1e-5); * scale.
+// mode 2: s = softmax over all logits; select the k largest; weights = s / (their sum + 1e-20) * scale.
+// `always` > 0 (any mode): experts E .. E + always - 1 follow the k selected ones with the weight sigmoid(logit[E])
+// (a gated shared expert, cut into slices); a row of logits is `ld` long.
 // ---------------------------------------------------------------------------------------------
 template <int PER>
 __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ sel_bias,
                                                         int T, int E, int k, int mode, int normalize, float scale,
-                                                        int* __restrict__ ids, float* __restrict__ wts) {
+                                                        int ld, int always, int* __restrict__ ids, float* __restrict__ wts) {
     const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     pdl_wait();
     pdl_trigger();
     if (t >= T) return;
     float sel[PER], val[PER];                   // PER = ceil(E / 32) rounded up to an instantiated size
-    const float* row = logits + (long)t * E;
+    const float* row = logits + (long)t * ld;
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
         const int e = i * 32 + lane;
@@ -57,6 +60,18 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
             val[i] = 0.f;
             sel[i] = -INFINITY;
         }
+    }
+    float denom = 1.f;                    // mode 2: the softmax's sum over all experts
+    float top = 0.f;
+    if (mode == 2) {
+        float mx = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) mx = fmaxf(mx, sel[i]);
+        top = warp_max(mx);
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) s += sel[i] == -INFINITY ? 0.f : expf(sel[i] - top);
+        denom = warp_sum(s);
     }
     float wk = 0.f;                       // lane j keeps the j-th selected weight
     int ik = 0;
@@ -89,6 +104,9 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
         const float ex = on ? __expf(wk - m) : 0.f;
         const float s = warp_sum(ex);
         wk = ex / s;
+    } else if (mode == 2) {
+        const float p = on ? expf(wk - top) / denom : 0.f;
+        wk = p / (warp_sum(p) + 1e-20f) * scale;
     } else {
         if (normalize) {
             const float s = warp_sum(on ? wk : 0.f);
@@ -96,25 +114,221 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
         }
         wk *= scale;
     }
+    const long o = (long)t * (k + always);
     if (on) {
-        ids[(long)t * k + lane] = ik;
-        wts[(long)t * k + lane] = wk;
+        ids[o + lane] = ik;
+        wts[o + lane] = wk;
+    }
+    if (always > 0) {
+        const float g = 1.f / (1.f + expf(-row[E]));
+        for (int i = lane; i < always; i += 32) {
+            ids[o + k + i] = E + i;
+            wts[o + k + i] = g;
+        }
     }
 }
 
-extern "C" int tsb_moe_route(const float* logits, const float* sel_bias, int T, int E, int k, int mode, int normalize,
-                             float scale, int* ids, float* wts, void* stream) {
+extern "C" int tsb_moe_route_ex(const float* logits, const float* sel_bias, int T, int E, int k, int mode, int normalize,
+                                float scale, int ld, int always, int* ids, float* wts, void* stream) {
+    TSB_CHECK_ARG(ld >= E + (always > 0 ? 1 : 0) && always >= 0, "moe_route: rows of %d logits for %d experts and %d always on", ld, E, always);
     TSB_CHECK_ARG(E > 0 && E <= MOE_MAX_E, "moe_route: %d experts (limit %d)", E, MOE_MAX_E);
     TSB_CHECK_ARG(k > 0 && k <= MOE_MAX_K && k <= E, "moe_route: top-%d of %d", k, E);
     if (T == 0) return TSB_OK;
     const dim3 grid((T + 3) / 4), block(128);
     cudaStream_t st = (cudaStream_t)stream;
-#define TSB_ROUTE(P) TSB_CHECK_CUDA(tsb_launch(moe_route_kernel<P>, grid, block, 0, st, logits, sel_bias, T, E, k, mode, normalize, scale, ids, wts))
+#define TSB_ROUTE(P) TSB_CHECK_CUDA(tsb_launch(moe_route_kernel<P>, grid, block, 0, st, logits, sel_bias, T, E, k, mode, normalize, scale, ld, always, ids, wts))
     if (E <= 32) TSB_ROUTE(1);
     else if (E <= 128) TSB_ROUTE(4);
     else if (E <= 256) TSB_ROUTE(8);
     else TSB_ROUTE(MOE_MAX_E / 32);
 #undef TSB_ROUTE
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}
+
+extern "C" int tsb_moe_route(const float* logits, const float* sel_bias, int T, int E, int k, int mode, int normalize,
+                             float scale, int* ids, float* wts, void* stream) {
+    return tsb_moe_route_ex(logits, sel_bias, T, E, k, mode, normalize, scale, E, 0, ids, wts, stream);
+}
+
+// ---------------------------------------------------------------------------------------------
+// Sorting the (token, slot) pairs by expert for the grouped GEMM, without a host read-back:
+//   order[i]  the pair at sorted place i       pos[p]  the sorted place of pair p
+//   tiles     {expert or -1, first place, end place} for pieces of at most bn places of one expert; a fixed number of
+//             entries (ceil(P / bn) + E), the surplus marked -1
+// Pairs of one expert come in no particular order (every row's product is its own).  Up to SORT_ONE_CTA pairs one CTA does
+// it all; more pairs take a histogram per 1024 pairs, one CTA that turns the counts into offsets, and a scatter.
+// ---------------------------------------------------------------------------------------------
+#define SORT_CHUNK 1024
+#define SORT_ONE_CTA 4096
+
+struct SortArgs {
+    const int* ids;          // [P], each in [0, E)
+    int* order; int* pos; int* tiles;
+    int* counts;             // [chunks, E] scratch (null for the one-CTA form)
+    int P, E, bn, n_tiles;
+};
+
+// exclusive scan of one value per thread over a CTA of 1024 threads; `sh` holds 33 ints.  Returns the prefix.
+__device__ __forceinline__ int scan1024(int v, int* sh) {
+    const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
+    int x = v;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const int y = __shfl_up_sync(0xffffffffu, x, o);
+        if (lane >= o) x += y;
+    }
+    __syncthreads();
+    if (lane == 31) sh[w] = x;
+    __syncthreads();
+    if (w == 0) {
+        int s = sh[lane];
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int y = __shfl_up_sync(0xffffffffu, s, o);
+            if (lane >= o) s += y;
+        }
+        sh[lane] = s;
+    }
+    __syncthreads();
+    return x - v + (w > 0 ? sh[w - 1] : 0);
+}
+
+// shared-memory counter of expert e, one atomic per warp and distinct expert; returns this thread's value before the add
+__device__ __forceinline__ int count_up(int* cnt, int e, bool on) {
+    const unsigned act = __ballot_sync(0xffffffffu, on);
+    if (!on) return 0;
+    const unsigned same = __match_any_sync(act, e);
+    const int lane = threadIdx.x & 31, lead = __ffs(same) - 1;
+    int base = 0;
+    if (lane == lead) base = atomicAdd(&cnt[e], __popc(same));
+    base = __shfl_sync(same, base, lead);
+    return base + __popc(same & ((1u << lane) - 1u));
+}
+
+// thread e holds expert e's pair count: offsets (returned) and the tile list
+__device__ __forceinline__ int sort_tiles(const SortArgs& a, int count, int* sh) {
+    const int e = threadIdx.x;
+    const int start = scan1024(count, sh);
+    const int nt = (count + a.bn - 1) / a.bn;
+    const int first = scan1024(nt, sh);
+    if (e < a.E)
+        for (int i = 0; i < nt; ++i) {
+            int* t = a.tiles + 3 * (first + i);
+            t[0] = e;
+            t[1] = start + i * a.bn;
+            t[2] = min(start + count, start + (i + 1) * a.bn);
+        }
+    __syncthreads();
+    const int used = sh[31];
+    for (int i = used + threadIdx.x; i < a.n_tiles; i += SORT_CHUNK) a.tiles[3 * i] = -1;
+    return start;
+}
+
+__global__ void __launch_bounds__(SORT_CHUNK) moe_sort_one_kernel(SortArgs a) {
+    __shared__ int cnt[MOE_MAX_E], sh[33];
+    pdl_wait();
+    pdl_trigger();
+    cnt[threadIdx.x] = 0;
+    __syncthreads();
+    for (int p0 = 0; p0 < a.P; p0 += SORT_CHUNK) {
+        const int p = p0 + threadIdx.x;
+        count_up(cnt, p < a.P ? a.ids[p] : 0, p < a.P);
+    }
+    __syncthreads();
+    const int start = sort_tiles(a, threadIdx.x < a.E ? cnt[threadIdx.x] : 0, sh);
+    __syncthreads();
+    cnt[threadIdx.x] = start;
+    __syncthreads();
+    for (int p0 = 0; p0 < a.P; p0 += SORT_CHUNK) {
+        const int p = p0 + threadIdx.x;
+        const int i = count_up(cnt, p < a.P ? a.ids[p] : 0, p < a.P);
+        if (p < a.P) {
+            a.order[i] = p;
+            a.pos[p] = i;
+        }
+    }
+}
+
+__global__ void __launch_bounds__(SORT_CHUNK) moe_sort_count_kernel(SortArgs a) {
+    __shared__ int cnt[MOE_MAX_E];
+    pdl_wait();
+    pdl_trigger();
+    cnt[threadIdx.x] = 0;
+    __syncthreads();
+    const int p = blockIdx.x * SORT_CHUNK + threadIdx.x;
+    count_up(cnt, p < a.P ? a.ids[p] : 0, p < a.P);
+    __syncthreads();
+    if (threadIdx.x < a.E) a.counts[(long)blockIdx.x * a.E + threadIdx.x] = cnt[threadIdx.x];
+}
+
+__global__ void __launch_bounds__(SORT_CHUNK) moe_sort_offsets_kernel(SortArgs a, int chunks) {
+    __shared__ int sh[33];
+    pdl_wait();
+    pdl_trigger();
+    const int e = threadIdx.x;
+    int total = 0;
+    if (e < a.E)
+        for (int c = 0; c < chunks; ++c) total += a.counts[(long)c * a.E + e];
+    int at = sort_tiles(a, total, sh);
+    if (e < a.E)
+        for (int c = 0; c < chunks; ++c) {
+            const int n = a.counts[(long)c * a.E + e];
+            a.counts[(long)c * a.E + e] = at;
+            at += n;
+        }
+}
+
+__global__ void __launch_bounds__(SORT_CHUNK) moe_sort_scatter_kernel(SortArgs a) {
+    __shared__ int cnt[MOE_MAX_E];
+    pdl_wait();
+    pdl_trigger();
+    if (threadIdx.x < a.E) cnt[threadIdx.x] = a.counts[(long)blockIdx.x * a.E + threadIdx.x];
+    __syncthreads();
+    const int p = blockIdx.x * SORT_CHUNK + threadIdx.x;
+    const int i = count_up(cnt, p < a.P ? a.ids[p] : 0, p < a.P);
+    if (p < a.P) {
+        a.order[i] = p;
+        a.pos[p] = i;
+    }
+}
+
+extern "C" int tsb_moe_sort(const int* ids, int P, int E, int bn, int* order, int* pos, int* tiles, int n_tiles, int* counts, void* stream) {
+    TSB_CHECK_ARG(E > 0 && E <= MOE_MAX_E, "moe_sort: %d experts (limit %d)", E, MOE_MAX_E);
+    TSB_CHECK_ARG(P >= 0 && bn > 0 && n_tiles >= (P + bn - 1) / bn + E, "moe_sort: %d tile entries for %d pairs of %d experts", n_tiles, P, E);
+    if (P == 0) return TSB_OK;
+    SortArgs a{ids, order, pos, tiles, counts, P, E, bn, n_tiles};
+    cudaStream_t s = (cudaStream_t)stream;
+    if (P <= SORT_ONE_CTA) {
+        TSB_CHECK_CUDA(tsb_launch(moe_sort_one_kernel, dim3(1), dim3(SORT_CHUNK), 0, s, a));
+    } else {
+        TSB_CHECK_ARG(counts != nullptr, "moe_sort: count scratch is missing");
+        const int chunks = (P + SORT_CHUNK - 1) / SORT_CHUNK;
+        TSB_CHECK_CUDA(tsb_launch(moe_sort_count_kernel, dim3(chunks), dim3(SORT_CHUNK), 0, s, a));
+        TSB_CHECK_CUDA(tsb_launch(moe_sort_offsets_kernel, dim3(1), dim3(SORT_CHUNK), 0, s, a, chunks));
+        TSB_CHECK_CUDA(tsb_launch(moe_sort_scatter_kernel, dim3(chunks), dim3(SORT_CHUNK), 0, s, a));
+    }
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}
+
+// out[i] = x[order[i] / div] (bf16 rows of K, a multiple of 8): the activation rows in sorted order, one warp per row.
+__global__ void __launch_bounds__(256) gather_bf16_rows_kernel(const bf16* __restrict__ x, const int* __restrict__ order, int P, int div,
+                                                               int K, bf16* __restrict__ out) {
+    pdl_wait();
+    pdl_trigger();
+    const int i = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (i >= P) return;
+    const uint4* s = reinterpret_cast<const uint4*>(x + (long)(order[i] / div) * K);
+    uint4* d = reinterpret_cast<uint4*>(out + (long)i * K);
+    for (int c = lane; c < K / 8; c += 32) d[c] = s[c];
+}
+
+extern "C" int tsb_gather_bf16_rows(const void* x, const int* order, int P, int div, int K, void* out, void* stream) {
+    TSB_CHECK_ARG(K > 0 && K % 8 == 0 && div > 0, "gather_bf16_rows: K=%d div=%d", K, div);
+    if (P == 0) return TSB_OK;
+    TSB_CHECK_CUDA(tsb_launch(gather_bf16_rows_kernel, dim3((P + 7) / 8), dim3(256), 0, (cudaStream_t)stream, (const bf16*)x, order, P, div, K,
+                              (bf16*)out));
     TSB_CHECK_LAUNCH();
     return TSB_OK;
 }

@@ -17,7 +17,7 @@ from typing import Callable, Dict, List, Optional, Sequence, Tuple
 import numpy as np
 import torch
 
-from ..gguf.reader import GGUFFile
+from ..gguf.folder import open_checkpoint
 from ..ops import functional as F
 from ..ops.functional import Batch
 from ..quant import codecs
@@ -63,14 +63,23 @@ class ModelBase:
     supports_kv_truncation = True
     supports_pipeline = False
     supports_context_parallel = False
+    supports_float32 = False           # compute_dtype float32 on the GPU
+    mixed_batches = False              # the continuous batcher may put prompt portions and decoded tokens into one step
+    native_sources: Optional[Tuple[str, ...]] = None     # kernel sources the family needs (None: the whole library)
 
     def __init__(self, path: str, device="cuda", *, max_context: Optional[int] = None, max_seqs: int = 1,
                  page_size: int = 64, kv_dtype: Optional[torch.dtype] = None, tp_rank: int = 0, tp_size: int = 1,
                  ep_rank: int = 0, ep_size: int = 1, comm=None, pp_rank: int = 0, pp_size: int = 1, pp_comm=None,
-                 cp_comm=None):
+                 cp_comm=None, kv_pages: Optional[int] = None, compute_dtype: Optional[torch.dtype] = None):
+        """``kv_pages`` fixes the size of the KV pool (default: ``max_context`` for each of ``max_seqs`` sequences);
+        ``compute_dtype`` float32 runs the whole model in 32 bits on families that support it (on the CPU all do)."""
         self.path = path
         self.device = torch.device(device)
-        self.gguf = GGUFFile(path)
+        self.kv_pages = kv_pages
+        self.compute_dtype = compute_dtype or (torch.bfloat16 if self.device.type == "cuda" else torch.float32)
+        if self.compute_dtype == torch.float32 and self.device.type == "cuda" and not self.supports_float32:
+            raise ValueError(f"{type(self).__name__} has no float32 path on the GPU")
+        self.gguf = open_checkpoint(path)
         self.tp_rank, self.tp_size, self.ep_rank, self.ep_size, self.comm = tp_rank, tp_size, ep_rank, ep_size, comm
         # pipeline parallelism: this process holds a contiguous range of layers (and only their KV cache);
         # the first stage owns the embedding, the last one the output norm and lm_head
@@ -328,7 +337,8 @@ class ModelBase:
     def is_last_stage(self) -> bool:
         return self.pp_rank == self.pp_size - 1
 
-    def kv_layer_shapes(self) -> List[Optional[Tuple[int, int]]]:
+    def kv_layer_shapes(self) -> List[Optional[Tuple[int, ...]]]:
+        """Per cached layer ``(KV heads, head size)`` or ``(KV heads, key size, value size)``; None: no cache."""
         c = self.cfg
         l0, l1 = self.layer_range
         return [(c.n_kv_heads // self.tp_size, c.head_dim) if l0 <= l < l1 else None for l in range(c.n_layers)]
@@ -347,14 +357,15 @@ class ModelBase:
         if (os.environ.get("TSB_KV_WINDOW_RING", "0") not in ("", "0") and self.cp_comm is None and self.pp_size == 1
                 and self.kv_dtype != torch.float8_e4m3fn):
             ring_chunk = max(self.page_size, int(os.environ.get("TSB_KV_RING_CHUNK", "2048")))
-        return PagedKV(self.kv_layer_shapes(), pages_per_seq * self.max_seqs, self.page_size, self.device,
+        return PagedKV(self.kv_layer_shapes(), self.kv_pages or pages_per_seq * self.max_seqs, self.page_size, self.device,
                        self.kv_dtype, self.kv_donors(), max_seqs=max(self.max_seqs, 1),
                        window_layers=self.kv_window_layers() if ring_chunk else None, ring_chunk=ring_chunk)
 
     # ------------------------------------------------------------------ execution
     def forward_batch(self, batch: Batch, want_logits: bool = True) -> Optional[torch.Tensor]:
         """Run the packed batch; returns float32 logits ``[B, vocab]`` for the last token of
-        every sequence (or ``None`` when ``want_logits`` is false: prefill chunks)."""
+        every sequence (or ``None`` when ``want_logits`` is false: prefill chunks).  A batch that was
+        built for other rows (``PagedKV.build_batch(rows=...)``) gives one row of logits for each."""
         raise NotImplementedError
 
     def recurrent_state_tensors(self) -> list:
@@ -598,9 +609,14 @@ class ModelBase:
     @staticmethod
     def create(path: str, device="cuda", **kw) -> "ModelBase":
         """Open ``path`` and instantiate the graph for its ``general.architecture``."""
+        return ModelBase.class_of(path)(path, device, **kw)
+
+    @staticmethod
+    def class_of(path: str):
+        """The model class for the ``general.architecture`` of the file or folder at ``path``."""
         from . import _load_all  # noqa: F401  (registers every architecture)
-        with GGUFFile(path) as g:
+        with open_checkpoint(path) as g:
             arch = g.get_str("general.architecture", "")
         if arch not in _REGISTRY:
             raise ValueError(f"unsupported architecture {arch!r}; supported: {supported_architectures()}")
-        return _REGISTRY[arch](path, device, **kw)
+        return _REGISTRY[arch]

@@ -31,7 +31,7 @@ DENSE_GEMV_MAX_M = min(GEMV_MAX_M, int(os.environ.get("TSB_GEMV_MAX_M", "8")))
 @dataclass
 class Act:
     """A (normalised) activation in the forms the linear kernels consume."""
-    b: Optional[torch.Tensor] = None      # [T, K] bf16 (CUDA) or f32 (CPU)
+    b: Optional[torch.Tensor] = None      # [T, K] bf16 (CUDA) or f32 (CPU, and CUDA models that run in 32 bits)
     q: Optional[torch.Tensor] = None      # [T, K] int8
     ds: Optional[torch.Tensor] = None     # [T, K/32, 2] f32 (scale, sum)
 
@@ -62,7 +62,7 @@ class Batch:
     cu_q: torch.Tensor            # [B+1] int32
     kv_lens: torch.Tensor         # [B] int32 (cache length after this step)
     block_table: torch.Tensor     # [B, P] int32
-    last_idx: torch.Tensor        # [B] int64 index of each sequence's last token in the packed dim
+    last_idx: torch.Tensor        # int64 rows of the packed dim whose logits are wanted ([B]: each sequence's last token)
     seq_slots: torch.Tensor       # [B] int64 recurrent-state slot per sequence
     max_q_len: int
     max_kv_len: int
@@ -132,6 +132,25 @@ def norm_add(x: torch.Tensor, w: Optional[torch.Tensor], eps: float, h: torch.Te
         _, yf, _, _ = _k().rmsnorm(x.contiguous(), w, eps, want_bf16=False, add=h)
         return yf
     return h + ref.rmsnorm(x, w, eps)
+
+
+def residual_layernorm(h: torch.Tensor, eps: float, n: int, *, y=None, post=None, add: Optional[torch.Tensor] = None, pre=None,
+                       dtype: Optional[torch.dtype] = None) -> Optional[Act]:
+    """The seam between two sublayers of a sandwich-normed decoder, one kernel on CUDA: ``h`` (f32 ``[T, D]``, in place)
+    gains the layer norm ``post`` of the sublayer's output ``y`` (a tensor or :class:`MoeParts`) and then the vector
+    ``add`` ``[D]``; returned is the layer norm ``pre`` of the new ``h`` as the next sublayer's input (None without
+    ``pre``).  ``post`` / ``pre`` are (weight, bias); statistics run over the first ``n`` columns, the rest is padding."""
+    if h.is_cuda:
+        parts = y if isinstance(y, MoeParts) else None
+        yt = parts.y if parts is not None else y
+        out = _k().residual_layernorm(h, eps, n, y=yt, pos=parts.pos if parts else None, wts=parts.w if parts else None,
+                                      parts=parts.k if parts else 1, post=post, add=add, pre=pre, out_dtype=dtype or torch.bfloat16)
+        return Act(out) if out is not None else None
+    if y is not None:
+        h.add_(ref.layernorm_n(y.sum() if isinstance(y, MoeParts) else y.float(), post[0], post[1], eps, n))
+    if add is not None:
+        h.add_(add)
+    return Act(ref.layernorm_n(h, pre[0], pre[1], eps, n)) if pre is not None else None
 
 
 def as_act(x, w: Optional[QuantWeight] = None) -> Act:
@@ -249,6 +268,12 @@ def linear(a: Act, w: QuantWeight, *, bias: Optional[torch.Tensor] = None, resid
     """y = a @ w^T (+ bias) (+ residual), optional GLU over the row halves of ``w``
     (rows [0, N/2) gate, [N/2, N) up).  ``residual`` is added in the output dtype."""
     T = a.T
+    if w.device.type == "cuda" and a.b is not None and a.b.dtype == torch.float32:      # a model that runs in 32 bits
+        y = _k().gemm_f32(w, a.b, bias=bias)
+        if act is not None:
+            half = w.N // 2
+            y = _k().glu_f32(y, None, act) if act in ("relu2", "silu") else _k().glu_f32(y[:, :half], y[:, half:], act)
+        return y if residual is None else y + residual
     if w.device.type != "cuda":
         y = a.b.float() @ w.dequantize().t()
         if bias is not None:
@@ -314,11 +339,16 @@ def glu(act: str, gate: torch.Tensor, up: Optional[torch.Tensor]) -> torch.Tenso
 def qkv_rope_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, *, Hq: int, Hkv: int, Dh: int,
                    batch: Batch, k_cache: torch.Tensor, v_cache: torch.Tensor, rope: Optional[RopeSpec],
                    qn: Optional[torch.Tensor] = None, kn: Optional[torch.Tensor] = None, v_norm: bool = False,
-                   eps: float = 1e-6, q_scale: float = 1.0, write_kv: bool = True) -> torch.Tensor:
+                   eps: float = 1e-6, q_scale: float = 1.0, write_kv: bool = True, Dv: Optional[int] = None,
+                   norm_n: Optional[int] = None, q_temp: Optional[Tuple[float, float]] = None) -> torch.Tensor:
     """Per-head norm on Q / K (and optionally V), RoPE on Q / K, write K / V into the paged
     cache at ``batch.slots``; returns the rotated queries ``[T, Hq, Dh]``.
-    ``q``, ``k``, ``v`` are ``[T, H*, Dh]`` views (any token / head stride, last dim dense)."""
+    ``q``, ``k``, ``v`` are ``[T, H*, Dh]`` views (any token / head stride, last dim dense).  ``Dv``: value head
+    size where it differs; ``norm_n``: the norm's divisor where the head is padded with zeros; ``q_temp``
+    (coef, every): position-dependent query factor (reference.py: query_temperature).  A float32 cache gets
+    float32 rows and gives float32 queries."""
     T = batch.T
+    Dv = Dv or Dh
     if q.is_cuda:
         kk = _k()
         rp = kk.RopeParams()
@@ -335,10 +365,13 @@ def qkv_rope_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, *, Hq: int
             if table is None:
                 table = kk.rope_table(batch.positions, rp, rope.freq_factors)
                 batch.cache[key] = table
-        q_out = torch.empty((T, Hq, Dh), dtype=torch.bfloat16, device=q.device)
+        f32 = k_cache.dtype == torch.float32
+        q_out = torch.empty((T, Hq, Dh), dtype=torch.float32 if f32 else torch.bfloat16, device=q.device)
         assert q.stride(-1) == 1 and k.stride(-1) == 1 and v.stride(-1) == 1 and q.dtype == k.dtype == v.dtype
         slots, kc, vc = batch.slots, k_cache, v_cache
         fp8 = write_kv and is_fp8(k_cache)
+        if fp8 and Dv != Dh:
+            raise ValueError("8-bit pages hold keys and values of one size")
         if fp8:
             # 8-bit pages: the kernel leaves the finished K / V rows in dense bf16 staging rows, which one more
             # kernel converts and scatters to their slots
@@ -352,15 +385,16 @@ def qkv_rope_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, *, Hq: int
                     pos=batch.positions, slot=slots,
                     q_out=q_out, k_cache=kc, v_cache=vc, qn=qn, kn=kn, v_norm=v_norm, eps=eps, rope=rp,
                     freq_factors=rope.freq_factors if rope is not None else None, q_scale=q_scale,
-                    cs_table=table)
+                    cs_table=table, Dv=Dv, norm_n=norm_n or Dh, q_temp=q_temp, out_f32=f32)
         if fp8:
             kk.kv_store_fp8(kc, vc, k_cache, v_cache, batch.slots)
         return q_out
     qf, kf, vf = q.float(), k.float(), v.float()
+    nn = norm_n or Dh
     if qn is not None:
-        qf = ref.rmsnorm(qf, qn, eps)
+        qf = torch.nn.functional.pad(ref.rmsnorm(qf[..., :nn], qn[:nn], eps), (0, Dh - nn))
     if kn is not None:
-        kf = ref.rmsnorm(kf, kn, eps)
+        kf = torch.nn.functional.pad(ref.rmsnorm(kf[..., :nn], kn[:nn], eps), (0, Dh - nn))
     if v_norm:
         vf = ref.rmsnorm(vf, None, eps)
     if rope is not None and rope.rot_dim > 0:
@@ -372,6 +406,8 @@ def qkv_rope_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, *, Hq: int
     if write_kv:
         kv_scatter(k_cache, batch.slots, kf)
         kv_scatter(v_cache, batch.slots, vf)
+    if q_temp is not None:
+        qf = qf * ref.query_temperature(batch.positions, *q_temp).view(-1, 1, 1)
     return qf * q_scale
 
 
@@ -445,11 +481,17 @@ def decode_splits(batch: Batch, Hkv: int, window: int) -> int:
 
 def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch: Batch, *, scale: float,
               Hq: int, Hkv: int, Dh: int, window: int = 0, sinks: Optional[torch.Tensor] = None,
-              softcap: float = 0.0, as_act: bool = False):
+              softcap: float = 0.0, as_act: bool = False, Dv: Optional[int] = None, gate: Optional[torch.Tensor] = None):
     """Causal attention of the packed queries against the paged cache -> [T, Hq * Dh].  ``as_act`` returns an
     ``Act``; on the CUDA decode path it already carries the int8 form written by the combine kernel, so
-    the quantised projection that follows needs no quantise launch."""
+    the quantised projection that follows needs no quantise launch.  ``Dv``: value head size where it differs from
+    ``Dh`` (the result is then [T, Hq * Dv]); ``gate`` [T, Hq] (a view, last dim dense): head h's output is
+    multiplied by sigmoid(gate[:, h]); float32 caches run in 32 bits."""
     T = q.shape[0]
+    Dv = Dv or Dh
+    if q.is_cuda and (Dv != Dh or gate is not None or k_cache.dtype == torch.float32):
+        return _gated_attention(q, k_cache, v_cache, batch, scale=scale, Hq=Hq, Hkv=Hkv, Dh=Dh, Dv=Dv, window=window,
+                                sinks=sinks, softcap=softcap, gate=gate)
     if as_act:
         if q.is_cuda and batch.is_decode and Dh % 32 == 0:
             sp = decode_splits(batch, Hkv, window)
@@ -484,7 +526,30 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, bat
         kb, vb = kv_gather(k_cache, idx), kv_gather(v_cache, idx)
         outs.append(ref.attention(q[q0:q1], kb, vb, batch.positions[q0:q1], scale=scale, window=window, sinks=sinks,
                                   softcap=softcap))
-    return torch.cat(outs, 0).reshape(T, Hq * Dh)
+    out = torch.cat(outs, 0)
+    if gate is not None:
+        out = out * torch.sigmoid(gate.float()).unsqueeze(-1)
+    return out.reshape(T, Hq * Dv)
+
+
+def _gated_attention(q, k_cache, v_cache, batch: Batch, *, scale, Hq, Hkv, Dh, Dv, window, sinks, softcap, gate) -> torch.Tensor:
+    """The CUDA side of :func:`attention` for the forms beyond one head size and bf16: keys and values of different
+    sizes, a sigmoid gate per head, 32-bit caches."""
+    kk = _k()
+    T = q.shape[0]
+    if is_fp8(k_cache):
+        raise ValueError("8-bit pages have no gated attention")
+    kw = dict(scale=scale, Hq=Hq, Hkv=Hkv, Dh=Dh, Dv=Dv, page_size=batch.page_size, sinks=sinks, softcap=softcap, window=window,
+              gate=gate)
+    if k_cache.dtype == torch.float32:
+        return kk.attn_f32(q, k_cache, v_cache, batch.block_table, batch.kv_lens, batch.cu_q, **kw).view(T, Hq * Dv)
+    if batch.is_decode:
+        sp = decode_splits(batch, Hkv, window)
+        out = kk.attn_decode(q, k_cache, v_cache, batch.block_table, batch.kv_lens, splits=sp,
+                             split_len=decode_split_len(batch, sp, window), **kw)
+    else:
+        out = kk.attn_prefill(q, k_cache, v_cache, batch.block_table, batch.kv_lens, batch.cu_q, batch.max_q_len, **kw)
+    return out.view(T, Hq * Dv)
 
 
 def argmax(logits: torch.Tensor) -> torch.Tensor:
@@ -525,6 +590,72 @@ def route_sigmoid(logits: torch.Tensor, k: int, bias: Optional[torch.Tensor], no
     if normalize:
         w = w / w.sum(-1, keepdim=True).clamp_min(6.103515625e-5)
     return ids.to(torch.int32), w * scale
+
+
+def route_softmax_renorm(logits: torch.Tensor, E: int, k: int, scale: float, n_always: int = 0):
+    """Softmax over the first ``E`` logits, the ``k`` largest, their scores divided by their sum (+ 1e-20) times
+    ``scale``.  ``n_always`` > 0 appends the experts ``E .. E + n_always - 1`` (slices of a shared expert) to every
+    token, each with the weight sigmoid(logits[:, E]).  -> (ids int32, weights f32), both [T, k + n_always]."""
+    if logits.is_cuda:
+        return _k().moe_route(logits, k, mode=2, scale=scale, n_experts=E, n_always=n_always)
+    s = torch.softmax(logits[:, :E].float(), -1)
+    val, ids = torch.topk(s, k, dim=-1)
+    w = val / (val.sum(-1, keepdim=True) + 1e-20) * scale
+    if n_always:
+        T = logits.shape[0]
+        ids = torch.cat([ids, torch.arange(E, E + n_always).expand(T, n_always)], 1)
+        w = torch.cat([w, torch.sigmoid(logits[:, E:E + 1].float()).expand(T, n_always)], 1)
+    return ids.to(torch.int32), w
+
+
+@dataclass
+class MoeParts:
+    """The experts' output rows before they are summed per token: token t's result is the sum over j < k of
+    ``w[t * k + j] * y[pos[t * k + j]]`` (``w`` None: rows are weighted already; ``pos`` None: row t * k + j)."""
+    y: torch.Tensor
+    k: int
+    pos: Optional[torch.Tensor] = None
+    w: Optional[torch.Tensor] = None
+
+    def sum(self) -> torch.Tensor:
+        y = self.y.float()
+        if self.pos is not None:
+            y = y[self.pos.long()]
+        if self.w is not None:
+            y = y * self.w.reshape(-1, 1)
+        return y.view(-1, self.k, y.shape[-1]).sum(1)
+
+
+def moe_expert_parts(a: Act, ids: torch.Tensor, weights: torch.Tensor, gate_up: QuantWeight, down: QuantWeight, *, act: str) -> MoeParts:
+    """:func:`moe_experts` without its last step, for a consumer that sums the rows itself (``residual_layernorm``):
+    every expert is local, there are no biases, and ``act`` is gated."""
+    T, k = ids.shape
+    if ids.device.type != "cuda":
+        return MoeParts(moe_experts(a, ids, weights, gate_up, down, act=act), 1)
+    kk = _k()
+    P, E, F_out, D = T * k, gate_up.experts, gate_up.N // 2, down.N
+    wts = weights.reshape(-1)
+    if a.b.dtype == torch.float32:
+        bn = 64
+        order, tiles, pos = kk.moe_sort(ids, E, bn)
+        y1 = kk.gemm_f32(gate_up, a.b, tiles=tiles, rows=order, row_div=k)
+        h = kk.glu_f32(y1[:, :F_out], y1[:, F_out:], act)
+        return MoeParts(kk.gemm_f32(down, h, tiles=tiles), k, pos, wts)
+    if P <= 4 * GEMV_MAX_M:
+        flat = ids.reshape(-1)
+        gu = torch.empty((P, F_out), dtype=torch.bfloat16, device=ids.device)
+        kk.gemv(gate_up, xb=a.b, M=1, ids=flat, x_div=k, act=act, out=gu)
+        y = torch.empty((P, D), dtype=torch.float32, device=ids.device)
+        kk.gemv(down, xb=gu, M=1, ids=flat, x_div=1, out=y)
+        return MoeParts(y, k, None, wts)
+    avg = max(1, P // E)
+    bn = 32 if avg <= 32 else 64 if avg <= 64 else 128 if avg <= 128 else 256
+    order, tiles, pos = kk.moe_sort(ids, E, bn)
+    xs = kk.gather_bf16_rows(a.b, order, k)
+    y1 = kk.gemm_bf16_grouped(_dequant_scratch(gate_up), E, xs, tiles, bn, out_dtype=torch.bfloat16, zero=False)
+    h, _, _ = kk.glu(y1, y1[:, F_out:], act, F_out, gate_up.N, gate_up.N, P)
+    y2 = kk.gemm_bf16_grouped(_dequant_scratch(down), E, h, tiles, bn, out_dtype=torch.bfloat16, zero=False)
+    return MoeParts(y2, k, pos, wts)
 
 
 def moe_experts(a: Act, ids: torch.Tensor, weights: torch.Tensor, gate_up: QuantWeight, down: QuantWeight, *,

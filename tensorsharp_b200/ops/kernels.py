@@ -69,7 +69,8 @@ class QkvArgs(C.Structure):
                 ("in_f32", C.c_int), ("qn", _vp), ("kn", _vp), ("v_norm", C.c_int), ("eps", C.c_float),
                 ("pos", _vp), ("slot", _vp), ("freq_factors", _vp), ("cs_table", _vp), ("q_out", _vp), ("k_cache", _vp),
                 ("v_cache", _vp), ("q_scale", C.c_float),
-                ("T", C.c_int), ("Hq", C.c_int), ("Hkv", C.c_int), ("Dh", C.c_int), ("rp", RopeParams)]
+                ("T", C.c_int), ("Hq", C.c_int), ("Hkv", C.c_int), ("Dh", C.c_int), ("rp", RopeParams),
+                ("Dv", C.c_int), ("norm_n", C.c_int), ("qt_coef", C.c_float), ("qt_every", C.c_float), ("out_f32", C.c_int)]
 
 
 class AttnArgs(C.Structure):
@@ -78,7 +79,8 @@ class AttnArgs(C.Structure):
                 ("scale", C.c_float), ("softcap", C.c_float), ("window", C.c_int),
                 ("B", C.c_int), ("Hq", C.c_int), ("Hkv", C.c_int), ("Dh", C.c_int), ("page_size", C.c_int),
                 ("max_pages", C.c_int), ("splits", C.c_int), ("q_pos0", _vp), ("lse_out", _vp),
-                ("out_q", _vp), ("out_ds", _vp), ("ticket", _vp), ("split_len", C.c_int)]
+                ("out_q", _vp), ("out_ds", _vp), ("ticket", _vp), ("split_len", C.c_int),
+                ("gate", _vp), ("gate_tok", C.c_long), ("gate_f32", C.c_int), ("Dv", C.c_int)]
 
 
 _configured = False
@@ -97,7 +99,9 @@ def _lib():
         for name in ("tsb_quantize_q8", "tsb_gemv", "tsb_rmsnorm", "tsb_qkv_rope", "tsb_glu", "tsb_gather_rows",
                      "tsb_argmax", "tsb_rope_table", "tsb_fused_gemv", "tsb_gemv_push", "tsb_tp_reduce_norm", "tsb_tpseq_push_rows", "tsb_decode_advance", "tsb_attn_decode", "tsb_attn_prefill", "tsb_gemm_bf16", "tsb_causal_conv1d", "tsb_gdn_recurrent",
                      "tsb_mamba2_recurrent"):
-            getattr(lib, name).restype = C.c_int
+            fn = getattr(lib, name, None)             # a library linked from a selection of sources lacks some
+            if fn is not None:
+                fn.restype = C.c_int
         _configured = True
     return lib
 
@@ -157,17 +161,50 @@ def gemv_multi(ws, *, xq=None, xds=None, xb=None, M: int, out_dtype=torch.float3
     return out
 
 
-def moe_route(logits: torch.Tensor, k: int, *, mode: int = 0, sel_bias=None, normalize: bool = False, scale: float = 1.0):
+def moe_route(logits: torch.Tensor, k: int, *, mode: int = 0, sel_bias=None, normalize: bool = False, scale: float = 1.0,
+              n_experts: Optional[int] = None, n_always: int = 0):
     """Router on the device: f32 logits [T, E] -> (ids int32 [T, k], weights f32 [T, k]).  mode 0: top-k
-    then softmax over the selected; mode 1: sigmoid, selection on p + sel_bias, optional renormalise, scale."""
+    then softmax over the selected; mode 1: sigmoid, selection on p + sel_bias, optional renormalise, scale;
+    mode 2: softmax over all, top-k, divided by the selected's sum (+ 1e-20), scale.  ``n_experts``: only the
+    first of the columns are routed experts; ``n_always``: that many further ids follow on every token,
+    weighted sigmoid(logits[:, n_experts])."""
     assert logits.is_cuda and logits.dtype == torch.float32 and logits.is_contiguous()
-    T, E = logits.shape
-    ids = torch.empty((T, k), dtype=torch.int32, device=logits.device)
-    w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
-    native.check(_lib().tsb_moe_route(_p(logits), _p(sel_bias), C.c_int(T), C.c_int(E), C.c_int(k), C.c_int(mode),
-                                      C.c_int(1 if normalize else 0), C.c_float(scale), _p(ids), _p(w), _stream()), "moe_route")
+    T, ld = logits.shape
+    E, ko = n_experts or ld, k + n_always
+    ids = torch.empty((T, ko), dtype=torch.int32, device=logits.device)
+    w = torch.empty((T, ko), dtype=torch.float32, device=logits.device)
+    native.check(_lib().tsb_moe_route_ex(_p(logits), _p(sel_bias), C.c_int(T), C.c_int(E), C.c_int(k), C.c_int(mode),
+                                         C.c_int(1 if normalize else 0), C.c_float(scale), C.c_int(ld), C.c_int(n_always), _p(ids), _p(w),
+                                         _stream()), "moe_route")
     _count(1)
     return ids, w
+
+
+def moe_sort(ids: torch.Tensor, E: int, bn: int):
+    """Sort the (token, slot) pairs of ``ids`` (int32, every value in [0, E)) by expert on the device.  Returns ``order``
+    (the pair at each sorted place), ``tiles`` int32 [ceil(P / bn) + E, 3] (expert or -1, first, end place; at most bn
+    places each) and ``pos`` (the sorted place of each pair)."""
+    assert ids.dtype == torch.int32 and ids.is_contiguous()
+    check_index("moe_sort", "expert id", ids, E)
+    P, dev = ids.numel(), ids.device
+    n_tiles = (P + bn - 1) // bn + E
+    order, pos = torch.empty(P, dtype=torch.int32, device=dev), torch.empty(P, dtype=torch.int32, device=dev)
+    tiles = torch.empty((n_tiles, 3), dtype=torch.int32, device=dev)
+    counts = torch.empty(((P + 1023) // 1024, E), dtype=torch.int32, device=dev) if P > 4096 else None
+    native.check(_lib().tsb_moe_sort(_p(ids), C.c_int(P), C.c_int(E), C.c_int(bn), _p(order), _p(pos), _p(tiles), C.c_int(n_tiles), _p(counts),
+                                     _stream()), "moe_sort")
+    _count(1 if counts is None else 3)
+    return order, tiles, pos
+
+
+def gather_bf16_rows(x: torch.Tensor, order: torch.Tensor, div: int) -> torch.Tensor:
+    """x[order // div] for bf16 rows."""
+    assert x.dtype == torch.bfloat16 and x.is_contiguous() and order.dtype == torch.int32
+    out = torch.empty((order.numel(), x.shape[1]), dtype=torch.bfloat16, device=x.device)
+    native.check(_lib().tsb_gather_bf16_rows(_p(x), _p(order), C.c_int(order.numel()), C.c_int(div), C.c_int(x.shape[1]), _p(out), _stream()),
+                 "gather_bf16_rows")
+    _count(1)
+    return out
 
 
 def moe_grouped(*, xq=None, xds=None, xb=None, ids: torch.Tensor, weights: torch.Tensor, gate_up: QuantWeight,
@@ -320,7 +357,7 @@ def yarn_corr_dims(n_dims: int, n_ctx_orig: int, freq_base: float, beta_fast: fl
 
 def qkv_rope(*, q, k, v, q_strides, k_strides, v_strides, Hq, Hkv, Dh, pos, slot, q_out, k_cache, v_cache,
              qn=None, kn=None, v_norm=False, eps=1e-6, rope: RopeParams, freq_factors=None, q_scale=1.0,
-             cs_table=None):
+             cs_table=None, Dv=None, norm_n=None, q_temp=None, out_f32=False):
     T = int(pos.numel())
     check_index("qkv_rope", "KV slot", slot, k_cache.shape[0] if k_cache is not None else 1 << 62)
     check_index("qkv_rope", "position", pos, 1 << 31)
@@ -339,6 +376,8 @@ def qkv_rope(*, q, k, v, q_strides, k_strides, v_strides, Hq, Hkv, Dh, pos, slot
     a.q_scale = q_scale
     a.T, a.Hq, a.Hkv, a.Dh = T, Hq, Hkv, Dh
     a.rp = rope
+    a.Dv, a.norm_n, a.out_f32 = Dv or Dh, norm_n or Dh, int(out_f32)
+    a.qt_coef, a.qt_every = q_temp or (0.0, 0.0)
     native.check(_lib().tsb_qkv_rope(C.byref(a), _stream()), "qkv_rope")
     _count(1)
 
@@ -404,7 +443,7 @@ def decode_advance(sampled, batch) -> None:
 
 
 def _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, cu_q, sinks, scale, softcap, window, Hq, Hkv, Dh,
-               page_size, B):
+               page_size, B, Dv=None, gate=None):
     check_index("attention", "block-table page", block_table, k_cache.shape[0] // page_size)
     check_index("attention", "cache length", kv_lens, block_table.shape[1] * page_size + 1)
     a = AttnArgs()
@@ -414,21 +453,26 @@ def _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, cu_q, sinks, scal
     a.B, a.Hq, a.Hkv, a.Dh, a.page_size = B, Hq, Hkv, Dh, page_size
     a.max_pages = block_table.shape[1]
     a.splits = 1
+    a.Dv = Dv or Dh
+    if gate is not None:
+        assert gate.shape == (q.shape[0], Hq) and gate.stride(1) == 1
+        a.gate, a.gate_tok, a.gate_f32 = gate.data_ptr(), gate.stride(0), int(gate.dtype == torch.float32)
     return a
 
 
 def attn_decode(q, k_cache, v_cache, block_table, kv_lens, *, scale, Hq, Hkv, Dh, page_size, splits, sinks=None,
-                softcap=0.0, window=0, out=None, want_q8=False, split_len=0):
+                softcap=0.0, window=0, out=None, want_q8=False, split_len=0, Dv=None, gate=None):
     """q [B, Hq, Dh] bf16; one query per sequence against the paged cache.  ``want_q8`` also returns the
     output as int8 groups of 32 with (scale, sum) written by the combine kernel: (out, q, ds)."""
     B = q.shape[0]
+    Dv = Dv or Dh
     if out is None:
-        out = torch.empty_like(q)
+        out = torch.empty((B, Hq, Dv), dtype=q.dtype, device=q.device)
     a = _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, None, sinks, scale, softcap, window, Hq, Hkv, Dh,
-                   page_size, B)
+                   page_size, B, Dv, gate)
     a.splits = splits
     a.split_len = split_len
-    part_o = torch.empty((B, Hq, splits, Dh), dtype=torch.float32, device=q.device)
+    part_o = torch.empty((B, Hq, splits, Dv), dtype=torch.float32, device=q.device)
     part_ml = torch.empty((B, Hq, splits, 2), dtype=torch.float32, device=q.device)
     a.part_o, a.part_ml = _p(part_o), _p(part_ml)
     oq = ods = None
@@ -478,18 +522,93 @@ def kv_load_fp8(k_cache: torch.Tensor, v_cache: torch.Tensor, idx: torch.Tensor)
 
 
 def attn_prefill(q, k_cache, v_cache, block_table, kv_lens, cu_q, max_q_len, *, scale, Hq, Hkv, Dh, page_size,
-                 sinks=None, softcap=0.0, window=0, out=None, q_pos0=None, lse_out=None):
+                 sinks=None, softcap=0.0, window=0, out=None, q_pos0=None, lse_out=None, Dv=None, gate=None):
     """q [T, Hq, Dh] bf16 packed over sequences (cu_q [B+1]).  ``q_pos0`` [B] int32 overrides the cache
     position of each sequence's first query (default kv_len - q_len); ``lse_out`` [T, Hq] f32 receives the
     log-sum-exp of the scores, for merging partial results over KV shards."""
     B = kv_lens.shape[0]
     if out is None:
-        out = torch.empty_like(q)
+        out = torch.empty((q.shape[0], Hq, Dv or Dh), dtype=q.dtype, device=q.device)
     a = _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, cu_q, sinks, scale, softcap, window, Hq, Hkv, Dh,
-                   page_size, B)
+                   page_size, B, Dv, gate)
     a.q_pos0 = q_pos0.data_ptr() if q_pos0 is not None else None
     a.lse_out = lse_out.data_ptr() if lse_out is not None else None
     native.check(_lib().tsb_attn_prefill(C.byref(a), C.c_int(max_q_len), _stream()), "attn_prefill")
+    _count(1)
+    return out
+
+
+def attn_f32(q, k_cache, v_cache, block_table, kv_lens, cu_q, *, scale, Hq, Hkv, Dh, page_size, Dv=None, sinks=None, softcap=0.0,
+             window=0, gate=None):
+    """Attention in 32 bits over a float32 cache, prompts and decode alike: q [T, Hq, Dh] -> [T, Hq, Dv]."""
+    assert q.dtype == k_cache.dtype == v_cache.dtype == torch.float32 and (gate is None or gate.dtype == torch.float32)
+    out = torch.empty((q.shape[0], Hq, Dv or Dh), dtype=torch.float32, device=q.device)
+    a = _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, cu_q, sinks, scale, softcap, window, Hq, Hkv, Dh, page_size,
+                   kv_lens.shape[0], Dv, gate)
+    native.check(_lib().tsb_attn_f32(C.byref(a), C.c_int(q.shape[0]), _stream()), "attn_f32")
+    _count(1)
+    return out
+
+
+class SandwichArgs(C.Structure):
+    _fields_ = [("h", _vp), ("y", _vp), ("pos", _vp), ("wts", _vp), ("post_w", _vp), ("post_b", _vp), ("add", _vp), ("pre_w", _vp),
+                ("pre_b", _vp), ("out", _vp), ("rows", C.c_long), ("D", C.c_int), ("n", C.c_int), ("parts", C.c_int),
+                ("y_f32", C.c_int), ("out_f32", C.c_int), ("eps", C.c_float)]
+
+
+def residual_layernorm(h: torch.Tensor, eps: float, n: int, *, y=None, pos=None, wts=None, parts: int = 1, post=None, add=None, pre=None,
+                       out_dtype=torch.bfloat16) -> Optional[torch.Tensor]:
+    """h (f32 [T, D], in place) += layernorm(sum of y's parts; post) (+ add); returns layernorm(h; pre) or None."""
+    assert h.dtype == torch.float32 and h.is_contiguous()
+    T, D = h.shape
+    a = SandwichArgs()
+    a.h, a.rows, a.D, a.n, a.parts, a.eps = _p(h), T, D, n, parts, eps
+    if y is not None:
+        assert y.is_contiguous() and y.shape[-1] == D and y.dtype in (torch.float32, torch.bfloat16)
+        assert (y.shape[0] == T * parts or pos is not None) and (pos is None or (pos.dtype == torch.int32 and pos.numel() == T * parts))
+        assert wts is None or (wts.dtype == torch.float32 and wts.is_contiguous() and wts.numel() == T * parts)
+        check_index("residual_layernorm", "part row", pos, y.shape[0], low=-1)
+        a.y, a.pos, a.wts, a.y_f32 = _p(y), _p(pos), _p(wts), int(y.dtype == torch.float32)
+        a.post_w, a.post_b = _p(post[0]), _p(post[1])
+    a.add = _p(add)
+    out = None
+    if pre is not None:
+        out = torch.empty((T, D), dtype=out_dtype, device=h.device)
+        a.pre_w, a.pre_b, a.out, a.out_f32 = _p(pre[0]), _p(pre[1]), _p(out), int(out_dtype == torch.float32)
+    native.check(_lib().tsb_sandwich_norm(C.byref(a), _stream()), "residual_layernorm")
+    _count(1)
+    return out
+
+
+class GemmF32Args(C.Structure):
+    _fields_ = [("W", _vp), ("X", _vp), ("out", _vp), ("bias", _vp), ("tiles", _vp), ("rows", _vp), ("ldx", C.c_long), ("ldo", C.c_long),
+                ("T", C.c_int), ("N", C.c_int), ("K", C.c_int), ("row_div", C.c_int)]
+
+
+def gemm_f32(w: QuantWeight, x: torch.Tensor, *, bias=None, tiles=None, rows=None, row_div: int = 1) -> torch.Tensor:
+    """x [T, K] float32 @ w^T in 32-bit arithmetic (weights as stored, bf16 or f32).  With ``tiles`` (int32 [n, 3] on the
+    device, pieces of at most 64 rows, see :func:`moe_sort`) ``w`` is a stack and row i of the result uses the matrix of its
+    tile; ``rows`` int32: result row i reads x row rows[i] // row_div."""
+    from ..gguf.constants import GGMLType
+    assert x.dtype == torch.float32 and x.stride(1) == 1 and x.shape[1] == w.K and w.ggml_type in (GGMLType.BF16, GGMLType.F32)
+    T = rows.numel() if rows is not None else x.shape[0]
+    out = torch.empty((T, w.N), dtype=torch.float32, device=x.device)
+    a = GemmF32Args()
+    a.W, a.X, a.out, a.bias, a.tiles, a.rows = _p(w.planes[0]), _p(x), _p(out), _p(bias), _p(tiles), _p(rows)
+    a.ldx, a.ldo, a.T, a.N, a.K, a.row_div = x.stride(0), w.N, T, w.N, w.K, row_div
+    native.check(_lib().tsb_gemm_f32(C.byref(a), C.c_int(w.ggml_type == GGMLType.BF16), C.c_int(tiles.shape[0] if tiles is not None else 0),
+                                     _stream()), "gemm_f32")
+    _count(1)
+    return out
+
+
+def glu_f32(gate: torch.Tensor, up: Optional[torch.Tensor], act: str) -> torch.Tensor:
+    """Gated activation of two float32 [T, F] views in 32 bits."""
+    T, F = gate.shape
+    assert gate.dtype == torch.float32 and gate.stride(1) == 1 and (up is None or (up.dtype == torch.float32 and up.stride(1) == 1))
+    out = torch.empty((T, F), dtype=torch.float32, device=gate.device)
+    native.check(_lib().tsb_glu_f32(_p(gate), _p(up), C.c_long(gate.stride(0)), C.c_long(up.stride(0) if up is not None else 0), C.c_long(T),
+                                    C.c_int(F), C.c_int(ACT[act]), _p(out), _stream()), "glu_f32")
     _count(1)
     return out
 
@@ -539,15 +658,15 @@ def gemm_bf16(W: torch.Tensor, X: torch.Tensor, *, out_dtype=torch.bfloat16, bia
 
 
 def gemm_bf16_grouped(W: torch.Tensor, E: int, X: torch.Tensor, tiles: torch.Tensor, bn: int, *, out_dtype=torch.bfloat16,
-                      bias=None) -> torch.Tensor:
+                      bias=None, zero: bool = True) -> torch.Tensor:
     """Grouped GEMM over a stack of ``E`` matrices: W [E * N, K] bf16, X [P, K] bf16 with each group's rows contiguous,
     ``tiles`` int32 [n_tiles, 3] on the device = (matrix index or -1, first row, end row) with at most ``bn`` rows per
-    tile -> out [P, N], zero where no tile covers a row."""
+    tile -> out [P, N], zero where no tile covers a row (``zero=False``: every row is covered)."""
     assert W.dtype == torch.bfloat16 and X.dtype == torch.bfloat16 and W.stride(1) == 1 and X.stride(1) == 1
     assert tiles.dtype == torch.int32 and tiles.is_contiguous() and tiles.shape[1] == 3
     N, K = W.shape[0] // E, W.shape[1]
     P = X.shape[0]
-    out = torch.zeros((P, N), dtype=out_dtype, device=X.device)
+    out = (torch.zeros if zero else torch.empty)((P, N), dtype=out_dtype, device=X.device)
     lib = _lib()
     lib.tsb_gemm_bf16_grouped.restype = C.c_int
     native.check(lib.tsb_gemm_bf16_grouped(_p(W), C.c_long(W.stride(0)), C.c_int(E), _p(X), C.c_long(X.stride(0)), _p(out),

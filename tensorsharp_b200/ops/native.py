@@ -16,7 +16,7 @@ import subprocess
 import sys
 from concurrent.futures import ThreadPoolExecutor
 from pathlib import Path
-from typing import List, Optional
+from typing import List, Optional, Sequence
 
 _PKG = Path(__file__).resolve().parent.parent
 CSRC = _PKG / "csrc"
@@ -56,13 +56,16 @@ def _stamp(src: Path) -> str:
     return h.hexdigest()
 
 
-def build(force: bool = False, verbose: bool = False, jobs: Optional[int] = None) -> Path:
+def build(force: bool = False, verbose: bool = False, jobs: Optional[int] = None, only: Optional[Sequence[str]] = None) -> Path:
     """Compile every source under ``csrc`` for sm_100a and link the shared library.
-    Objects are cached by content hash, so an unchanged tree is a no-op."""
+    Objects are cached by content hash, so an unchanged tree is a no-op.  ``only`` (source file names, closed
+    under their references to one another) compiles those and links them as a library of their own."""
     OUT_DIR.mkdir(exist_ok=True)
     nvcc = _nvcc()
     objs, todo = [], []
-    for src in sources():
+    wanted = sources() if only is None else [CSRC / n for n in only]
+    lib_path = LIB_PATH if only is None else _part_path(only)
+    for src in wanted:
         obj = OUT_DIR / (src.stem + ".o")
         stamp = OUT_DIR / (src.stem + ".stamp")
         objs.append(obj)
@@ -84,13 +87,33 @@ def build(force: bool = False, verbose: bool = False, jobs: Optional[int] = None
     if todo:
         with ThreadPoolExecutor(max_workers=jobs or min(8, os.cpu_count() or 2)) as ex:
             list(ex.map(compile_one, todo))
-    if todo or not LIB_PATH.exists():
-        cmd = [nvcc, "-shared", "-o", str(LIB_PATH), *map(str, objs), "-gencode",
+    if todo or not lib_path.exists():
+        part = lib_path.with_suffix(f".{os.getpid()}.part")
+        cmd = [nvcc, "-shared", "-o", str(part), *map(str, objs), "-gencode",
                "arch=compute_100a,code=sm_100a", "-ldl"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise NativeLibraryError(f"link failed:\n{r.stderr[-4000:]}")
-    return LIB_PATH
+        os.replace(part, lib_path)
+    return lib_path
+
+
+def _part_path(only: Sequence[str]) -> Path:
+    """The library of a selection of sources; its name holds what it was linked from."""
+    h = hashlib.sha1(" ".join(f"{n} {_stamp(CSRC / n)}" for n in sorted(only)).encode()).hexdigest()[:12]
+    return OUT_DIR / f"libtsb200-part-{h}.so"
+
+
+def ensure(only: Optional[Sequence[str]] = None) -> None:
+    """Have kernels to run: the whole library where it is built and current, otherwise the selection ``only`` (compiled
+    now if it is not there yet), otherwise the whole library built now."""
+    global _lib
+    if _lib is not None or (LIB_PATH.exists() and not is_stale()):
+        return
+    if only is None:
+        build()
+        return
+    _lib = _open(build(only=only))
 
 
 def build_tests(force: bool = False) -> List[Path]:
@@ -136,9 +159,14 @@ def lib() -> ctypes.CDLL:
             raise NativeLibraryError(
                 f"{LIB_PATH} is missing: run `python -c 'import __graft_entry__ as g; g.build()'` "
                 "(or tensorsharp_b200.ops.native.build()) before using the CUDA path")
-        _lib = ctypes.CDLL(str(LIB_PATH))
-        _lib.tsb_last_error.restype = ctypes.c_char_p
+        _lib = _open(LIB_PATH)
     return _lib
+
+
+def _open(path: Path) -> ctypes.CDLL:
+    handle = ctypes.CDLL(str(path))
+    handle.tsb_last_error.restype = ctypes.c_char_p
+    return handle
 
 
 def available() -> bool:

@@ -30,6 +30,18 @@ def layernorm(x, w, b, eps):
     return torch.nn.functional.layer_norm(x.float(), (x.shape[-1],), w, b, eps)
 
 
+def layernorm_n(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float, n: int) -> torch.Tensor:
+    """Layer norm over the first ``n`` columns of rows that are padded with zeros (so are ``w`` and ``b``)."""
+    y = torch.zeros(x.shape, dtype=torch.float32, device=x.device)
+    y[..., :n] = layernorm(x[..., :n], w[:n], b[:n], eps)
+    return y
+
+
+def query_temperature(pos: torch.Tensor, coef: float, every: float) -> torch.Tensor:
+    """1 + coef ln(floor((p + 1) / every) + 1): the factor that keeps attention sharp at far positions."""
+    return 1.0 + coef * torch.log1p(torch.floor((pos.float() + 1.0) / every))
+
+
 def rope_cos_sin(pos: torch.Tensor, rot_dim: int, theta_base: float, freq_scale: float = 1.0,
                  ext_factor: float = 0.0, attn_factor: float = 1.0, corr_lo: float = 0.0, corr_hi: float = 0.0,
                  freq_factors: Optional[torch.Tensor] = None):

@@ -40,11 +40,11 @@ class SeqState:
 
 
 class PagedKV:
-    def __init__(self, layer_shapes: Sequence[Optional[Tuple[int, int]]], n_pages: int, page_size: int = 64,
+    def __init__(self, layer_shapes: Sequence[Optional[Tuple[int, ...]]], n_pages: int, page_size: int = 64,
                  device="cpu", dtype=torch.bfloat16, donors: Optional[Dict[int, int]] = None, max_seqs: int = 64,
                  window_layers: Optional[Dict[int, int]] = None, ring_chunk: int = 0):
-        """``layer_shapes[l]`` is ``(Hkv, Dh)`` for attention layers, ``None`` for layers
-        without a KV cache; ``donors[l] = m`` makes layer ``l`` read layer ``m``'s cache.
+        """``layer_shapes[l]`` is ``(Hkv, Dh)``, or ``(Hkv, Dk, Dv)`` where keys and values have different
+        sizes, for attention layers, ``None`` for layers without a KV cache; ``donors[l] = m`` makes layer ``l`` read layer ``m``'s cache.
         ``window_layers[l] = W`` with ``ring_chunk > 0`` gives those layers the ring pool."""
         self.page_size = page_size
         self.n_pages = n_pages
@@ -64,10 +64,10 @@ class PagedKV:
                 self.k.append(None)
                 self.v.append(None)
                 continue
-            hkv, dh = shp
+            hkv, dh, dv = shp[0], shp[1], shp[-1]
             rows = (self.n_wpages if l in self.window_layers else n_pages) * page_size
             self.k.append(torch.zeros((rows, hkv, dh), dtype=dtype, device=self.device))
-            self.v.append(torch.zeros((rows, hkv, dh), dtype=dtype, device=self.device))
+            self.v.append(torch.zeros((rows, hkv, dv), dtype=dtype, device=self.device))
         self._wfree: List[int] = list(range(self.n_wpages - 1, -1, -1))
         for l, m in donors.items():
             self.k[l], self.v[l] = self.k[m], self.v[m]
@@ -152,10 +152,18 @@ class PagedKV:
 
     # ------------------------------------------------------------------ batches
     def build_batch(self, seqs: Sequence[SeqState], new_tokens: Sequence[Sequence[int]],
-                    table_width: Optional[int] = None) -> Batch:
+                    table_width: Optional[int] = None, rows: Optional[Sequence[Sequence[int]]] = None) -> Batch:
         """Reserve pages for the new tokens of each sequence and assemble the packed batch.
-        Sequence lengths are advanced; the caller runs the model right after."""
+        Sequence lengths are advanced; the caller runs the model right after.  ``rows[i]`` lists the places
+        among sequence i's new tokens whose logits are wanted (default: its last token).  When the pool is
+        short of pages for the whole batch it raises before any sequence is touched."""
         ps = self.page_size
+        need = sum(max(0, (s.length + len(nt) + ps - 1) // ps - len(s.pages)) for s, nt in zip(seqs, new_tokens))
+        if need > len(self._free):
+            raise OutOfPagesError(f"need {need} pages, {len(self._free)} free")
+        for want, nt in zip(rows or (), new_tokens):
+            if any(not 0 <= r < len(nt) for r in want):
+                raise ValueError(f"rows {list(want)} are not all among the {len(nt)} new tokens")
         toks: List[int] = []
         pos: List[int] = []
         slots: List[int] = []
@@ -178,7 +186,10 @@ class PagedKV:
             s.length += n
             cu.append(cu[-1] + n)
             lens.append(s.length)
-            last.append(cu[-1] - 1)
+            if rows is None:
+                last.append(cu[-1] - 1)
+            else:
+                last.extend(cu[-2] + r for r in rows[len(cu) - 2])
         width = table_width or max(1, max(len(s.pages) for s in seqs))
         table = torch.zeros((len(seqs), width), dtype=torch.int32)
         for i, s in enumerate(seqs):
