@@ -15,7 +15,7 @@ from typing import List, Optional, Sequence
 
 from ..runtime.sampling import SamplingConfig
 
-USAGE = ("Usage: python -m tensorsharp_b200.cli --model <path.gguf> [--input <input.txt>] "
+USAGE = ("Usage: python -m tensorsharp_b200.cli --model <path.gguf | model folder> [--input <input.txt>] "
          "[--input-jsonl <requests.jsonl>] [--multi-turn-jsonl <turns.jsonl>] [--image <image.png>] [--audio <a.wav>] "
          "[--video <v.mp4>] [--mmproj <path.gguf>] [--output <output.txt>] [--max-tokens N] [--test] "
          "[--backend b200|cpu] [--interactive] [--system <text>] [--system-file <path>] "
@@ -24,7 +24,7 @@ USAGE = ("Usage: python -m tensorsharp_b200.cli --model <path.gguf> [--input <in
          "[--benchmark [--bench-prefill N] [--bench-decode N] [--bench-runs N] [--bench-chunked]] "
          "[--test-chunked-prefill [--correct-prefill N] [--correct-decode N]] [--bench-kvcache [--bench-kv-turns N]] "
          "[--test-templates <dir>] [--log-level info|debug|trace] [--log-dir <path>] [--log-file off] [--log-console off] "
-         "[--batch-size N] [--max-context N] [--kv-dtype bf16|fp8] [--tp N | --pp N | --cp N  (one process per GPU: python -m torch.distributed.run "
+         "[--batch-size N] [--max-context N] [--kv-dtype bf16|fp8] [--dtype bfloat16|float32] [--tp N | --pp N | --cp N  (one process per GPU: python -m torch.distributed.run "
          "--nproc-per-node N -m tensorsharp_b200.cli ...)]")
 
 
@@ -68,6 +68,7 @@ class CliOptions:
     cp: int = 1                       # context-parallel ranks: long prompts are dealt to them slice by slice
     batch_size: int = 1               # JSONL mode: requests decoded together (continuous batching)
     max_context: Optional[int] = None
+    dtype: Optional[str] = None             # "float32": everything in 32 bits, on families that have such a path
     kv_dtype: Optional[str] = None          # "bf16" or "fp8" (exported as TSB_KV_DTYPE before the model loads)
     unknown: List[str] = field(default_factory=list)
 
@@ -131,6 +132,10 @@ def parse_cli_args(args: Sequence[str]) -> CliOptions:
             o.sampling.stop_sequences = (o.sampling.stop_sequences or []) + [value(a)]
         elif a == "--backend":
             o.backend = value(a).lower()
+        elif a == "--dtype":
+            o.dtype = value(a)
+            if o.dtype not in ("bfloat16", "float32"):
+                raise ValueError(f"Invalid value for --dtype: '{o.dtype}' (bfloat16 or float32).")
         elif a == "--kv-dtype":
             o.kv_dtype = kv_dtype_name(value(a))
         elif a == "--system-file":

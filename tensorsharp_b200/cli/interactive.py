@@ -15,6 +15,7 @@ import signal
 import time
 from typing import Callable, List, Optional, Tuple
 
+from ..gguf.folder import is_checkpoint
 from ..runtime import media
 from ..runtime.chat import ChatMessage, ToolFunction
 from ..runtime.kv_cache import KVCache
@@ -484,7 +485,7 @@ class InteractiveSession:
 
     def load_different_model(self, arg: str) -> None:
         path = _strip_quotes(arg)
-        if not path or not os.path.isfile(path):
+        if not path or not is_checkpoint(path):
             self.say(f"Model file not found: {path}")
             return
         self._reload(path, self.backend, None, f"Loading {os.path.basename(path)}")

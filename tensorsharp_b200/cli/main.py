@@ -15,6 +15,7 @@ import sys
 import time
 from typing import Any, Dict, List, Optional, Sequence
 
+from ..gguf.folder import is_checkpoint
 from ..runtime import media
 from ..runtime.chat import ChatMessage, ToolFunction, ToolParameter, dotnet_json
 from ..runtime.chat_template import build_jinja_context, render_hardcoded
@@ -596,6 +597,9 @@ def load_model(o: CliOptions, log):
         kw["max_context"] = o.max_context
     if o.kv_dtype:
         os.environ["TSB_KV_DTYPE"] = o.kv_dtype       # read by ModelBase (every rank parses the same command line)
+    if o.dtype == "float32":
+        import torch
+        kw["compute_dtype"] = torch.float32
     if o.batch_size > 1:
         kw["max_seqs"] = o.batch_size + 1          # one KV sequence per request in flight, plus the default one
     world = int(os.environ.get("WORLD_SIZE", "1"))
@@ -694,7 +698,7 @@ def _run(o: CliOptions, con: Console, log) -> int:
                  ToolsFile=o.tools_file)
     if o.test_templates_dir is not None:
         return 1 if test_chat_templates(o.test_templates_dir, con, log)["failed"] else 0
-    if o.model is None or not os.path.isfile(o.model):
+    if o.model is None or not is_checkpoint(o.model):
         log.error(Ev.CliFailed, "Model file not found: {ModelPath}", ModelPath=o.model or "(none)")
         con.error(f"Model file not found: {o.model or '(none)'}")
         con.error(USAGE)

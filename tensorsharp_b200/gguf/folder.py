@@ -31,6 +31,16 @@ def is_model_folder(path: str) -> bool:
     return os.path.isdir(path) and os.path.isfile(os.path.join(path, CONFIG_NAME))
 
 
+def is_checkpoint(path: str) -> bool:
+    """Whether ``path`` is something a model can be loaded from: a file, or a model folder."""
+    return os.path.isfile(path) or is_model_folder(path)
+
+
+def checkpoint_bytes(path: str) -> int:
+    """Size on disk of a model file, or of the weights of a model folder."""
+    return os.path.getsize(os.path.join(path, WEIGHTS_NAME) if os.path.isdir(path) else path)
+
+
 class ModelFolder(GGUFFile):
     """An open model folder; ``offset`` of a tensor is relative to ``data_offset``, as in a GGUF file."""
 

@@ -146,10 +146,11 @@ class ModelBase:
 
     @property
     def tokenizer(self):
-        """The tokenizer described by the file's ``tokenizer.*`` metadata (built on first use)."""
+        """The tokenizer described by the file's ``tokenizer.*`` metadata (built on first use); token ids as
+        text for a model folder, which has none."""
         if getattr(self, "_tokenizer", None) is None:
             from ..runtime.tokenizer import tokenizer_from_gguf
-            self._tokenizer = tokenizer_from_gguf(self.gguf)
+            self._tokenizer = tokenizer_from_gguf(self.gguf, self.cfg.vocab)
         return self._tokenizer
 
     # ------------------------------------------------------------------ multimodal

@@ -483,3 +483,80 @@ def write_nemotron_h(path: str, *, pattern="MAFMEM", hidden=256, n_heads=4, n_kv
             b.weight(p + "ffn_up.weight", (ffn, hidden), ft(p + "ffn_up.weight", l))
             b.weight(p + "ffn_down.weight", (hidden, ffn), ft(p + "ffn_down.weight", l))
     return b.write()
+
+
+def fobolorn_config(*, n_layers=3, width=128, heads=4, kv_heads=2, dim=32, vdim=48, ff=64, experts=4, top=2, shared_ff=64, vocab=512,
+                    loop=None, scale=None, router_scale=1.5, q_coef=0.4, q_every=64, eps=1e-5, no_mlp=()) -> dict:
+    """A config.json of the Fobolorn architecture with equal layers; ``loop`` = (start, stop, times) or None, ``no_mlp``:
+    layers without a feed-forward."""
+    def spec(i):
+        mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "scale": router_scale},
+               "shared": {"ff": shared_ff}}
+        return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim,
+                                               "scale": scale if scale is not None else dim ** -0.5,
+                                               "q_temp": {"coef": q_coef, "every": q_every}},
+                "mlp": None if i in no_mlp else mlp}
+    cfg = {"architecture": "Fobolorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": [spec(i) for i in range(n_layers)]}
+    if loop is not None:
+        cfg["loop"] = {"start": loop[0], "stop": loop[1], "times": loop[2]}
+    return cfg
+
+
+def write_fobolorn(folder: str, config: Optional[dict] = None, *, seed=0, device=None, gain=1.0, **sizes) -> None:
+    """A model folder with random bf16 weights for ``config`` (default: :func:`fobolorn_config` of ``sizes``): matrices
+    N(0, gain / fan-in), norm weights around 1, biases and loop vectors small."""
+    import json
+    import os
+
+    from ..gguf.folder import CONFIG_NAME, WEIGHTS_NAME, write_safetensors
+    cfg = config if config is not None else fobolorn_config(**sizes)
+    dev = torch.device(device or ("cuda" if torch.cuda.is_available() else "cpu"))
+    gen = torch.Generator(device=dev)
+    gen.manual_seed(seed)
+    t = {}
+
+    def mat(name, rows, cols, std=None):
+        w = torch.randn((rows, cols), generator=gen, device=dev) * (std if std is not None else math.sqrt(gain / cols))
+        t[name] = w.to(torch.bfloat16).cpu()
+
+    def vec(name, n, mean, std):
+        t[name] = (mean + std * torch.randn(n, generator=gen, device=dev)).to(torch.bfloat16).cpu()
+
+    D = cfg["width"]
+    mat("embed", cfg["vocab"], D, 1.0)
+    if cfg.get("loop"):
+        mat("loop.step", cfg["loop"]["times"], D, 0.3)
+
+    def norm(name):
+        vec(name, D, 1.0, 0.15)
+        vec(name + ".b", D, 0.0, 0.15)
+
+    def expert(p, ff):
+        mat(p + "gate", ff, D)
+        mat(p + "up", ff, D)
+        mat(p + "down", D, ff)
+    for i, s in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", s["mixer"]
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if s["mlp"] is not None else ()):
+            norm(p + n)
+        mat(p + "mix.q", m["heads"] * m["dim"], D)
+        mat(p + "mix.k", m["kv_heads"] * m["dim"], D)
+        mat(p + "mix.v", m["kv_heads"] * m["vdim"], D)
+        vec(p + "mix.q.norm", m["dim"], 1.4, 0.2)
+        vec(p + "mix.k.norm", m["dim"], 1.4, 0.2)
+        mat(p + "mix.g", m["heads"], D)
+        mat(p + "mix.o", D, m["heads"] * m["vdim"])
+        if s["mlp"] is not None:
+            f = s["mlp"]
+            for e in range(f["router"]["experts"]):
+                expert(f"{p}mlp.e{e}.", f["expert"]["ff"])
+            mat(p + "mlp.router", f["router"]["experts"], D)
+            if f.get("shared"):
+                expert(p + "mlp.shared.", f["shared"]["ff"])
+                mat(p + "mlp.shared.sg", 1, D)
+    norm("final.norm")
+    mat("head", cfg["vocab"], D)
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, CONFIG_NAME), "w", encoding="utf-8") as f:
+        json.dump(cfg, f, indent=1)
+    write_safetensors(os.path.join(folder, WEIGHTS_NAME), t)

@@ -7,12 +7,16 @@ to the end-of-sequence set), anything else the byte-level BPE tokenizer with
 """
 from __future__ import annotations
 
+from ..gguf.folder import ModelFolder
 from ..gguf.reader import GGUFFile
 from .tokenizer_bpe import BpeTokenizer
+from .tokenizer_ids import IdTokenizer
 from .tokenizer_spm import SentencePieceTokenizer
 
 
-def tokenizer_from_gguf(g: GGUFFile):
+def tokenizer_from_gguf(g: GGUFFile, vocab_size: int = 0):
+    if isinstance(g, ModelFolder):
+        return IdTokenizer(vocab_size)
     vocab = g.get_array("tokenizer.ggml.tokens") or []
     types = g.get_array("tokenizer.ggml.token_type")
     bos = g.get_int("tokenizer.ggml.bos_token_id", -1)

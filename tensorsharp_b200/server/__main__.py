@@ -10,6 +10,7 @@ import os
 import sys
 import time
 
+from ..gguf.folder import is_checkpoint
 from ..runtime import media
 from ..runtime.logging import Ev, setup_file_logging
 from .app import ServerApp, serve
@@ -29,7 +30,7 @@ ENDPOINT_SUMMARY = (
     "GET  /api/models                - Show hosted model state (Web UI)",
 )
 
-USAGE = ("No startup model configured. Launch with --model <path.gguf> --backend <type> [--mmproj <path>] "
+USAGE = ("No startup model configured. Launch with --model <path.gguf | model folder> --backend <type> [--mmproj <path>] "
          "[--max-tokens 20000] [--temperature F] [--top-k N] [--top-p F] [--min-p F] [--repeat-penalty F] "
          "[--presence-penalty F] [--frequency-penalty F] [--seed N] [--stop <text>] [--max-context N] [--kv-dtype bf16|fp8] [--max-sessions N] "
          "[--max-batch N] [--replicas N] to use the Web UI.")
@@ -73,7 +74,7 @@ def load_startup_model(options, svc, configured_backend, log) -> None:
     backend, err = try_resolve_supported_backend(options, configured_backend)
     if err:
         raise RuntimeError(err)
-    if not os.path.isfile(options.startup_model_path):
+    if not is_checkpoint(options.startup_model_path):
         raise FileNotFoundError(f"Configured model file not found: {options.startup_model_path}")
     if options.startup_mmproj_path and not os.path.isfile(options.startup_mmproj_path):
         raise FileNotFoundError(f"Configured mmproj file not found: {options.startup_mmproj_path}")

@@ -29,6 +29,7 @@ from http.server import BaseHTTPRequestHandler, ThreadingHTTPServer
 from typing import Any, Callable, Dict, List, Optional, Tuple
 from urllib.parse import unquote, urlsplit
 
+from ..gguf.folder import checkpoint_bytes, is_checkpoint
 from ..runtime import media
 from ..runtime.logging import Ev, FileLoggerProvider, Logger, NULL_LOGGER, log_scope
 from ..runtime.output_parser import create_output_parser, is_always_required
@@ -331,11 +332,11 @@ class ServerApp:
         models = []
         p = self.options.startup_model_path
         if p and p.strip():
-            exists = os.path.isfile(p)
+            exists = is_checkpoint(p)
             fn = os.path.basename(p)
             import datetime as _dt
             mod = iso_o(_dt.datetime.fromtimestamp(os.path.getmtime(p), _dt.timezone.utc)) if exists else ""
-            models.append({"name": os.path.splitext(fn)[0], "model": fn, "size": os.path.getsize(p) if exists else 0,
+            models.append({"name": os.path.splitext(fn)[0], "model": fn, "size": checkpoint_bytes(p) if exists else 0,
                            "modified_at": mod})
         ex.send_json({"models": models})
 
@@ -355,8 +356,8 @@ class ServerApp:
             ex.send_json({"error": err}, 404)
             return
         fam = self.svc.architecture if self.svc.is_loaded and self.svc.loaded_model_name == os.path.basename(path) else ""
-        ex.send_json({"modelfile": "", "parameters": "", "template": "", "details": {"format": "gguf", "family": fam},
-                      "model_info": {"file": os.path.basename(path), "size": os.path.getsize(path)}})
+        ex.send_json({"modelfile": "", "parameters": "", "template": "", "details": {"format": "safetensors" if os.path.isdir(path) else "gguf", "family": fam},
+                      "model_info": {"file": os.path.basename(path), "size": checkpoint_bytes(path)}})
 
     @staticmethod
     def _num_predict(body: Dict[str, Any], default: int = 200) -> int:

@@ -20,6 +20,7 @@ import os
 import time
 from typing import Iterator, List, NamedTuple, Optional, Sequence
 
+from ..gguf.folder import is_model_folder
 from ..runtime import media
 from ..runtime.chat import ChatMessage, ToolFunction
 from ..runtime.kv_cache import ReusePlanKind
@@ -647,7 +648,8 @@ class ModelService:
     def scan_models(self, directory: str) -> List[str]:
         if not os.path.isdir(directory):
             return []
-        return sorted(f for f in os.listdir(directory) if f.endswith(".gguf") and not self._is_mmproj(f))
+        return sorted(f for f in os.listdir(directory) if (f.endswith(".gguf") and not self._is_mmproj(f))
+                      or is_model_folder(os.path.join(directory, f)))
 
     def scan_mmproj_models(self, directory: str) -> List[str]:
         if not os.path.isdir(directory):

@@ -35,10 +35,11 @@ def causal_attention(q, k, v, scale):
     out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
     for h in range(H):
         g = h // (H // G)
+        s = (q[:, h] @ k[:, g].T) * scale
         for i in range(T):
-            s = (k[:i + 1, g] @ q[i, h]) * scale
-            p = torch.exp(s - s.max())
-            out[i, h] = (p / p.sum()) @ v[:i + 1, g]
+            s[i, i + 1:] = -math.inf
+        p = torch.exp(s - s.max(1, keepdim=True).values)
+        out[:, h] = (p / p.sum(1, keepdim=True)) @ v[:, g]
     return out
 
 
