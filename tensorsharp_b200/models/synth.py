@@ -542,8 +542,8 @@ def write_fobolorn(folder: str, config: Optional[dict] = None, *, seed=0, device
         mat(p + "mix.q", m["heads"] * m["dim"], D)
         mat(p + "mix.k", m["kv_heads"] * m["dim"], D)
         mat(p + "mix.v", m["kv_heads"] * m["vdim"], D)
-        vec(p + "mix.q.norm", m["dim"], 1.4, 0.2)
-        vec(p + "mix.k.norm", m["dim"], 1.4, 0.2)
+        vec(p + "mix.q.norm", m["dim"], 1.2, 0.2)
+        vec(p + "mix.k.norm", m["dim"], 1.2, 0.2)
         mat(p + "mix.g", m["heads"], D)
         mat(p + "mix.o", D, m["heads"] * m["vdim"])
         if s["mlp"] is not None:
