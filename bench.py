@@ -57,6 +57,11 @@ def parse_args():
     ap.add_argument("--trace", default=None, metavar="FILE",
                     help="after the timed runs, record three more graph replays with the CUDA activity tracer, write the "
                          "kernel events of the middle one to FILE (JSON) and print its per-kernel table to stderr")
+    ap.add_argument("--design", default=None, choices=["fobolorn"],
+                    help="measure this design at several sizes beside the closest other model at equal size (one JSON line per "
+                         "size and model) instead of the headline workload")
+    ap.add_argument("--design-size", default=None, help="with --design: only this size")
+    ap.add_argument("--design-kernels", default=None, metavar="FILE", help="with --design: write per-kernel tables to FILE")
     ap.add_argument("--cache-dir", default=os.environ.get("TSB_BENCH_CACHE", os.path.join(tempfile.gettempdir(), "tsb_bench")))
     a = ap.parse_args()
     if a.batch is None:
@@ -488,8 +493,130 @@ def run_reference(args) -> dict:
     return ref_run(args, MODEL_SHAPES[args.model])
 
 
+# Fobolorn beside gpt-oss (the framework's other mixture of experts with plain attention in every layer), both with bf16
+# weights: same width, heads, experts and layers; gpt-oss gets one routed expert more in place of the shared one, and a window
+# that never bites.  "uneven" has key and value heads of different sizes, beside gpt-oss heads of the larger size.
+DESIGN_SIZES = {
+    "2048x8": (dict(n_layers=8, width=2048, heads=16, kv_heads=4, dim=128, vdim=128, ff=1024, shared_ff=1024, experts=32, top=4, vocab=32000),
+               dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, expert_ffn=1024, n_experts=33, top_k=5, vocab=32000)),
+    "2880x6": (dict(n_layers=6, width=2880, heads=64, kv_heads=8, dim=64, vdim=64, ff=2880, shared_ff=2880, experts=32, top=4, vocab=32000),
+               dict(n_layers=6, hidden=2880, n_heads=64, n_kv_heads=8, head_dim=64, expert_ffn=2880, n_experts=33, top_k=5, vocab=32000)),
+    "uneven": (dict(n_layers=8, width=2048, heads=16, kv_heads=4, dim=96, vdim=128, ff=1024, shared_ff=2048, experts=32, top=4, vocab=32000),
+               dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, expert_ffn=1024, n_experts=34, top_k=6, vocab=32000)),
+}
+
+
+def kernel_table(run, repeats: int = 3):
+    """[(kernel, launches, total us)] of one call of ``run`` under the CUDA activity tracer, longest first."""
+    import collections
+    import re
+
+    import torch
+    from torch.profiler import ProfilerActivity, profile
+    with profile(activities=[ProfilerActivity.CUDA]) as prof:
+        for _ in range(repeats):
+            run()
+        torch.cuda.synchronize()
+    rows = collections.OrderedDict()
+    for e in prof.events():
+        if e.device_type == torch.autograd.DeviceType.CUDA:
+            r = rows.setdefault(re.sub(r"\(.*", "", e.name)[:70], [0, 0.0])
+            r[0] += 1
+            r[1] += e.time_range.end - e.time_range.start
+    return sorted(((k, n / repeats, us / repeats) for k, (n, us) in rows.items()), key=lambda x: -x[2])
+
+
+def run_design(args) -> None:
+    """Prefill (1 x 2048 and 1 x 8192 tokens, nothing cached) and greedy decode (batch 1 and 16 after 2048 tokens each)."""
+    import shutil
+
+    import torch
+    from tensorsharp_b200.models import synth
+    from tensorsharp_b200.models.base import ModelBase
+    from tensorsharp_b200.ops import functional as F
+    from tensorsharp_b200.ops import kernels
+    from tensorsharp_b200.runtime.engine import DecodeGraph
+    dev, K, W = torch.device("cuda", 0), args.steps, max(3, args.warmup)
+    torch.cuda.set_device(0)
+    tables = []
+
+    def timed(fn, n):
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(n):
+            fn()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / n
+    os.makedirs(args.cache_dir, exist_ok=True)
+    for size, (ours, closest) in DESIGN_SIZES.items():
+        if args.design_size not in (None, size):
+            continue
+        for name in ("fobolorn", "gpt-oss"):
+            path = os.path.join(args.cache_dir, f"design-{name}-{size}")
+            if name == "fobolorn":
+                synth.write_fobolorn(path, seed=0, **ours)
+            else:
+                path += ".gguf"
+                synth.write_gptoss(path, seed=0, expert_scheme="BF16", window=1 << 20, **closest)
+            model = ModelBase.create(path, dev, max_context=8192 + 64, max_seqs=18, kv_pages=16 * (2048 + 2 * K + 2 * W + 128) // 64 + 160)
+            res = {"design": name, "size": size, "layers": len(getattr(model, "runs", model.layers)), "dtype": "bf16", "data": "synthetic",
+                   "l2": "every step reads more weight bytes than L2 holds"}
+            g = torch.Generator().manual_seed(1)
+            clocks = ClockSampler(0)
+            clocks.start()
+            for P in (2048, 8192):
+                ids = torch.randint(0, model.cfg.vocab, (P,), generator=g).tolist()
+
+                def prefill():
+                    s = model.kv.new_seq()
+                    out = model.forward_batch(model.kv.build_batch([s], [ids]))
+                    model.kv.free_seq(s)
+                    return out
+                for _ in range(W):
+                    prefill()
+                res[f"prefill_{P}_tok_s"] = P / (sorted(timed(prefill, 1) for _ in range(5))[2] / 1e3)
+                if args.design_kernels:
+                    tables.append((f"{size} {name} prefill {P}", kernel_table(prefill)))
+            for B in (1, 16):
+                seqs = [model.kv.new_seq() for _ in range(B)]
+                first = []
+                for s in seqs:
+                    ids = torch.randint(0, model.cfg.vocab, (2048,), generator=g).tolist()
+                    first.append(int(F.argmax(model.forward_batch(model.kv.build_batch([s], [ids])))[0]))
+                dg = DecodeGraph(model, seqs, K + W + 16)
+                dg.set_tokens(first)
+                dg.capture()
+                for _ in range(W):
+                    dg.step()
+                ms = timed(dg.step, K)
+                res[f"decode_b{B}_tok_s"], res[f"decode_b{B}_ms"] = B / (ms / 1e3), ms
+                if args.design_kernels:
+                    tables.append((f"{size} {name} decode batch {B}, context 2048", kernel_table(dg.step)))
+                dg.graph = None
+                for s in seqs:
+                    model.kv.free_seq(s)
+            res["clocks"] = clocks.stop()
+            res["kernel_status"] = int(kernels.gemm_status(dev).item())
+            print(json.dumps(res), flush=True)
+            model.close()
+            del model
+            torch.cuda.empty_cache()
+            (shutil.rmtree if os.path.isdir(path) else os.unlink)(path)
+    if args.design_kernels:
+        with open(args.design_kernels, "w") as f:
+            for title, rows in tables:
+                total = sum(us for _, _, us in rows)
+                f.write(f"{title}: {sum(n for _, n, _ in rows):.0f} kernels, {total:.1f} us\n")
+                for k, n, us in rows[:16]:
+                    f.write(f"  {k:70s} {n:6.1f} x {us / n:9.2f} us = {us:9.1f} us\n")
+
+
 def main():
     args = parse_args()
+    if args.design:
+        return run_design(args)
     dump = os.environ.get("TSB_BENCH_STACK_DUMP_AFTER")
     if dump:          # diagnostics: print every thread's Python stack if the run is still going after N seconds
         import faulthandler
