@@ -507,7 +507,8 @@ DESIGN_SIZES = {
 
 
 def kernel_table(run, repeats: int = 3):
-    """[(kernel, launches, total us)] of one call of ``run`` under the CUDA activity tracer, longest first."""
+    """[(kernel, launches, us)] of one call of ``run`` under the CUDA activity tracer, longest first.  The time is exclusive
+    (see trace_step): what a kernel adds after every earlier one has ended, since a waiting kernel is already resident."""
     import collections
     import re
 
@@ -517,12 +518,12 @@ def kernel_table(run, repeats: int = 3):
         for _ in range(repeats):
             run()
         torch.cuda.synchronize()
-    rows = collections.OrderedDict()
-    for e in prof.events():
-        if e.device_type == torch.autograd.DeviceType.CUDA:
-            r = rows.setdefault(re.sub(r"\(.*", "", e.name)[:70], [0, 0.0])
-            r[0] += 1
-            r[1] += e.time_range.end - e.time_range.start
+    rows, prev = collections.OrderedDict(), 0.0
+    for e in sorted((e for e in prof.events() if e.device_type == torch.autograd.DeviceType.CUDA), key=lambda e: e.time_range.start):
+        r = rows.setdefault(re.sub(r"\(.*", "", e.name)[:70], [0, 0.0])
+        r[0] += 1
+        r[1] += max(0.0, e.time_range.end - max(prev, e.time_range.start))
+        prev = max(prev, e.time_range.end)
     return sorted(((k, n / repeats, us / repeats) for k, (n, us) in rows.items()), key=lambda x: -x[2])
 
 

@@ -483,6 +483,28 @@ __global__ void glu_kernel(const T* gate, const T* up, long g_stride, long u_str
     }
 }
 
+// Long bf16 inputs (prompts): eight columns per thread, 16-byte loads and stores.
+__global__ void __launch_bounds__(256) glu_vec_kernel(const bf16* gate, const bf16* up, long g_stride, long u_stride, int F8, int act,
+                                                      bf16* out, unsigned total) {
+    pdl_wait();
+    pdl_trigger();
+    const unsigned idx = blockIdx.x * 256u + threadIdx.x;
+    if (idx >= total) return;
+    const unsigned t = idx / (unsigned)F8, c = (idx - t * F8) * 8;
+    const uint4 gv = *reinterpret_cast<const uint4*>(gate + (long)t * g_stride + c);
+    const uint4 uv = up ? *reinterpret_cast<const uint4*>(up + (long)t * u_stride + c) : make_uint4(0u, 0u, 0u, 0u);
+    const bf162* g2 = reinterpret_cast<const bf162*>(&gv);
+    const bf162* u2 = reinterpret_cast<const bf162*>(&uv);
+    uint4 ov;
+    bf162* o2 = reinterpret_cast<bf162*>(&ov);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 g = __bfloat1622float2(g2[i]), u = __bfloat1622float2(u2[i]);
+        o2[i] = __floats2bfloat162_rn(glu_apply(act, g.x, u.x), glu_apply(act, g.y, u.y));
+    }
+    reinterpret_cast<uint4*>(out)[idx] = ov;
+}
+
 extern "C" int tsb_glu(const void* gate, const void* up, int in_f32, long g_stride, long u_stride, long rows, int F,
                        int act, void* out, void* yq, void* yds, void* stream) {
     TSB_CHECK_ARG(!yq || F % 32 == 0, "glu: q8 output needs F %% 32 == 0, got %d", F);
@@ -490,6 +512,14 @@ extern "C" int tsb_glu(const void* gate, const void* up, int in_f32, long g_stri
     const long total = rows * ((F + 31) & ~31);
     dim3 grid((unsigned)((total + 255) / 256));
     cudaStream_t s = (cudaStream_t)stream;
+    const bool aligned = ((reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(up) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    if (!in_f32 && !yq && out && aligned && F % 8 == 0 && g_stride % 8 == 0 && u_stride % 8 == 0 && rows * (F / 8) < (1L << 31)) {
+        const unsigned n = (unsigned)(rows * (F / 8));
+        TSB_CHECK_CUDA(tsb_launch(glu_vec_kernel, dim3((n + 255) / 256), dim3(256), 0, s, (const bf16*)gate, (const bf16*)up, g_stride, u_stride,
+                                  F / 8, act, (bf16*)out, n));
+        TSB_CHECK_LAUNCH();
+        return TSB_OK;
+    }
     if (in_f32)
         TSB_CHECK_CUDA(tsb_launch(glu_kernel<float>, grid, dim3(256), 0, s, (const float*)gate, (const float*)up, g_stride,
                                   u_stride, F, act, (bf16*)out, (int8_t*)yq, (float2*)yds, rows));

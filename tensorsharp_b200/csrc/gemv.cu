@@ -285,6 +285,8 @@ bool tsb_gemv_stream_eligible(const GemvArgs& a);                     // gemv_st
 int tsb_gemv_stream_launch(const GemvArgs& a, bool glu, cudaStream_t s);
 bool tsb_gemv_mma_eligible(const GemvArgs& a);                        // gemv_mma.cu
 int tsb_gemv_mma_launch(const GemvArgs& a, bool glu, cudaStream_t s);
+bool tsb_gemv_bf16_eligible(const GemvArgs& a);                       // gemv_bf16.cu
+int tsb_gemv_bf16_launch(const GemvArgs& a, bool glu, int problems, cudaStream_t s);
 
 template <bool GLU>
 static int launch_gemv(const GemvArgs& a, int problems, cudaStream_t s) {
@@ -356,6 +358,7 @@ extern "C" int tsb_gemv_push(const void* p0, const void* p1, const void* p2, con
     a.M = M; a.x_div = x_div > 0 ? x_div : 1; a.out_f32 = out_f32; a.act = act;
     a.n_out = glu ? N / 2 : N;
     a.push = (const TpPush*)push;
+    if (tsb_gemv_bf16_eligible(a)) return tsb_gemv_bf16_launch(a, glu, problems, (cudaStream_t)stream);
     if (tsb_gemv_mma_eligible(a)) return tsb_gemv_mma_launch(a, glu, (cudaStream_t)stream);
     if (tsb_gemv_stream_eligible(a)) return tsb_gemv_stream_launch(a, glu, (cudaStream_t)stream);
     return glu ? launch_gemv<true>(a, problems, (cudaStream_t)stream)

@@ -299,10 +299,67 @@ __device__ __forceinline__ void comp_q4_32(const QW& w, const WQ432& t, int u, c
         }                                                                         \
     }
 
+// bf16 weights: R rows (the row, or the gate and up rows of a pair) in groups of four 8-value units per lane, all of a
+// group's weight loads issued before any is used (the first group's before `pre`), so a warp has 2 or 4 KB in flight.
+template <int M, int R, class Pre>
+__device__ __forceinline__ void dot_bf16(const QW& w, const long (&rows)[R], int lane, const bf16* xb, float* const (&acc)[R], int mv, Pre pre,
+                                         int part = 0, int parts = 1) {
+    constexpr int U = 4;
+    const int K = w.K, units = K >> 3, step = 32 * parts;
+    const uint4* wp[R];
+#pragma unroll
+    for (int r = 0; r < R; ++r) wp[r] = reinterpret_cast<const uint4*>(w.p0) + rows[r] * units;
+    uint4 wv[R][U];
+    auto fetch = [&](int u0) {
+#pragma unroll
+        for (int i = 0; i < U; ++i)
+#pragma unroll
+            for (int r = 0; r < R; ++r) {
+                const int u = u0 + i * step;
+                wv[r][i] = u < units ? ld_stream_u4(wp[r] + u) : make_uint4(0u, 0u, 0u, 0u);
+            }
+    };
+    int u0 = lane + 32 * part;
+    fetch(u0);
+    pre();
+    for (; u0 < units; u0 += U * step) {
+        if (u0 != lane + 32 * part) fetch(u0);
+#pragma unroll
+        for (int i = 0; i < U; ++i) {
+            const int u = u0 + i * step;
+            if (u < units) {
+#pragma unroll
+                for (int m = 0; m < M; ++m) {
+                    const int mr = m < mv ? m : 0;
+                    const uint4 xv = *reinterpret_cast<const uint4*>(xb + (long)mr * K + 8 * u);
+                    const uint32_t* xw = reinterpret_cast<const uint32_t*>(&xv);
+#pragma unroll
+                    for (int r = 0; r < R; ++r) {
+                        const uint32_t* ww = reinterpret_cast<const uint32_t*>(&wv[r][i]);
+                        float s = 0.f;
+#pragma unroll
+                        for (int c = 0; c < 4; ++c) {
+                            s = fmaf(__uint_as_float(ww[c] << 16), __uint_as_float(xw[c] << 16), s);
+                            s = fmaf(__uint_as_float(ww[c] & 0xffff0000u), __uint_as_float(xw[c] & 0xffff0000u), s);
+                        }
+                        acc[r][m] += s;
+                    }
+                }
+            }
+        }
+    }
+}
+
 // Float-weight types (BF16 / F16 / F32) against bf16 activations.
 template <int M, class Pre>
 __device__ __forceinline__ void dot_float(const QW& w, long row, int lane, const bf16* xb, float* acc, int mv,
                                           Pre pre, int part = 0, int parts = 1) {
+    if (w.type == TSB_BF16) {
+        const long rows[1] = {row};
+        float* const a[1] = {acc};
+        dot_bf16<M, 1>(w, rows, lane, xb, a, mv, pre, part, parts);
+        return;
+    }
     const int K = w.K, units = K >> 3;
     pre();
     for (int u = lane + 32 * part; u < units; u += 32 * parts) {
@@ -385,6 +442,12 @@ __device__ __forceinline__ void dot_row2(const QW& w, long row_a, long row_b, in
     case TSB_Q8_0: TSB_ROW_LOOP2(WQ80, load_q8_0, comp_q8_0<M>, w.K >> 5) break;
     case TSB_MXFP4: TSB_ROW_LOOP2(WQ432, load_q4_32<true>, (comp_q4_32<M, true>), w.K >> 5) break;
     case TSB_Q4_0: TSB_ROW_LOOP2(WQ432, load_q4_32<false>, (comp_q4_32<M, false>), w.K >> 5) break;
+    case TSB_BF16: {
+        const long rows[2] = {row_a, row_b};
+        float* const a[2] = {acc_a, acc_b};
+        dot_bf16<M, 2>(w, rows, lane, xb, a, mv, pre);
+        break;
+    }
     default:
         dot_float<M>(w, row_a, lane, xb, acc_a, mv, pre);
         dot_float<M>(w, row_b, lane, xb, acc_b, mv, PdlWait{false});

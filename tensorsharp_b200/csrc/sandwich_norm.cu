@@ -35,6 +35,17 @@ __device__ __forceinline__ float4 ld4_any(const void* p, long row, int D, int i,
     return make_float4(a.x, a.y, b.x, b.y);
 }
 
+// Block-wide sum with one barrier: the caller alternates between two halves of `red` (32 floats each), so a half is written
+// again only after a barrier that every thread reaches after reading it.
+__device__ __forceinline__ float block_sum_half(float v, float* half) {
+    const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    v = warp_sum(v);
+    if (nw == 1) return v;
+    if (lane == 0) half[w] = v;
+    __syncthreads();
+    return warp_sum(lane < nw ? half[lane] : 0.f);
+}
+
 // v <- (v - mean) * rstd for the columns below n, 0 beyond
 template <int V>
 __device__ __forceinline__ void ln_rows(float4 (&v)[V], int n, float eps, float* red) {
@@ -42,7 +53,7 @@ __device__ __forceinline__ void ln_rows(float4 (&v)[V], int n, float eps, float*
     float s = 0.f;
 #pragma unroll
     for (int j = 0; j < V; ++j) s += v[j].x + v[j].y + v[j].z + v[j].w;      // columns past n hold zeros
-    const float mean = block_sum(s, red) / (float)n;
+    const float mean = block_sum_half(s, red) / (float)n;
     float q = 0.f;
 #pragma unroll
     for (int j = 0; j < V; ++j) {
@@ -53,14 +64,14 @@ __device__ __forceinline__ void ln_rows(float4 (&v)[V], int n, float eps, float*
         v[j].w = c + 3 < n ? v[j].w - mean : 0.f;
         q += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
     }
-    const float rs = 1.f / sqrtf(block_sum(q, red) / (float)n + eps);
+    const float rs = 1.f / sqrtf(block_sum_half(q, red + 32) / (float)n + eps);
 #pragma unroll
     for (int j = 0; j < V; ++j) { v[j].x *= rs; v[j].y *= rs; v[j].z *= rs; v[j].w *= rs; }
 }
 
 template <int V>
-__global__ void __launch_bounds__(V == 1 ? 1024 : 256) sandwich_norm_kernel(SandwichArgs a) {
-    __shared__ float red[32];
+__global__ void __launch_bounds__(V == 1 ? 1024 : 512, V == 2 ? 3 : 1) sandwich_norm_kernel(SandwichArgs a) {
+    __shared__ float red[64];
     const long row = blockIdx.x;
     const int nvec = a.D >> 2, nt = blockDim.x;
     float4 pw[V], pb[V];                       // the weights do not depend on the previous kernel
@@ -82,17 +93,27 @@ __global__ void __launch_bounds__(V == 1 ? 1024 : 256) sandwich_norm_kernel(Sand
         if (i < nvec) h[j] = reinterpret_cast<const float4*>(a.h + row * a.D)[i];
     }
     if (a.y != nullptr) {
-        for (int p = 0; p < a.parts; ++p) {
-            const long k = row * a.parts + p;
-            const long src = a.pos ? (long)a.pos[k] : k;
-            if (src < 0) continue;
-            const float w = a.wts ? a.wts[k] : 1.f;
+        constexpr int PB = V <= 4 ? 4 : 2;                     // parts in flight together
+        for (int p0 = 0; p0 < a.parts; p0 += PB) {
+            long src[PB];
+            float w[PB];
+#pragma unroll
+            for (int q = 0; q < PB; ++q) {
+                const long k = row * a.parts + p0 + q;
+                const bool on = p0 + q < a.parts;
+                src[q] = !on ? -1 : a.pos ? (long)a.pos[k] : k;
+                w[q] = on && a.wts ? a.wts[k] : 1.f;
+            }
 #pragma unroll
             for (int j = 0; j < V; ++j) {
                 const int i = threadIdx.x + j * nt;
-                if (i < nvec) {
-                    const float4 t = ld4_any(a.y, src, a.D, i, a.y_f32);
-                    x[j].x += w * t.x; x[j].y += w * t.y; x[j].z += w * t.z; x[j].w += w * t.w;
+                float4 t[PB];
+#pragma unroll
+                for (int q = 0; q < PB; ++q)
+                    t[q] = i < nvec && src[q] >= 0 ? ld4_any(a.y, src[q], a.D, i, a.y_f32) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                for (int q = 0; q < PB; ++q) {
+                    x[j].x += w[q] * t[q].x; x[j].y += w[q] * t[q].y; x[j].z += w[q] * t[q].z; x[j].w += w[q] * t[q].w;
                 }
             }
         }
@@ -145,17 +166,17 @@ extern "C" int tsb_sandwich_norm(const SandwichArgs* args, void* stream) {
     cudaStream_t s = (cudaStream_t)stream;
     const int nvec = a.D / 4;
     const dim3 grid((unsigned)a.rows);
-    // few rows (decode): a float4 per thread, for latency; many rows: 256 threads with several each, so that more rows are
-    // in flight per SM
+    // few rows (decode): a float4 per thread, for latency; many rows: two or more each (measured at 8192 x 2048, five parts:
+    // one 151 us, two at three CTAs per SM 105 us, three 155, four 150)
     if (nvec <= 256 || (a.rows < 296 && nvec <= 1024)) {
         TSB_CHECK_CUDA(tsb_launch(sandwich_norm_kernel<1>, grid, dim3((nvec + 31) & ~31), 0, s, a));
     } else {
-        const int v = (nvec + 255) / 256;
-        TSB_CHECK_ARG(v <= 16, "sandwich_norm: rows of %d columns (limit 16384)", a.D);
-        if (v <= 2) TSB_CHECK_CUDA(tsb_launch(sandwich_norm_kernel<2>, grid, dim3(256), 0, s, a));
-        else if (v <= 4) TSB_CHECK_CUDA(tsb_launch(sandwich_norm_kernel<4>, grid, dim3(256), 0, s, a));
-        else if (v <= 8) TSB_CHECK_CUDA(tsb_launch(sandwich_norm_kernel<8>, grid, dim3(256), 0, s, a));
-        else TSB_CHECK_CUDA(tsb_launch(sandwich_norm_kernel<16>, grid, dim3(256), 0, s, a));
+        TSB_CHECK_ARG(nvec <= 4096, "sandwich_norm: rows of %d columns (limit 16384)", a.D);
+        const int v = nvec <= 1024 ? 2 : nvec <= 2048 ? 4 : 8;
+        const dim3 block((((nvec + v - 1) / v) + 31) & ~31);
+        if (v == 2) TSB_CHECK_CUDA(tsb_launch(sandwich_norm_kernel<2>, grid, block, 0, s, a));
+        else if (v == 4) TSB_CHECK_CUDA(tsb_launch(sandwich_norm_kernel<4>, grid, block, 0, s, a));
+        else TSB_CHECK_CUDA(tsb_launch(sandwich_norm_kernel<8>, grid, block, 0, s, a));
     }
     TSB_CHECK_LAUNCH();
     return TSB_OK;

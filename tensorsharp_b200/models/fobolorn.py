@@ -59,7 +59,7 @@ class FobolornModel(ModelBase):
     supports_float32 = True
     mixed_batches = True
     native_sources = ("error.cpp", "elementwise.cu", "sandwich_norm.cu", "float32.cu", "attention.cu", "attention_vd.cu",
-                      "attention_decode_mma.cu", "gemm_tcgen05.cu", "gemv.cu", "gemv_mma.cu", "gemv_stream.cu", "moe.cu", "sampler.cu")
+                      "attention_decode_mma.cu", "gemm_tcgen05.cu", "gemv.cu", "gemv_bf16.cu", "gemv_mma.cu", "gemv_stream.cu", "moe.cu", "sampler.cu")
 
     # ------------------------------------------------------------------ configuration
     def parse_base_config(self) -> ModelConfig:
