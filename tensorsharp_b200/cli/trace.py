@@ -2,7 +2,7 @@
 
     bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N  < steps.jsonl
 
-Every line of standard input is one step, ``{"step": 0, "entries": [{"id": "a", "tokens": [5, 17], "want": [1]}], "end": []}``:
+Every line of standard input is one step, ``{"step": 7, "entries": [{"id": "x", "tokens": [31, 8], "want": [1]}], "end": ["y"]}``:
 the entries are one batch of the engine (portions of prompts beside single tokens; ``want``: places among the entry's tokens
 whose logits are wanted), the requests of ``end`` give their pages and slot back afterwards.  The wanted logits go to
 ``DIR/<step>.f32`` (little-endian float32, [wanted, vocab]); ``done <step>`` is printed after every step.  Nothing is

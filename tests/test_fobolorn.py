@@ -148,7 +148,7 @@ def test_query_temperature_and_head_norm(place):
     assert steps[0] == 1.0 and steps[1] == steps[2] > 1.0 and steps[3] > steps[2]
 
 
-HEADS = [(6, 1, 64, 80), (4, 2, 32, 48), (8, 2, 64, 64), (4, 4, 128, 128), (3, 3, 16, 112), (20, 1, 208, 256), (5, 5, 96, 16),
+HEADS = [(9, 3, 64, 80), (4, 2, 32, 48), (8, 2, 64, 64), (4, 4, 128, 128), (3, 3, 16, 112), (20, 1, 208, 256), (5, 5, 96, 16),
          (17, 1, 128, 64), (24, 1, 64, 64), (2, 1, 256, 256)]
 
 
