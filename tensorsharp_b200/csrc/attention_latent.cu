@@ -1,0 +1,483 @@
+// Latent attention: keys and values of all heads are linear maps of one cached row per token, [latent c (R) | rotated key
+// part (rot) | zeros], Lp elements.  Query heads are laid out [dim unrotated | rot rotated | zeros], Dk elements.
+//
+//   score = (q_c . W_uk c + q_r . k_r) scale = ((W_uk^T q_c) . c + q_r . k_r) scale;   W_uv sum_j p_j c_j = sum_j p_j W_uv c_j
+//
+// Prompts expand the rows that their queries can see with one matrix product over the cached rows, [W_uk 0; 0 I; W_uv 0],
+// and run the ordinary prefill kernel.  Decoding keeps the rows as they are: every query head is mapped into the row's
+// space (latent_absorb_kernel), all heads share one row per key, which serves as key and as value
+// (latent_decode_kernel, tensor cores), and latent_out_kernel merges the splits with the sink and applies W_uv.
+#include "attn_mma.cuh"
+#include "common.cuh"
+
+namespace {
+__device__ __forceinline__ float la_ld(const void* p, long i, int f32) {
+    return f32 ? reinterpret_cast<const float*>(p)[i] : bf2f(reinterpret_cast<const bf16*>(p)[i]);
+}
+__device__ __forceinline__ void la_st(void* p, long i, int f32, float v) {
+    if (f32) reinterpret_cast<float*>(p)[i] = v;
+    else reinterpret_cast<bf16*>(p)[i] = f2bf(v);
+}
+}  // namespace
+
+// ------------------------------------------------------------------------------------------
+// (cos, sin) of position * freq per (token, pair).  The angle is formed and reduced to one turn in double precision: in
+// f32 the product alone is off by 3e-5 at position 1000.
+// ------------------------------------------------------------------------------------------
+__global__ void rotary_table_kernel(const int* pos, const double* freq, float2* out, int T, int half) {
+    pdl_wait();
+    pdl_trigger();
+    const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (long)T * half) return;
+    constexpr double TURN = 6.283185307179586476925;
+    double a = (double)pos[i / half] * freq[i % half];
+    a -= TURN * rint(a / TURN);
+    float s, c;
+    sincosf((float)a, &s, &c);
+    out[i] = make_float2(c, s);
+}
+
+extern "C" int tsb_rotary_table(const int* pos, const double* freq, void* out, int T, int half, void* stream) {
+    TSB_CHECK_ARG(T >= 0 && half >= 0, "rotary_table: T=%d half=%d", T, half);
+    const long n = (long)T * half;
+    if (n == 0) return TSB_OK;
+    TSB_CHECK_CUDA(tsb_launch(rotary_table_kernel, dim3((unsigned)((n + 127) / 128)), dim3(128), 0, (cudaStream_t)stream, pos, freq, (float2*)out,
+                              T, half));
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}
+
+struct LatentArgs {
+    // rows [query latent (qr, padded to qp) | latent (R) | rotated part (rot)]
+    const void* y; long y_s; int y_f32;
+    const float* qn; const float* kn;        // norm weights [qr], [R]
+    const float2* cs;                        // [T, rot / 2]
+    const long* slots;                       // [T]
+    void* cache;                             // [slots, Lp]
+    void* cq;                                // [T, qp]
+    int f32;                                 // cache, cq, absorbed queries and results are f32 (else bf16)
+    int T, qr, qp, R, rot, Lp;
+    float eps;
+    // queries
+    void* q; int q_f32;                      // [T, H, Dk], not rotated
+    const void* wuk; const void* wuv; int w_f32;      // [H * dim, Rp], [H * Dv, Rp]
+    void* qa;                                // [T, H, Lp]
+    int H, dim, Dk, Rp, Dv;
+    // decoding
+    const int* block_table; const int* kv_lens;
+    float* part_o; float* part_ml;           // [T, H, splits, Ro], [T, H, splits, 2] (null: part_o is the finished result)
+    const float* sinks;                      // [H] or null
+    void* out;                               // [T, H, Dv]
+    float scale;
+    int window, page_size, max_pages, splits, Ro;
+};
+
+// ------------------------------------------------------------------------------------------
+// Norms of both latents, rotation of the shared key part, cache write.  One CTA per token.
+// ------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) latent_prep_kernel(LatentArgs a) {
+    __shared__ float red[2][32];
+    pdl_wait();
+    pdl_trigger();
+    const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, w = tid >> 5, nw = blockDim.x >> 5;
+    const long row = (long)t * a.y_s, lat = row + a.qp;
+    float sq = 0.f, sc = 0.f;
+    for (int i = tid; i < a.qr; i += blockDim.x) { const float v = la_ld(a.y, row + i, a.y_f32); sq = fmaf(v, v, sq); }
+    for (int i = tid; i < a.R; i += blockDim.x) { const float v = la_ld(a.y, lat + i, a.y_f32); sc = fmaf(v, v, sc); }
+    sq = warp_sum(sq);
+    sc = warp_sum(sc);
+    if (lane == 0) { red[0][w] = sq; red[1][w] = sc; }
+    __syncthreads();
+    sq = warp_sum(lane < nw ? red[0][lane] : 0.f);
+    sc = warp_sum(lane < nw ? red[1][lane] : 0.f);
+    const float rq = 1.f / sqrtf(sq / (float)a.qr + a.eps), rc = 1.f / sqrtf(sc / (float)a.R + a.eps);
+    for (int i = tid; i < a.qp; i += blockDim.x)
+        la_st(a.cq, (long)t * a.qp + i, a.f32, i < a.qr ? la_ld(a.y, row + i, a.y_f32) * rq * a.qn[i] : 0.f);
+    const long dst = a.slots[t] * a.Lp;
+    const int half = a.rot >> 1;
+    for (int i = tid; i < a.Lp; i += blockDim.x) {
+        float v = 0.f;
+        if (i < a.R) {
+            v = la_ld(a.y, lat + i, a.y_f32) * rc * a.kn[i];
+        } else if (i < a.R + a.rot) {
+            const int e = i - a.R, pair = e < half ? e : e - half;
+            const float2 cs = a.cs[(long)t * half + pair];
+            const float x0 = la_ld(a.y, lat + a.R + pair, a.y_f32), x1 = la_ld(a.y, lat + a.R + half + pair, a.y_f32);
+            v = e < half ? x0 * cs.x - x1 * cs.y : x1 * cs.x + x0 * cs.y;
+        }
+        la_st(a.cache, dst + i, a.f32, v);
+    }
+}
+
+extern "C" int tsb_latent_prep(const LatentArgs* args, void* stream) {
+    const LatentArgs& a = *args;
+    TSB_CHECK_ARG(a.qr > 0 && a.qp >= a.qr && a.R > 0 && a.rot >= 0 && a.rot % 2 == 0 && a.Lp >= a.R + a.rot, "latent_prep: sizes %d / %d / %d in %d",
+                  a.qr, a.R, a.rot, a.Lp);
+    if (a.T == 0) return TSB_OK;
+    TSB_CHECK_CUDA(tsb_launch(latent_prep_kernel, dim3(a.T), dim3(256), 0, (cudaStream_t)stream, a));
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}
+
+// ------------------------------------------------------------------------------------------
+// Rotation of the queries' rotated parts in place (prompts).
+// ------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) latent_rotate_kernel(LatentArgs a) {
+    pdl_wait();
+    pdl_trigger();
+    const int half = a.rot >> 1;
+    const long i = (long)blockIdx.x * 256 + threadIdx.x;
+    if (i >= (long)a.T * a.H * half) return;
+    const int pair = (int)(i % half);
+    const long th = i / half;
+    const float2 cs = a.cs[(th / a.H) * half + pair];
+    const long p0 = th * a.Dk + a.dim + pair, p1 = p0 + half;
+    const float x0 = la_ld(a.q, p0, a.q_f32), x1 = la_ld(a.q, p1, a.q_f32);
+    la_st(a.q, p0, a.q_f32, x0 * cs.x - x1 * cs.y);
+    la_st(a.q, p1, a.q_f32, x1 * cs.x + x0 * cs.y);
+}
+
+extern "C" int tsb_latent_rotate(const LatentArgs* args, void* stream) {
+    const LatentArgs& a = *args;
+    TSB_CHECK_ARG(a.rot % 2 == 0 && a.Dk >= a.dim + a.rot, "latent_rotate: head of %d + %d in %d", a.dim, a.rot, a.Dk);
+    const long n = (long)a.T * a.H * (a.rot >> 1);
+    if (n == 0) return TSB_OK;
+    TSB_CHECK_CUDA(tsb_launch(latent_rotate_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, (cudaStream_t)stream, a));
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}
+
+// ------------------------------------------------------------------------------------------
+// Queries into the row's space: qa[r] = sum_d W_uk[h, d, r] q[d] for r < R, then the rotated part.  Grid (ceil(Lp / 64), H,
+// ceil(T / TT)); eight warps share the d range, a lane holds two neighbouring r.
+// ------------------------------------------------------------------------------------------
+template <typename TW, int TT>
+__global__ void __launch_bounds__(256) latent_absorb_kernel(LatentArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    float* sq = sm;                          // [TT][Dk]
+    float* sp = sm + TT * a.Dk;              // [8][TT][64]
+    const int h = blockIdx.y, r0 = blockIdx.x * 64, t0 = blockIdx.z * TT, tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
+    const int nt = min(TT, a.T - t0);
+    pdl_wait();
+    pdl_trigger();
+    for (int i = tid; i < TT * a.Dk; i += 256) {
+        const int m = i / a.Dk, d = i % a.Dk;
+        sq[i] = m < nt ? la_ld(a.q, ((long)(t0 + m) * a.H + h) * a.Dk + d, a.q_f32) : 0.f;
+    }
+    __syncthreads();
+    const int r = r0 + 2 * lane;
+    float acc[TT][2];
+#pragma unroll
+    for (int m = 0; m < TT; ++m) acc[m][0] = acc[m][1] = 0.f;
+    if (r < a.Rp) {                          // Rp is even, columns R .. Rp - 1 are zero
+        const TW* wp = reinterpret_cast<const TW*>(a.wuk) + (long)h * a.dim * a.Rp + r;
+#pragma unroll 8
+        for (int d = w; d < a.dim; d += 8) {
+            float w0, w1;
+            if (sizeof(TW) == 2) {
+                const float2 v = __bfloat1622float2(*reinterpret_cast<const bf162*>(wp + (long)d * a.Rp));
+                w0 = v.x; w1 = v.y;
+            } else {
+                const float2 v = *reinterpret_cast<const float2*>(wp + (long)d * a.Rp);
+                w0 = v.x; w1 = v.y;
+            }
+#pragma unroll
+            for (int m = 0; m < TT; ++m) {
+                acc[m][0] = fmaf(w0, sq[m * a.Dk + d], acc[m][0]);
+                acc[m][1] = fmaf(w1, sq[m * a.Dk + d], acc[m][1]);
+            }
+        }
+    }
+#pragma unroll
+    for (int m = 0; m < TT; ++m) *reinterpret_cast<float2*>(sp + (w * TT + m) * 64 + 2 * lane) = make_float2(acc[m][0], acc[m][1]);
+    __syncthreads();
+    const int half = a.rot >> 1;
+    for (int i = tid; i < nt * 64; i += 256) {
+        const int m = i / 64, c = i % 64, rr = r0 + c, t = t0 + m;
+        if (rr >= a.Lp) continue;
+        float v = 0.f;
+        if (rr < a.R) {
+#pragma unroll
+            for (int u = 0; u < 8; ++u) v += sp[(u * TT + m) * 64 + c];
+        } else if (rr < a.R + a.rot) {
+            const int e = rr - a.R, pair = e < half ? e : e - half;
+            const float2 cs = a.cs[(long)t * half + pair];
+            const float x0 = sq[m * a.Dk + a.dim + pair], x1 = sq[m * a.Dk + a.dim + half + pair];
+            v = e < half ? x0 * cs.x - x1 * cs.y : x1 * cs.x + x0 * cs.y;
+        }
+        la_st(a.qa, ((long)t * a.H + h) * a.Lp + rr, a.f32, v);
+    }
+}
+
+template <typename TW>
+static int launch_absorb(const LatentArgs& a, cudaStream_t s) {
+    const int bx = (a.Lp + 63) / 64;
+    // tokens per CTA: each shares the head's weights between its tokens; few tokens keep one for parallelism
+    if (a.T <= 2) {
+        const size_t smem = sizeof(float) * (a.Dk + 8 * 64);
+        TSB_CHECK_CUDA(tsb_launch(latent_absorb_kernel<TW, 1>, dim3(bx, a.H, a.T), dim3(256), smem, s, a));
+    } else {
+        const size_t smem = sizeof(float) * 4 * (a.Dk + 8 * 64);
+        TSB_CHECK_CUDA(tsb_launch(latent_absorb_kernel<TW, 4>, dim3(bx, a.H, (a.T + 3) / 4), dim3(256), smem, s, a));
+    }
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}
+
+extern "C" int tsb_latent_absorb(const LatentArgs* args, void* stream) {
+    const LatentArgs& a = *args;
+    TSB_CHECK_ARG(a.Rp % 2 == 0 && a.Rp >= a.R && a.Lp >= a.R + a.rot && a.Dk >= a.dim + a.rot && a.Dk <= 1024 && a.H <= 65535 && a.T <= 4 * 65535,
+                  "latent_absorb: latent %d (%d), head %d + %d in %d", a.R, a.Rp, a.dim, a.rot, a.Dk);
+    if (a.T == 0) return TSB_OK;
+    return a.w_f32 ? launch_absorb<float>(a, (cudaStream_t)stream) : launch_absorb<bf16>(a, (cudaStream_t)stream);
+}
+
+// ------------------------------------------------------------------------------------------
+// Decode attention over the cached rows.  Grid (splits, ceil(H / 16), B), eight warps; the 16 query heads are the rows of
+// one m16 tile.  Rows arrive in tiles of 64 keys through cp.async, two stages.  Warp w scores keys 8 w .. 8 w + 7 over the
+// whole row; the probabilities meet in shared memory, and warp w accumulates the latent columns 16 (w NV + i).
+// ------------------------------------------------------------------------------------------
+template <int NV>
+__global__ void __launch_bounds__(256) latent_decode_kernel(LatentArgs a) {
+    constexpr int KT = 64, LDP = KT + 8;
+    constexpr float LOG2E = 1.4426950408889634f;
+    extern __shared__ __align__(128) unsigned char smem_raw[];
+    __shared__ float red[8][16];
+    const int ld = a.Lp + 8, cl = a.Lp / 8;
+    bf16* sQ = reinterpret_cast<bf16*>(smem_raw);       // [16][ld]
+    bf16* sP = sQ + 16 * ld;                            // [16][LDP]
+    bf16* sK = sP + 16 * LDP;                           // [2][64][ld]
+    const int split = blockIdx.x, h0 = blockIdx.y * 16, b = blockIdx.z, G = min(16, a.H - h0);
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    pdl_wait();
+    pdl_trigger();
+    const int len = a.kv_lens[b];
+    const int lo = (a.window > 0 && len > a.window) ? len - a.window : 0;
+    const int per = (((len - lo + a.splits - 1) / a.splits) + 31) & ~31;
+    const int s0 = lo + split * per, s1 = min(len, s0 + per);
+    const bf16* cache = reinterpret_cast<const bf16*>(a.cache);
+    auto load_tile = [&](int base, int stage) {
+        const int r = tid >> 2, j = base + r;           // four threads per row
+        bf16* dst = sK + (stage * KT + r) * ld;
+        if (j < s1) {
+            const long slot = (long)a.block_table[(long)b * a.max_pages + j / a.page_size] * a.page_size + j % a.page_size;
+            for (int c = tid & 3; c < cl; c += 4) cp_async16(dst + c * 8, cache + slot * a.Lp + c * 8);
+        } else {
+            for (int c = tid & 3; c < cl; c += 4) *reinterpret_cast<uint4*>(dst + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+        }
+        cp_async_commit();
+    };
+    float o[2 * NV][4];
+#pragma unroll
+    for (int i = 0; i < 2 * NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
+    if (s0 < s1) {
+        load_tile(s0, 0);
+        for (int i = tid; i < 16 * cl; i += 256) {
+            const int r = i / cl, c = i % cl;
+            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+            if (r < G) v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.qa) + ((long)b * a.H + h0 + r) * a.Lp + c * 8);
+            *reinterpret_cast<uint4*>(sQ + r * ld + c * 8) = v;
+        }
+    }
+    int stage = 0;
+    for (int base = s0; base < s1; base += KT, stage ^= 1) {
+        if (base + KT < s1) {
+            load_tile(base + KT, stage ^ 1);
+            cp_async_wait<1>();
+        } else {
+            cp_async_wait<0>();
+        }
+        __syncthreads();
+        const bf16* tK = sK + stage * KT * ld;
+        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        {
+            const bf16* qrow = sQ + (lane & 15) * ld + ((lane >> 4) << 3);
+            const bf16* krow = tK + (warp * 8 + (lane & 7)) * ld + ((lane >> 3) << 3);
+#pragma unroll 2
+            for (int kk = 0; kk < a.Lp; kk += 32) {      // Lp is a multiple of 32
+                uint32_t q0[4], q1[4], kb[4];
+                ldsm_x4(q0, qrow + kk);
+                ldsm_x4(q1, qrow + kk + 16);
+                ldsm_x4(kb, krow + kk);
+                mma_bf16(s[0], q0, kb[0], kb[1]);
+                mma_bf16(s[1], q1, kb[2], kb[3]);
+            }
+        }
+        const int key = base + warp * 8 + (lane & 3) * 2;
+        float p[4], mx[2];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) p[e] = key + (e & 1) < s1 ? (s[0][e] + s[1][e]) * a.scale : -INFINITY;
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            mx[r] = fmaxf(p[2 * r], p[2 * r + 1]);
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+            if ((lane & 3) == 0) red[warp][(lane >> 2) + 8 * r] = mx[r];
+        }
+        __syncthreads();
+        float corr[2];
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            float m = mrow[r];
+#pragma unroll
+            for (int w = 0; w < 8; ++w) m = fmaxf(m, red[w][(lane >> 2) + 8 * r]);      // the tile has a valid key: finite
+            corr[r] = mrow[r] == -INFINITY ? 0.f : exp2f((mrow[r] - m) * LOG2E);
+            mrow[r] = m;
+            const float e0 = exp2f((p[2 * r] - m) * LOG2E), e1 = exp2f((p[2 * r + 1] - m) * LOG2E);
+            lrow[r] = lrow[r] * corr[r] + e0 + e1;
+            *reinterpret_cast<uint32_t*>(sP + ((lane >> 2) + 8 * r) * LDP + warp * 8 + (lane & 3) * 2) = pack_bf16(e0, e1);
+        }
+#pragma unroll
+        for (int i = 0; i < 2 * NV; ++i) {
+            o[i][0] *= corr[0]; o[i][1] *= corr[0];
+            o[i][2] *= corr[1]; o[i][3] *= corr[1];
+        }
+        __syncthreads();
+#pragma unroll
+        for (int kt = 0; kt < KT / 16; ++kt) {
+            uint32_t pa[4];
+            ldsm_x4(pa, sP + (lane & 15) * LDP + kt * 16 + ((lane >> 4) << 3));
+            const bf16* row = tK + (kt * 16 + (((lane >> 3) & 1) << 3) + (lane & 7)) * ld + ((lane >> 4) << 3);
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+                const int c = (warp * NV + i) * 16;
+                if (c >= a.R) break;
+                uint32_t vb[4];
+                ldsm_x4_t(vb, row + c);
+                mma_bf16(o[2 * i], pa, vb[0], vb[1]);
+                mma_bf16(o[2 * i + 1], pa, vb[2], vb[3]);
+            }
+        }
+        __syncthreads();                                 // before the stage, the maxima and P are written again
+    }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        lrow[r] += __shfl_xor_sync(0xffffffffu, lrow[r], 1);
+        lrow[r] += __shfl_xor_sync(0xffffffffu, lrow[r], 2);
+        if ((lane & 3) == 0) red[warp][(lane >> 2) + 8 * r] = lrow[r];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        const int row = (lane >> 2) + 8 * r;
+        if (row >= G) continue;
+        const long pi = ((long)b * a.H + h0 + row) * a.splits + split;
+        if (warp == 0 && (lane & 3) == 0) {
+            float l = 0.f;
+#pragma unroll
+            for (int w = 0; w < 8; ++w) l += red[w][row];
+            a.part_ml[pi * 2] = mrow[r];
+            a.part_ml[pi * 2 + 1] = l;
+        }
+#pragma unroll
+        for (int i = 0; i < 2 * NV; ++i) {
+            const int c = (warp * NV + (i >> 1)) * 16 + (i & 1) * 8 + (lane & 3) * 2;
+            if (c < a.Ro) *reinterpret_cast<float2*>(a.part_o + pi * a.Ro + c) = make_float2(o[i][2 * r], o[i][2 * r + 1]);
+        }
+    }
+}
+
+template <int NV>
+static int launch_latent_decode(const LatentArgs& a, cudaStream_t s) {
+    const int ld = a.Lp + 8;
+    const size_t smem = (size_t)(16 * ld + 16 * 72 + 2 * 64 * ld) * sizeof(bf16);
+    static size_t configured = 0;
+    if (smem > configured) {
+        TSB_CHECK_CUDA(cudaFuncSetAttribute(latent_decode_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        configured = smem;
+    }
+    TSB_CHECK_CUDA(tsb_launch(latent_decode_kernel<NV>, dim3(a.splits, (a.H + 15) / 16, a.T), dim3(256), smem, s, a));
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}
+
+// One query per sequence (T sequences); leaves the split partials in part_o / part_ml.
+extern "C" int tsb_latent_decode(const LatentArgs* args, void* stream) {
+    const LatentArgs& a = *args;
+    TSB_CHECK_ARG(!a.f32 && a.Lp % 32 == 0 && a.Lp <= 704 && a.R > 0 && a.R <= 512 && a.Lp >= a.R + a.rot, "latent_decode: latent %d + %d in %d (limits 512, 704)",
+                  a.R, a.rot, a.Lp);
+    TSB_CHECK_ARG(a.splits >= 1 && a.splits <= 64 && a.part_o && a.part_ml && a.Ro % 8 == 0 && a.Ro >= a.R && a.Ro <= ((a.R + 15) & ~15),
+                  "latent_decode: %d splits, partial rows of %d", a.splits, a.Ro);
+    if (a.T == 0) return TSB_OK;
+    cudaStream_t s = (cudaStream_t)stream;
+    switch ((a.R + 127) / 128) {
+    case 1: return launch_latent_decode<1>(a, s);
+    case 2: return launch_latent_decode<2>(a, s);
+    case 3: return launch_latent_decode<3>(a, s);
+    default: return launch_latent_decode<4>(a, s);
+    }
+}
+
+// ------------------------------------------------------------------------------------------
+// Merge of the splits (with the sink) and the value map.  Grid (parts of Dv, H, T), eight warps: the merged latent in shared
+// memory, one output row of W_uv per warp at a time.
+// ------------------------------------------------------------------------------------------
+template <typename TW>
+__global__ void __launch_bounds__(256) latent_out_kernel(LatentArgs a, int rows) {
+    extern __shared__ __align__(16) float sm[];          // [Rp]
+    const int e0 = blockIdx.x * rows, e1 = min(a.Dv, e0 + rows), h = blockIdx.y, t = blockIdx.z;
+    const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
+    pdl_wait();
+    pdl_trigger();
+    const long th = (long)t * a.H + h;
+    if (a.part_ml == nullptr) {
+        for (int r = tid; r < a.Rp; r += 256) sm[r] = r < a.R ? a.part_o[th * a.Ro + r] : 0.f;
+    } else {
+        const float* ml = a.part_ml + th * a.splits * 2;
+        float m = a.sinks ? a.sinks[h] : -INFINITY;
+        for (int i = 0; i < a.splits; ++i) m = fmaxf(m, ml[2 * i]);
+        float l = a.sinks ? expf(a.sinks[h] - m) : 0.f;
+        for (int i = 0; i < a.splits; ++i) l += ml[2 * i] == -INFINITY ? 0.f : ml[2 * i + 1] * expf(ml[2 * i] - m);
+        const float inv = 1.f / l;
+        for (int r = tid; r < a.Rp; r += 256) {
+            float v = 0.f;
+            if (r < a.R)
+                for (int i = 0; i < a.splits; ++i)
+                    if (ml[2 * i] != -INFINITY) v = fmaf(a.part_o[(th * a.splits + i) * a.Ro + r], expf(ml[2 * i] - m), v);
+            sm[r] = v * inv;
+        }
+    }
+    __syncthreads();
+    for (int e = e0 + w; e < e1; e += 8) {
+        const TW* wp = reinterpret_cast<const TW*>(a.wuv) + ((long)h * a.Dv + e) * a.Rp;
+        float acc = 0.f;
+        for (int u = lane * 8; u < a.Rp; u += 256) {     // Rp is a multiple of 8
+            float wv[8];
+            if (sizeof(TW) == 2) {
+                const uint4 v = *reinterpret_cast<const uint4*>(wp + u);
+                const uint32_t* x = reinterpret_cast<const uint32_t*>(&v);
+#pragma unroll
+                for (int c = 0; c < 4; ++c) {
+                    wv[2 * c] = __uint_as_float(x[c] << 16);
+                    wv[2 * c + 1] = __uint_as_float(x[c] & 0xffff0000u);
+                }
+            } else {
+#pragma unroll
+                for (int c = 0; c < 8; ++c) wv[c] = (float)wp[u + c];
+            }
+            const float4 x0 = *reinterpret_cast<const float4*>(sm + u), x1 = *reinterpret_cast<const float4*>(sm + u + 4);
+            acc = fmaf(wv[0], x0.x, acc); acc = fmaf(wv[1], x0.y, acc); acc = fmaf(wv[2], x0.z, acc); acc = fmaf(wv[3], x0.w, acc);
+            acc = fmaf(wv[4], x1.x, acc); acc = fmaf(wv[5], x1.y, acc); acc = fmaf(wv[6], x1.z, acc); acc = fmaf(wv[7], x1.w, acc);
+        }
+        acc = warp_sum(acc);
+        if (lane == 0) la_st(a.out, th * a.Dv + e, a.f32, acc);
+    }
+}
+
+extern "C" int tsb_latent_out(const LatentArgs* args, void* stream) {
+    const LatentArgs& a = *args;
+    TSB_CHECK_ARG(a.Rp % 8 == 0 && a.Rp >= a.R && a.Rp <= 4096 && a.Dv > 0 && a.T <= 65535 && a.H <= 65535, "latent_out: latent %d (%d), values %d, %d rows",
+                  a.R, a.Rp, a.Dv, a.T);
+    if (a.T == 0) return TSB_OK;
+    // output rows per CTA: all of a head's when there are heads and tokens enough for the SMs, else a share
+    int rows = a.Dv;
+    while (rows > 8 && (long)a.T * a.H * ((a.Dv + rows - 1) / rows) < 296) rows = (rows / 2 + 7) & ~7;
+    const dim3 grid((a.Dv + rows - 1) / rows, a.H, a.T);
+    cudaStream_t s = (cudaStream_t)stream;
+    const size_t smem = sizeof(float) * a.Rp;
+    if (a.w_f32) TSB_CHECK_CUDA(tsb_launch(latent_out_kernel<float>, grid, dim3(256), smem, s, a, rows));
+    else TSB_CHECK_CUDA(tsb_launch(latent_out_kernel<bf16>, grid, dim3(256), smem, s, a, rows));
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}

@@ -133,9 +133,9 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
         bf16* pk = sK + stage * BN * ldk + r * ldk;
         bf16* pv = sV + stage * BN * ldv + r * ldv;
         if (j < kvlen) {
-            const long row = vd_slot(a, b, j) * a.Hkv + hk;
-            const bf16* gk = a.k_cache + row * dk;
-            const bf16* gv = a.v_cache + row * DV;
+            const long slot = vd_slot(a, b, j);
+            const bf16* gk = a.k_cache + slot * a.k_ld + hk * dk;
+            const bf16* gv = a.v_cache + slot * a.v_ld + hk * DV;
             for (int c = half; c < ck; c += 2) cp_async16(pk + c * 8, gk + c * 8);
 #pragma unroll
             for (int c = 0; c < cv; c += 2) cp_async16(pv + (c + half) * 8, gv + (c + half) * 8);
@@ -259,21 +259,21 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
 
     for (int base = s0 + warp * KT; base < s1; base += 4 * KT) {
         const int j = base + lane;
-        const long row = j < s1 ? vd_slot(a, b, j) * a.Hkv + hk : 0;
+        const long slot = j < s1 ? vd_slot(a, b, j) : 0;
         // consecutive lanes copy consecutive pieces of a row; rows past the end are zero
         for (int i = lane; i < KT * ck; i += 32) {
             const int key = i / ck, c = i % ck;
-            const long rw = __shfl_sync(0xffffffffu, row, key);
+            const long sl = __shfl_sync(0xffffffffu, slot, key);
             bf16* p = sK + key * ldk + c * 8;
-            if (base + key < s1) cp_async16(p, a.k_cache + rw * dk + c * 8);
+            if (base + key < s1) cp_async16(p, a.k_cache + sl * a.k_ld + hk * dk + c * 8);
             else *reinterpret_cast<uint4*>(p) = make_uint4(0u, 0u, 0u, 0u);
         }
 #pragma unroll 4
         for (int i = lane; i < KT * cv; i += 32) {
             const int key = i / cv, c = i % cv;
-            const long rw = __shfl_sync(0xffffffffu, row, key);
+            const long sl = __shfl_sync(0xffffffffu, slot, key);
             bf16* p = sV + key * ldv + c * 8;
-            if (base + key < s1) cp_async16(p, a.v_cache + rw * DV + c * 8);
+            if (base + key < s1) cp_async16(p, a.v_cache + sl * a.v_ld + hk * DV + c * 8);
             else *reinterpret_cast<uint4*>(p) = make_uint4(0u, 0u, 0u, 0u);
         }
         cp_async_commit();
@@ -363,6 +363,9 @@ static int launch_vd(const AttnArgs& a, int max_q, cudaStream_t s) {
 static int dispatch_vd(const AttnArgs& in, int max_q, cudaStream_t s) {
     AttnArgs a = in;
     if (a.Dv == 0) a.Dv = a.Dh;
+    if (a.k_ld == 0) a.k_ld = (long)a.Hkv * a.Dh;
+    if (a.v_ld == 0) a.v_ld = (long)a.Hkv * a.Dv;
+    TSB_CHECK_ARG(a.k_ld % 8 == 0 && a.v_ld % 8 == 0, "attention: cache rows of %ld / %ld elements are not 16-byte aligned", a.k_ld, a.v_ld);
     if (a.Dh <= 0 || a.Dh > 256 || a.Dh % 16 || a.Dv <= 0 || a.Dv > 256 || a.Dv % 16) {
         tsb_set_error("attention: unsupported head sizes %d / %d (multiples of 16 up to 256, or 512 with equal sizes)", a.Dh, a.Dv);
         return TSB_ERR_UNSUPPORTED;

@@ -36,6 +36,9 @@ struct AttnArgs {
     long gate_tok;            // elements between query rows
     int gate_f32;
     int Dv;                   // value head size (0 = Dh): v_cache [slots, Hkv, Dv], out [Tq, Hq, Dv]
+    // Elements between slots where the rows of a slot are not dense (attention_vd.cu and the 32-bit kernel): 0 = Hkv * Dh
+    // and Hkv * Dv.  Multiples of 8.
+    long k_ld, v_ld;
 };
 
 #ifdef __CUDACC__

@@ -456,6 +456,22 @@ extern "C" int tsb_glu_f32(const float* gate, const float* up, long g_stride, lo
     return TSB_OK;
 }
 
+// out = cap tanh(x / cap)
+__global__ void __launch_bounds__(256) softcap_kernel(const float* x, float* out, long n, float cap, float inv) {
+    pdl_wait();
+    pdl_trigger();
+    const long i = (long)blockIdx.x * 256 + threadIdx.x;
+    if (i < n) out[i] = cap * tanhf(x[i] * inv);
+}
+
+extern "C" int tsb_softcap(const float* x, float* out, long n, float cap, void* stream) {
+    TSB_CHECK_ARG(cap > 0.f, "softcap: cap %f", cap);
+    if (n == 0) return TSB_OK;
+    TSB_CHECK_CUDA(tsb_launch(softcap_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, (cudaStream_t)stream, x, out, n, cap, 1.f / cap));
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}
+
 template <typename T>
 __global__ void glu_kernel(const T* gate, const T* up, long g_stride, long u_stride, int F, int act, bf16* out,
                            int8_t* yq, float2* yds, long rows) {

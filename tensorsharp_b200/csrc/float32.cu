@@ -120,11 +120,11 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnArgs a) {
     for (int base = lo + warp * 32; base <= pos; base += 128) {
         const int j = base + lane;
         const bool ok = j <= pos;
-        const long row = ok ? ((long)a.block_table[(long)b * a.max_pages + j / a.page_size] * a.page_size + j % a.page_size) * a.Hkv + hk : 0;
+        const long slot = ok ? (long)a.block_table[(long)b * a.max_pages + j / a.page_size] * a.page_size + j % a.page_size : 0;
         float s = -INFINITY;
         if (ok) {
             s = 0.f;
-            const float* kp = kc + row * a.Dh;
+            const float* kp = kc + slot * a.k_ld + hk * a.Dh;
             for (int d = 0; d < a.Dh; ++d) s = fmaf(sq[d], kp[d], s);
             s *= a.scale;
             if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
@@ -139,8 +139,8 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnArgs a) {
         const int cnt = min(32, pos - base + 1);
         for (int u = 0; u < cnt; ++u) {
             const float pu = __shfl_sync(0xffffffffu, p, u);
-            const long ru = __shfl_sync(0xffffffffu, row, u);
-            const float* vp = vc + ru * a.Dv;
+            const long su = __shfl_sync(0xffffffffu, slot, u);
+            const float* vp = vc + su * a.v_ld + hk * a.Dv;
 #pragma unroll
             for (int i = 0; i < NJ; ++i) {
                 const int d = lane + 32 * i;
@@ -174,6 +174,8 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnArgs a) {
 extern "C" int tsb_attn_f32(const AttnArgs* args, int T, void* stream) {
     AttnArgs a = *args;
     if (a.Dv == 0) a.Dv = a.Dh;
+    if (a.k_ld == 0) a.k_ld = (long)a.Hkv * a.Dh;
+    if (a.v_ld == 0) a.v_ld = (long)a.Hkv * a.Dv;
     TSB_CHECK_ARG(a.Hkv > 0 && a.Hq % a.Hkv == 0 && a.cu_q != nullptr, "attn_f32: Hq=%d Hkv=%d", a.Hq, a.Hkv);
     TSB_CHECK_ARG(a.Dh > 0 && a.Dh <= 1024 && a.Dv > 0 && a.Dv <= ATTN_F32_MAX_DV, "attn_f32: head sizes %d / %d", a.Dh, a.Dv);
     TSB_CHECK_ARG(a.gate == nullptr || a.gate_f32, "attn_f32: the gate must be float32");

@@ -64,6 +64,7 @@ class ModelBase:
     supports_pipeline = False
     supports_context_parallel = False
     supports_float32 = False           # compute_dtype float32 on the GPU
+    graphs_with_state = False          # single-token steps may be captured although the model has recurrent state
     mixed_batches = False              # the continuous batcher may put prompt portions and decoded tokens into one step
     native_sources: Optional[Tuple[str, ...]] = None     # kernel sources the family needs (None: the whole library)
 
@@ -432,7 +433,7 @@ class ModelBase:
         with recurrent state, and not while multimodal embeddings wait to be injected."""
         if self.device.type != "cuda" or self.tp_size > 1 or self.pp_size > 1 or self._pending_embeddings:
             return False
-        if not self.supports_kv_truncation:             # recurrent state: the capture's warm-up step would advance it
+        if not (self.supports_kv_truncation or self.graphs_with_state):      # (recurrent state)
             return False
         if self.kv.ring:                                # the steppers rewrite block-table rows themselves (full table only)
             return False

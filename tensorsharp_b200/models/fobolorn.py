@@ -22,15 +22,10 @@ from typing import Dict, List, Optional, Tuple
 import torch
 import torch.nn.functional as TF
 
-from ..gguf.constants import GGMLType
 from ..ops import functional as F
 from ..ops.functional import Act, Batch
-from ..quant.qweight import QuantWeight
-from .base import ModelBase, ModelConfig, register_architecture
-
-
-def _up(n: int, m: int) -> int:
-    return (n + m - 1) // m * m
+from .base import ModelConfig, register_architecture
+from .folder import FolderModel, round_up
 
 
 @dataclass
@@ -55,36 +50,21 @@ class MoeSpec:
 
 
 @register_architecture("fobolorn")
-class FobolornModel(ModelBase):
-    supports_float32 = True
-    mixed_batches = True
+class FobolornModel(FolderModel):
     native_sources = ("error.cpp", "elementwise.cu", "sandwich_norm.cu", "float32.cu", "attention.cu", "attention_vd.cu",
                       "attention_decode_mma.cu", "gemm_tcgen05.cu", "gemv.cu", "gemv_bf16.cu", "gemv_mma.cu", "gemv_stream.cu", "moe.cu", "sampler.cu")
 
     # ------------------------------------------------------------------ configuration
     def parse_base_config(self) -> ModelConfig:
-        j = self.gguf.config
-        self.layer_specs: List[dict] = list(j["layers"])
-        n = len(self.layer_specs)
-        loop = j.get("loop") or {}
-        self.loop = (int(loop.get("start", 0)), int(loop.get("stop", 0)), int(loop.get("times", 1))) if loop else (0, 0, 1)
-        a, b, times = self.loop
-        if not (0 <= a <= b <= n and times >= 0):
-            raise ValueError(f"{self.path}: loop {loop} does not fit {n} layers")
-        # (layer, pass number at the start of a pass): the layer runs in execution order
-        self.runs: List[Tuple[int, Optional[int]]] = [(i, None) for i in range(a)]
-        for t in range(times):
-            self.runs += [(i, t if loop and i == a else None) for i in range(a, b)]
-        self.runs += [(i, None) for i in range(b, n)]
-        self.width = int(j["width"])
+        self.parse_layers()
+        j, n = self.gguf.config, len(self.layer_specs)
         first = self.layer_specs[0]["mixer"] if n else {}
-        return ModelConfig(arch=self.arch, n_layers=len(self.runs), hidden=_up(self.width, 8), n_heads=int(first.get("heads", 0)),
+        return ModelConfig(arch=self.arch, n_layers=len(self.runs), hidden=round_up(self.width, 8), n_heads=int(first.get("heads", 0)),
                            n_kv_heads=int(first.get("kv_heads", 0)), head_dim=int(first.get("dim", 0)), vocab=int(j["vocab"]),
                            eps=float(j["norm"]["eps"]), context_length=int(j.get("context_length", 4096)))
 
     def parse_config(self) -> None:
-        if self.tp_size > 1 or self.ep_size > 1:
-            raise ValueError("Fobolorn runs on one GPU (no tensor- or expert-parallel path)")
+        self.refuse_parallel()
         for i, s in enumerate(self.layer_specs):
             if s["type"] != "attention":
                 raise ValueError(f"{self.path}: layer {i} has unknown type {s['type']!r}")
@@ -92,32 +72,6 @@ class FobolornModel(ModelBase):
                 raise ValueError(f"{self.path}: layer {i} has unknown feed-forward {s['mlp'].get('kind')!r}")
 
     # ------------------------------------------------------------------ weights
-    def _host(self, name: str) -> torch.Tensor:
-        """A stored matrix or vector on the host, in its stored float type."""
-        ti = self.gguf.tensors.get(name)
-        if ti is None:
-            raise KeyError(f"{self.path}: tensor {name!r} not found")
-        kinds = {GGMLType.BF16: torch.bfloat16, GGMLType.F16: torch.float16, GGMLType.F32: torch.float32}
-        if ti.ggml_type not in kinds:
-            raise ValueError(f"{self.path}: tensor {name!r} has type {ti.ggml_type.name}, a float type is needed")
-        raw = torch.frombuffer(bytearray(self.gguf.tensor_bytes_view(name)), dtype=kinds[ti.ggml_type])
-        return raw.view(ti.shape)
-
-    def _mat(self, name: str, rows: Optional[int] = None, cols: Optional[int] = None) -> torch.Tensor:
-        """A stored matrix, padded with zero rows / columns."""
-        w = self._host(name)
-        return TF.pad(w, (0, (cols or w.shape[1]) - w.shape[1], 0, (rows or w.shape[0]) - w.shape[0]))
-
-    def _vec(self, name: str, n: int) -> torch.Tensor:
-        w = self._host(name).float()
-        return TF.pad(w, (0, n - w.shape[-1])).to(self.device).contiguous()
-
-    def _qw(self, w: torch.Tensor, name: str) -> QuantWeight:
-        """A float matrix ``[N, K]`` or stack ``[E, N, K]`` as the linear kernels take it."""
-        t = GGMLType.BF16 if w.dtype == torch.bfloat16 else GGMLType.F32
-        w = w if t == GGMLType.BF16 else w.float()
-        return QuantWeight.from_raw(w.contiguous().view(-1).view(torch.uint8), t, tuple(w.shape), self.device, name)
-
     def _norm(self, name: str) -> Tuple[torch.Tensor, torch.Tensor]:
         return self._vec(name, self.cfg.hidden), self._vec(name + ".b", self.cfg.hidden)
 
@@ -126,7 +80,7 @@ class FobolornModel(ModelBase):
         H, G, dim, vdim = int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])
         if H % G:
             raise ValueError(f"{p}: {H} heads are not a multiple of {G} key / value heads")
-        s = AttnSpec(H, G, dim, vdim, _up(dim, 16), _up(vdim, 16), float(m["scale"]),
+        s = AttnSpec(H, G, dim, vdim, round_up(dim, 16), round_up(vdim, 16), float(m["scale"]),
                      (float(m["q_temp"]["coef"]), float(m["q_temp"]["every"])) if m.get("q_temp") else None)
         if max(s.Dk, s.Dv) > 256:
             raise ValueError(f"{p}: head sizes {dim} / {vdim} are above 256")
@@ -136,7 +90,7 @@ class FobolornModel(ModelBase):
             return TF.pad(w, (0, 0, 0, dp - d)).reshape(n * dp, D)
         parts = [heads("q", H, dim, s.Dk), heads("k", G, dim, s.Dk), heads("v", G, vdim, s.Dv), self._mat(p + "g", cols=D)]
         w = torch.cat(parts)
-        w = TF.pad(w, (0, 0, 0, _up(w.shape[0], 8) - w.shape[0]))            # rows of the result stay 16-byte aligned
+        w = TF.pad(w, (0, 0, 0, round_up(w.shape[0], 8) - w.shape[0]))            # rows of the result stay 16-byte aligned
         wo = TF.pad(self._mat(p + "o", rows=D).view(D, H, vdim), (0, s.Dv - vdim)).reshape(D, H * s.Dv)
         return {"spec": s, "wqkvg": self._qw(w, p + "qkvg"), "wo": self._qw(wo, p + "o"),
                 "qn": self._vec(p + "q.norm", s.Dk), "kn": self._vec(p + "k.norm", s.Dk)}
@@ -144,7 +98,7 @@ class FobolornModel(ModelBase):
     def _moe(self, p: str, m: dict) -> Dict[str, object]:
         D = self.cfg.hidden
         r = m["router"]
-        E, top, ff = int(r["experts"]), int(r["top"]), _up(int(m["expert"]["ff"]), 8)
+        E, top, ff = int(r["experts"]), int(r["top"]), round_up(int(m["expert"]["ff"]), 8)
         shared = m.get("shared")
         gate = [self._mat(f"{p}e{e}.gate", ff, D) for e in range(E)]
         up = [self._mat(f"{p}e{e}.up", ff, D) for e in range(E)]
@@ -207,10 +161,6 @@ class FobolornModel(ModelBase):
         logits = F.linear(a, m["router"], out_dtype=torch.float32)
         ids, w = F.route_softmax_renorm(logits, s.E, s.top, s.scale, s.shared)
         return F.moe_expert_parts(a, ids, w, m["gate_up"], m["down"], act="swiglu")
-
-    @property
-    def bf16(self) -> bool:
-        return self.device.type == "cuda" and self.compute_dtype == torch.bfloat16
 
     def forward_batch(self, batch: Batch, want_logits: bool = True) -> Optional[torch.Tensor]:
         c, n, dt = self.cfg, self.width, self.compute_dtype

@@ -153,6 +153,43 @@ def residual_layernorm(h: torch.Tensor, eps: float, n: int, *, y=None, post=None
     return Act(ref.layernorm_n(h, pre[0], pre[1], eps, n)) if pre is not None else None
 
 
+def parallel_seam(h: torch.Tensor, eps: float, n: int, *, y=(None, None), scale=(None, None), w=(None, None), out=(None, None),
+                  outputs: int = 2, dtype: Optional[torch.dtype] = None, shift: Optional[torch.Tensor] = None,
+                  state: Optional[torch.Tensor] = None, batch: Optional[Batch] = None):
+    """The seam between two layers whose sublayers read the same residual (one kernel on CUDA): ``h`` (f32 ``[T, D]``) plus
+    ``scale[0] * y[0] + scale[1] * y[1]`` (vectors ``[D]``; None: no such sublayer), and the next layer's inputs, the RMS
+    norms of the sum with the weights ``w``.  The first input moves towards the previous token's by ``shift`` per channel;
+    ``state`` (f32, a row per slot) holds that of the last token of each sequence between calls.  An output without a
+    weight is the sum itself; ``out`` are buffers to write to, else the first ``outputs`` of them are made.  The norm runs
+    over the first ``n`` columns, the rest is padding.  Returns (new h, first output, second output)."""
+    out = list(out)
+    if h.is_cuda:
+        for i in range(outputs):
+            if out[i] is None:
+                out[i] = torch.empty(h.shape, dtype=dtype or torch.bfloat16, device=h.device)
+        kw = dict(shift=shift, state=state, cu_q=batch.cu_q, seq_slots=batch.seq_slots) if shift is not None else {}
+        return (_k().parallel_norm(h, eps, n, y=y, scale=scale, w=w, out=out, **kw),) + tuple(out)
+    for t, s in zip(y, scale):
+        if t is not None:
+            h = h + s * t.float()
+    rs = torch.rsqrt((h * h).sum(-1, keepdim=True) / n + eps)
+    res = [h * rs * wi if wi is not None else h for wi in w]
+    if shift is not None:
+        v = res[0]
+        before = torch.empty_like(v)
+        before[1:] = v[:-1]
+        for b, slot in enumerate(batch.seq_slots.tolist()):
+            before[batch.h_cu_q[b]] = state[slot]
+            state[slot] = v[batch.h_cu_q[b + 1] - 1]
+        res[0] = v + (before - v) * shift
+    for i in range(2):
+        if out[i] is not None:
+            out[i].copy_(res[i])
+        elif i < outputs:
+            out[i] = res[i]
+    return h, out[0], out[1]
+
+
 def as_act(x, w: Optional[QuantWeight] = None) -> Act:
     """Wrap a plain activation tensor (an ``Act`` passes through)."""
     if isinstance(x, Act):
@@ -558,7 +595,150 @@ def argmax(logits: torch.Tensor) -> torch.Tensor:
     return logits.argmax(-1).to(torch.int32)
 
 
+# --------------------------------------------------------------------------------------------
+# Latent attention: one cached row [latent | rotated key part] per token serves every head
+# --------------------------------------------------------------------------------------------
+@dataclass
+class LatentSpec:
+    """Sizes of a latent-attention mixer.  A cached row is [latent (rank) | rotated part (rot) | zeros] of ``row`` elements, a
+    query head [unrotated (dim) | rotated (rot) | zeros] of ``Dk``, a value head ``Dv``; ``qp``, ``rank_p``: padded ranks."""
+    heads: int
+    dim: int
+    rot: int
+    vdim: int
+    rank: int
+    q_rank: int
+    scale: float
+    window: int                           # 0: the whole context
+    base: float
+    freq: torch.Tensor                    # float64 [rot / 2] on the compute device
+
+    def __post_init__(self):
+        self.Dk, self.Dv = (self.dim + self.rot + 15) // 16 * 16, (self.vdim + 15) // 16 * 16
+        self.row = (self.rank + self.rot + 31) // 32 * 32
+        self.qp, self.rank_p = (self.q_rank + 7) // 8 * 8, (self.rank + 7) // 8 * 8
+
+
+def rotary_freqs(dims: int, base: float, device) -> torch.Tensor:
+    """base^(-2 i / dims) of every pair, float64."""
+    return torch.tensor([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64, device=device)
+
+
+def rotary_table(batch: Batch, s: LatentSpec) -> torch.Tensor:
+    """(cos, sin) [T, rot / 2, 2] of the batch's positions, made once per step for all layers with these frequencies."""
+    key = ("rotary", s.base, s.rot)
+    t = batch.cache.get(key)
+    if t is None:
+        if batch.positions.is_cuda:
+            t = _k().rotary_table(batch.positions, s.freq)
+        else:
+            ang = batch.positions.double().unsqueeze(1) * s.freq
+            t = torch.stack([ang.cos(), ang.sin()], -1).float()
+        batch.cache[key] = t
+    return t
+
+
+def _rotate_half(x: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
+    """x [T, ..., R] with the columns i and i + R / 2 as pairs."""
+    half = x.shape[-1] // 2
+    t = table.view(table.shape[0], *([1] * (x.dim() - 2)), half, 2)
+    c, s = t[..., 0], t[..., 1]
+    x0, x1 = x[..., :half], x[..., half:]
+    return torch.cat([x0 * c - x1 * s, x1 * c + x0 * s], -1)
+
+
+def latent_cache(y: torch.Tensor, s: LatentSpec, qn: torch.Tensor, kn: torch.Tensor, cache: torch.Tensor, batch: Batch, eps: float) -> Act:
+    """Projection rows [query latent (qp) | latent (rank) | rotated part (rot)] -> the normed query latent; the normed latent
+    and the rotated key part are written to the paged cache ``[slots, 1, row]`` at ``batch.slots``."""
+    table = rotary_table(batch, s)
+    if y.is_cuda:
+        return Act(_k().latent_prep(y, s, qn, kn, table, cache, batch.slots, eps))
+    T = y.shape[0]
+    cq = torch.zeros((T, s.qp))
+    cq[:, :s.q_rank] = ref.rmsnorm(y[:, :s.q_rank], qn, eps)
+    row = torch.zeros((T, s.row))
+    row[:, :s.rank] = ref.rmsnorm(y[:, s.qp:s.qp + s.rank], kn, eps)
+    row[:, s.rank:s.rank + s.rot] = _rotate_half(y[:, s.qp + s.rank:s.qp + s.rank + s.rot].float(), table)
+    kv_scatter(cache, batch.slots, row.unsqueeze(1))
+    return Act(cq)
+
+
+def visible_rows(batch: Batch, window: int):
+    """The cache rows that some query of the batch can see, packed sequence after sequence: (cache slot of each packed row
+    int32, block table of the packed rows in pages of 64).  A sequence's rows start at a multiple of 64 positions, and its
+    last page is filled up with copies of its last row; memoised per step."""
+    key = ("visible", id(batch.block_table), window)
+    hit = batch.cache.get(key)
+    if hit is not None:
+        return hit
+    seq, pos, table, n = [], [], [], 0
+    width = max((L + 63) // 64 for L in batch.h_kv_lens)
+    for b, L in enumerate(batch.h_kv_lens):
+        first = L - (batch.h_cu_q[b + 1] - batch.h_cu_q[b])                 # position of the first query
+        lo = max(0, first - window + 1) // 64 if window else 0
+        hi = (L + 63) // 64
+        table.append([0] * lo + list(range(n, n + hi - lo)) + [0] * (width - hi))
+        p = torch.arange(lo * 64, hi * 64).clamp_(max=L - 1)
+        pos.append(p)
+        seq.append(torch.full_like(p, b))
+        n += hi - lo
+    dev, ps = batch.block_table.device, batch.page_size
+    p, b = torch.cat(pos).to(dev), torch.cat(seq).to(dev)
+    slots = (batch.block_table[b, p // ps].long() * ps + p % ps).to(torch.int32)
+    hit = batch.cache[key] = (slots, torch.tensor(table, dtype=torch.int32).to(dev))
+    return hit
+
+
+def latent_attention(q: torch.Tensor, cache: torch.Tensor, batch: Batch, s: LatentSpec, *, wuk: torch.Tensor, wuv: torch.Tensor,
+                     expand: Optional[QuantWeight], sinks: Optional[torch.Tensor]) -> torch.Tensor:
+    """Causal attention of the queries ``[T, heads * Dk]`` (not rotated yet) over the cached rows -> ``[T, heads * Dv]``.
+    ``wuk`` [heads * dim, rank_p], ``wuv`` [heads * Dv, rank_p]: key and value maps; ``expand``: both as one matrix over
+    whole rows, [heads * Dk + heads * Dv, row], the rotated part passed on to every head.
+
+    CUDA, bf16: decode steps work on the rows themselves; prompts expand the rows in sight and take the ordinary prefill
+    kernel.  CUDA, float32: on the rows themselves, prompts too."""
+    T, H = q.shape[0], s.heads
+    table = rotary_table(batch, s)
+    if not q.is_cuda:
+        qh = q.float().view(T, H, s.Dk)
+        qh = torch.cat([qh[..., :s.dim], _rotate_half(qh[..., s.dim:s.dim + s.rot], table)], -1)
+        uk, uv = wuk.float().view(H, s.dim, -1)[..., :s.rank], wuv.float().view(H, s.Dv, -1)[..., :s.rank]
+        outs, ps = [], batch.page_size
+        for b, L in enumerate(batch.h_kv_lens):
+            q0, q1 = batch.h_cu_q[b], batch.h_cu_q[b + 1]
+            p = torch.arange(L)
+            rows = cache[batch.block_table[b].long()[p // ps] * ps + p % ps, 0].float()
+            if s.window:
+                rows[:max(0, L - (q1 - q0) - s.window + 1)] = 0                # out of every query's sight; may be stale
+            k = torch.cat([torch.einsum("tr,hdr->thd", rows[:, :s.rank], uk),
+                           rows[:, None, s.rank:s.rank + s.rot].expand(L, H, s.rot)], -1)
+            v = torch.einsum("tr,hdr->thd", rows[:, :s.rank], uv)
+            outs.append(ref.attention(qh[q0:q1], k, v, batch.positions[q0:q1], scale=s.scale, window=s.window, sinks=sinks))
+        return torch.cat(outs).reshape(T, H * s.Dv)
+    kk = _k()
+    if cache.dtype == torch.float32:
+        qa = kk.latent_absorb(q, s, wuk, table, cache)
+        o = kk.attn_f32(qa, cache, cache[:, :, :s.rank], batch.block_table, batch.kv_lens, batch.cu_q, scale=s.scale, Hq=H, Hkv=1, Dh=s.row,
+                        Dv=s.rank, page_size=batch.page_size, sinks=sinks, window=s.window)
+        return kk.latent_out(o, None, s, wuv, None, table, cache)
+    if batch.is_decode:
+        qa = kk.latent_absorb(q, s, wuk, table, cache)
+        part_o, part_ml = kk.latent_decode(qa, s, table, cache, batch.block_table, batch.kv_lens, batch.page_size,
+                                           decode_splits(batch, (H + 15) // 16, s.window))
+        return kk.latent_out(part_o, part_ml, s, wuv, sinks, table, cache)
+    kk.latent_rotate(q, s, table, cache)
+    slots, pages = visible_rows(batch, s.window)
+    rows = kk.gather_bf16_rows(cache.view(-1, s.row), slots, 1)
+    kv = kk.gemm_bf16(_dequant_scratch(expand), rows)
+    k, v = kv[:, :H * s.Dk].unflatten(1, (H, s.Dk)), kv[:, H * s.Dk:].unflatten(1, (H, s.Dv))
+    out = kk.attn_prefill(q.view(T, H, s.Dk), k, v, pages, batch.kv_lens, batch.cu_q, batch.max_q_len, scale=s.scale, Hq=H, Hkv=H, Dh=s.Dk,
+                          Dv=s.Dv, page_size=64, sinks=sinks, window=s.window)
+    return out.view(T, H * s.Dv)
+
+
 def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    if cap and cap > 0 and x.is_cuda and x.dtype == torch.float32 and x.is_contiguous():
+        return _k().softcap(x, cap)
     return torch.tanh(x / cap) * cap if cap and cap > 0 else x
 
 
@@ -880,6 +1060,43 @@ def gdn(qkv: torch.Tensor, z: torch.Tensor, beta: torch.Tensor, alpha: torch.Ten
         outs.append(ref.gdn_recurrent(qkv[q0:q1], z[q0:q1], beta[q0:q1], alpha[q0:q1], dt_bias, a_log, norm_w, state[slots[b]],
                                       Hk=Hk, Hv=Hv, Dk=Dk, Dv=Dv, eps=eps))
     return torch.cat(outs, 0).to(torch.bfloat16 if qkv.is_cuda else torch.float32)     # the kernel's output types
+
+
+GENERAL_DELTA_SCAN_MIN = 8          # tokens of the longest portion from which the prompt kernels beat the one-kernel step
+
+
+def general_delta(y: torch.Tensor, w2: QuantWeight, w0: torch.Tensor, ab: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, batch: Batch,
+                  *, H: int, D: int, n: int, rank: int, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """Generalized delta rule with a decay and a removal rate per key channel over the packed tokens -> gated output
+    [T, H * D].  ``y`` rows: r | k | v | removal | gate (H * D each) | low-rank part of the decay (``rank``); ``w2``
+    [H * D, rank up to 8], ``w0``: the decay's second map and offset; ``ab``: the removal's offset.  ``state`` f32
+    [slots, H, values, keys].  Heads of ``n`` channels are padded with zeros to ``D``."""
+    HD = H * D
+    if y.is_cuda:
+        kk = _k()
+        kw = dict(H=H, D=D, n=n, eps=eps, out_dtype=dtype)
+        if batch.max_q_len < GENERAL_DELTA_SCAN_MIN:
+            return kk.general_delta_short(y, _weight_matrix(w2), w0, ab, norm_w, state, batch.cu_q, batch.seq_slots, rank=w2.K, **kw)
+        t = kk.tanh_rows(y, 5 * HD, rank, w2.K, dtype)
+        z = linear(Act(t), w2, out_dtype=torch.float32)
+        # a CTA holds 16 or 32 value channels of a head: the narrower slices while the wider ones would leave SMs idle
+        return kk.general_delta_prompt(y, z, w0, ab, norm_w, state, batch.cu_q, batch.seq_slots, warps=4 if batch.B * HD // 32 >= 148 else 2, **kw)
+    T, y = y.shape[0], y.float()
+    z = torch.tanh(y[:, 5 * HD:5 * HD + rank]) @ w2.dequantize()[:, :rank].t() + w0
+    r, k, v, a = (y[:, i * HD:(i + 1) * HD].view(T, H, D) for i in range(4))
+    o, slots = torch.empty((T, H, D)), batch.seq_slots.tolist()
+    decay, a = ref.delta_decay(z).view(T, H, D), torch.sigmoid(a + ab.view(H, D))
+    for b in range(batch.B):
+        q0, q1 = batch.h_cu_q[b], batch.h_cu_q[b + 1]
+        o[q0:q1] = ref.general_delta(r[q0:q1], k[q0:q1], v[q0:q1], decay[q0:q1], a[q0:q1], state[slots[b]])
+    o = o * torch.rsqrt((o * o).sum(-1, keepdim=True) / n + eps)
+    return o.reshape(T, HD) * norm_w * torch.sigmoid(y[:, 4 * HD:5 * HD])
+
+
+def _weight_matrix(w: QuantWeight) -> torch.Tensor:
+    """The [N, K] tensor of a bf16 or f32 weight."""
+    from ..gguf.constants import GGMLType
+    return w.planes[0].view(torch.bfloat16 if w.ggml_type == GGMLType.BF16 else torch.float32).view(w.rows, w.K)
 
 
 def mamba2(xbc: torch.Tensor, dt: torch.Tensor, dt_bias, A, D, state: torch.Tensor, batch: Batch, *, H: int, P: int,

@@ -80,7 +80,8 @@ class AttnArgs(C.Structure):
                 ("B", C.c_int), ("Hq", C.c_int), ("Hkv", C.c_int), ("Dh", C.c_int), ("page_size", C.c_int),
                 ("max_pages", C.c_int), ("splits", C.c_int), ("q_pos0", _vp), ("lse_out", _vp),
                 ("out_q", _vp), ("out_ds", _vp), ("ticket", _vp), ("split_len", C.c_int),
-                ("gate", _vp), ("gate_tok", C.c_long), ("gate_f32", C.c_int), ("Dv", C.c_int)]
+                ("gate", _vp), ("gate_tok", C.c_long), ("gate_f32", C.c_int), ("Dv", C.c_int),
+                ("k_ld", C.c_long), ("v_ld", C.c_long)]
 
 
 _configured = False
@@ -454,6 +455,11 @@ def _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, cu_q, sinks, scal
     a.max_pages = block_table.shape[1]
     a.splits = 1
     a.Dv = Dv or Dh
+    # a slot's rows may be a slice of a wider row (no gaps between the heads)
+    for c, heads, d, ld in ((k_cache, Hkv, Dh, "k_ld"), (v_cache, Hkv, Dv or Dh, "v_ld")):
+        if c.dim() == 3 and c.stride(0) != heads * d:
+            assert c.stride(2) == 1 and (heads == 1 or c.stride(1) == d)
+            setattr(a, ld, c.stride(0))
     if gate is not None:
         assert gate.shape == (q.shape[0], Hq) and gate.stride(1) == 1
         a.gate, a.gate_tok, a.gate_f32 = gate.data_ptr(), gate.stride(0), int(gate.dtype == torch.float32)
@@ -576,6 +582,204 @@ def residual_layernorm(h: torch.Tensor, eps: float, n: int, *, y=None, pos=None,
         out = torch.empty((T, D), dtype=out_dtype, device=h.device)
         a.pre_w, a.pre_b, a.out, a.out_f32 = _p(pre[0]), _p(pre[1]), _p(out), int(out_dtype == torch.float32)
     native.check(_lib().tsb_sandwich_norm(C.byref(a), _stream()), "residual_layernorm")
+    _count(1)
+    return out
+
+
+class ParallelNormArgs(C.Structure):
+    _fields_ = [("h", _vp), ("h_out", _vp), ("y1", _vp), ("y2", _vp), ("s1", _vp), ("s2", _vp), ("w1", _vp), ("w2", _vp),
+                ("out1", _vp), ("out2", _vp), ("shift", _vp), ("state", _vp), ("cu_q", _vp), ("seq_slots", _vp),
+                ("rows", C.c_long), ("ld1", C.c_long), ("ld2", C.c_long), ("state_s", C.c_long),
+                ("D", C.c_int), ("n", C.c_int), ("B", C.c_int), ("y_f32", C.c_int), ("out1_f32", C.c_int), ("out2_f32", C.c_int),
+                ("span", C.c_int), ("eps", C.c_float)]
+
+
+def parallel_norm(h, eps: float, n: int, *, y=(None, None), scale=(None, None), w=(None, None), out=(None, None), shift=None, state=None,
+                  cu_q=None, seq_slots=None) -> torch.Tensor:
+    """The seam of csrc/parallel_norm.cu: returns the new residual (``h`` itself when there is nothing to add) and fills the
+    ``out`` tensors (rows may be strided)."""
+    assert h.dtype == torch.float32 and h.is_contiguous()
+    T, D = h.shape
+    a = ParallelNormArgs()
+    a.h, a.rows, a.D, a.n, a.eps = _p(h), T, D, n, eps
+    res = h
+    if y[0] is not None:
+        res = torch.empty_like(h)
+        a.h_out, a.y_f32 = _p(res), int(y[0].dtype == torch.float32)
+        for t in y:
+            assert t is None or (t.shape == h.shape and t.is_contiguous() and t.dtype == y[0].dtype and t.dtype in (torch.float32, torch.bfloat16))
+        a.y1, a.y2, a.s1, a.s2 = _p(y[0]), _p(y[1]), _p(scale[0]), _p(scale[1])
+    a.w1, a.w2 = _p(w[0]), _p(w[1])
+    for i, o in enumerate(out, 1):
+        if o is not None:
+            assert o.shape == h.shape and o.stride(1) == 1 and o.dtype in (torch.float32, torch.bfloat16)
+            setattr(a, f"out{i}", _p(o))
+            setattr(a, f"ld{i}", o.stride(0))
+            setattr(a, f"out{i}_f32", int(o.dtype == torch.float32))
+    if shift is not None:
+        check_index("parallel_norm", "state slot", seq_slots, state.shape[0])
+        check_index("parallel_norm", "row offset", cu_q, T + 1)
+        assert state.dtype == torch.float32 and state.stride(1) == 1 and seq_slots.dtype == torch.int64 and cu_q.dtype == torch.int32
+        a.shift, a.state, a.state_s, a.cu_q, a.seq_slots, a.B = _p(shift), _p(state), state.stride(0), _p(cu_q), _p(seq_slots), cu_q.numel() - 1
+    native.check(_lib().tsb_parallel_norm(C.byref(a), _stream()), "parallel_norm")
+    _count(1)
+    return res
+
+
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """cap tanh(x / cap) (f32)."""
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    out = torch.empty_like(x)
+    native.check(_lib().tsb_softcap(_p(x), _p(out), C.c_long(x.numel()), C.c_float(cap), _stream()), "softcap")
+    _count(1)
+    return out
+
+
+class LatentArgs(C.Structure):
+    _fields_ = [("y", _vp), ("y_s", C.c_long), ("y_f32", C.c_int), ("qn", _vp), ("kn", _vp), ("cs", _vp), ("slots", _vp), ("cache", _vp),
+                ("cq", _vp), ("f32", C.c_int), ("T", C.c_int), ("qr", C.c_int), ("qp", C.c_int), ("R", C.c_int), ("rot", C.c_int),
+                ("Lp", C.c_int), ("eps", C.c_float),
+                ("q", _vp), ("q_f32", C.c_int), ("wuk", _vp), ("wuv", _vp), ("w_f32", C.c_int), ("qa", _vp),
+                ("H", C.c_int), ("dim", C.c_int), ("Dk", C.c_int), ("Rp", C.c_int), ("Dv", C.c_int),
+                ("block_table", _vp), ("kv_lens", _vp), ("part_o", _vp), ("part_ml", _vp), ("sinks", _vp), ("out", _vp),
+                ("scale", C.c_float), ("window", C.c_int), ("page_size", C.c_int), ("max_pages", C.c_int), ("splits", C.c_int),
+                ("Ro", C.c_int)]
+
+
+def rotary_table(pos: torch.Tensor, freq: torch.Tensor) -> torch.Tensor:
+    """(cos, sin) of pos * freq: float32 [T, pairs, 2]; ``freq`` float64 on the device."""
+    assert pos.dtype == torch.int32 and freq.dtype == torch.float64
+    out = torch.empty((pos.numel(), freq.numel(), 2), dtype=torch.float32, device=pos.device)
+    native.check(_lib().tsb_rotary_table(_p(pos), _p(freq), _p(out), C.c_int(pos.numel()), C.c_int(freq.numel()), _stream()), "rotary_table")
+    _count(1)
+    return out
+
+
+def _latent_args(s, T: int, cs: torch.Tensor, cache: torch.Tensor) -> LatentArgs:
+    a = LatentArgs()
+    a.T, a.qr, a.qp, a.R, a.rot, a.Lp, a.cs = T, s.q_rank, s.qp, s.rank, s.rot, s.row, _p(cs)
+    a.H, a.dim, a.Dk, a.Rp, a.Dv, a.scale, a.window = s.heads, s.dim, s.Dk, s.rank_p, s.Dv, s.scale, s.window
+    assert cache.shape[-1] == s.row and cache.is_contiguous() and cache.dtype in (torch.float32, torch.bfloat16)
+    a.cache, a.f32 = _p(cache), int(cache.dtype == torch.float32)
+    return a
+
+
+def latent_prep(y: torch.Tensor, s, qn, kn, cs, cache, slots, eps: float) -> torch.Tensor:
+    """Rows [query latent | key / value latent | rotated part] -> the normed query latent [T, qp]; the normed latent and the
+    rotated key part go to the cache rows ``slots``."""
+    T = y.shape[0]
+    check_index("latent_prep", "cache slot", slots, cache.shape[0])
+    assert y.stride(1) == 1 and y.shape[1] >= s.qp + s.rank + s.rot and slots.dtype == torch.int64
+    a = _latent_args(s, T, cs, cache)
+    cq = torch.empty((T, s.qp), dtype=cache.dtype, device=y.device)
+    a.y, a.y_s, a.y_f32, a.qn, a.kn, a.slots, a.cq, a.eps = _p(y), y.stride(0), int(y.dtype == torch.float32), _p(qn), _p(kn), _p(slots), _p(cq), eps
+    native.check(_lib().tsb_latent_prep(C.byref(a), _stream()), "latent_prep")
+    _count(1)
+    return cq
+
+
+def latent_rotate(q: torch.Tensor, s, cs, cache) -> torch.Tensor:
+    """Rotate the rotated parts of queries [T, H * Dk] in place."""
+    a = _latent_args(s, q.shape[0], cs, cache)
+    assert q.is_contiguous() and q.shape[1] == s.heads * s.Dk
+    a.q, a.q_f32 = _p(q), int(q.dtype == torch.float32)
+    native.check(_lib().tsb_latent_rotate(C.byref(a), _stream()), "latent_rotate")
+    _count(1)
+    return q
+
+
+def latent_absorb(q: torch.Tensor, s, wuk: torch.Tensor, cs, cache) -> torch.Tensor:
+    """Queries [T, H * Dk] (not rotated) in the space of the cached rows: [T, H, row]."""
+    T = q.shape[0]
+    a = _latent_args(s, T, cs, cache)
+    assert q.is_contiguous() and q.shape[1] == s.heads * s.Dk and wuk.is_contiguous() and wuk.shape == (s.heads * s.dim, s.rank_p)
+    qa = torch.empty((T, s.heads, s.row), dtype=cache.dtype, device=q.device)
+    a.q, a.q_f32, a.wuk, a.w_f32, a.qa = _p(q), int(q.dtype == torch.float32), _p(wuk), int(wuk.dtype == torch.float32), _p(qa)
+    native.check(_lib().tsb_latent_absorb(C.byref(a), _stream()), "latent_absorb")
+    _count(1)
+    return qa
+
+
+def latent_decode(qa: torch.Tensor, s, cs, cache, block_table, kv_lens, page_size: int, splits: int):
+    """One query per sequence against the cached bf16 rows -> split partials (o [B, H, splits, Ro], (max, sum))."""
+    B = qa.shape[0]
+    check_index("latent_decode", "block-table page", block_table, cache.shape[0] // page_size)
+    check_index("latent_decode", "cache length", kv_lens, block_table.shape[1] * page_size + 1)
+    a = _latent_args(s, B, cs, cache)
+    Ro = (s.rank + 7) // 8 * 8
+    part_o = torch.empty((B, s.heads, splits, Ro), dtype=torch.float32, device=qa.device)
+    part_ml = torch.empty((B, s.heads, splits, 2), dtype=torch.float32, device=qa.device)
+    a.qa, a.block_table, a.kv_lens, a.part_o, a.part_ml = _p(qa), _p(block_table), _p(kv_lens), _p(part_o), _p(part_ml)
+    a.page_size, a.max_pages, a.splits, a.Ro = page_size, block_table.shape[1], splits, Ro
+    native.check(_lib().tsb_latent_decode(C.byref(a), _stream()), "latent_decode")
+    _count(1)
+    return part_o, part_ml
+
+
+def latent_out(part_o: torch.Tensor, part_ml: Optional[torch.Tensor], s, wuv: torch.Tensor, sinks, cs, cache) -> torch.Tensor:
+    """Merge split partials (``part_ml`` None: finished rows [T, H, rank]) and apply the value map -> [T, H * Dv]."""
+    T = part_o.shape[0]
+    a = _latent_args(s, T, cs, cache)
+    assert wuv.is_contiguous() and wuv.shape == (s.heads * s.Dv, s.rank_p) and part_o.dtype == torch.float32 and part_o.is_contiguous()
+    out = torch.empty((T, s.heads * s.Dv), dtype=cache.dtype, device=part_o.device)
+    a.part_o, a.part_ml, a.wuv, a.w_f32, a.sinks, a.out = _p(part_o), _p(part_ml), _p(wuv), int(wuv.dtype == torch.float32), _p(sinks), _p(out)
+    a.splits, a.Ro = part_o.shape[2] if part_ml is not None else 1, part_o.shape[-1]
+    native.check(_lib().tsb_latent_out(C.byref(a), _stream()), "latent_out")
+    _count(1)
+    return out
+
+
+class GdrArgs(C.Structure):
+    _fields_ = [("y", _vp), ("y_s", C.c_long), ("y_f32", C.c_int), ("z", _vp), ("z_s", C.c_long), ("w2", _vp), ("w2_f32", C.c_int),
+                ("w0", _vp), ("ab", _vp), ("norm_w", _vp), ("state", _vp), ("state_s", C.c_long), ("cu_q", _vp), ("seq_slots", _vp),
+                ("pack", _vp), ("core", _vp), ("out", _vp), ("out_s", C.c_long), ("out_f32", C.c_int),
+                ("T", C.c_int), ("B", C.c_int), ("H", C.c_int), ("D", C.c_int), ("n", C.c_int), ("rank", C.c_int), ("eps", C.c_float)]
+
+
+def _gdr_args(y, w0, ab, norm_w, state, cu_q, seq_slots, *, H, D, n, rank, eps, out_dtype):
+    T = y.shape[0]
+    check_index("general_delta", "state slot", seq_slots, state.shape[0])
+    check_index("general_delta", "row offset", cu_q, T + 1)
+    assert y.stride(1) == 1 and y.shape[1] >= 5 * H * D + rank and state.dtype == torch.float32 and state.shape[1:] == (H, D, D)
+    assert state.stride(1) == D * D and state.stride(2) == D and seq_slots.dtype == torch.int64
+    a = GdrArgs()
+    a.y, a.y_s, a.y_f32, a.w0, a.ab, a.norm_w = _p(y), y.stride(0), int(y.dtype == torch.float32), _p(w0), _p(ab), _p(norm_w)
+    a.state, a.state_s, a.cu_q, a.seq_slots = _p(state), state.stride(0), _p(cu_q), _p(seq_slots)
+    out = torch.empty((T, H * D), dtype=out_dtype, device=y.device)
+    a.out, a.out_s, a.out_f32 = _p(out), H * D, int(out_dtype == torch.float32)
+    a.T, a.B, a.H, a.D, a.n, a.rank, a.eps = T, cu_q.numel() - 1, H, D, n, rank, eps
+    return a, out
+
+
+def general_delta_short(y, w2: torch.Tensor, w0, ab, norm_w, state, cu_q, seq_slots, *, H, D, n, rank, eps, out_dtype) -> torch.Tensor:
+    """Decode steps and short portions of the generalized delta rule (csrc/general_delta.cu), everything in one kernel."""
+    assert w2.is_contiguous() and w2.shape == (H * D, rank)
+    a, out = _gdr_args(y, w0, ab, norm_w, state, cu_q, seq_slots, H=H, D=D, n=n, rank=rank, eps=eps, out_dtype=out_dtype)
+    a.w2, a.w2_f32 = _p(w2), int(w2.dtype == torch.float32)
+    native.check(_lib().tsb_general_delta_short(C.byref(a), _stream()), "general_delta_short")
+    _count(1)
+    return out
+
+
+def general_delta_prompt(y, z: torch.Tensor, w0, ab, norm_w, state, cu_q, seq_slots, *, H, D, n, eps, out_dtype, warps: int = 4) -> torch.Tensor:
+    """Prompts: per-token vectors, recurrence, norm and gate in three kernels; ``z`` f32 [T, H * D] is the decay's projection."""
+    T = y.shape[0]
+    assert z.dtype == torch.float32 and z.shape == (T, H * D) and z.stride(1) == 1
+    a, out = _gdr_args(y, w0, ab, norm_w, state, cu_q, seq_slots, H=H, D=D, n=n, rank=0, eps=eps, out_dtype=out_dtype)
+    pack = torch.empty((T, H, 5, D), dtype=torch.float32, device=y.device)
+    core = torch.empty((T, H, D), dtype=torch.float32, device=y.device)
+    a.z, a.z_s, a.pack, a.core = _p(z), z.stride(0), _p(pack), _p(core)
+    native.check(_lib().tsb_general_delta_prompt(C.byref(a), C.c_int(warps), _stream()), "general_delta_prompt")
+    _count(3)
+    return out
+
+
+def tanh_rows(y: torch.Tensor, off: int, cols: int, ld: int, out_dtype) -> torch.Tensor:
+    """tanh of ``cols`` columns of y from ``off`` on as dense rows [T, ld], zero past the columns."""
+    assert y.stride(1) == 1 and off + cols <= y.shape[1]
+    out = torch.empty((y.shape[0], ld), dtype=out_dtype, device=y.device)
+    native.check(_lib().tsb_tanh_rows(_p(y), C.c_long(y.stride(0)), C.c_int(y.dtype == torch.float32), C.c_long(off), C.c_int(y.shape[0]),
+                                      C.c_int(cols), C.c_int(ld), _p(out), C.c_int(out_dtype == torch.float32), _stream()), "tanh_rows")
     _count(1)
     return out
 

@@ -128,6 +128,24 @@ def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_pos: torch.Te
     return torch.matmul(pr, vf).permute(1, 0, 2).contiguous()
 
 
+def delta_decay(z: torch.Tensor) -> torch.Tensor:
+    """exp(-e^(-1/2) sigmoid(z)): the decay of a key channel per token."""
+    return torch.exp(-math.exp(-0.5) * torch.sigmoid(z))
+
+
+def general_delta(r, k, v, decay, a, state: torch.Tensor) -> torch.Tensor:
+    """Generalized delta rule of one sequence, [T, H, D] each; ``state`` [H, values, keys] is advanced in place.  Per token:
+    S <- S diag(decay) - (S u)(a u)^T + v k^T with u = k / sqrt(sum(k^2) + 1e-6);  o = S r."""
+    out = torch.empty_like(r)
+    u = k * torch.rsqrt((k * k).sum(-1, keepdim=True) + 1e-6)
+    au = a * u
+    for t in range(r.shape[0]):
+        read = torch.einsum("hvk,hk->hv", state, u[t])
+        state.mul_(decay[t].unsqueeze(1)).sub_(read.unsqueeze(2) * au[t].unsqueeze(1)).add_(v[t].unsqueeze(2) * k[t].unsqueeze(1))
+        out[t] = torch.einsum("hvk,hk->hv", state, r[t])
+    return out
+
+
 def quantize_q8_dequant(x: torch.Tensor) -> torch.Tensor:
     """What the GEMV kernels see: x rounded to int8 in groups of 32 (scale amax/127)."""
     xf = x.float()
