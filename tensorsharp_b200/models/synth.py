@@ -560,3 +560,92 @@ def write_fobolorn(folder: str, config: Optional[dict] = None, *, seed=0, device
     with open(os.path.join(folder, CONFIG_NAME), "w", encoding="utf-8") as f:
         json.dump(cfg, f, indent=1)
     write_safetensors(os.path.join(folder, WEIGHTS_NAME), t)
+
+
+def sogulix_config(*, layers="lglg", width=128, heads=4, dim=32, rot_dim=16, vdim=32, q_rank=48, kv_rank=40, window=24, rot_base=10000.0,
+                   scale=None, delta_heads=3, delta_dim=32, decay_rank=8, ff=64, vocab=512, loop=None, residual_mult=0.5, softcap=30.0, eps=1e-5,
+                   no_mlp=()) -> dict:
+    """A config.json of the Sogulix architecture: ``layers`` has an ``l`` (latent attention) or a ``g`` (generalized delta
+    rule) per layer, ``loop`` = (start, stop, times) or None, ``no_mlp``: layers without a feed-forward.  The ranks of the
+    queries and of the decay are read off the tensors; the configuration names them for the writer."""
+    def spec(i, kind):
+        if kind == "l":
+            mixer = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank,
+                     "scale": scale if scale is not None else (dim + rot_dim) ** -0.5, "mask": {"size": window},
+                     "rot": {"dims": rot_dim, "base": rot_base}}
+        else:
+            mixer = {"heads": delta_heads, "dim": delta_dim, "decay_rank": decay_rank}
+        return {"type": "latent_attention" if kind == "l" else "general_delta", "mixer": mixer,
+                "mlp": None if i in no_mlp else {"kind": "dense", "ff": ff}}
+    cfg = {"architecture": "Sogulix", "vocab": vocab, "width": width, "norm": {"eps": eps}, "residual_mult": residual_mult,
+           "logit_softcap": softcap, "layers": [spec(i, k) for i, k in enumerate(layers)]}
+    if loop is not None:
+        cfg["loop"] = {"start": loop[0], "stop": loop[1], "times": loop[2]}
+    return cfg
+
+
+def write_sogulix(folder: str, config: Optional[dict] = None, *, seed=0, device=None, gain=1.0, **sizes) -> None:
+    """A model folder with random bf16 weights for ``config`` (default: :func:`sogulix_config` of ``sizes``): matrices
+    N(0, gain / fan-in), norm weights around their neutral value, shifts between 0 and 1, decays and removal rates spread
+    over their range."""
+    import json
+    import os
+
+    from ..gguf.folder import CONFIG_NAME, WEIGHTS_NAME, write_safetensors
+    cfg = config if config is not None else sogulix_config(**sizes)
+    dev = torch.device(device or ("cuda" if torch.cuda.is_available() else "cpu"))
+    gen = torch.Generator(device=dev)
+    gen.manual_seed(seed)
+    t = {}
+
+    def mat(name, rows, cols, std=None):
+        w = torch.randn((rows, cols), generator=gen, device=dev) * (std if std is not None else math.sqrt(gain / cols))
+        t[name] = w.to(torch.bfloat16).cpu()
+
+    def vec(name, n, mean, std):
+        t[name] = (mean + std * torch.randn(n, generator=gen, device=dev)).to(torch.bfloat16).cpu()
+
+    D = cfg["width"]
+    mat("embed", cfg["vocab"], D, 1.0)
+    vec("embed.norm", D, 0.0, 0.15)
+    if cfg.get("loop"):
+        mat("loop.in", D, 2 * D)
+    for i, s in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", s["mixer"]
+        q = p + "mix."
+        vec(p + "norm1", D, 0.0, 0.15)
+        vec(p + "ls1", D, 1.0, 0.2)
+        vec(p + "shift", D, 0.4, 0.2)
+        if s["type"] == "latent_attention":
+            H, R = m["heads"], m["kv_rank"]
+            mat(q + "dq", m["q_rank"], D)
+            vec(q + "dq.norm", m["q_rank"], 1.2, 0.2)
+            mat(q + "uq", H * (m["dim"] + m["rot_dim"]), m["q_rank"])
+            mat(q + "dkv", R + m["rot_dim"], D)
+            vec(q + "dkv.norm", R, 1.2, 0.2)
+            mat(q + "uk", H * m["dim"], R)
+            mat(q + "uv", H * m["vdim"], R)
+            vec(q + "sink", H, 0.5, 1.0)
+            mat(q + "o", D, H * m["vdim"])
+        else:
+            n, r = m["heads"] * m["dim"], m["decay_rank"]
+            for x in "rkvga":
+                mat(q + x, n, D)
+            vec(q + "a.b", n, -1.0, 1.0)
+            mat(q + "w1", r, D)
+            mat(q + "w2", n, r)
+            vec(q + "w0", n, -2.0, 2.0)
+            vec(q + "norm", n, 1.0, 0.15)
+            mat(q + "o", D, n)
+        if s["mlp"] is not None:
+            vec(p + "norm2", D, 0.0, 0.15)
+            vec(p + "ls2", D, 1.0, 0.2)
+            for x in ("gate", "up"):
+                mat(p + "mlp." + x, s["mlp"]["ff"], D)
+            mat(p + "mlp.down", D, s["mlp"]["ff"])
+    vec("final.norm", D, 0.0, 0.15)
+    mat("head", cfg["vocab"], D)
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, CONFIG_NAME), "w", encoding="utf-8") as f:
+        json.dump(cfg, f, indent=1)
+    write_safetensors(os.path.join(folder, WEIGHTS_NAME), t)
