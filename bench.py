@@ -57,7 +57,7 @@ def parse_args():
     ap.add_argument("--trace", default=None, metavar="FILE",
                     help="after the timed runs, record three more graph replays with the CUDA activity tracer, write the "
                          "kernel events of the middle one to FILE (JSON) and print its per-kernel table to stderr")
-    ap.add_argument("--design", default=None, choices=["fobolorn"],
+    ap.add_argument("--design", default=None, choices=["fobolorn", "sogulix"],
                     help="measure this design at several sizes beside the closest other model at equal size (one JSON line per "
                          "size and model) instead of the headline workload")
     ap.add_argument("--design-size", default=None, help="with --design: only this size")
@@ -493,17 +493,48 @@ def run_reference(args) -> dict:
     return ref_run(args, MODEL_SHAPES[args.model])
 
 
-# Fobolorn beside gpt-oss (the framework's other mixture of experts with plain attention in every layer), both with bf16
-# weights: same width, heads, experts and layers; gpt-oss gets one routed expert more in place of the shared one, and a window
-# that never bites.  "uneven" has key and value heads of different sizes, beside gpt-oss heads of the larger size.
-DESIGN_SIZES = {
-    "2048x8": (dict(n_layers=8, width=2048, heads=16, kv_heads=4, dim=128, vdim=128, ff=1024, shared_ff=1024, experts=32, top=4, vocab=32000),
-               dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, expert_ffn=1024, n_experts=33, top_k=5, vocab=32000)),
-    "2880x6": (dict(n_layers=6, width=2880, heads=64, kv_heads=8, dim=64, vdim=64, ff=2880, shared_ff=2880, experts=32, top=4, vocab=32000),
-               dict(n_layers=6, hidden=2880, n_heads=64, n_kv_heads=8, head_dim=64, expert_ffn=2880, n_experts=33, top_k=5, vocab=32000)),
-    "uneven": (dict(n_layers=8, width=2048, heads=16, kv_heads=4, dim=96, vdim=128, ff=1024, shared_ff=2048, experts=32, top=4, vocab=32000),
-               dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, expert_ffn=1024, n_experts=34, top_k=6, vocab=32000)),
+# Designs beside the closest other model, both with bf16 weights at equal sizes: design -> (that model, sizes).
+# Fobolorn beside gpt-oss (the framework's other mixture of experts with plain attention in every layer): gpt-oss gets one
+# routed expert more in place of the shared one, and a window that never bites; "uneven" has key and value heads of different
+# sizes, beside gpt-oss heads of the larger size.
+# Sogulix beside dense Qwen3.5 (the other hybrid of a delta rule and attention): as many heads of the same size in the
+# recurrent layers, one attention layer in four; "looped" runs its first four layers twice, beside as many layers as it runs.
+_Q35 = dict(n_experts=0, interval=4, vocab=32000, context=16384)
+DESIGNS = {
+    "fobolorn": ("gpt-oss", {
+        "2048x8": (dict(n_layers=8, width=2048, heads=16, kv_heads=4, dim=128, vdim=128, ff=1024, shared_ff=1024, experts=32, top=4, vocab=32000),
+                   dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, expert_ffn=1024, n_experts=33, top_k=5, vocab=32000)),
+        "2880x6": (dict(n_layers=6, width=2880, heads=64, kv_heads=8, dim=64, vdim=64, ff=2880, shared_ff=2880, experts=32, top=4, vocab=32000),
+                   dict(n_layers=6, hidden=2880, n_heads=64, n_kv_heads=8, head_dim=64, expert_ffn=2880, n_experts=33, top_k=5, vocab=32000)),
+        "uneven": (dict(n_layers=8, width=2048, heads=16, kv_heads=4, dim=96, vdim=128, ff=1024, shared_ff=2048, experts=32, top=4, vocab=32000),
+                   dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, expert_ffn=1024, n_experts=34, top_k=6, vocab=32000)),
+    }),
+    "sogulix": ("qwen3.5", {
+        "2048x8": (dict(layers="gggl" * 2, width=2048, heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=512, window=1 << 20,
+                        delta_heads=16, delta_dim=128, decay_rank=64, ff=6144, vocab=32000),
+                   dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, rope_dims=64, hk=16, hv=16, dk=128, dv=128, ffn=6144, **_Q35)),
+        "4096x4": (dict(layers="gggl", width=4096, heads=32, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, window=4096,
+                        delta_heads=64, delta_dim=64, decay_rank=96, ff=12288, vocab=32000),
+                   dict(n_layers=4, hidden=4096, n_heads=32, n_kv_heads=8, head_dim=128, rope_dims=64, hk=64, hv=64, dk=64, dv=64, ffn=12288, **_Q35)),
+        "looped": (dict(layers="gggl" * 2, width=1536, heads=12, dim=64, rot_dim=32, vdim=64, q_rank=384, kv_rank=256, window=1 << 20, loop=(0, 4, 2),
+                        delta_heads=24, delta_dim=64, decay_rank=48, ff=4096, vocab=32000),
+                   dict(n_layers=12, hidden=1536, n_heads=12, n_kv_heads=4, head_dim=64, rope_dims=32, hk=24, hv=24, dk=64, dv=64, ffn=4096, **_Q35)),
+    }),
 }
+
+
+def write_design(name: str, path: str, sizes: dict) -> str:
+    """The synthetic model ``name`` of these sizes at ``path`` (a folder, or a GGUF file of that stem); returns where it is."""
+    from tensorsharp_b200.models import synth
+    if name in ("fobolorn", "sogulix"):
+        getattr(synth, f"write_{name}")(path, seed=0, **sizes)
+        return path
+    path += ".gguf"
+    if name == "gpt-oss":
+        synth.write_gptoss(path, seed=0, expert_scheme="BF16", window=1 << 20, **sizes)
+    else:
+        synth.write_qwen35(path, seed=0, scheme="BF16", **sizes)
+    return path
 
 
 def kernel_table(run, repeats: int = 3):
@@ -532,7 +563,6 @@ def run_design(args) -> None:
     import shutil
 
     import torch
-    from tensorsharp_b200.models import synth
     from tensorsharp_b200.models.base import ModelBase
     from tensorsharp_b200.ops import functional as F
     from tensorsharp_b200.ops import kernels
@@ -551,16 +581,12 @@ def run_design(args) -> None:
         torch.cuda.synchronize()
         return e0.elapsed_time(e1) / n
     os.makedirs(args.cache_dir, exist_ok=True)
-    for size, (ours, closest) in DESIGN_SIZES.items():
+    other, sizes = DESIGNS[args.design]
+    for size, pair in sizes.items():
         if args.design_size not in (None, size):
             continue
-        for name in ("fobolorn", "gpt-oss"):
-            path = os.path.join(args.cache_dir, f"design-{name}-{size}")
-            if name == "fobolorn":
-                synth.write_fobolorn(path, seed=0, **ours)
-            else:
-                path += ".gguf"
-                synth.write_gptoss(path, seed=0, expert_scheme="BF16", window=1 << 20, **closest)
+        for name, what in zip((args.design, other), pair):
+            path = write_design(name, os.path.join(args.cache_dir, f"design-{name}-{size}"), what)
             model = ModelBase.create(path, dev, max_context=8192 + 64, max_seqs=18, kv_pages=16 * (2048 + 2 * K + 2 * W + 128) // 64 + 160)
             res = {"design": name, "size": size, "layers": len(getattr(model, "runs", model.layers)), "dtype": "bf16", "data": "synthetic",
                    "l2": "every step reads more weight bytes than L2 holds"}
@@ -571,9 +597,9 @@ def run_design(args) -> None:
                 ids = torch.randint(0, model.cfg.vocab, (P,), generator=g).tolist()
 
                 def prefill():
-                    s = model.kv.new_seq()
+                    s = model.new_sequence()
                     out = model.forward_batch(model.kv.build_batch([s], [ids]))
-                    model.kv.free_seq(s)
+                    model.free_sequence(s)
                     return out
                 for _ in range(W):
                     prefill()
@@ -581,7 +607,7 @@ def run_design(args) -> None:
                 if args.design_kernels:
                     tables.append((f"{size} {name} prefill {P}", kernel_table(prefill)))
             for B in (1, 16):
-                seqs = [model.kv.new_seq() for _ in range(B)]
+                seqs = [model.new_sequence() for _ in range(B)]
                 first = []
                 for s in seqs:
                     ids = torch.randint(0, model.cfg.vocab, (2048,), generator=g).tolist()
@@ -597,7 +623,7 @@ def run_design(args) -> None:
                     tables.append((f"{size} {name} decode batch {B}, context 2048", kernel_table(dg.step)))
                 dg.graph = None
                 for s in seqs:
-                    model.kv.free_seq(s)
+                    model.free_sequence(s)
             res["clocks"] = clocks.stop()
             res["kernel_status"] = int(kernels.gemm_status(dev).item())
             print(json.dumps(res), flush=True)

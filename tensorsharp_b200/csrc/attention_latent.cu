@@ -154,15 +154,15 @@ extern "C" int tsb_latent_rotate(const LatentArgs* args, void* stream) {
 template <typename TW, int TT>
 __global__ void __launch_bounds__(256) latent_absorb_kernel(LatentArgs a) {
     extern __shared__ __align__(16) float sm[];
-    float* sq = sm;                          // [TT][Dk]
+    float* sq = sm;                          // [Dk][TT]
     float* sp = sm + TT * a.Dk;              // [8][TT][64]
     const int h = blockIdx.y, r0 = blockIdx.x * 64, t0 = blockIdx.z * TT, tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
     const int nt = min(TT, a.T - t0);
     pdl_wait();
     pdl_trigger();
     for (int i = tid; i < TT * a.Dk; i += 256) {
-        const int m = i / a.Dk, d = i % a.Dk;
-        sq[i] = m < nt ? la_ld(a.q, ((long)(t0 + m) * a.H + h) * a.Dk + d, a.q_f32) : 0.f;
+        const int m = i / a.Dk, d = i - m * a.Dk;
+        sq[d * TT + m] = m < nt ? la_ld(a.q, ((long)(t0 + m) * a.H + h) * a.Dk + d, a.q_f32) : 0.f;
     }
     __syncthreads();
     const int r = r0 + 2 * lane;
@@ -171,20 +171,25 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(LatentArgs a) {
     for (int m = 0; m < TT; ++m) acc[m][0] = acc[m][1] = 0.f;
     if (r < a.Rp) {                          // Rp is even, columns R .. Rp - 1 are zero
         const TW* wp = reinterpret_cast<const TW*>(a.wuk) + (long)h * a.dim * a.Rp + r;
-#pragma unroll 8
-        for (int d = w; d < a.dim; d += 8) {
-            float w0, w1;
-            if (sizeof(TW) == 2) {
-                const float2 v = __bfloat1622float2(*reinterpret_cast<const bf162*>(wp + (long)d * a.Rp));
-                w0 = v.x; w1 = v.y;
-            } else {
-                const float2 v = *reinterpret_cast<const float2*>(wp + (long)d * a.Rp);
-                w0 = v.x; w1 = v.y;
+        for (int d0 = w; d0 < a.dim; d0 += 64) {         // eight rows of the map in flight per warp
+            float2 wv[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int d = d0 + 8 * i;
+                wv[i] = make_float2(0.f, 0.f);
+                if (d < a.dim) {
+                    if (sizeof(TW) == 2) wv[i] = __bfloat1622float2(*reinterpret_cast<const bf162*>(wp + (long)d * a.Rp));
+                    else wv[i] = *reinterpret_cast<const float2*>(wp + (long)d * a.Rp);
+                }
             }
 #pragma unroll
-            for (int m = 0; m < TT; ++m) {
-                acc[m][0] = fmaf(w0, sq[m * a.Dk + d], acc[m][0]);
-                acc[m][1] = fmaf(w1, sq[m * a.Dk + d], acc[m][1]);
+            for (int i = 0; i < 8; ++i) {
+                const float* x = sq + min(d0 + 8 * i, a.dim - 1) * TT;
+#pragma unroll
+                for (int m = 0; m < TT; ++m) {
+                    acc[m][0] = fmaf(wv[i].x, x[m], acc[m][0]);
+                    acc[m][1] = fmaf(wv[i].y, x[m], acc[m][1]);
+                }
             }
         }
     }
@@ -202,7 +207,7 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(LatentArgs a) {
         } else if (rr < a.R + a.rot) {
             const int e = rr - a.R, pair = e < half ? e : e - half;
             const float2 cs = a.cs[(long)t * half + pair];
-            const float x0 = sq[m * a.Dk + a.dim + pair], x1 = sq[m * a.Dk + a.dim + half + pair];
+            const float x0 = sq[(a.dim + pair) * TT + m], x1 = sq[(a.dim + half + pair) * TT + m];
             v = e < half ? x0 * cs.x - x1 * cs.y : x1 * cs.x + x0 * cs.y;
         }
         la_st(a.qa, ((long)t * a.H + h) * a.Lp + rr, a.f32, v);
@@ -416,6 +421,7 @@ extern "C" int tsb_latent_decode(const LatentArgs* args, void* stream) {
 template <typename TW>
 __global__ void __launch_bounds__(256) latent_out_kernel(LatentArgs a, int rows) {
     extern __shared__ __align__(16) float sm[];          // [Rp]
+    __shared__ float cw[64];
     const int e0 = blockIdx.x * rows, e1 = min(a.Dv, e0 + rows), h = blockIdx.y, t = blockIdx.z;
     const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
     pdl_wait();
@@ -425,17 +431,25 @@ __global__ void __launch_bounds__(256) latent_out_kernel(LatentArgs a, int rows)
         for (int r = tid; r < a.Rp; r += 256) sm[r] = r < a.R ? a.part_o[th * a.Ro + r] : 0.f;
     } else {
         const float* ml = a.part_ml + th * a.splits * 2;
-        float m = a.sinks ? a.sinks[h] : -INFINITY;
-        for (int i = 0; i < a.splits; ++i) m = fmaxf(m, ml[2 * i]);
-        float l = a.sinks ? expf(a.sinks[h] - m) : 0.f;
-        for (int i = 0; i < a.splits; ++i) l += ml[2 * i] == -INFINITY ? 0.f : ml[2 * i + 1] * expf(ml[2 * i] - m);
-        const float inv = 1.f / l;
+        if (w == 0) {                                    // the splits' weights, at most 64
+            const float s0 = a.sinks ? a.sinks[h] : -INFINITY;
+            const float m0 = lane < a.splits ? ml[2 * lane] : -INFINITY, m1 = lane + 32 < a.splits ? ml[2 * lane + 64] : -INFINITY;
+            const float l0 = lane < a.splits ? ml[2 * lane + 1] : 0.f, l1 = lane + 32 < a.splits ? ml[2 * lane + 65] : 0.f;
+            const float m = fmaxf(s0, warp_max(fmaxf(m0, m1)));
+            const float c0 = m0 == -INFINITY ? 0.f : expf(m0 - m), c1 = m1 == -INFINITY ? 0.f : expf(m1 - m);
+            const float inv = 1.f / (warp_sum(l0 * c0 + l1 * c1) + (a.sinks ? expf(s0 - m) : 0.f));
+            cw[lane] = c0 * inv;
+            cw[lane + 32] = c1 * inv;
+        }
+        __syncthreads();
+        const float* po = a.part_o + th * a.splits * a.Ro;
         for (int r = tid; r < a.Rp; r += 256) {
             float v = 0.f;
-            if (r < a.R)
-                for (int i = 0; i < a.splits; ++i)
-                    if (ml[2 * i] != -INFINITY) v = fmaf(a.part_o[(th * a.splits + i) * a.Ro + r], expf(ml[2 * i] - m), v);
-            sm[r] = v * inv;
+            if (r < a.R) {
+#pragma unroll 8
+                for (int i = 0; i < a.splits; ++i) v = fmaf(po[(long)i * a.Ro + r], cw[i], v);      // an empty split holds zeros
+            }
+            sm[r] = v;
         }
     }
     __syncthreads();

@@ -732,7 +732,7 @@ def latent_out(part_o: torch.Tensor, part_ml: Optional[torch.Tensor], s, wuv: to
 class GdrArgs(C.Structure):
     _fields_ = [("y", _vp), ("y_s", C.c_long), ("y_f32", C.c_int), ("z", _vp), ("z_s", C.c_long), ("w2", _vp), ("w2_f32", C.c_int),
                 ("w0", _vp), ("ab", _vp), ("norm_w", _vp), ("state", _vp), ("state_s", C.c_long), ("cu_q", _vp), ("seq_slots", _vp),
-                ("pack", _vp), ("core", _vp), ("out", _vp), ("out_s", C.c_long), ("out_f32", C.c_int),
+                ("pack", _vp), ("link", _vp), ("core", _vp), ("out", _vp), ("out_s", C.c_long), ("out_f32", C.c_int),
                 ("T", C.c_int), ("B", C.c_int), ("H", C.c_int), ("D", C.c_int), ("n", C.c_int), ("rank", C.c_int), ("eps", C.c_float)]
 
 
@@ -761,15 +761,17 @@ def general_delta_short(y, w2: torch.Tensor, w0, ab, norm_w, state, cu_q, seq_sl
     return out
 
 
-def general_delta_prompt(y, z: torch.Tensor, w0, ab, norm_w, state, cu_q, seq_slots, *, H, D, n, eps, out_dtype, warps: int = 4) -> torch.Tensor:
-    """Prompts: per-token vectors, recurrence, norm and gate in three kernels; ``z`` f32 [T, H * D] is the decay's projection."""
+def general_delta_prompt(y, z: torch.Tensor, w0, ab, norm_w, state, cu_q, seq_slots, *, H, D, n, eps, out_dtype, wide: bool = True) -> torch.Tensor:
+    """Prompts: per-token vectors, recurrence, norm and gate in three kernels; ``z`` f32 [T, H * D] is the decay's projection.
+    ``wide``: twice the value channels per warp."""
     T = y.shape[0]
     assert z.dtype == torch.float32 and z.shape == (T, H * D) and z.stride(1) == 1
     a, out = _gdr_args(y, w0, ab, norm_w, state, cu_q, seq_slots, H=H, D=D, n=n, rank=0, eps=eps, out_dtype=out_dtype)
-    pack = torch.empty((T, H, 5, D), dtype=torch.float32, device=y.device)
+    pack = torch.empty((T + 1, H, 5, D), dtype=torch.float32, device=y.device)
     core = torch.empty((T, H, D), dtype=torch.float32, device=y.device)
-    a.z, a.z_s, a.pack, a.core = _p(z), z.stride(0), _p(pack), _p(core)
-    native.check(_lib().tsb_general_delta_prompt(C.byref(a), C.c_int(warps), _stream()), "general_delta_prompt")
+    link = torch.empty((T + 1, H, 4), dtype=torch.float32, device=y.device)
+    a.z, a.z_s, a.pack, a.link, a.core = _p(z), z.stride(0), _p(pack), _p(link), _p(core)
+    native.check(_lib().tsb_general_delta_prompt(C.byref(a), C.c_int(wide), _stream()), "general_delta_prompt")
     _count(3)
     return out
 

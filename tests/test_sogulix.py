@@ -295,7 +295,7 @@ def test_delta_rule_in_portions(place, H, n, rank):
             assert (batch.max_q_len < F.GENERAL_DELTA_SCAN_MIN) == (p in (1, 4))
             y = torch.cat([torch.cat([heads(x[b][k][lo:hi]) for k in names] +
                                      [torch.nn.functional.pad(low[b][lo:hi], (0, rp - rank))], 1) for b, lo, hi in part])
-            y = torch.nn.functional.pad(y, (0, 3)).to(dev)[:, :-3]                # a row stride of its own
+            y = torch.nn.functional.pad(y, (0, 4)).to(dev)[:, :-4]                # a row stride of its own
             out = F.general_delta(y, w2d, *vecs, state, batch, H=H, D=D, n=n, rank=rank, eps=eps, dtype=dtype(place))
             got = out.double().cpu().view(-1, H, D)
             ref = torch.cat([want[b][lo:hi] for b, lo, hi in part]).view(-1, H, n)
