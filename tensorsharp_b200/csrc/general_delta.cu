@@ -17,43 +17,9 @@
 //                          memory by cp.async; gdr_finish_kernel: norm and gate
 #include "attn_mma.cuh"
 #include "common.cuh"
-
-struct GdrArgs {
-    const void* y; long y_s; int y_f32;      // rows [r | k | v | a' | g | t]: five parts of H * D, then the decay's low rank part
-    const float* z; long z_s;                // prompts: the decay's projection [T, H * D] without w0
-    const void* w2; int w2_f32;              // short steps: [H * D, rank], z = w2 tanh(t)
-    const float* w0; const float* ab; const float* norm_w;      // [H * D]
-    float* state; long state_s;              // slot stride
-    const int* cu_q; const long* seq_slots;
-    float* pack;                             // [T + 1, H, 5, D]: u | w | a | r | v * |k|; record T changes nothing
-    float* link;                             // [T + 1, H, 4]: u' . (a u) and u' . u with the next token's key u'
-    float* core;                             // [T, H, D]
-    void* out; long out_s; int out_f32;      // [T, H * D]
-    int T, B, H, D, n, rank;
-    float eps;
-};
+#include "general_delta.cuh"
 
 namespace {
-constexpr float KEY_EPS = 1e-6f;
-
-__device__ __forceinline__ float gd_ld(const void* p, long i, int f32) {
-    return f32 ? reinterpret_cast<const float*>(p)[i] : bf2f(reinterpret_cast<const bf16*>(p)[i]);
-}
-__device__ __forceinline__ float4 gd_ld4(const void* p, long i, int f32) {
-    if (f32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + i);
-    const uint2 r = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(p) + i);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const bf162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const bf162*>(&r.y));
-    return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ void gd_st(void* p, long i, int f32, float v) {
-    if (f32) reinterpret_cast<float*>(p)[i] = v;
-    else reinterpret_cast<bf16*>(p)[i] = f2bf(v);
-}
-__device__ __forceinline__ float gd_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float gd_decay(float z) {
-    constexpr float C = 0.60653065971263342f;            // e^(-1/2)
-    return expf(-C * gd_sigmoid(z));
-}
 __device__ __forceinline__ float sum8(float v) {
     v += __shfl_xor_sync(0xffffffffu, v, 1);
     v += __shfl_xor_sync(0xffffffffu, v, 2);
@@ -138,7 +104,7 @@ __global__ void __launch_bounds__(gdr_short_threads<KPL>()) gdr_short_kernel(Gdr
         float kk = 0.f;
 #pragma unroll
         for (int i = 0; i < D / 32; ++i) { const float v = sk[lane + 32 * i]; kk = fmaf(v, v, kk); }
-        const float inv = 1.f / sqrtf(warp_sum(kk) + KEY_EPS);
+        const float inv = 1.f / sqrtf(warp_sum(kk) + GDR_KEY_EPS);
         __syncthreads();
 #pragma unroll 1
         for (int pass = 0; pass < PASSES; ++pass) {
@@ -232,7 +198,7 @@ __global__ void __launch_bounds__(256) gdr_prep_kernel(GdrArgs p) {
         }
 #pragma unroll
         for (int i = 0; i < 4 * NV; ++i) kk = fmaf(k[i], k[i], kk);
-        const float len = sqrtf(warp_sum(kk) + KEY_EPS), inv = 1.f / len;
+        const float len = sqrtf(warp_sum(kk) + GDR_KEY_EPS), inv = 1.f / len;
 #pragma unroll
         for (int i = 0; i < 4 * NV; ++i) k[i] *= inv;
         if (t > t0) {
@@ -244,6 +210,7 @@ __global__ void __launch_bounds__(256) gdr_prep_kernel(GdrArgs p) {
             if (lane == 0) *reinterpret_cast<float4*>(p.link + ((long)(t - 1) * p.H + h) * 4) = make_float4(g, f, 0.f, 0.f);
         }
         if (t == t0 + PREP_T) return;
+        if (t == p.T - 1 && lane == 0) *reinterpret_cast<float4*>(p.link + ((long)t * p.H + h) * 4) = make_float4(0.f, 0.f, 0.f, 0.f);
         float* dst = p.pack + ((long)t * p.H + h) * 5 * D;
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
@@ -528,13 +495,6 @@ __global__ void __launch_bounds__(256) gdr_tanh_kernel(const void* y, long y_s, 
     gd_st(out, i, out_f32, c < cols ? tanhf(gd_ld(y, (long)t * y_s + off + c, y_f32)) : 0.f);
 }
 
-static int gdr_check(const GdrArgs& a, const char* what) {
-    TSB_CHECK_ARG(a.H > 0 && a.D >= 32 && a.D <= 256 && a.D % 32 == 0 && a.n > 0 && a.n <= a.D && a.rank >= 0 && a.rank <= 4096,
-                  "%s: heads %d of %d (true size %d), rank %d", what, a.H, a.D, a.n, a.rank);
-    TSB_CHECK_ARG(a.B <= 65535 && a.H <= 65535 && a.state_s % 4 == 0, "%s: %d sequences, %d heads", what, a.B, a.H);
-    return TSB_OK;
-}
-
 #define GDR_SIZES(X) X(4) X(8) X(12) X(16) X(20) X(24) X(28) X(32)
 
 extern "C" int tsb_general_delta_short(const GdrArgs* args, void* stream) {
@@ -561,7 +521,17 @@ static int launch_scan(const GdrArgs& a, cudaStream_t s) {
         TSB_CHECK_CUDA(cudaFuncSetAttribute(gdr_scan_kernel<D, G, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Z::smem));
         configured = true;
     }
-    TSB_CHECK_CUDA(tsb_launch(gdr_scan_kernel<D, G, C>, dim3(D / Z::COLS, a.H, a.B), dim3(128), Z::smem, s, a));
+    // not as a dependent launch: its long-lived CTAs would take the first places that the other kernel's CTAs leave, several
+    // on one SM with others idle
+    gdr_scan_kernel<D, G, C><<<dim3(D / Z::COLS, a.H, a.B), 128, Z::smem, s>>>(a);
+    return TSB_OK;
+}
+
+int tsb_gdr_finish_launch(const GdrArgs& a, cudaStream_t s) {
+    const dim3 rows((unsigned)(((long)a.T * a.H + 7) / 8));
+    if (a.D <= 128) TSB_CHECK_CUDA(tsb_launch(gdr_finish_kernel<1>, rows, dim3(256), 0, s, a));
+    else TSB_CHECK_CUDA(tsb_launch(gdr_finish_kernel<2>, rows, dim3(256), 0, s, a));
+    TSB_CHECK_LAUNCH();
     return TSB_OK;
 }
 
@@ -575,7 +545,7 @@ extern "C" int tsb_general_delta_prompt(const GdrArgs* args, int wide, void* str
     if (a.B == 0 || a.T == 0) return TSB_OK;
     cudaStream_t s = (cudaStream_t)stream;
     const long groups = ((long)a.T + PREP_T - 1) / PREP_T + 1;
-    const dim3 prep((unsigned)((groups * a.H + 7) / 8)), rows((unsigned)(((long)a.T * a.H + 7) / 8));
+    const dim3 prep((unsigned)((groups * a.H + 7) / 8));
     if (a.D <= 128) TSB_CHECK_CUDA(tsb_launch(gdr_prep_kernel<1>, prep, dim3(256), 0, s, a));
     else TSB_CHECK_CUDA(tsb_launch(gdr_prep_kernel<2>, prep, dim3(256), 0, s, a));
     switch (a.D) {
@@ -584,10 +554,7 @@ extern "C" int tsb_general_delta_prompt(const GdrArgs* args, int wide, void* str
 #undef X
     }
     if (rc != TSB_OK) return rc;
-    if (a.D <= 128) TSB_CHECK_CUDA(tsb_launch(gdr_finish_kernel<1>, rows, dim3(256), 0, s, a));
-    else TSB_CHECK_CUDA(tsb_launch(gdr_finish_kernel<2>, rows, dim3(256), 0, s, a));
-    TSB_CHECK_LAUNCH();
-    return TSB_OK;
+    return tsb_gdr_finish_launch(a, s);
 }
 
 extern "C" int tsb_tanh_rows(const void* y, long y_s, int y_f32, long off, int T, int cols, int ld, void* out, int out_f32, void* stream) {

@@ -43,7 +43,7 @@ class DeltaSpec:
 class SogulixModel(FolderModel):
     supports_kv_truncation = False           # recurrent state and the token shift's previous row
     graphs_with_state = True
-    native_sources = ("error.cpp", "elementwise.cu", "parallel_norm.cu", "general_delta.cu", "attention_latent.cu", "float32.cu", "attention.cu",
+    native_sources = ("error.cpp", "elementwise.cu", "parallel_norm.cu", "general_delta.cu", "general_delta_chunk.cu", "attention_latent.cu", "float32.cu", "attention.cu",
                       "attention_vd.cu", "attention_decode_mma.cu", "gemm_tcgen05.cu", "gemv.cu", "gemv_bf16.cu", "gemv_mma.cu", "gemv_stream.cu",
                       "moe.cu", "sampler.cu")
 

@@ -1079,7 +1079,9 @@ def general_delta(y: torch.Tensor, w2: QuantWeight, w0: torch.Tensor, ab: torch.
             return kk.general_delta_short(y, _weight_matrix(w2), w0, ab, norm_w, state, batch.cu_q, batch.seq_slots, rank=w2.K, **kw)
         t = kk.tanh_rows(y, 5 * HD, rank, w2.K, dtype)
         z = linear(Act(t), w2, out_dtype=torch.float32)
-        return kk.general_delta_prompt(y, z, w0, ab, norm_w, state, batch.cu_q, batch.seq_slots, wide=True, **kw)
+        if dtype == torch.bfloat16:
+            return kk.general_delta_chunk(y, z, w0, ab, norm_w, state, batch.cu_q, batch.seq_slots, max_q=batch.max_q_len, **kw)
+        return kk.general_delta_prompt(y, z, w0, ab, norm_w, state, batch.cu_q, batch.seq_slots, wide=batch.B * HD >= 2048, **kw)
     T, y = y.shape[0], y.float()
     z = torch.tanh(y[:, 5 * HD:5 * HD + rank]) @ w2.dequantize()[:, :rank].t() + w0
     r, k, v, a = (y[:, i * HD:(i + 1) * HD].view(T, H, D) for i in range(4))

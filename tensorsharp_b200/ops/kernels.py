@@ -776,6 +776,22 @@ def general_delta_prompt(y, z: torch.Tensor, w0, ab, norm_w, state, cu_q, seq_sl
     return out
 
 
+def general_delta_chunk(y, z: torch.Tensor, w0, ab, norm_w, state, cu_q, seq_slots, *, H, D, n, eps, max_q: int, out_dtype) -> torch.Tensor:
+    """:func:`general_delta_prompt` in chunks of eight tokens on the tensor cores (csrc/general_delta_chunk.cu: split tf32
+    operands, f32 accuracy); ``max_q``: the longest portion of the batch."""
+    T = y.shape[0]
+    assert z.dtype == torch.float32 and z.shape == (T, H * D) and z.stride(1) == 1
+    a, out = _gdr_args(y, w0, ab, norm_w, state, cu_q, seq_slots, H=H, D=D, n=n, rank=0, eps=eps, out_dtype=out_dtype)
+    lib = _lib()
+    lib.tsb_general_delta_chunk_floats.restype = C.c_long
+    pack = torch.empty((T // 8 + a.B + 1) * H * int(lib.tsb_general_delta_chunk_floats(C.c_int(D))), dtype=torch.float32, device=y.device)
+    core = torch.empty((T, H, D), dtype=torch.float32, device=y.device)
+    a.z, a.z_s, a.pack, a.core = _p(z), z.stride(0), _p(pack), _p(core)
+    native.check(lib.tsb_general_delta_chunk(C.byref(a), C.c_int(max_q), _stream()), "general_delta_chunk")
+    _count(3)
+    return out
+
+
 def tanh_rows(y: torch.Tensor, off: int, cols: int, ld: int, out_dtype) -> torch.Tensor:
     """tanh of ``cols`` columns of y from ``off`` on as dense rows [T, ld], zero past the columns."""
     assert y.stride(1) == 1 and off + cols <= y.shape[1]

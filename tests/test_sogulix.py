@@ -252,6 +252,47 @@ def test_latent_attention_with_keys_that_stand_out(place, H, dim, rot, vdim, ran
 DELTA = [(3, 20, 5), (2, 64, 16), (5, 96, 33), (4, 128, 64), (1, 150, 3), (2, 256, 8), (40, 32, 8)]
 
 
+@gpu
+@pytest.mark.parametrize("H,n", [(h, n) for h, n, _ in DELTA])
+def test_delta_rule_prompt_kernels_keep_32_bits(H, n):
+    """Both prompt paths, the tensor-core one included, against the oracle with 32-bit outputs: unequal sequences with full,
+    short and one-token chunks, and the state they leave."""
+    from tensorsharp_b200.ops import kernels as K
+    D, eps = (n + 31) // 32 * 32, 1e-5
+    g = torch.Generator().manual_seed(n)
+    cu, T = [0, 1, 44, 52, 68, 75], 75
+    x = {k: torch.randn(T, H, n, generator=g) for k in "rkvagz"}
+    x["z"] = x["z"] * 3 - 2
+    x["z"][:, :, ::2] -= 14                                                # half of the channels forget next to nothing
+    s0 = torch.randn(6, H, n, n, generator=g)
+    w0, ab, on = (torch.randn(H, n, generator=g) for _ in range(3))
+
+    def pad(v):
+        return torch.nn.functional.pad(v, (0, D - n)).reshape(*v.shape[:-2], H * D).contiguous().cuda()
+    y, z = torch.cat([pad(x[k]) for k in "rkvag"], 1), pad(x["z"])
+    state = torch.zeros(6, H, D, D)
+    state[:, :, :n, :n] = s0
+    slots = torch.tensor([4, 0, 5, 2, 1])
+    outs, states = [], []
+    for kind in ("scan", "wide", "chunk"):
+        st = state.cuda()
+        args = (y, z, pad(w0), pad(ab), pad(on), st, torch.tensor(cu, dtype=torch.int32).cuda(), slots.cuda())
+        kw = dict(H=H, D=D, n=n, eps=eps, out_dtype=torch.float32)
+        out = K.general_delta_chunk(*args, max_q=43, **kw) if kind == "chunk" else K.general_delta_prompt(*args, wide=kind == "wide", **kw)
+        outs.append(out.cpu().double().view(T, H, D))
+        states.append(st.cpu().double())
+    x = {k: v.double() for k, v in x.items()}
+    decay = torch.exp(-torch.exp(torch.tensor(-0.5).double()) * O.sigmoid(x["z"] + w0))
+    for b, (lo, hi) in enumerate(zip(cu, cu[1:])):
+        o, S = O.delta_rule(x["r"][lo:hi], x["k"][lo:hi], x["v"][lo:hi], decay[lo:hi], O.sigmoid(x["a"][lo:hi] + ab), s0[slots[b]].double().transpose(1, 2))
+        want = O.rms(o, eps) * on * O.sigmoid(x["g"][lo:hi])
+        for out, st in zip(outs, states):
+            assert torch.allclose(out[lo:hi, :, :n], want, rtol=3e-5, atol=3e-5), (b, (out[lo:hi, :, :n] - want).abs().max())
+            assert torch.allclose(st[slots[b], :, :n, :n].transpose(1, 2), S, rtol=3e-5, atol=3e-5)
+            assert not out[lo:hi, :, n:].any() and not st[slots[b], :, n:].any() and not st[slots[b], :, :, n:].any()
+    assert all(torch.equal(st[3], state[3].double()) for st in states)      # nobody's slot
+
+
 @pytest.mark.parametrize("place", PLACES)
 @pytest.mark.parametrize("H,n,rank", DELTA)
 def test_delta_rule_in_portions(place, H, n, rank):
