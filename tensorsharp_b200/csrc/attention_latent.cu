@@ -158,38 +158,38 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(LatentArgs a) {
     float* sp = sm + TT * a.Dk;              // [8][TT][64]
     const int h = blockIdx.y, r0 = blockIdx.x * 64, t0 = blockIdx.z * TT, tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
     const int nt = min(TT, a.T - t0);
+    const int r = r0 + 2 * lane;             // Rp is even, columns R .. Rp - 1 are zero
+    const TW* wp = reinterpret_cast<const TW*>(a.wuk) + (long)h * a.dim * a.Rp + r;
+    float2 wv[8];                            // eight rows of the map in flight per warp, the first ones before the queries are there
+    auto fetch = [&](int d0) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int d = d0 + 8 * i;
+            wv[i] = make_float2(0.f, 0.f);
+            if (d < a.dim && r < a.Rp) {
+                if (sizeof(TW) == 2) wv[i] = __bfloat1622float2(*reinterpret_cast<const bf162*>(wp + (long)d * a.Rp));
+                else wv[i] = *reinterpret_cast<const float2*>(wp + (long)d * a.Rp);
+            }
+        }
+    };
+    fetch(w);
     pdl_wait();
     pdl_trigger();
-    for (int i = tid; i < TT * a.Dk; i += 256) {
-        const int m = i / a.Dk, d = i - m * a.Dk;
-        sq[d * TT + m] = m < nt ? la_ld(a.q, ((long)(t0 + m) * a.H + h) * a.Dk + d, a.q_f32) : 0.f;
-    }
+    for (int m = 0; m < TT; ++m)
+        for (int d = tid; d < a.Dk; d += 256) sq[d * TT + m] = m < nt ? la_ld(a.q, ((long)(t0 + m) * a.H + h) * a.Dk + d, a.q_f32) : 0.f;
     __syncthreads();
-    const int r = r0 + 2 * lane;
     float acc[TT][2];
 #pragma unroll
     for (int m = 0; m < TT; ++m) acc[m][0] = acc[m][1] = 0.f;
-    if (r < a.Rp) {                          // Rp is even, columns R .. Rp - 1 are zero
-        const TW* wp = reinterpret_cast<const TW*>(a.wuk) + (long)h * a.dim * a.Rp + r;
-        for (int d0 = w; d0 < a.dim; d0 += 64) {         // eight rows of the map in flight per warp
-            float2 wv[8];
+    for (int d0 = w; d0 < a.dim; d0 += 64) {
+        if (d0 != w) fetch(d0);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) {
-                const int d = d0 + 8 * i;
-                wv[i] = make_float2(0.f, 0.f);
-                if (d < a.dim) {
-                    if (sizeof(TW) == 2) wv[i] = __bfloat1622float2(*reinterpret_cast<const bf162*>(wp + (long)d * a.Rp));
-                    else wv[i] = *reinterpret_cast<const float2*>(wp + (long)d * a.Rp);
-                }
-            }
+        for (int i = 0; i < 8; ++i) {
+            const float* x = sq + min(d0 + 8 * i, a.dim - 1) * TT;
 #pragma unroll
-            for (int i = 0; i < 8; ++i) {
-                const float* x = sq + min(d0 + 8 * i, a.dim - 1) * TT;
-#pragma unroll
-                for (int m = 0; m < TT; ++m) {
-                    acc[m][0] = fmaf(wv[i].x, x[m], acc[m][0]);
-                    acc[m][1] = fmaf(wv[i].y, x[m], acc[m][1]);
-                }
+            for (int m = 0; m < TT; ++m) {
+                acc[m][0] = fmaf(wv[i].x, x[m], acc[m][0]);
+                acc[m][1] = fmaf(wv[i].y, x[m], acc[m][1]);
             }
         }
     }
@@ -254,8 +254,8 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(LatentArgs a) {
     bf16* sK = sP + 16 * LDP;                           // [2][64][ld]
     const int split = blockIdx.x, h0 = blockIdx.y * 16, b = blockIdx.z, G = min(16, a.H - h0);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    pdl_wait();
-    pdl_trigger();
+    // The cached rows and the batch's metadata are not written by the kernel launched directly before (the one that makes
+    // qa), and all kernels before that one have ended: the first tile is on its way before the queries are there.
     const int len = a.kv_lens[b];
     const int lo = (a.window > 0 && len > a.window) ? len - a.window : 0;
     const int per = (((len - lo + a.splits - 1) / a.splits) + 31) & ~31;
@@ -276,8 +276,10 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(LatentArgs a) {
 #pragma unroll
     for (int i = 0; i < 2 * NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
+    if (s0 < s1) load_tile(s0, 0);
+    pdl_wait();
+    pdl_trigger();
     if (s0 < s1) {
-        load_tile(s0, 0);
         for (int i = tid; i < 16 * cl; i += 256) {
             const int r = i / cl, c = i % cl;
             uint4 v = make_uint4(0u, 0u, 0u, 0u);
@@ -295,24 +297,30 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(LatentArgs a) {
         }
         __syncthreads();
         const bf16* tK = sK + stage * KT * ld;
-        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        float s[4][4] = {};                              // four chains of products
         {
             const bf16* qrow = sQ + (lane & 15) * ld + ((lane >> 4) << 3);
             const bf16* krow = tK + (warp * 8 + (lane & 7)) * ld + ((lane >> 3) << 3);
-#pragma unroll 2
-            for (int kk = 0; kk < a.Lp; kk += 32) {      // Lp is a multiple of 32
+            auto step = [&](int kk, float* s0, float* s1) {
                 uint32_t q0[4], q1[4], kb[4];
                 ldsm_x4(q0, qrow + kk);
                 ldsm_x4(q1, qrow + kk + 16);
                 ldsm_x4(kb, krow + kk);
-                mma_bf16(s[0], q0, kb[0], kb[1]);
-                mma_bf16(s[1], q1, kb[2], kb[3]);
+                mma_bf16(s0, q0, kb[0], kb[1]);
+                mma_bf16(s1, q1, kb[2], kb[3]);
+            };
+            int kk = 0;                                  // Lp is a multiple of 32
+#pragma unroll 2
+            for (; kk + 64 <= a.Lp; kk += 64) {
+                step(kk, s[0], s[1]);
+                step(kk + 32, s[2], s[3]);
             }
+            if (kk < a.Lp) step(kk, s[0], s[1]);
         }
         const int key = base + warp * 8 + (lane & 3) * 2;
         float p[4], mx[2];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) p[e] = key + (e & 1) < s1 ? (s[0][e] + s[1][e]) * a.scale : -INFINITY;
+        for (int e = 0; e < 4; ++e) p[e] = key + (e & 1) < s1 ? ((s[0][e] + s[2][e]) + (s[1][e] + s[3][e])) * a.scale : -INFINITY;
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
             mx[r] = fmaxf(p[2 * r], p[2 * r + 1]);
@@ -415,15 +423,48 @@ extern "C" int tsb_latent_decode(const LatentArgs* args, void* stream) {
 }
 
 // ------------------------------------------------------------------------------------------
-// Merge of the splits (with the sink) and the value map.  Grid (parts of Dv, H, T), eight warps: the merged latent in shared
-// memory, one output row of W_uv per warp at a time.
+// Merge of the splits (with the sink) and the value map.  A cluster of CTAs per (head, token), eight warps each: every CTA
+// merges a share of the latent columns, hands them to the others through distributed shared memory, and then computes a
+// share of the output rows, one row of W_uv per warp at a time.
 // ------------------------------------------------------------------------------------------
+// *p of CTA `rank` of the cluster = v
+__device__ __forceinline__ void cluster_store(float* p, int rank, float v) {
+    uint32_t a;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"((uint32_t)__cvta_generic_to_shared(p)), "r"(rank));
+    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(a), "f"(v) : "memory");
+}
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+
+template <typename TW>
+__device__ __forceinline__ void la_row8(const TW* p, float (&v)[8]) {
+    if (sizeof(TW) == 2) {
+        const uint4 r = *reinterpret_cast<const uint4*>(p);
+        const uint32_t* x = reinterpret_cast<const uint32_t*>(&r);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            v[2 * c] = __uint_as_float(x[c] << 16);
+            v[2 * c + 1] = __uint_as_float(x[c] & 0xffff0000u);
+        }
+    } else {
+#pragma unroll
+        for (int c = 0; c < 8; ++c) v[c] = (float)p[c];
+    }
+}
+
 template <typename TW>
 __global__ void __launch_bounds__(256) latent_out_kernel(LatentArgs a, int rows) {
     extern __shared__ __align__(16) float sm[];          // [Rp]
-    __shared__ float cw[64];
-    const int e0 = blockIdx.x * rows, e1 = min(a.Dv, e0 + rows), h = blockIdx.y, t = blockIdx.z;
+    __shared__ float cw[64], share[256];
+    const int cs = gridDim.x, rank = blockIdx.x;         // the cluster spans the grid's x
+    const int e0 = rank * rows, e1 = min(a.Dv, e0 + rows), h = blockIdx.y, t = blockIdx.z;
     const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
+    if (cs > 1) cluster_arrive();
+    const TW* wuv = reinterpret_cast<const TW*>(a.wuv) + (long)h * a.Dv * a.Rp;
+    float first[2][8];                                   // this warp's first row, up to 512 columns of it
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+        if (e0 + w < e1 && lane * 8 + 256 * i < a.Rp) la_row8(wuv + (long)(e0 + w) * a.Rp + lane * 8 + 256 * i, first[i]);
     pdl_wait();
     pdl_trigger();
     const long th = (long)t * a.H + h;
@@ -442,40 +483,64 @@ __global__ void __launch_bounds__(256) latent_out_kernel(LatentArgs a, int rows)
             cw[lane + 32] = c1 * inv;
         }
         __syncthreads();
+        if (cs > 1) cluster_wait();                      // the other CTAs have started: their memory may be written
+        // this CTA's columns [c0, c1): G groups of threads share the splits of a column
         const float* po = a.part_o + th * a.splits * a.Ro;
-        for (int r = tid; r < a.Rp; r += 256) {
+        const int per = (((a.Rp + cs - 1) / cs) + 63) & ~63, c0 = min(a.Rp, rank * per), c1 = min(a.Rp, c0 + per);
+        const int G = per == 64 ? 4 : per == 128 ? 2 : 1, lanes = 256 / G, grp = tid / lanes;
+        for (int r = c0 + tid % lanes; r < c0 + per; r += lanes) {        // with G > 1 one turn for every thread
             float v = 0.f;
-            if (r < a.R) {
+            if (r < a.R && r < c1) {
 #pragma unroll 8
-                for (int i = 0; i < a.splits; ++i) v = fmaf(po[(long)i * a.Ro + r], cw[i], v);      // an empty split holds zeros
+                for (int i = grp; i < a.splits; i += G) v = fmaf(po[(long)i * a.Ro + r], cw[i], v);      // an empty split holds zeros
             }
-            sm[r] = v;
+            if (G > 1) {
+                share[tid] = v;
+                __syncthreads();
+                if (grp == 0)
+                    for (int i = 1; i < G; ++i) v += share[tid + i * lanes];
+            }
+            if (grp == 0 && r < c1)
+                for (int c = 0; c < cs; ++c) cluster_store(sm + r, c, v);
         }
     }
+    if (cs > 1) {
+        cluster_arrive();
+        cluster_wait();
+    }
     __syncthreads();
-    for (int e = e0 + w; e < e1; e += 8) {
-        const TW* wp = reinterpret_cast<const TW*>(a.wuv) + ((long)h * a.Dv + e) * a.Rp;
+    auto dot8 = [&](const float (&v)[8], int u, float acc) {
+        const float4 x0 = *reinterpret_cast<const float4*>(sm + u), x1 = *reinterpret_cast<const float4*>(sm + u + 4);
+        acc = fmaf(v[0], x0.x, acc); acc = fmaf(v[1], x0.y, acc); acc = fmaf(v[2], x0.z, acc); acc = fmaf(v[3], x0.w, acc);
+        acc = fmaf(v[4], x1.x, acc); acc = fmaf(v[5], x1.y, acc); acc = fmaf(v[6], x1.z, acc); return fmaf(v[7], x1.w, acc);
+    };
+    if (e0 + w < e1) {
         float acc = 0.f;
-        for (int u = lane * 8; u < a.Rp; u += 256) {     // Rp is a multiple of 8
-            float wv[8];
-            if (sizeof(TW) == 2) {
-                const uint4 v = *reinterpret_cast<const uint4*>(wp + u);
-                const uint32_t* x = reinterpret_cast<const uint32_t*>(&v);
 #pragma unroll
-                for (int c = 0; c < 4; ++c) {
-                    wv[2 * c] = __uint_as_float(x[c] << 16);
-                    wv[2 * c + 1] = __uint_as_float(x[c] & 0xffff0000u);
-                }
-            } else {
-#pragma unroll
-                for (int c = 0; c < 8; ++c) wv[c] = (float)wp[u + c];
-            }
-            const float4 x0 = *reinterpret_cast<const float4*>(sm + u), x1 = *reinterpret_cast<const float4*>(sm + u + 4);
-            acc = fmaf(wv[0], x0.x, acc); acc = fmaf(wv[1], x0.y, acc); acc = fmaf(wv[2], x0.z, acc); acc = fmaf(wv[3], x0.w, acc);
-            acc = fmaf(wv[4], x1.x, acc); acc = fmaf(wv[5], x1.y, acc); acc = fmaf(wv[6], x1.z, acc); acc = fmaf(wv[7], x1.w, acc);
+        for (int i = 0; i < 2; ++i)
+            if (lane * 8 + 256 * i < a.Rp) acc = dot8(first[i], lane * 8 + 256 * i, acc);
+        for (int u = lane * 8 + 512; u < a.Rp; u += 256) {
+            float v[8];
+            la_row8(wuv + (long)(e0 + w) * a.Rp + u, v);
+            acc = dot8(v, u, acc);
         }
         acc = warp_sum(acc);
-        if (lane == 0) la_st(a.out, th * a.Dv + e, a.f32, acc);
+        if (lane == 0) la_st(a.out, th * a.Dv + e0 + w, a.f32, acc);
+    }
+    for (int e = e0 + w + 8; e < e1; e += 32) {          // the others, four at a time
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int u = lane * 8; u < a.Rp; u += 256) {     // Rp is a multiple of 8
+            float v[4][8];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) la_row8(wuv + (long)min(e + 8 * j, e1 - 1) * a.Rp + u, v[j]);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[j] = dot8(v[j], u, acc[j]);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            acc[j] = warp_sum(acc[j]);
+            if (lane == 0 && e + 8 * j < e1) la_st(a.out, th * a.Dv + e + 8 * j, a.f32, acc[j]);
+        }
     }
 }
 
@@ -484,14 +549,25 @@ extern "C" int tsb_latent_out(const LatentArgs* args, void* stream) {
     TSB_CHECK_ARG(a.Rp % 8 == 0 && a.Rp >= a.R && a.Rp <= 4096 && a.Dv > 0 && a.T <= 65535 && a.H <= 65535, "latent_out: latent %d (%d), values %d, %d rows",
                   a.R, a.Rp, a.Dv, a.T);
     if (a.T == 0) return TSB_OK;
-    // output rows per CTA: all of a head's when there are heads and tokens enough for the SMs, else a share
-    int rows = a.Dv;
-    while (rows > 8 && (long)a.T * a.H * ((a.Dv + rows - 1) / rows) < 296) rows = (rows / 2 + 7) & ~7;
-    const dim3 grid((a.Dv + rows - 1) / rows, a.H, a.T);
-    cudaStream_t s = (cudaStream_t)stream;
-    const size_t smem = sizeof(float) * a.Rp;
-    if (a.w_f32) TSB_CHECK_CUDA(tsb_launch(latent_out_kernel<float>, grid, dim3(256), smem, s, a, rows));
-    else TSB_CHECK_CUDA(tsb_launch(latent_out_kernel<bf16>, grid, dim3(256), smem, s, a, rows));
+    // CTAs per (head, token): as many as keep all of them on the SMs together
+    int cs = 1;
+    while (cs < 8 && a.part_ml != nullptr && (long)a.T * a.H * cs * 2 <= 1184) cs *= 2;
+    const int rows = (((a.Dv + cs - 1) / cs) + 7) & ~7;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(cs, a.H, a.T);
+    cfg.blockDim = dim3(256);
+    cfg.dynamicSmemBytes = sizeof(float) * a.Rp;
+    cfg.stream = (cudaStream_t)stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = cs;
+    attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = tsb_pdl_enabled() ? 2 : 1;
+    if (a.w_f32) TSB_CHECK_CUDA(cudaLaunchKernelEx(&cfg, latent_out_kernel<float>, a, rows));
+    else TSB_CHECK_CUDA(cudaLaunchKernelEx(&cfg, latent_out_kernel<bf16>, a, rows));
     TSB_CHECK_LAUNCH();
     return TSB_OK;
 }

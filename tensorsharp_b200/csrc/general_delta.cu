@@ -71,8 +71,8 @@ __global__ void __launch_bounds__(gdr_short_threads<KPL>()) gdr_short_kernel(Gdr
     float* st = so + D;          // [rank] tanh of the low rank part
     const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, l8 = tid & 7, grp = tid >> 3;
     const long HD = (long)p.H * D, hc = (long)h * D;
-    pdl_wait();
-    pdl_trigger();
+    // The state and the batch's metadata are not written by the kernel launched directly before (the projection that makes
+    // y), and all kernels before that one have ended: the state is on its way while the projection still runs.
     const int q0 = p.cu_q[b], n = p.cu_q[b + 1] - q0;
     float* S = p.state + p.seq_slots[b] * p.state_s + hc * D + 4 * l8;
     float4 s[C][NF];
@@ -82,6 +82,8 @@ __global__ void __launch_bounds__(gdr_short_threads<KPL>()) gdr_short_kernel(Gdr
 #pragma unroll
             for (int i = 0; i < NF; ++i) s[j][i] = *reinterpret_cast<const float4*>(S + (long)(grp + j * GROUPS) * D + 32 * i);
     }
+    pdl_wait();
+    pdl_trigger();
     for (int t = q0; t < q0 + n; ++t) {
         const long row = (long)t * p.y_s;
         for (int i = tid; i < p.rank; i += NT) st[i] = tanhf(gd_ld(p.y, row + 5 * HD + i, p.y_f32));

@@ -58,8 +58,25 @@ __device__ __forceinline__ float4 pn_mul(float4 a, float r, float4 w) { return m
 
 // The new residual row in registers and the reciprocal of its root mean square.  `red`: 64 floats; two calls in a row use
 // its halves in turn (`flip`), so one barrier per call is enough.
+// The vectors that do not depend on earlier kernels.  With one float4 per thread (decode, narrow rows) they are loaded ahead
+// of the dependency wait; otherwise where they are used, for the registers' sake.
 template <int V>
-__device__ __forceinline__ float pn_row(const ParallelNormArgs& a, long row, float4 (&x)[V], float* red, int& flip) {
+struct PnVecs {
+    float4 s1, s2, w1, w2, sh;
+    __device__ __forceinline__ void load(const ParallelNormArgs& a) {
+        const int i = threadIdx.x;
+        if (V > 1 || i >= (a.D >> 2)) return;
+        if (a.y1 != nullptr) s1 = pn_ld4(a.s1, i);
+        if (a.y2 != nullptr) s2 = pn_ld4(a.s2, i);
+        if (a.w1 != nullptr) w1 = pn_ld4(a.w1, i);
+        if (a.w2 != nullptr) w2 = pn_ld4(a.w2, i);
+        if (a.shift != nullptr) sh = pn_ld4(a.shift, i);
+    }
+    static __device__ __forceinline__ float4 get(const float4& held, const float* p, int i) { return V == 1 ? held : pn_ld4(p, i); }
+};
+
+template <int V>
+__device__ __forceinline__ float pn_row(const ParallelNormArgs& a, const PnVecs<V>& c, long row, float4 (&x)[V], float* red, int& flip) {
     const int nvec = a.D >> 2, nt = blockDim.x;
     float q = 0.f;
 #pragma unroll
@@ -68,8 +85,8 @@ __device__ __forceinline__ float pn_row(const ParallelNormArgs& a, long row, flo
         x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (i < nvec) {
             x[j] = reinterpret_cast<const float4*>(a.h + row * a.D)[i];
-            if (a.y1 != nullptr) pn_axpy(x[j], pn_ld4(a.s1, i), pn_ld4_any(a.y1, row, a.D, i, a.y_f32));
-            if (a.y2 != nullptr) pn_axpy(x[j], pn_ld4(a.s2, i), pn_ld4_any(a.y2, row, a.D, i, a.y_f32));
+            if (a.y1 != nullptr) pn_axpy(x[j], c.get(c.s1, a.s1, i), pn_ld4_any(a.y1, row, a.D, i, a.y_f32));
+            if (a.y2 != nullptr) pn_axpy(x[j], c.get(c.s2, a.s2, i), pn_ld4_any(a.y2, row, a.D, i, a.y_f32));
         }
         q += x[j].x * x[j].x + x[j].y * x[j].y + x[j].z * x[j].z + x[j].w * x[j].w;       // padding is zero
     }
@@ -89,6 +106,8 @@ __device__ __forceinline__ float pn_row(const ParallelNormArgs& a, long row, flo
 template <int V>
 __global__ void __launch_bounds__(V == 1 ? 1024 : 512) parallel_norm_kernel(ParallelNormArgs a) {
     __shared__ float red[64];
+    PnVecs<V> vec;
+    vec.load(a);
     pdl_wait();
     pdl_trigger();
     const int nvec = a.D >> 2, nt = blockDim.x;
@@ -106,11 +125,11 @@ __global__ void __launch_bounds__(V == 1 ? 1024 : 512) parallel_norm_kernel(Para
         first = a.cu_q[b];
         last = a.cu_q[b + 1] - 1;
         if (r0 > first) {                                  // the row ahead of this block's first one
-            const float rs = pn_row<V>(a, r0 - 1, x, red, flip);
+            const float rs = pn_row<V>(a, vec, r0 - 1, x, red, flip);
 #pragma unroll
             for (int j = 0; j < V; ++j) {
                 const int i = threadIdx.x + j * nt;
-                if (i < nvec) prev[j] = pn_mul(x[j], rs, pn_ld4(a.w1, i));
+                if (i < nvec) prev[j] = pn_mul(x[j], rs, vec.get(vec.w1, a.w1, i));
             }
         }
     }
@@ -129,26 +148,26 @@ __global__ void __launch_bounds__(V == 1 ? 1024 : 512) parallel_norm_kernel(Para
                     if (i < nvec) prev[j] = reinterpret_cast<const float4*>(st)[i];
                 }
                 if (last > first) {                        // the slot's next value, by the block that has read the old one
-                    const float rs = pn_row<V>(a, last, x, red, flip);
+                    const float rs = pn_row<V>(a, vec, last, x, red, flip);
 #pragma unroll
                     for (int j = 0; j < V; ++j) {
                         const int i = threadIdx.x + j * nt;
-                        if (i < nvec) reinterpret_cast<float4*>(st)[i] = pn_mul(x[j], rs, pn_ld4(a.w1, i));
+                        if (i < nvec) reinterpret_cast<float4*>(st)[i] = pn_mul(x[j], rs, vec.get(vec.w1, a.w1, i));
                     }
                 }
             }
         }
-        const float rs = pn_row<V>(a, row, x, red, flip);
+        const float rs = pn_row<V>(a, vec, row, x, red, flip);
 #pragma unroll
         for (int j = 0; j < V; ++j) {
             const int i = threadIdx.x + j * nt;
             if (i >= nvec) continue;
             if (a.h_out != nullptr) reinterpret_cast<float4*>(a.h_out + row * a.D)[i] = x[j];
-            if (a.out2 != nullptr) pn_st4(a.out2, row * a.ld2, i, a.out2_f32, a.w2 != nullptr ? pn_mul(x[j], rs, pn_ld4(a.w2, i)) : x[j]);
+            if (a.out2 != nullptr) pn_st4(a.out2, row * a.ld2, i, a.out2_f32, a.w2 != nullptr ? pn_mul(x[j], rs, vec.get(vec.w2, a.w2, i)) : x[j]);
             if (a.out1 == nullptr) continue;
-            float4 v = a.w1 != nullptr ? pn_mul(x[j], rs, pn_ld4(a.w1, i)) : x[j];
+            float4 v = a.w1 != nullptr ? pn_mul(x[j], rs, vec.get(vec.w1, a.w1, i)) : x[j];
             if (a.shift != nullptr) {
-                const float4 m = pn_ld4(a.shift, i), p = prev[j];
+                const float4 m = vec.get(vec.sh, a.shift, i), p = prev[j];
                 if (first == last) reinterpret_cast<float4*>(a.state + a.seq_slots[b] * a.state_s)[i] = v;
                 prev[j] = v;
                 v = make_float4(v.x + (p.x - v.x) * m.x, v.y + (p.y - v.y) * m.y, v.z + (p.z - v.z) * m.z, v.w + (p.w - v.w) * m.w);

@@ -689,6 +689,14 @@ def visible_rows(batch: Batch, window: int):
     return hit
 
 
+def latent_splits(batch: Batch, s: LatentSpec) -> int:
+    """Split-KV factor of the latent decode kernel: as many CTAs as the SMs hold at once (its tiles of 64 keys take up to
+    most of an SM's shared memory), at least one tile each."""
+    span = min(batch.max_kv_len, s.window) if s.window else batch.max_kv_len
+    per_sm = max(1, min(4, (220 << 10) // (2 * (s.row + 8) * 144 + 3072)))
+    return max(1, min(148 * per_sm // max(1, batch.B * ((s.heads + 15) // 16)), (span + 63) // 64, 64))
+
+
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, batch: Batch, s: LatentSpec, *, wuk: torch.Tensor, wuv: torch.Tensor,
                      expand: Optional[QuantWeight], sinks: Optional[torch.Tensor]) -> torch.Tensor:
     """Causal attention of the queries ``[T, heads * Dk]`` (not rotated yet) over the cached rows -> ``[T, heads * Dv]``.
@@ -724,7 +732,7 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, batch: Batch, s: Late
     if batch.is_decode:
         qa = kk.latent_absorb(q, s, wuk, table, cache)
         part_o, part_ml = kk.latent_decode(qa, s, table, cache, batch.block_table, batch.kv_lens, batch.page_size,
-                                           decode_splits(batch, (H + 15) // 16, s.window))
+                                           latent_splits(batch, s))
         return kk.latent_out(part_o, part_ml, s, wuv, sinks, table, cache)
     kk.latent_rotate(q, s, table, cache)
     slots, pages = visible_rows(batch, s.window)

@@ -37,6 +37,21 @@ CONFIGS = {
 }
 
 
+def mixed():
+    """No two layers alike: sizes, windows, rotations, scales and feed-forwards differ from layer to layer."""
+    c = synth.sogulix_config(layers="lglg", width=96, loop=(1, 4, 2), residual_mult=0.6, softcap=15.0)
+    a, b, d, e = c["layers"]
+    a["mixer"].update(heads=5, dim=24, vdim=40, kv_rank=24, q_rank=40, mask={"size": 9})
+    d["mixer"].update(heads=2, dim=40, rot_dim=24, rot={"dims": 24, "base": 200.0}, kv_rank=56, scale=0.3, mask={"size": 90})
+    b["mixer"].update(heads=2, dim=64, decay_rank=20)
+    e["mixer"].update(heads=4, dim=16, decay_rank=3)
+    d["mlp"]["ff"], e["mlp"] = 120, None
+    return c
+
+
+CONFIGS["mixed"] = dict(config=mixed())
+
+
 def device(place):
     return "cpu" if place == "cpu" else "cuda"
 
@@ -406,7 +421,7 @@ def test_order_of_layer_runs(models):
 
 
 @pytest.mark.parametrize("place", PLACES)
-@pytest.mark.parametrize("name", ["odd", "plain", "wide"])
+@pytest.mark.parametrize("name", ["odd", "plain", "wide", "mixed"])
 @pytest.mark.parametrize("cut", [[1], [2], [3, 2, 61], [64], [23, 1, 24, 2, 70]])
 def test_portions_and_token_by_token(models, place, name, cut):
     """However a prompt is cut, its logits are the same."""
