@@ -238,22 +238,25 @@ extern "C" int tsb_latent_absorb(const LatentArgs* args, void* stream) {
 }
 
 // ------------------------------------------------------------------------------------------
-// Decode attention over the cached rows.  Grid (splits, ceil(H / 16), B), eight warps; the 16 query heads are the rows of
-// one m16 tile.  Rows arrive in tiles of 64 keys through cp.async, two stages.  Warp w scores keys 8 w .. 8 w + 7 over the
-// whole row; the probabilities meet in shared memory, and warp w accumulates the latent columns 16 (w NV + i).
+// Decode attention over the cached rows.  Grid (splits, ceil(H / (16 MT)), B), eight warps; 16 MT query heads are the rows of
+// MT m16 tiles.  Rows of the cache arrive in tiles of 64 keys through cp.async, two stages.  For the scores a warp takes half
+// of the keys and a quarter of the row's columns, for which it keeps the queries in registers (QS k-steps of 16 at most), so a
+// tile's keys are read from shared memory once; the quarters are added where the softmax is taken.  For the values warp w
+// accumulates the latent columns 16 (w NV + i).
 // ------------------------------------------------------------------------------------------
-template <int NV>
+template <int NV, int QS, int MT>
 __global__ void __launch_bounds__(256) latent_decode_kernel(LatentArgs a) {
-    constexpr int KT = 64, LDP = KT + 8;
+    constexpr int KT = 64, LDP = KT + 8, LDS_ = KT + 8, ROWS = 16 * MT, TPR = 256 / ROWS, KPT = KT / TPR;      // threads per row, keys each
     constexpr float LOG2E = 1.4426950408889634f;
     extern __shared__ __align__(128) unsigned char smem_raw[];
-    __shared__ float red[8][16];
+    __shared__ float scorr[ROWS];
     const int ld = a.Lp + 8, cl = a.Lp / 8;
-    bf16* sQ = reinterpret_cast<bf16*>(smem_raw);       // [16][ld]
-    bf16* sP = sQ + 16 * ld;                            // [16][LDP]
-    bf16* sK = sP + 16 * LDP;                           // [2][64][ld]
-    const int split = blockIdx.x, h0 = blockIdx.y * 16, b = blockIdx.z, G = min(16, a.H - h0);
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    bf16* sK = reinterpret_cast<bf16*>(smem_raw);       // [2][64][ld]
+    bf16* sP = sK + 2 * KT * ld;                        // [ROWS][LDP]
+    bf16* sQ = sP + ROWS * LDP;                         // [ROWS][ld], later:
+    float* sS = reinterpret_cast<float*>(sQ);           // [4][ROWS][LDS_] scores by quarters
+    const int split = blockIdx.x, h0 = blockIdx.y * ROWS, b = blockIdx.z, G = min(ROWS, a.H - h0);
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, kq = warp & 3, kg = warp >> 2;
     // The cached rows and the batch's metadata are not written by the kernel launched directly before (the one that makes
     // qa), and all kernels before that one have ended: the first tile is on its way before the queries are there.
     const int len = a.kv_lens[b];
@@ -272,137 +275,181 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(LatentArgs a) {
         }
         cp_async_commit();
     };
-    float o[2 * NV][4];
-#pragma unroll
-    for (int i = 0; i < 2 * NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-    float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
+    const int steps = a.Lp / 16, qs = (steps + 3) / 4, k_lo = kq * qs, k_n = max(0, min(qs, steps - k_lo));      // k-steps of this warp
+    uint32_t qf[MT][QS][4];
     if (s0 < s1) load_tile(s0, 0);
     pdl_wait();
     pdl_trigger();
     if (s0 < s1) {
-        for (int i = tid; i < 16 * cl; i += 256) {
-            const int r = i / cl, c = i % cl;
+        for (int i = tid; i < ROWS * cl; i += 256) {
+            const int r = i / cl, c = i - r * cl;
             uint4 v = make_uint4(0u, 0u, 0u, 0u);
             if (r < G) v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.qa) + ((long)b * a.H + h0 + r) * a.Lp + c * 8);
             *reinterpret_cast<uint4*>(sQ + r * ld + c * 8) = v;
         }
+        __syncthreads();
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int i = 0; i < QS; ++i)
+                if (i < k_n) ldsm_x4(qf[m][i], sQ + (16 * m + (lane & 15)) * ld + (k_lo + i) * 16 + ((lane >> 4) << 3));
+        __syncthreads();                                 // the queries' place is the scores' from here on
     }
+    float o[MT][2 * NV][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int i = 0; i < 2 * NV; ++i) o[m][i][0] = o[m][i][1] = o[m][i][2] = o[m][i][3] = 0.f;
+    const int row = tid / TPR, key0 = (tid % TPR) * KPT;             // this thread's part of the softmax
+    float mrow = -INFINITY, lrow = 0.f;
     int stage = 0;
     for (int base = s0; base < s1; base += KT, stage ^= 1) {
-        if (base + KT < s1) {
-            load_tile(base + KT, stage ^ 1);
-            cp_async_wait<1>();
-        } else {
-            cp_async_wait<0>();
-        }
-        __syncthreads();
+        cp_async_wait<0>();
+        __syncthreads();                                 // the tile is there, and the last one is done with
+        if (base + KT < s1) load_tile(base + KT, stage ^ 1);
         const bf16* tK = sK + stage * KT * ld;
-        float s[4][4] = {};                              // four chains of products
         {
-            const bf16* qrow = sQ + (lane & 15) * ld + ((lane >> 4) << 3);
-            const bf16* krow = tK + (warp * 8 + (lane & 7)) * ld + ((lane >> 3) << 3);
-            auto step = [&](int kk, float* s0, float* s1) {
-                uint32_t q0[4], q1[4], kb[4];
-                ldsm_x4(q0, qrow + kk);
-                ldsm_x4(q1, qrow + kk + 16);
-                ldsm_x4(kb, krow + kk);
-                mma_bf16(s0, q0, kb[0], kb[1]);
-                mma_bf16(s1, q1, kb[2], kb[3]);
-            };
-            int kk = 0;                                  // Lp is a multiple of 32
-#pragma unroll 2
-            for (; kk + 64 <= a.Lp; kk += 64) {
-                step(kk, s[0], s[1]);
-                step(kk + 32, s[2], s[3]);
+            float s[MT][4][4];
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) s[m][i][0] = s[m][i][1] = s[m][i][2] = s[m][i][3] = 0.f;
+            const bf16* krow = tK + (kg * 32 + ((lane >> 4) << 3) + (lane & 7)) * ld + k_lo * 16 + (((lane >> 3) & 1) << 3);
+#pragma unroll
+            for (int i = 0; i < QS; ++i) {
+                if (i >= k_n) break;
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    uint32_t kb[4];
+                    ldsm_x4(kb, krow + half * 16 * ld + i * 16);
+#pragma unroll
+                    for (int m = 0; m < MT; ++m) {
+                        mma_bf16(s[m][2 * half], qf[m][i], kb[0], kb[1]);
+                        mma_bf16(s[m][2 * half + 1], qf[m][i], kb[2], kb[3]);
+                    }
+                }
             }
-            if (kk < a.Lp) step(kk, s[0], s[1]);
-        }
-        const int key = base + warp * 8 + (lane & 3) * 2;
-        float p[4], mx[2];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) p[e] = key + (e & 1) < s1 ? ((s[0][e] + s[2][e]) + (s[1][e] + s[3][e])) * a.scale : -INFINITY;
+            for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            mx[r] = fmaxf(p[2 * r], p[2 * r + 1]);
-            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
-            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
-            if ((lane & 3) == 0) red[warp][(lane >> 2) + 8 * r] = mx[r];
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int r = 0; r < 2; ++r)
+                        *reinterpret_cast<float2*>(sS + (kq * ROWS + 16 * m + (lane >> 2) + 8 * r) * LDS_ + kg * 32 + i * 8 + (lane & 3) * 2) =
+                            make_float2(s[m][i][2 * r], s[m][i][2 * r + 1]);
         }
         __syncthreads();
-        float corr[2];
+        {
+            float p[KPT], m = mrow;
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            float m = mrow[r];
+            for (int j = 0; j < KPT; j += 4) {
+                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-            for (int w = 0; w < 8; ++w) m = fmaxf(m, red[w][(lane >> 2) + 8 * r]);      // the tile has a valid key: finite
-            corr[r] = mrow[r] == -INFINITY ? 0.f : exp2f((mrow[r] - m) * LOG2E);
-            mrow[r] = m;
-            const float e0 = exp2f((p[2 * r] - m) * LOG2E), e1 = exp2f((p[2 * r + 1] - m) * LOG2E);
-            lrow[r] = lrow[r] * corr[r] + e0 + e1;
-            *reinterpret_cast<uint32_t*>(sP + ((lane >> 2) + 8 * r) * LDP + warp * 8 + (lane & 3) * 2) = pack_bf16(e0, e1);
-        }
+                for (int q = 0; q < 4; ++q) {
+                    const float4 x = *reinterpret_cast<const float4*>(sS + (q * ROWS + row) * LDS_ + key0 + j);
+                    v.x += x.x; v.y += x.y; v.z += x.z; v.w += x.w;
+                }
+                p[j] = v.x; p[j + 1] = v.y; p[j + 2] = v.z; p[j + 3] = v.w;
+            }
 #pragma unroll
-        for (int i = 0; i < 2 * NV; ++i) {
-            o[i][0] *= corr[0]; o[i][1] *= corr[0];
-            o[i][2] *= corr[1]; o[i][3] *= corr[1];
+            for (int j = 0; j < KPT; ++j) {
+                p[j] = base + key0 + j < s1 ? p[j] * a.scale : -INFINITY;
+                m = fmaxf(m, p[j]);
+            }
+#pragma unroll
+            for (int x = TPR / 2; x >= 1; x >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, x));      // the tile has a valid key: finite
+            const float corr = mrow == -INFINITY ? 0.f : exp2f((mrow - m) * LOG2E);
+            mrow = m;
+            lrow *= corr;
+#pragma unroll
+            for (int j = 0; j < KPT; j += 2) {
+                const float e0 = exp2f((p[j] - m) * LOG2E), e1 = exp2f((p[j + 1] - m) * LOG2E);
+                lrow += e0 + e1;
+                *reinterpret_cast<uint32_t*>(sP + row * LDP + key0 + j) = pack_bf16(e0, e1);
+            }
+            if (tid % TPR == 0) scorr[row] = corr;
         }
         __syncthreads();
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+            const float c0 = scorr[16 * m + (lane >> 2)], c1 = scorr[16 * m + (lane >> 2) + 8];
+#pragma unroll
+            for (int i = 0; i < 2 * NV; ++i) {
+                o[m][i][0] *= c0; o[m][i][1] *= c0;
+                o[m][i][2] *= c1; o[m][i][3] *= c1;
+            }
+        }
 #pragma unroll
         for (int kt = 0; kt < KT / 16; ++kt) {
-            uint32_t pa[4];
-            ldsm_x4(pa, sP + (lane & 15) * LDP + kt * 16 + ((lane >> 4) << 3));
-            const bf16* row = tK + (kt * 16 + (((lane >> 3) & 1) << 3) + (lane & 7)) * ld + ((lane >> 4) << 3);
+            uint32_t pa[MT][4];
+#pragma unroll
+            for (int m = 0; m < MT; ++m) ldsm_x4(pa[m], sP + (16 * m + (lane & 15)) * LDP + kt * 16 + ((lane >> 4) << 3));
+            const bf16* vrow = tK + (kt * 16 + (((lane >> 3) & 1) << 3) + (lane & 7)) * ld + ((lane >> 4) << 3);
 #pragma unroll
             for (int i = 0; i < NV; ++i) {
                 const int c = (warp * NV + i) * 16;
                 if (c >= a.R) break;
                 uint32_t vb[4];
-                ldsm_x4_t(vb, row + c);
-                mma_bf16(o[2 * i], pa, vb[0], vb[1]);
-                mma_bf16(o[2 * i + 1], pa, vb[2], vb[3]);
+                ldsm_x4_t(vb, vrow + c);
+#pragma unroll
+                for (int m = 0; m < MT; ++m) {
+                    mma_bf16(o[m][2 * i], pa[m], vb[0], vb[1]);
+                    mma_bf16(o[m][2 * i + 1], pa[m], vb[2], vb[3]);
+                }
             }
         }
-        __syncthreads();                                 // before the stage, the maxima and P are written again
     }
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-        lrow[r] += __shfl_xor_sync(0xffffffffu, lrow[r], 1);
-        lrow[r] += __shfl_xor_sync(0xffffffffu, lrow[r], 2);
-        if ((lane & 3) == 0) red[warp][(lane >> 2) + 8 * r] = lrow[r];
+    for (int x = TPR / 2; x >= 1; x >>= 1) lrow += __shfl_xor_sync(0xffffffffu, lrow, x);
+    const long p0 = ((long)b * a.H + h0) * a.splits + split;             // partial of head h0 + r: p0 + r * splits
+    if (row < G && tid % TPR == 0) {
+        a.part_ml[(p0 + (long)row * a.splits) * 2] = mrow;
+        a.part_ml[(p0 + (long)row * a.splits) * 2 + 1] = lrow;
     }
-    __syncthreads();
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-        const int row = (lane >> 2) + 8 * r;
-        if (row >= G) continue;
-        const long pi = ((long)b * a.H + h0 + row) * a.splits + split;
-        if (warp == 0 && (lane & 3) == 0) {
-            float l = 0.f;
+    for (int m = 0; m < MT; ++m)
 #pragma unroll
-            for (int w = 0; w < 8; ++w) l += red[w][row];
-            a.part_ml[pi * 2] = mrow[r];
-            a.part_ml[pi * 2 + 1] = l;
+        for (int r = 0; r < 2; ++r) {
+            const int hr = 16 * m + (lane >> 2) + 8 * r;
+            if (hr >= G) continue;
+#pragma unroll
+            for (int i = 0; i < 2 * NV; ++i) {
+                const int c = (warp * NV + (i >> 1)) * 16 + (i & 1) * 8 + (lane & 3) * 2;
+                if (c < a.Ro) *reinterpret_cast<float2*>(a.part_o + (p0 + (long)hr * a.splits) * a.Ro + c) = make_float2(o[m][i][2 * r], o[m][i][2 * r + 1]);
+            }
         }
-#pragma unroll
-        for (int i = 0; i < 2 * NV; ++i) {
-            const int c = (warp * NV + (i >> 1)) * 16 + (i & 1) * 8 + (lane & 3) * 2;
-            if (c < a.Ro) *reinterpret_cast<float2*>(a.part_o + pi * a.Ro + c) = make_float2(o[i][2 * r], o[i][2 * r + 1]);
-        }
-    }
 }
 
-template <int NV>
+static size_t latent_decode_smem(int Lp, int MT) {
+    const size_t ld = Lp + 8, q = 16 * MT * ld * sizeof(bf16), sc = (size_t)4 * 16 * MT * 72 * sizeof(float);
+    return (2 * 64 * ld + 16 * MT * 72) * sizeof(bf16) + (q > sc ? q : sc);
+}
+
+template <int NV, int QS, int MT>
 static int launch_latent_decode(const LatentArgs& a, cudaStream_t s) {
-    const int ld = a.Lp + 8;
-    const size_t smem = (size_t)(16 * ld + 16 * 72 + 2 * 64 * ld) * sizeof(bf16);
+    const size_t smem = latent_decode_smem(a.Lp, MT);
     static size_t configured = 0;
     if (smem > configured) {
-        TSB_CHECK_CUDA(cudaFuncSetAttribute(latent_decode_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        TSB_CHECK_CUDA(cudaFuncSetAttribute(latent_decode_kernel<NV, QS, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         configured = smem;
     }
-    TSB_CHECK_CUDA(tsb_launch(latent_decode_kernel<NV>, dim3(a.splits, (a.H + 15) / 16, a.T), dim3(256), smem, s, a));
+    TSB_CHECK_CUDA(tsb_launch(latent_decode_kernel<NV, QS, MT>, dim3(a.splits, (a.H + 16 * MT - 1) / (16 * MT), a.T), dim3(256), smem, s, a));
     TSB_CHECK_LAUNCH();
     return TSB_OK;
+}
+
+// Tiles of 16 query heads per CTA of the decode kernel: two where there are more than 16 heads, sequences enough to fill the
+// SMs all the same, and room
+static int latent_head_tiles(int B, int H, int Lp) { return H > 16 && B >= 4 && latent_decode_smem(Lp, 2) <= 226 * 1024 ? 2 : 1; }
+extern "C" int tsb_latent_heads_per_cta(int B, int H, int Lp) { return 16 * latent_head_tiles(B, H, Lp); }
+extern "C" long tsb_latent_decode_smem(int B, int H, int Lp) { return (long)latent_decode_smem(Lp, latent_head_tiles(B, H, Lp)); }
+
+template <int NV, int QS>
+static int launch_latent_decode_mt(const LatentArgs& a, cudaStream_t s) {
+    // rows with a wide rotated part need more k-steps than the latent size suggests
+    const bool two = latent_head_tiles(a.T, a.H, a.Lp) == 2;
+    if (a.Lp > 64 * QS) return two ? launch_latent_decode<NV, 11, 2>(a, s) : launch_latent_decode<NV, 11, 1>(a, s);
+    return two ? launch_latent_decode<NV, QS, 2>(a, s) : launch_latent_decode<NV, QS, 1>(a, s);
 }
 
 // One query per sequence (T sequences); leaves the split partials in part_o / part_ml.
@@ -415,10 +462,10 @@ extern "C" int tsb_latent_decode(const LatentArgs* args, void* stream) {
     if (a.T == 0) return TSB_OK;
     cudaStream_t s = (cudaStream_t)stream;
     switch ((a.R + 127) / 128) {
-    case 1: return launch_latent_decode<1>(a, s);
-    case 2: return launch_latent_decode<2>(a, s);
-    case 3: return launch_latent_decode<3>(a, s);
-    default: return launch_latent_decode<4>(a, s);
+    case 1: return launch_latent_decode_mt<1, 3>(a, s);
+    case 2: return launch_latent_decode_mt<2, 5>(a, s);
+    case 3: return launch_latent_decode_mt<3, 7>(a, s);
+    default: return launch_latent_decode_mt<4, 9>(a, s);
     }
 }
 

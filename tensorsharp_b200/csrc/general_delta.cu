@@ -5,16 +5,16 @@
 //   S <- diag(w) S - (a u)(u^T S) + k v^T                          both terms read the old state
 //   o = S^T r;   out = o / rms(o) * norm * sigmoid(g)
 //
-// Every column of S (one value channel) evolves by itself, so a head is spread over groups of eight lanes, each holding
-// one or two columns in registers (lane l: keys 4 l + 32 i .. + 3); the only exchange is the sum u^T S over eight lanes.
-// Everything here is f32.  Head sizes are padded with zeros to a multiple of 32 (zero r, k, v keep the padding of S zero);
+// Every column of S (one value channel) evolves by itself, so a head is spread over groups of lanes that hold a few columns
+// in registers, each lane a share of the keys; the only exchange is the sum u^T S over a group.  Everything here is f32.  Head sizes are padded with zeros to a multiple of 32 (zero r, k, v keep the padding of S zero);
 // the norm divides by the true size n.  The state of a slot is [H][value][key].
 //
 //   short steps (decode)   gdr_short_kernel: one CTA per (head, sequence); decay projection, unit key, recurrence, norm
 //                          and gate in one kernel
-//   prompts                gdr_prep_kernel: the per-token vectors (u, w, a, r, and v times the key's length);
-//                          gdr_scan_kernel: the recurrence, 32 value channels of a head per CTA, tokens staged in shared
-//                          memory by cp.async; gdr_finish_kernel: norm and gate
+//   prompts, f32 models    gdr_prep_kernel: the per-token vectors (u, w, a, r, and v times the key's length);
+//                          gdr_scan_kernel: the recurrence token by token, tokens staged in shared memory by cp.async;
+//                          gdr_finish_kernel: norm and gate
+//   prompts, bf16 models   general_delta_chunk.cu: eight tokens at a time on the tensor cores; gdr_finish_kernel
 #include "attn_mma.cuh"
 #include "common.cuh"
 #include "general_delta.cuh"

@@ -693,8 +693,9 @@ def latent_splits(batch: Batch, s: LatentSpec) -> int:
     """Split-KV factor of the latent decode kernel: as many CTAs as the SMs hold at once (its tiles of 64 keys take up to
     most of an SM's shared memory), at least one tile each."""
     span = min(batch.max_kv_len, s.window) if s.window else batch.max_kv_len
-    per_sm = max(1, min(4, (220 << 10) // (2 * (s.row + 8) * 144 + 3072)))
-    return max(1, min(148 * per_sm // max(1, batch.B * ((s.heads + 15) // 16)), (span + 63) // 64, 64))
+    heads, smem = _k().latent_decode_shape(batch.B, s.heads, s.row)
+    per_sm = max(1, min(4, (226 << 10) // smem))
+    return max(1, min(148 * per_sm // max(1, batch.B * -(-s.heads // heads)), (span + 63) // 64, 64))
 
 
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, batch: Batch, s: LatentSpec, *, wuk: torch.Tensor, wuv: torch.Tensor,

@@ -700,6 +700,14 @@ def latent_absorb(q: torch.Tensor, s, wuk: torch.Tensor, cs, cache) -> torch.Ten
     return qa
 
 
+def latent_decode_shape(B: int, heads: int, row: int):
+    """(query heads per CTA, bytes of shared memory) of the latent decode kernel."""
+    lib = _lib()
+    lib.tsb_latent_decode_smem.restype = C.c_long
+    n = (C.c_int(B), C.c_int(heads), C.c_int(row))
+    return int(lib.tsb_latent_heads_per_cta(*n)), int(lib.tsb_latent_decode_smem(*n))
+
+
 def latent_decode(qa: torch.Tensor, s, cs, cache, block_table, kv_lens, page_size: int, splits: int):
     """One query per sequence against the cached bf16 rows -> split partials (o [B, H, splits, Ro], (max, sum))."""
     B = qa.shape[0]

@@ -378,6 +378,45 @@ def test_what_the_delta_rule_keeps():
     assert torch.allclose(o[T - 1, 0], v[T - 3], atol=1e-5)                        # (the same key was written three times)
 
 
+@gpu
+@pytest.mark.parametrize("H,dim,rot,vdim,rank,window", [(20, 32, 16, 48, 512, 300), (40, 24, 160, 16, 64, 0), (33, 64, 64, 32, 300, 97), (64, 16, 200, 16, 500, 0),
+                                                        (16, 32, 96, 32, 200, 0)])
+def test_latent_decoding_of_many_heads_and_sequences(H, dim, rot, vdim, rank, window):
+    """Six sequences of very different lengths in one step: every head tile, row width and split count of the decode kernel
+    against the attention written out."""
+    g = torch.Generator().manual_seed(H + rank)
+    s = spec(H, dim, rot, vdim, rank, 8, window, "cuda", scale=0.2)
+    lens = [1, 700, 64, 65, 333, 1500]
+    kv = PagedKV([(1, s.row, 0)], 60, 64, "cuda", torch.bfloat16, max_seqs=6)
+    kv._free = torch.randperm(60, generator=g).tolist()
+    kv.k[0].fill_(float("nan"))
+    seqs = [kv.new_seq() for _ in lens]
+    uk, uv = (torch.randn(H * d, rank, generator=g).div(rank ** 0.5).bfloat16() for d in (dim, vdim))
+    sinks = torch.randn(H, generator=g)
+    rows = [torch.nn.functional.pad(torch.randn(n, rank + rot, generator=g), (0, s.row - rank - rot)).bfloat16() for n in lens]
+    q = torch.randn(6, H, dim + rot, generator=g) * 0.5
+    kv.build_batch([x for x, n in zip(seqs, lens) if n > 1], [[0] * (n - 1) for n in lens if n > 1])
+    batch = kv.build_batch(seqs, [[0]] * 6)
+    for x, r in zip(seqs, rows):
+        at = torch.tensor([x.pages[j // 64] * 64 + j % 64 for j in range(len(r))])
+        kv.k[0][at.cuda(), 0] = r.cuda()
+    wuk = torch.nn.functional.pad(uk, (0, s.rank_p - rank)).cuda()
+    wuv = torch.zeros(H, s.Dv, s.rank_p, dtype=torch.bfloat16)
+    wuv[:, :vdim, :rank] = uv.view(H, vdim, rank)
+    out = F.latent_attention(torch.nn.functional.pad(q, (0, s.Dk - dim - rot)).view(6, -1).cuda(), kv.k[0], batch, s, wuk=wuk,
+                             wuv=wuv.view(H * s.Dv, s.rank_p).cuda(), expand=None, sinks=sinks.cuda()).view(6, H, s.Dv)
+    for b, (n, r) in enumerate(zip(lens, rows)):
+        lo = max(0, n - window) if window else 0
+        r = r.double()[lo:]
+        qr = torch.cat([q[b, :, :dim].double(), O.rotate_half(q[b, :, dim:].double()[None], torch.tensor([n - 1]), 3000.0)[0]], -1)
+        k = torch.cat([(r[:, :rank] @ uk.double().T).view(-1, H, dim), r[:, None, rank:rank + rot].expand(-1, H, rot)], -1)
+        v = (r[:, :rank] @ uv.double().T).view(-1, H, vdim)
+        sc = torch.einsum("hd,thd->ht", qr, k) * 0.2
+        e = torch.exp(sc - 20)
+        want = torch.einsum("ht,thv->hv", e / (e.sum(1, keepdim=True) + torch.exp(sinks.double() - 20)[:, None]), v)
+        assert (out[b, :, :vdim].double().cpu() - want).abs().max() < 0.05, b
+
+
 @pytest.mark.parametrize("place", PLACES)
 def test_logit_cap(place):
     z = torch.linspace(-200, 200, 999).to(device(place))
