@@ -194,7 +194,7 @@ def test_latent_rows_and_rotation(place):
     assert torch.allclose(row[:, 21:31], O.rotate_half(x[:, 48:].double(), torch.tensor(pos), 3000.0), **tol) and not row[:, 31:].any()
 
 
-LATENT = [(4, 32, 16, 32, 40, 24), (3, 20, 6, 24, 36, 70), (8, 64, 32, 64, 96, 33), (17, 48, 2, 16, 130, 64), (1, 16, 0, 80, 256, 1), (33, 128, 64, 128, 512, 65),
+LATENT = [(4, 32, 16, 32, 40, 24), (3, 20, 6, 24, 36, 70), (7, 64, 32, 48, 88, 33), (17, 48, 2, 16, 130, 64), (1, 16, 0, 80, 256, 1), (33, 128, 64, 128, 512, 65),
           (2, 64, 64, 48, 64, 0), (5, 8, 8, 8, 390, 16)]
 
 
