@@ -1,7 +1,7 @@
 """Sogulix: a hybrid of latent attention and a generalized delta rule in parallel layers, with a range of layers that runs
 several times with the same weights.
 
-A layer:  x += m (ls1 mixer(shift(norm1(x))) + ls2 ff(norm2(x)))  with RMS norms whose weights are stored around zero
+A layer:  x += m (ls1 mixer(shift(norm1(x))) + ls2 ff(norm2(x)))  with RMS norms whose weights are offsets from 1
 (factor 1 + w); ``shift`` moves every channel towards the previous token's normalised value.
   latent_attention   queries through a normed latent; one normed latent per token for the keys and values of all heads, plus
                      one rotated key part they share; sliding window, a sink per head in the softmax
@@ -68,7 +68,7 @@ class SogulixModel(FolderModel):
 
     # ------------------------------------------------------------------ weights
     def _norm1p(self, name: str) -> torch.Tensor:
-        """The factor 1 + w of a norm stored around zero (0 in the padding)."""
+        """The factor 1 + w of a norm stored as its offset from 1 (0 in the padding)."""
         w = self._host(name).float() + 1.0
         return TF.pad(w, (0, self.cfg.hidden - w.shape[0])).to(self.device).contiguous()
 
