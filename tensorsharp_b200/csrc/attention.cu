@@ -313,7 +313,7 @@ __global__ void attn_combine_kernel(AttnArgs a) {
             o += pv[i] * c;
         }
     }
-    const bf16 ob = f2bf(ll > 0.f ? o / ll * attn_gate(a, b, h) : 0.f);
+    const bf16 ob = f2bf(ll > 0.f ? o / ll * attn_gate(a, b, h, dd) : 0.f);
     if (d < a.Dh) a.out[((long)b * a.Hq + h) * a.Dh + d] = ob;
     if (a.out_q != nullptr) {
         // a warp holds 32 consecutive dims = one group (Dh is a multiple of 32); same arithmetic as quantize_q8_kernel
@@ -406,7 +406,7 @@ static int attn_decode_impl(const AttnArgs* args, void* stream, bool allow_fused
     cudaStream_t s = (cudaStream_t)stream;
     int rc;
     if (a.gate != nullptr) a.ticket = nullptr;          // the in-kernel merges know no gate
-    if ((a.Dv != 0 && a.Dv != a.Dh) || a.k_ld != 0 || a.v_ld != 0 || (a.Dh != 64 && a.Dh != 128 && a.Dh != 256 && a.Dh != 512)) {
+    if (attn_needs_vd(a)) {
         if (a.Dv == 0) a.Dv = a.Dh;
         rc = tsb_attn_decode_vd_launch(a, s);
         if (rc != TSB_OK) return rc;
@@ -745,7 +745,7 @@ extern "C" int tsb_attn_prefill(const AttnArgs* args, int max_q_len, void* strea
     TSB_CHECK_ARG(a.cu_q != nullptr, "attn_prefill: cu_q is required");
     if (a.B == 0 || max_q_len == 0) return TSB_OK;
     cudaStream_t s = (cudaStream_t)stream;
-    if ((a.Dv != 0 && a.Dv != a.Dh) || a.k_ld != 0 || a.v_ld != 0 || (a.Dh != 64 && a.Dh != 128 && a.Dh != 256 && a.Dh != 512))
+    if (attn_needs_vd(a))
         return tsb_attn_prefill_vd_launch(a, max_q_len, s);
     switch (a.Dh) {
     case 64: return launch_prefill<64>(a, max_q_len, s);

@@ -20,33 +20,6 @@ __device__ __forceinline__ void la_st(void* p, long i, int f32, float v) {
 }
 }  // namespace
 
-// ------------------------------------------------------------------------------------------
-// (cos, sin) of position * freq per (token, pair).  The angle is formed and reduced to one turn in double precision: in
-// f32 the product alone is off by 3e-5 at position 1000.
-// ------------------------------------------------------------------------------------------
-__global__ void rotary_table_kernel(const int* pos, const double* freq, float2* out, int T, int half) {
-    pdl_wait();
-    pdl_trigger();
-    const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= (long)T * half) return;
-    constexpr double TURN = 6.283185307179586476925;
-    double a = (double)pos[i / half] * freq[i % half];
-    a -= TURN * rint(a / TURN);
-    float s, c;
-    sincosf((float)a, &s, &c);
-    out[i] = make_float2(c, s);
-}
-
-extern "C" int tsb_rotary_table(const int* pos, const double* freq, void* out, int T, int half, void* stream) {
-    TSB_CHECK_ARG(T >= 0 && half >= 0, "rotary_table: T=%d half=%d", T, half);
-    const long n = (long)T * half;
-    if (n == 0) return TSB_OK;
-    TSB_CHECK_CUDA(tsb_launch(rotary_table_kernel, dim3((unsigned)((n + 127) / 128)), dim3(128), 0, (cudaStream_t)stream, pos, freq, (float2*)out,
-                              T, half));
-    TSB_CHECK_LAUNCH();
-    return TSB_OK;
-}
-
 struct LatentArgs {
     // rows [query latent (qr, padded to qp) | latent (R) | rotated part (rot)]
     const void* y; long y_s; int y_f32;

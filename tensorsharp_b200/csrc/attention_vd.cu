@@ -7,6 +7,10 @@
 // from shared memory where they are used; only the accumulators, whose number depends on Dv, are registers), and tile rows
 // are padded by 16 bytes instead of XOR-swizzled: with an even number of 16-byte pieces per row the padded row length is
 // odd in units of 16 bytes, so the eight rows of an ldmatrix start in eight different bank groups.
+//
+// These kernels also know a window with kept first positions (two ranges of key tiles), a distance bias per head, a gate per
+// output column, and caches whose rows are key and value at once (AttnArgs::kv_scale): one tile is then staged and read both
+// ways, and the scores get the factor of their key.
 #include "attn_args.cuh"
 #include "attn_mma.cuh"
 #include "common.cuh"
@@ -120,6 +124,11 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
     const int j_lo = a.window > 0 ? max(0, pos0 + m0 - a.window + 1) : 0;
     const int j_hi = min(pos0 + m0 + rows, kvlen);
     const int t_lo = j_lo / BN, t_hi = (j_hi + BN - 1) / BN;
+    // tiles in order: those of the kept first positions that lie ahead of the window, then the window's
+    const int n_first = a.keep_first > 0 ? min(t_lo, (a.keep_first + BN - 1) / BN) : 0, n_tiles = n_first + t_hi - t_lo;
+    const bool one_row = a.kv_scale != 0;
+    float* sF = reinterpret_cast<float*>(sV);                          // 2 stages of key factors, in place of the value tiles
+    const float slope = a.slopes ? a.slopes[h] : 0.f;
 
     for (int i = threadIdx.x; i < BM * ck; i += 128) {
         const int r = i / ck, c = i % ck;
@@ -137,15 +146,24 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
             const bf16* gk = a.k_cache + slot * a.k_ld + hk * dk;
             const bf16* gv = a.v_cache + slot * a.v_ld + hk * DV;
             for (int c = half; c < ck; c += 2) cp_async16(pk + c * 8, gk + c * 8);
+            if (one_row) {
+                if (half == 0) cp_async4(sF + stage * BN + r, attn_key_factor(a, slot));
+                return;
+            }
 #pragma unroll
             for (int c = 0; c < cv; c += 2) cp_async16(pv + (c + half) * 8, gv + (c + half) * 8);
         } else {
             for (int c = half; c < ck; c += 2) *reinterpret_cast<uint4*>(pk + c * 8) = make_uint4(0, 0, 0, 0);
+            if (one_row) {
+                if (half == 0) sF[stage * BN + r] = 0.f;
+                return;
+            }
 #pragma unroll
             for (int c = 0; c < cv; c += 2) *reinterpret_cast<uint4*>(pv + (c + half) * 8) = make_uint4(0, 0, 0, 0);
         }
     };
-    load_kv(t_lo, 0);
+    auto tile = [&](int u) { return u < n_first ? u : t_lo + u - n_first; };
+    load_kv(tile(0), 0);
     cp_async_commit();
 
     float o[DV / 8][4];
@@ -156,14 +174,21 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
     const int qpos_a = pos0 + m0 + r_lo, qpos_b = qpos_a + 8;
     const int q_first = pos0 + m0 + warp * 16;
 
-    for (int t = t_lo; t < t_hi; ++t) {
-        const int stage = (t - t_lo) & 1;
-        if (t + 1 < t_hi) load_kv(t + 1, stage ^ 1);
+    for (int u = 0; u < n_tiles; ++u) {
+        const int stage = u & 1, t = tile(u);
+        if (u + 1 < n_tiles) load_kv(tile(u + 1), stage ^ 1);
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
         float s[BN / 8][4];
         vd_qk<BN>(s, sQ + warp * 16 * ldk, ldk, sK + stage * BN * ldk, ldk, dk, lane);
+        if (one_row) {
+#pragma unroll
+            for (int nt = 0; nt < BN / 8; ++nt) {
+                const float2 kf = *reinterpret_cast<const float2*>(sF + stage * BN + nt * 8 + (lane & 3) * 2);
+                s[nt][0] *= kf.x; s[nt][1] *= kf.y; s[nt][2] *= kf.x; s[nt][3] *= kf.y;
+            }
+        }
         float f = a.scale;
         if (a.softcap > 0.f) {
             const float inv_cap = a.scale / a.softcap;
@@ -171,6 +196,14 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
             for (int nt = 0; nt < BN / 8; ++nt)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) s[nt][e] = a.softcap * tanhf(s[nt][e] * inv_cap);
+            f = 1.f;
+        }
+        if (a.slopes != nullptr) {
+            const int d0 = t * BN + (lane & 3) * 2 - qpos_a;                        // key minus query
+#pragma unroll
+            for (int nt = 0; nt < BN / 8; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[nt][e] = fmaf(slope, (float)(d0 + nt * 8 + (e & 1) - (e < 2 ? 0 : 8)), s[nt][e] * f);
             f = 1.f;
         }
         const bool need_mask = (t * BN + BN - 1 > q_first) || ((t + 1) * BN > kvlen) ||
@@ -182,12 +215,12 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
                 for (int e = 0; e < 4; ++e) {
                     const int j = t * BN + nt * 8 + (lane & 3) * 2 + (e & 1);
                     const int qp = (e < 2) ? qpos_a : qpos_b;
-                    const bool ok = j <= qp && j < kvlen && (a.window <= 0 || j > qp - a.window);
+                    const bool ok = j <= qp && j < kvlen && (a.window <= 0 || j > qp - a.window || j < a.keep_first);
                     s[nt][e] = ok ? s[nt][e] : -INFINITY;
                 }
         }
         vd_softmax<BN, DV / 8>(s, o, mrow, lrow, f);
-        vd_pv<BN, DV>(s, o, sV + stage * BN * ldv, ldv, lane);
+        vd_pv<BN, DV>(s, o, one_row ? sK + stage * BN * ldk : sV + stage * BN * ldv, ldv, lane);      // one row: ldk = ldv
         __syncthreads();
     }
     cp_async_wait<0>();
@@ -205,7 +238,7 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
         inv[r] = ll > 0.f ? oc / ll : 0.f;
         const int row = r_lo + 8 * r;
         if (row < rows) {
-            inv[r] *= attn_gate(a, q0 + m0 + row, h);
+            if (!a.gate_cols) inv[r] *= attn_gate(a, q0 + m0 + row, h);
             if (a.lse_out != nullptr && (lane & 3) == 0)
                 a.lse_out[(long)(q0 + m0 + row) * a.Hq + h] = lrow[r] > 0.f ? mrow[r] + __logf(lrow[r]) : -INFINITY;
         }
@@ -213,6 +246,11 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i) {
         const int d = i * 8 + (lane & 3) * 2;
+        if (a.gate_cols) {
+            const long t = q0 + m0 + r_lo;
+            if (r_lo < rows) { o[i][0] *= attn_gate(a, t, h, d); o[i][1] *= attn_gate(a, t, h, d + 1); }
+            if (r_lo + 8 < rows) { o[i][2] *= attn_gate(a, t + 8, h, d); o[i][3] *= attn_gate(a, t + 8, h, d + 1); }
+        }
         if (r_lo < rows)
             *reinterpret_cast<uint32_t*>(a.out + ((long)(q0 + m0 + r_lo) * a.Hq + h) * DV + d) = pack_bf16(o[i][0] * inv[0], o[i][1] * inv[0]);
         if (r_lo + 8 < rows)
@@ -233,7 +271,7 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
     const int dk = a.Dh, ldk = dk + 8, ldv = DV + 8, ck = dk / 8;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     bf16* sQ = reinterpret_cast<bf16*>(smem_raw);                       // [16][ldk]
-    bf16* sK = sQ + 16 * ldk + warp * KT * (ldk + ldv);                 // this warp's K tile
+    bf16* sK = sQ + 16 * ldk + warp * KT * (a.kv_scale ? ldk : ldk + ldv);                 // this warp's K tile
     bf16* sV = sK + KT * ldk;                                           // and V tile
     const int split = blockIdx.x, hk = blockIdx.y / chunks, b = blockIdx.z;
     const int group = a.Hq / a.Hkv, first = (blockIdx.y % chunks) * 16;
@@ -245,11 +283,19 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
         if (r < G) v = *reinterpret_cast<const uint4*>(a.q + ((long)b * a.Hq + h0 + r) * dk + c * 8);
         *reinterpret_cast<uint4*>(sQ + r * ldk + c * 8) = v;
     }
+    // the visible positions, numbered without a gap: the kept first ones ahead of the window, then the window
     const int len = a.kv_lens[b];
-    const int lo = (a.window > 0 && len > a.window) ? len - a.window : 0;
-    const int span = len - lo;
+    const int lo = (a.window > 0 && len > a.window) ? len - a.window : 0, nf = min(a.keep_first, lo), gap = lo - nf;
+    const int span = len - gap;
     const int per = a.split_len > 0 ? a.split_len : ((((span + a.splits - 1) / a.splits) + 31) & ~31);
-    const int s0 = lo + split * per, s1 = min(len, s0 + per);
+    const int s0 = split * per, s1 = min(span, s0 + per);
+    const bool one_row = a.kv_scale != 0;
+    float slope[2] = {0.f, 0.f};
+    if (a.slopes != nullptr) {
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+            if ((lane >> 2) + 8 * r < G) slope[r] = a.slopes[h0 + (lane >> 2) + 8 * r];
+    }
     __syncthreads();
 
     float o[DV / 8][4];
@@ -259,7 +305,8 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
 
     for (int base = s0 + warp * KT; base < s1; base += 4 * KT) {
         const int j = base + lane;
-        const long slot = j < s1 ? vd_slot(a, b, j) : 0;
+        const long slot = j < s1 ? vd_slot(a, b, j < nf ? j : j + gap) : 0;
+        const float kf = one_row && j < s1 ? *attn_key_factor(a, slot) : 0.f;
         // consecutive lanes copy consecutive pieces of a row; rows past the end are zero
         for (int i = lane; i < KT * ck; i += 32) {
             const int key = i / ck, c = i % ck;
@@ -268,6 +315,7 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
             if (base + key < s1) cp_async16(p, a.k_cache + sl * a.k_ld + hk * dk + c * 8);
             else *reinterpret_cast<uint4*>(p) = make_uint4(0u, 0u, 0u, 0u);
         }
+        if (!one_row)
 #pragma unroll 4
         for (int i = lane; i < KT * cv; i += 32) {
             const int key = i / cv, c = i % cv;
@@ -281,6 +329,13 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
         __syncwarp();
         float s[KT / 8][4];
         vd_qk<KT>(s, sQ, ldk, sK, ldk, dk, lane);
+        if (one_row) {
+#pragma unroll
+            for (int nt = 0; nt < KT / 8; ++nt) {
+                const float k0 = __shfl_sync(0xffffffffu, kf, nt * 8 + (lane & 3) * 2), k1 = __shfl_sync(0xffffffffu, kf, nt * 8 + (lane & 3) * 2 + 1);
+                s[nt][0] *= k0; s[nt][1] *= k1; s[nt][2] *= k0; s[nt][3] *= k1;
+            }
+        }
         float f = a.scale;
         if (a.softcap > 0.f) {
 #pragma unroll
@@ -289,13 +344,23 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
                 for (int e = 0; e < 4; ++e) s[nt][e] = a.softcap * tanhf(s[nt][e] * a.scale / a.softcap);
             f = 1.f;
         }
+        if (a.slopes != nullptr) {
+#pragma unroll
+            for (int nt = 0; nt < KT / 8; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int i = base + nt * 8 + (lane & 3) * 2 + (e & 1);
+                    s[nt][e] = fmaf(slope[e >> 1], (float)((i < nf ? i : i + gap) - (len - 1)), s[nt][e] * f);
+                }
+            f = 1.f;
+        }
 #pragma unroll
         for (int nt = 0; nt < KT / 8; ++nt)
 #pragma unroll
             for (int e = 0; e < 4; ++e)
                 if (base + nt * 8 + (lane & 3) * 2 + (e & 1) >= s1) s[nt][e] = -INFINITY;
         vd_softmax<KT, DV / 8>(s, o, mrow, lrow, f);
-        vd_pv<KT, DV>(s, o, sV, ldv, lane);
+        vd_pv<KT, DV>(s, o, one_row ? sK : sV, ldv, lane);
         __syncwarp();
     }
 #pragma unroll
@@ -348,11 +413,11 @@ static int launch_vd(const AttnArgs& a, int max_q, cudaStream_t s) {
         configured = true;
     }
     if (max_q > 0) {
-        const size_t smem = (size_t)(64 * ldk + 2 * 64 * (ldk + ldv)) * sizeof(bf16);
+        const size_t smem = (size_t)(64 * ldk + 2 * 64 * (a.kv_scale ? ldk + 2 : ldk + ldv)) * sizeof(bf16);       // (a factor per row: two elements)
         TSB_CHECK_CUDA(tsb_launch(attn_prefill_vd_kernel<DV>, dim3((max_q + 63) / 64, a.Hq, a.B), dim3(128), smem, s, a));
     } else {
         const int chunks = (a.Hq / a.Hkv + 15) / 16;
-        const size_t stage = (size_t)(16 * ldk + 4 * 32 * (ldk + ldv)) * sizeof(bf16), merge = (size_t)(128 + 4 * 16 * DV) * sizeof(float);
+        const size_t stage = (size_t)(16 * ldk + 4 * 32 * (a.kv_scale ? ldk : ldk + ldv)) * sizeof(bf16), merge = (size_t)(128 + 4 * 16 * DV) * sizeof(float);
         TSB_CHECK_CUDA(tsb_launch(attn_decode_vd_kernel<DV>, dim3(a.splits, a.Hkv * chunks, a.B), dim3(128), stage > merge ? stage : merge, s,
                                   a, chunks));
     }
@@ -365,6 +430,9 @@ static int dispatch_vd(const AttnArgs& in, int max_q, cudaStream_t s) {
     if (a.Dv == 0) a.Dv = a.Dh;
     if (a.k_ld == 0) a.k_ld = (long)a.Hkv * a.Dh;
     if (a.v_ld == 0) a.v_ld = (long)a.Hkv * a.Dv;
+    TSB_CHECK_ARG(a.kv_scale == 0 || (a.Dv == a.Dh && a.kv_scale % 2 == 0), "attention: rows of %d / %d elements are not key and value at once", a.Dh, a.Dv);
+    TSB_CHECK_ARG(a.keep_first >= 0 && (a.keep_first == 0 || a.window > 0), "attention: kept first positions without a window");
+    TSB_CHECK_ARG(a.split_len == 0 || a.window <= 0, "attention: fixed splits with a window");
     TSB_CHECK_ARG(a.k_ld % 8 == 0 && a.v_ld % 8 == 0, "attention: cache rows of %ld / %ld elements are not 16-byte aligned", a.k_ld, a.v_ld);
     if (a.Dh <= 0 || a.Dh > 256 || a.Dh % 16 || a.Dv <= 0 || a.Dv > 256 || a.Dv % 16) {
         tsb_set_error("attention: unsupported head sizes %d / %d (multiples of 16 up to 256, or 512 with equal sizes)", a.Dh, a.Dv);

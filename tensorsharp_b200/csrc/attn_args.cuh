@@ -39,14 +39,30 @@ struct AttnArgs {
     // Elements between slots where the rows of a slot are not dense (attention_vd.cu and the 32-bit kernel): 0 = Hkv * Dh
     // and Hkv * Dv.  Multiples of 8.
     long k_ld, v_ld;
+    // The forms below are served by attention_vd.cu and the 32-bit kernel.
+    int keep_first;           // with a window: these first positions stay visible as well
+    const float* slopes;      // [Hq] or null: slopes[h] * (query position - key position) is taken off the scaled score
+    int gate_cols;            // 1: the gate has a value per output column, gate[t * gate_tok + h * Dv + d]
+    int kv_scale;             // != 0: a row of k_cache is key and value at once (Dv = Dh; v_cache is not read), and the score of a
+                              // key is multiplied by the f32 number that starts at element kv_scale of its row
 };
 
+// Whether only the kernels for head sizes of their own know a form that these arguments ask for.
+static inline bool attn_needs_vd(const AttnArgs& a) {
+    return (a.Dv != 0 && a.Dv != a.Dh) || a.k_ld != 0 || a.v_ld != 0 || a.keep_first > 0 || a.slopes != nullptr || a.gate_cols || a.kv_scale ||
+           (a.Dh != 64 && a.Dh != 128 && a.Dh != 256 && a.Dh != 512);
+}
+
 #ifdef __CUDACC__
-__device__ __forceinline__ float attn_gate(const AttnArgs& a, long t, int h) {
+// the gate of head h, or with gate_cols of its column d
+__device__ __forceinline__ float attn_gate(const AttnArgs& a, long t, int h, int d = 0) {
     if (a.gate == nullptr) return 1.f;
-    const float g = a.gate_f32 ? reinterpret_cast<const float*>(a.gate)[t * a.gate_tok + h]
-                               : bf2f(reinterpret_cast<const bf16*>(a.gate)[t * a.gate_tok + h]);
+    const long i = t * a.gate_tok + (a.gate_cols ? (long)h * a.Dv + d : h);
+    const float g = a.gate_f32 ? reinterpret_cast<const float*>(a.gate)[i] : bf2f(reinterpret_cast<const bf16*>(a.gate)[i]);
     return 1.f / (1.f + __expf(-g));
+}
+__device__ __forceinline__ const float* attn_key_factor(const AttnArgs& a, long slot) {
+    return reinterpret_cast<const float*>(a.k_cache + slot * a.k_ld + a.kv_scale);
 }
 #endif
 

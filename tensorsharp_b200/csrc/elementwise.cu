@@ -263,6 +263,33 @@ extern "C" int tsb_rope_table(const int* pos, const RopeParams* rp, const float*
     return TSB_OK;
 }
 
+// ------------------------------------------------------------------------------------------
+// (cos, sin) of position * freq per (token, pair).  The angle is formed and reduced to one turn in double precision: in
+// f32 the product alone is off by 3e-5 at position 1000.  Both are multiplied by `gain`.
+// ------------------------------------------------------------------------------------------
+__global__ void rotary_table_kernel(const int* pos, const double* freq, float2* out, int T, int half, float gain) {
+    pdl_wait();
+    pdl_trigger();
+    const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (long)T * half) return;
+    constexpr double TURN = 6.283185307179586476925;
+    double a = (double)pos[i / half] * freq[i % half];
+    a -= TURN * rint(a / TURN);
+    float s, c;
+    sincosf((float)a, &s, &c);
+    out[i] = make_float2(c * gain, s * gain);
+}
+
+extern "C" int tsb_rotary_table(const int* pos, const double* freq, void* out, int T, int half, float gain, void* stream) {
+    TSB_CHECK_ARG(T >= 0 && half >= 0, "rotary_table: T=%d half=%d", T, half);
+    const long n = (long)T * half;
+    if (n == 0) return TSB_OK;
+    TSB_CHECK_CUDA(tsb_launch(rotary_table_kernel, dim3((unsigned)((n + 127) / 128)), dim3(128), 0, (cudaStream_t)stream, pos, freq, (float2*)out,
+                              T, half, gain));
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}
+
 __device__ __forceinline__ void rope_lookup(const QkvArgs& a, int t, int pair, float pos, float& c, float& s) {
     if (a.cs_table) {
         const float2 cs = a.cs_table[(long)t * (a.rp.rot_dim >> 1) + pair];
@@ -413,9 +440,104 @@ extern "C" int tsb_qkv_rope(const QkvArgs* args, void* stream) {
 }
 
 // ------------------------------------------------------------------------------------------
+// Query and key norms over whole projections (all heads together), for attention whose values are the keys ahead of their
+// norm: a cached row is [keys as projected | f32 factor 1 / rms of the row | zeros], and the keys' norm weight is multiplied
+// into the queries, so that (q rms_q^-1 w) . k times the row's factor is the score of the two normed vectors.
+// One block per token; rows of y are [q (H * Dh) | k (G * Dh)], heads padded with zeros.
+// ------------------------------------------------------------------------------------------
+struct JointNormArgs {
+    const void* y; long y_s; int y_f32;
+    const float* w;           // [H * Dh]: query norm weight times the key norm weight of the head's key head
+    const long* slot;         // [T]
+    void* q;                  // [T, H * Dh]
+    void* cache;              // rows of ld elements
+    long ld;
+    int T, nq, nk;            // H * Dh, G * Dh
+    int q_n, k_n;             // the same without padding: the norms' divisors
+    int out_f32;              // 1: q and the cache are float
+    float eps;
+};
+
+__device__ __forceinline__ float4 jn_ld4(const void* p, long at, int f32) {
+    if (f32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + at);
+    const uint2 r = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(p) + at);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const bf162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const bf162*>(&r.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void jn_st4(void* p, long at, int f32, float4 v) {
+    if (f32) {
+        *reinterpret_cast<float4*>(reinterpret_cast<float*>(p) + at) = v;
+    } else {
+        uint2 r;
+        *reinterpret_cast<bf162*>(&r.x) = __floats2bfloat162_rn(v.x, v.y);
+        *reinterpret_cast<bf162*>(&r.y) = __floats2bfloat162_rn(v.z, v.w);
+        *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(p) + at) = r;
+    }
+}
+
+__global__ void __launch_bounds__(512) joint_norm_kernel(JointNormArgs a) {
+    constexpr int HELD = 4;                                  // float4s of the queries a thread keeps; the rest is read again
+    __shared__ float red[32];
+    pdl_wait();
+    pdl_trigger();
+    const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+    const long row = t * a.y_s, dst = a.slot[t] * a.ld;
+    float4 v[HELD];
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int j = 0; j < HELD; ++j) {
+        const int i = tid + j * nt;
+        v[j] = 4 * i < a.nq ? jn_ld4(a.y, row + 4 * i, a.y_f32) : make_float4(0.f, 0.f, 0.f, 0.f);
+        sq += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+    }
+    for (int i = tid + HELD * nt; 4 * i < a.nq; i += nt) {
+        const float4 x = jn_ld4(a.y, row + 4 * i, a.y_f32);
+        sq += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+    }
+    for (int i = tid; 4 * i < a.nk; i += nt) {
+        const float4 x = jn_ld4(a.y, row + a.nq + 4 * i, a.y_f32);
+        sk += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+        jn_st4(a.cache, dst + 4 * i, a.out_f32, x);
+    }
+    sq = block_sum(sq, red);
+    sk = block_sum(sk, red);
+    const float rq = 1.f / sqrtf(sq / (float)a.q_n + a.eps);
+    auto put = [&](int i, float4 x) {
+        const float4 w = reinterpret_cast<const float4*>(a.w)[i];
+        jn_st4(a.q, (long)t * a.nq + 4 * i, a.out_f32, make_float4(x.x * rq * w.x, x.y * rq * w.y, x.z * rq * w.z, x.w * rq * w.w));
+    };
+#pragma unroll
+    for (int j = 0; j < HELD; ++j)
+        if (4 * (tid + j * nt) < a.nq) put(tid + j * nt, v[j]);
+    for (int i = tid + HELD * nt; 4 * i < a.nq; i += nt) put(i, jn_ld4(a.y, row + 4 * i, a.y_f32));
+    if (tid < 8) {
+        // the tail of the row: 16 bytes of bf16 elements, 32 of float
+        const float f = 1.f / sqrtf(sk / (float)a.k_n + a.eps);
+        if (a.out_f32) reinterpret_cast<float*>(a.cache)[dst + a.nk + tid] = tid == 0 ? f : 0.f;
+        else if (tid < 4) reinterpret_cast<float*>(reinterpret_cast<bf16*>(a.cache) + dst + a.nk)[tid] = tid == 0 ? f : 0.f;
+    }
+}
+
+extern "C" int tsb_joint_norm(const JointNormArgs* args, void* stream) {
+    const JointNormArgs& a = *args;
+    TSB_CHECK_ARG(a.nq > 0 && a.nk > 0 && a.nq % 8 == 0 && a.nk % 8 == 0 && a.q_n > 0 && a.k_n > 0 && a.y_s % 4 == 0 && a.ld == a.nk + 8,
+                  "joint_norm: %d query and %d key columns, cache rows of %ld", a.nq, a.nk, a.ld);
+    if (a.T == 0) return TSB_OK;
+    const int vecs = a.nq / 4, per = a.T < 296 ? 1 : 4;               // few rows: one float4 per thread, for latency
+    int nt = ((vecs + per - 1) / per + 31) & ~31;
+    nt = nt < 64 ? 64 : nt > 512 ? 512 : nt;
+    TSB_CHECK_CUDA(tsb_launch(joint_norm_kernel, dim3(a.T), dim3(nt), 0, (cudaStream_t)stream, a));
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}
+
+// ------------------------------------------------------------------------------------------
 // Gated activation: out[t, f] = act(gate[t, f] (+bg[f])) * (up[t, f] (+bu[f])), optional q8 output.
 // ------------------------------------------------------------------------------------------
-__device__ __forceinline__ float glu_apply(int act, float g, float u) {
+// Clamp of activation 4: `first` for the rows below `rows`, `lim` for the others.
+struct GluClamp { float lim, first; long rows; };
+
+__device__ __forceinline__ float glu_apply(int act, float g, float u, float lim) {
     switch (act) {
     case 1: return g / (1.f + __expf(-g)) * u;
     case 2: {
@@ -424,7 +546,7 @@ __device__ __forceinline__ float glu_apply(int act, float g, float u) {
     }
     case 3: return 0.5f * g * (1.f + erff(g * 0.7071067811865476f)) * u;
     case 4: {
-        const float x = fminf(g, 7.f), y = fminf(fmaxf(u, -7.f), 7.f);
+        const float x = fminf(g, lim), y = fminf(fmaxf(u, -lim), lim);
         return x / (1.f + __expf(-1.702f * x)) * (y + 1.f);
     }
     case 5: { const float r = fmaxf(g, 0.f); return r * r; }             // ReLU^2 (no gate)
@@ -435,7 +557,7 @@ __device__ __forceinline__ float glu_apply(int act, float g, float u) {
 }
 
 // 32-bit in and out (models that run in float32).
-__global__ void glu_f32_kernel(const float* gate, const float* up, long g_stride, long u_stride, int F, int act, float* out, long rows) {
+__global__ void glu_f32_kernel(const float* gate, const float* up, long g_stride, long u_stride, int F, int act, float* out, long rows, GluClamp cl) {
     pdl_wait();
     pdl_trigger();
     const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -443,15 +565,22 @@ __global__ void glu_f32_kernel(const float* gate, const float* up, long g_stride
     const long t = idx / F;
     const int f = (int)(idx % F);
     const float g = gate[t * g_stride + f], u = up ? up[t * u_stride + f] : 0.f;
-    out[idx] = act == 1 ? g / (1.f + expf(-g)) * u : glu_apply(act, g, u);
+    if (act == 1) {
+        out[idx] = g / (1.f + expf(-g)) * u;
+    } else if (act == 4) {
+        const float lim = t < cl.rows ? cl.first : cl.lim, x = fminf(g, lim), y = fminf(fmaxf(u, -lim), lim);
+        out[idx] = x / (1.f + expf(-1.702f * x)) * (y + 1.f);
+    } else {
+        out[idx] = glu_apply(act, g, u, cl.lim);
+    }
 }
 
 extern "C" int tsb_glu_f32(const float* gate, const float* up, long g_stride, long u_stride, long rows, int F, int act, float* out,
-                           void* stream) {
+                           float lim, float lim_first, long rows_first, void* stream) {
     TSB_CHECK_ARG(gate && out && rows >= 0 && F >= 0, "glu_f32: bad shape rows=%ld F=%d", rows, F);
     if (rows == 0 || F == 0) return TSB_OK;
     TSB_CHECK_CUDA(tsb_launch(glu_f32_kernel, dim3((unsigned)((rows * F + 255) / 256)), dim3(256), 0, (cudaStream_t)stream, gate, up,
-                              g_stride, u_stride, F, act, out, rows));
+                              g_stride, u_stride, F, act, out, rows, GluClamp{lim, lim_first, rows_first}));
     TSB_CHECK_LAUNCH();
     return TSB_OK;
 }
@@ -474,7 +603,7 @@ extern "C" int tsb_softcap(const float* x, float* out, long n, float cap, void* 
 
 template <typename T>
 __global__ void glu_kernel(const T* gate, const T* up, long g_stride, long u_stride, int F, int act, bf16* out,
-                           int8_t* yq, float2* yds, long rows) {
+                           int8_t* yq, float2* yds, long rows, GluClamp cl) {
     pdl_wait();
     pdl_trigger();
     const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -487,7 +616,7 @@ __global__ void glu_kernel(const T* gate, const T* up, long g_stride, long u_str
     if (f < F) {
         const float g = (float)gate[t * g_stride + f];
         const float u = up ? (float)up[t * u_stride + f] : 0.f;
-        r = glu_apply(act, g, u);
+        r = glu_apply(act, g, u, t < cl.rows ? cl.first : cl.lim);
         if (out) out[t * F + f] = f2bf(r);
     }
     if (yq) {
@@ -501,12 +630,13 @@ __global__ void glu_kernel(const T* gate, const T* up, long g_stride, long u_str
 
 // Long bf16 inputs (prompts): eight columns per thread, 16-byte loads and stores.
 __global__ void __launch_bounds__(256) glu_vec_kernel(const bf16* gate, const bf16* up, long g_stride, long u_stride, int F8, int act,
-                                                      bf16* out, unsigned total) {
+                                                      bf16* out, unsigned total, GluClamp cl) {
     pdl_wait();
     pdl_trigger();
     const unsigned idx = blockIdx.x * 256u + threadIdx.x;
     if (idx >= total) return;
     const unsigned t = idx / (unsigned)F8, c = (idx - t * F8) * 8;
+    const float lim = (long)t < cl.rows ? cl.first : cl.lim;
     const uint4 gv = *reinterpret_cast<const uint4*>(gate + (long)t * g_stride + c);
     const uint4 uv = up ? *reinterpret_cast<const uint4*>(up + (long)t * u_stride + c) : make_uint4(0u, 0u, 0u, 0u);
     const bf162* g2 = reinterpret_cast<const bf162*>(&gv);
@@ -516,13 +646,14 @@ __global__ void __launch_bounds__(256) glu_vec_kernel(const bf16* gate, const bf
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const float2 g = __bfloat1622float2(g2[i]), u = __bfloat1622float2(u2[i]);
-        o2[i] = __floats2bfloat162_rn(glu_apply(act, g.x, u.x), glu_apply(act, g.y, u.y));
+        o2[i] = __floats2bfloat162_rn(glu_apply(act, g.x, u.x, lim), glu_apply(act, g.y, u.y, lim));
     }
     reinterpret_cast<uint4*>(out)[idx] = ov;
 }
 
 extern "C" int tsb_glu(const void* gate, const void* up, int in_f32, long g_stride, long u_stride, long rows, int F,
-                       int act, void* out, void* yq, void* yds, void* stream) {
+                       int act, void* out, void* yq, void* yds, float lim, float lim_first, long rows_first, void* stream) {
+    const GluClamp cl{lim, lim_first, rows_first};
     TSB_CHECK_ARG(!yq || F % 32 == 0, "glu: q8 output needs F %% 32 == 0, got %d", F);
     if (rows == 0 || F == 0) return TSB_OK;
     const long total = rows * ((F + 31) & ~31);
@@ -532,16 +663,16 @@ extern "C" int tsb_glu(const void* gate, const void* up, int in_f32, long g_stri
     if (!in_f32 && !yq && out && aligned && F % 8 == 0 && g_stride % 8 == 0 && u_stride % 8 == 0 && rows * (F / 8) < (1L << 31)) {
         const unsigned n = (unsigned)(rows * (F / 8));
         TSB_CHECK_CUDA(tsb_launch(glu_vec_kernel, dim3((n + 255) / 256), dim3(256), 0, s, (const bf16*)gate, (const bf16*)up, g_stride, u_stride,
-                                  F / 8, act, (bf16*)out, n));
+                                  F / 8, act, (bf16*)out, n, cl));
         TSB_CHECK_LAUNCH();
         return TSB_OK;
     }
     if (in_f32)
         TSB_CHECK_CUDA(tsb_launch(glu_kernel<float>, grid, dim3(256), 0, s, (const float*)gate, (const float*)up, g_stride,
-                                  u_stride, F, act, (bf16*)out, (int8_t*)yq, (float2*)yds, rows));
+                                  u_stride, F, act, (bf16*)out, (int8_t*)yq, (float2*)yds, rows, cl));
     else
         TSB_CHECK_CUDA(tsb_launch(glu_kernel<bf16>, grid, dim3(256), 0, s, (const bf16*)gate, (const bf16*)up, g_stride,
-                                  u_stride, F, act, (bf16*)out, (int8_t*)yq, (float2*)yds, rows));
+                                  u_stride, F, act, (bf16*)out, (int8_t*)yq, (float2*)yds, rows, cl));
     TSB_CHECK_LAUNCH();
     return TSB_OK;
 }
@@ -586,6 +717,72 @@ extern "C" int tsb_gather_rows(const void* p0, const void* p1, const void* p2, c
         TSB_CHECK_CUDA(tsb_launch(gather_rows_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, w, ids, n_rows, scale, (float*)out));
     else
         TSB_CHECK_CUDA(tsb_launch(gather_rows_kernel<bf16>, grid, dim3(256), 0, (cudaStream_t)stream, w, ids, n_rows, scale, (bf16*)out));
+    TSB_CHECK_LAUNCH();
+    return TSB_OK;
+}
+
+// ------------------------------------------------------------------------------------------
+// Embedding with a bigram table: h[t] = token row + pair row (previous * mul_prev + current * mul_cur) mod buckets, the last
+// row of the pair table where a sequence begins.  The token ahead of a sequence's first one in the batch is in `prev` (int32
+// per slot, negative: none); the block that reads it leaves the sequence's last token there.  One block per token.
+// ------------------------------------------------------------------------------------------
+struct PairEmbedArgs {
+    QW tok, pair;             // [vocab, D], [buckets + 1, D]
+    const int* ids; const int* cu_q; const long* seq_slots;
+    int* prev;
+    float* h;                 // [T, D]
+    void* out;                // the same as the next product's input (bf16 or f32), or null
+    int T, B, out_f32;
+    long buckets, mul_prev, mul_cur;
+};
+
+__global__ void __launch_bounds__(256) pair_embed_kernel(PairEmbedArgs a) {
+    pdl_wait();
+    pdl_trigger();
+    const int t = blockIdx.x;
+    int lo = 0, hi = a.B - 1;                                 // the sequence that holds row t
+    while (lo < hi) {
+        const int mid = (lo + hi + 1) >> 1;
+        if (a.cu_q[mid] <= t) lo = mid; else hi = mid - 1;
+    }
+    const long cur = a.ids[t];
+    long before;
+    if (t == a.cu_q[lo]) {
+        int* slot = a.prev + a.seq_slots[lo];
+        before = *slot;
+        __syncthreads();                                      // every thread has read it
+        if (threadIdx.x == 0) *slot = a.ids[a.cu_q[lo + 1] - 1];
+    } else {
+        before = a.ids[t - 1];
+    }
+    long pair = before < 0 ? a.buckets : (before * a.mul_prev + cur * a.mul_cur) % a.buckets;
+    if (pair < 0) pair += a.buckets;
+    const long row = cur < 0 || cur >= a.tok.N ? 0 : cur;
+    for (int k8 = threadIdx.x; k8 < a.tok.K >> 3; k8 += blockDim.x) {
+        float x[8], y[8];
+        dequant8(a.tok, row, k8, x);
+        dequant8(a.pair, pair, k8, y);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) x[i] += y[i];
+        const long at = (long)t * a.tok.K + 8 * k8;
+        *reinterpret_cast<float4*>(a.h + at) = make_float4(x[0], x[1], x[2], x[3]);
+        *reinterpret_cast<float4*>(a.h + at + 4) = make_float4(x[4], x[5], x[6], x[7]);
+        if (a.out == nullptr) continue;
+        jn_st4(a.out, at, a.out_f32, make_float4(x[0], x[1], x[2], x[3]));
+        jn_st4(a.out, at + 4, a.out_f32, make_float4(x[4], x[5], x[6], x[7]));
+    }
+}
+
+extern "C" int tsb_pair_embed(const void* tok, const void* pair, int type, int vocab, int D, const int* ids, const int* cu_q, const long* seq_slots,
+                              int* prev, float* h, void* out, int out_f32, int T, int B, long buckets, long mul_prev, long mul_cur, void* stream) {
+    TSB_CHECK_ARG(D > 0 && D % 8 == 0 && vocab > 0 && buckets > 0 && B > 0, "pair_embed: D=%d vocab=%d buckets=%ld", D, vocab, buckets);
+    TSB_CHECK_ARG(type == TSB_BF16 || type == TSB_F32, "pair_embed: table type %d", type);
+    if (T == 0) return TSB_OK;
+    PairEmbedArgs a{QW{(const uint8_t*)tok, nullptr, nullptr, nullptr, type, vocab, D}, QW{(const uint8_t*)pair, nullptr, nullptr, nullptr, type, (int)buckets + 1, D},
+                    ids, cu_q, seq_slots, prev, h, out, T, B, out_f32, buckets, mul_prev, mul_cur};
+    int nt = (D / 8 + 31) & ~31;
+    nt = nt > 256 ? 256 : nt;
+    TSB_CHECK_CUDA(tsb_launch(pair_embed_kernel, dim3(T), dim3(nt), 0, (cudaStream_t)stream, a));
     TSB_CHECK_LAUNCH();
     return TSB_OK;
 }

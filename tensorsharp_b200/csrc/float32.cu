@@ -113,21 +113,26 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnArgs a) {
     for (int d = threadIdx.x; d < a.Dh; d += 128) sq[d] = q[d];
     __syncthreads();
     const int pos = a.kv_lens[b] - (a.cu_q[b + 1] - t);                   // this row's position
-    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    // the visible positions, numbered without a gap: the kept first ones ahead of the window, then the window
+    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0, nf = min(a.keep_first, lo), gap = lo - nf, last = pos - gap;
+    const float slope = a.slopes ? a.slopes[h] : 0.f;
+    const bool one_row = a.kv_scale != 0;
     float m = -INFINITY, l = 0.f, acc[NJ];
 #pragma unroll
     for (int j = 0; j < NJ; ++j) acc[j] = 0.f;
-    for (int base = lo + warp * 32; base <= pos; base += 128) {
-        const int j = base + lane;
-        const bool ok = j <= pos;
+    for (int base = warp * 32; base <= last; base += 128) {
+        const int i = base + lane, j = i < nf ? i : i + gap;
+        const bool ok = i <= last;
         const long slot = ok ? (long)a.block_table[(long)b * a.max_pages + j / a.page_size] * a.page_size + j % a.page_size : 0;
         float s = -INFINITY;
         if (ok) {
             s = 0.f;
             const float* kp = kc + slot * a.k_ld + hk * a.Dh;
             for (int d = 0; d < a.Dh; ++d) s = fmaf(sq[d], kp[d], s);
+            if (one_row) s *= kc[slot * a.k_ld + a.kv_scale];
             s *= a.scale;
             if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+            s = fmaf(slope, (float)(j - pos), s);
         }
         const float mx = fmaxf(m, warp_max(s));
         const float corr = m == -INFINITY ? 0.f : expf(m - mx);
@@ -136,11 +141,11 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnArgs a) {
         m = mx;
 #pragma unroll
         for (int i = 0; i < NJ; ++i) acc[i] *= corr;
-        const int cnt = min(32, pos - base + 1);
+        const int cnt = min(32, last - base + 1);
         for (int u = 0; u < cnt; ++u) {
             const float pu = __shfl_sync(0xffffffffu, p, u);
             const long su = __shfl_sync(0xffffffffu, slot, u);
-            const float* vp = vc + su * a.v_ld + hk * a.Dv;
+            const float* vp = one_row ? kc + su * a.k_ld + hk * a.Dh : vc + su * a.v_ld + hk * a.Dv;
 #pragma unroll
             for (int i = 0; i < NJ; ++i) {
                 const int d = lane + 32 * i;
@@ -163,10 +168,12 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnArgs a) {
         ll += sml[w][1] * c[w];
     }
     float g = 1.f;
-    if (a.gate != nullptr) g = 1.f / (1.f + expf(-reinterpret_cast<const float*>(a.gate)[(long)t * a.gate_tok + h]));
+    const float* gate = reinterpret_cast<const float*>(a.gate);
+    if (gate != nullptr && !a.gate_cols) g = 1.f / (1.f + expf(-gate[(long)t * a.gate_tok + h]));
     float* out = reinterpret_cast<float*>(a.out) + ((long)t * a.Hq + h) * a.Dv;
     for (int d = threadIdx.x; d < a.Dv; d += 128) {
         const float o = so[d] * c[0] + so[a.Dv + d] * c[1] + so[2 * a.Dv + d] * c[2] + so[3 * a.Dv + d] * c[3];
+        if (a.gate_cols) g = 1.f / (1.f + expf(-gate[(long)t * a.gate_tok + h * a.Dv + d]));
         out[d] = o / ll * g;
     }
 }
@@ -178,6 +185,8 @@ extern "C" int tsb_attn_f32(const AttnArgs* args, int T, void* stream) {
     if (a.v_ld == 0) a.v_ld = (long)a.Hkv * a.Dv;
     TSB_CHECK_ARG(a.Hkv > 0 && a.Hq % a.Hkv == 0 && a.cu_q != nullptr, "attn_f32: Hq=%d Hkv=%d", a.Hq, a.Hkv);
     TSB_CHECK_ARG(a.Dh > 0 && a.Dh <= 1024 && a.Dv > 0 && a.Dv <= ATTN_F32_MAX_DV, "attn_f32: head sizes %d / %d", a.Dh, a.Dv);
+    TSB_CHECK_ARG(a.kv_scale == 0 || a.Dv == a.Dh, "attn_f32: rows of %d / %d elements are not key and value at once", a.Dh, a.Dv);
+    TSB_CHECK_ARG(a.gate != nullptr || !a.gate_cols, "attn_f32: no gate given");
     TSB_CHECK_ARG(a.gate == nullptr || a.gate_f32, "attn_f32: the gate must be float32");
     if (T == 0) return TSB_OK;
     cudaStream_t s = (cudaStream_t)stream;

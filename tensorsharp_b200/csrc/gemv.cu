@@ -324,6 +324,11 @@ extern "C" int tsb_gemv_push(const void* p0, const void* p1, const void* p2, con
                              const void* residual, const int* ids, const float* row_scale, int M, int problems,
                              int x_div, int out_f32, int act, const void* push, void* stream);
 
+extern "C" int tsb_gemv_clamped(const void* p0, const void* p1, const void* p2, const void* p3, int type, int N, int K,
+                                const void* xq, const void* xds, const void* xb, void* out, const float* bias,
+                                const void* residual, const int* ids, const float* row_scale, int M, int problems,
+                                int x_div, int out_f32, int act, const void* push, float lim, float lim_first, int n_first, void* stream);
+
 // out = act(W x + bias) * row_scale + residual.  See GemvArgs for the meaning of each field.
 extern "C" int tsb_gemv(const void* p0, const void* p1, const void* p2, const void* p3, int type, int N, int K,
                         const void* xq, const void* xds, const void* xb, void* out, const float* bias,
@@ -340,6 +345,16 @@ extern "C" int tsb_gemv_push(const void* p0, const void* p1, const void* p2, con
                              const void* xq, const void* xds, const void* xb, void* out, const float* bias,
                              const void* residual, const int* ids, const float* row_scale, int M, int problems,
                              int x_div, int out_f32, int act, const void* push, void* stream) {
+    return tsb_gemv_clamped(p0, p1, p2, p3, type, N, K, xq, xds, xb, out, bias, residual, ids, row_scale, M, problems, x_div, out_f32, act, push,
+                            7.f, 7.f, 0, stream);
+}
+
+// Same with the clamp of ACT_SWIGLU_OAI given: `lim_first` for the experts below n_first (a shared expert's slices), `lim` for
+// the others.  Other limits than 7 need bf16 weights.
+extern "C" int tsb_gemv_clamped(const void* p0, const void* p1, const void* p2, const void* p3, int type, int N, int K,
+                                const void* xq, const void* xds, const void* xb, void* out, const float* bias,
+                                const void* residual, const int* ids, const float* row_scale, int M, int problems,
+                                int x_div, int out_f32, int act, const void* push, float lim, float lim_first, int n_first, void* stream) {
     TSB_CHECK_ARG(N > 0 && K > 0 && M >= 0, "gemv: bad shape N=%d K=%d M=%d", N, K, M);
     TSB_CHECK_ARG(!push || (!residual && act == 0), "gemv: push mode takes no residual / act");
     TSB_CHECK_ARG(!push || ids || !row_scale, "gemv: push mode takes a row scale only with expert ids");
@@ -358,7 +373,9 @@ extern "C" int tsb_gemv_push(const void* p0, const void* p1, const void* p2, con
     a.M = M; a.x_div = x_div > 0 ? x_div : 1; a.out_f32 = out_f32; a.act = act;
     a.n_out = glu ? N / 2 : N;
     a.push = (const TpPush*)push;
+    a.lim = lim; a.lim_first = lim_first; a.n_first = n_first;
     if (tsb_gemv_bf16_eligible(a)) return tsb_gemv_bf16_launch(a, glu, problems, (cudaStream_t)stream);
+    TSB_CHECK_ARG(act != ACT_SWIGLU_OAI || (lim == 7.f && n_first == 0), "gemv: clamp %f for weight type %d", lim, type);
     if (tsb_gemv_mma_eligible(a)) return tsb_gemv_mma_launch(a, glu, (cudaStream_t)stream);
     if (tsb_gemv_stream_eligible(a)) return tsb_gemv_stream_launch(a, glu, (cudaStream_t)stream);
     return glu ? launch_gemv<true>(a, problems, (cudaStream_t)stream)

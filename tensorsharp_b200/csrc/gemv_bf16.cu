@@ -45,7 +45,7 @@ __global__ void __launch_bounds__(128) gemv_bf16_kernel(GemvArgs a) {
         float v = acc[m];
         if (a.bias) v += a.bias[wrow];
         if (GLU) {
-            v = act_glu(a.act, v, acc2[m] + (a.bias ? a.bias[wrow + a.n_out] : 0.f));
+            v = act_glu(a.act, v, acc2[m] + (a.bias ? a.bias[wrow + a.n_out] : 0.f), expert < a.n_first ? a.lim_first : a.lim);
         } else if (a.act == ACT_RELU2) {
             v = fmaxf(v, 0.f);
             v = v * v;

@@ -9,7 +9,8 @@
 enum { ACT_NONE = 0, ACT_SWIGLU = 1, ACT_GEGLU_TANH = 2, ACT_GEGLU_ERF = 3, ACT_SWIGLU_OAI = 4,
        ACT_RELU2 = 5, ACT_SILU = 6 };
 
-__device__ __forceinline__ float act_glu(int act, float g, float u) {
+// `lim`: clamp of the OAI form
+__device__ __forceinline__ float act_glu(int act, float g, float u, float lim = 7.f) {
     switch (act) {
     case ACT_SWIGLU: return g / (1.f + __expf(-g)) * u;
     case ACT_GEGLU_TANH: {
@@ -19,7 +20,7 @@ __device__ __forceinline__ float act_glu(int act, float g, float u) {
     }
     case ACT_GEGLU_ERF: return 0.5f * g * (1.f + erff(g * 0.7071067811865476f)) * u;
     case ACT_SWIGLU_OAI: {
-        float x = fminf(g, 7.f), y = fminf(fmaxf(u, -7.f), 7.f);
+        float x = fminf(g, lim), y = fminf(fmaxf(u, -lim), lim);
         return x / (1.f + __expf(-1.702f * x)) * (y + 1.f);
     }
     default: return g * u;
@@ -43,6 +44,9 @@ struct GemvArgs {
     int n_out;             // N, or N/2 with GLU
     const TpPush* push;    // tensor-parallel exchange: store the f32 result into every rank's mailbox
                            // instead of `out` (see tp_fused.cuh); null for an ordinary GEMV
+    // clamp of ACT_SWIGLU_OAI, read by the bf16 kernel: `lim_first` for the experts below n_first, `lim` for the others
+    float lim = 7.f, lim_first = 7.f;
+    int n_first = 0;
 };
 
 // Each quantised type is split into a weight *load* (global, streaming, independent of the

@@ -30,13 +30,49 @@
 // mode 0: top-k of the logits, weights = softmax over the selected logits.
 // mode 1: p = sigmoid(logit); select on p + sel_bias; weights = p, optionally / max(sum, 6.1e-5); * scale.
 // mode 2: s = softmax over all logits; select the k largest; weights = s / (their sum + 1e-20) * scale.
-// `always` > 0 (any mode): experts E .. E + always - 1 follow the k selected ones with the weight sigmoid(logit[E])
+// mode 3: s = softmax over all logits; select on s + sel_bias, only in the `keep` best of `groups` equal groups of neighbours (a
+// group is as good as its best choice score); weights = s * scale, not renormalised.  Entries from n_real on are identity
+// experts (the layer's input itself): their id is -1.  `always` here: the ids 0 .. always - 1 come first on every token with
+// weight 1 (slices of a shared expert), and the routed experts' ids start at `always`.
+// `always` > 0 (modes 0 to 2): experts E .. E + always - 1 follow the k selected ones with the weight sigmoid(logit[E])
 // (a gated shared expert, cut into slices); a row of logits is `ld` long.
 // ---------------------------------------------------------------------------------------------
+struct RouteGroups { int groups, keep, n_real; };
+
+// Mode 3: the choice scores of the entries whose group is not among the best become -inf.  `sh`: 2 x MOE_MAX_E floats of this warp.
+template <int PER>
+__device__ __forceinline__ void keep_best_groups(float (&sel)[PER], int E, const RouteGroups& rg, float* sh, int lane) {
+    const int size = E / rg.groups;
+    float* gs = sh + MOE_MAX_E;                                   // score per group
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+        if (i * 32 + lane < E) sh[i * 32 + lane] = sel[i];
+    __syncwarp();
+    for (int g = lane; g < rg.groups; g += 32) {
+        float m = -INFINITY;
+        for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, sh[e]);
+        gs[g] = m;
+    }
+    __syncwarp();
+    for (int g = lane; g < rg.groups; g += 32) {                  // a group is kept when fewer than `keep` are ahead of it
+        const float m = gs[g];
+        int ahead = 0;
+        for (int o = 0; o < rg.groups; ++o) ahead += gs[o] > m || (gs[o] == m && o < g);
+        if (ahead >= rg.keep)
+            for (int e = g * size; e < (g + 1) * size; ++e) sh[e] = -INFINITY;
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+        if (i * 32 + lane < E) sel[i] = sh[i * 32 + lane];
+}
+
 template <int PER>
 __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ sel_bias,
                                                         int T, int E, int k, int mode, int normalize, float scale,
-                                                        int ld, int always, int* __restrict__ ids, float* __restrict__ wts) {
+                                                        int ld, int always, RouteGroups rg, int* __restrict__ ids,
+                                                        float* __restrict__ wts) {
+    extern __shared__ float group_sh[];         // mode 3 with groups: [4 warps][2 MOE_MAX_E]
     const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     pdl_wait();
     pdl_trigger();
@@ -63,7 +99,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
     }
     float denom = 1.f;                    // mode 2: the softmax's sum over all experts
     float top = 0.f;
-    if (mode == 2) {
+    if (mode >= 2) {
         float mx = -INFINITY;
 #pragma unroll
         for (int i = 0; i < PER; ++i) mx = fmaxf(mx, sel[i]);
@@ -72,6 +108,17 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
 #pragma unroll
         for (int i = 0; i < PER; ++i) s += sel[i] == -INFINITY ? 0.f : expf(sel[i] - top);
         denom = warp_sum(s);
+    }
+    if (mode == 3) {
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int e = i * 32 + lane;
+            if (e < E) {
+                val[i] = expf(sel[i] - top) / denom;
+                sel[i] = sel_bias ? val[i] + sel_bias[e] : val[i];
+            }
+        }
+        if (rg.keep < rg.groups) keep_best_groups<PER>(sel, E, rg, group_sh + (threadIdx.x >> 5) * 2 * MOE_MAX_E, lane);
     }
     float wk = 0.f;                       // lane j keeps the j-th selected weight
     int ik = 0;
@@ -107,6 +154,17 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
     } else if (mode == 2) {
         const float p = on ? expf(wk - top) / denom : 0.f;
         wk = p / (warp_sum(p) + 1e-20f) * scale;
+    } else if (mode == 3) {
+        const long o = (long)t * (k + always);
+        if (on) {
+            ids[o + always + lane] = ik < rg.n_real ? always + ik : -1;
+            wts[o + always + lane] = wk * scale;
+        }
+        for (int i = lane; i < always; i += 32) {
+            ids[o + i] = i;
+            wts[o + i] = 1.f;
+        }
+        return;
     } else {
         if (normalize) {
             const float s = warp_sum(on ? wk : 0.f);
@@ -128,15 +186,16 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
     }
 }
 
-extern "C" int tsb_moe_route_ex(const float* logits, const float* sel_bias, int T, int E, int k, int mode, int normalize,
-                                float scale, int ld, int always, int* ids, float* wts, void* stream) {
-    TSB_CHECK_ARG(ld >= E + (always > 0 ? 1 : 0) && always >= 0, "moe_route: rows of %d logits for %d experts and %d always on", ld, E, always);
+static int route_launch(const float* logits, const float* sel_bias, int T, int E, int k, int mode, int normalize, float scale, int ld, int always,
+                        RouteGroups rg, int* ids, float* wts, void* stream) {
+    const size_t smem = mode == 3 && rg.keep < rg.groups ? 4 * 2 * MOE_MAX_E * sizeof(float) : 0;
+    TSB_CHECK_ARG(mode == 3 || ld >= E + (always > 0 ? 1 : 0) && always >= 0, "moe_route: rows of %d logits for %d experts and %d always on", ld, E, always);
     TSB_CHECK_ARG(E > 0 && E <= MOE_MAX_E, "moe_route: %d experts (limit %d)", E, MOE_MAX_E);
     TSB_CHECK_ARG(k > 0 && k <= MOE_MAX_K && k <= E, "moe_route: top-%d of %d", k, E);
     if (T == 0) return TSB_OK;
     const dim3 grid((T + 3) / 4), block(128);
     cudaStream_t st = (cudaStream_t)stream;
-#define TSB_ROUTE(P) TSB_CHECK_CUDA(tsb_launch(moe_route_kernel<P>, grid, block, 0, st, logits, sel_bias, T, E, k, mode, normalize, scale, ld, always, ids, wts))
+#define TSB_ROUTE(P) TSB_CHECK_CUDA(tsb_launch(moe_route_kernel<P>, grid, block, smem, st, logits, sel_bias, T, E, k, mode, normalize, scale, ld, always, rg, ids, wts))
     if (E <= 32) TSB_ROUTE(1);
     else if (E <= 128) TSB_ROUTE(4);
     else if (E <= 256) TSB_ROUTE(8);
@@ -144,6 +203,21 @@ extern "C" int tsb_moe_route_ex(const float* logits, const float* sel_bias, int 
 #undef TSB_ROUTE
     TSB_CHECK_LAUNCH();
     return TSB_OK;
+}
+
+extern "C" int tsb_moe_route_ex(const float* logits, const float* sel_bias, int T, int E, int k, int mode, int normalize,
+                                float scale, int ld, int always, int* ids, float* wts, void* stream) {
+    TSB_CHECK_ARG(mode >= 0 && mode <= 2, "moe_route: mode %d", mode);
+    return route_launch(logits, sel_bias, T, E, k, mode, normalize, scale, ld, always, RouteGroups{1, 1, E}, ids, wts, stream);
+}
+
+// Mode 3: E logits per row, the last E - n_real of them identity experts.
+extern "C" int tsb_moe_route_grouped(const float* logits, const float* sel_bias, int T, int E, int n_real, int k, int groups, int keep, float scale,
+                                     int always, int* ids, float* wts, void* stream) {
+    TSB_CHECK_ARG(groups > 0 && E % groups == 0 && keep > 0 && keep <= groups && k <= keep * (E / groups),
+                  "moe_route: top-%d of %d experts in %d of %d groups", k, E, keep, groups);
+    TSB_CHECK_ARG(n_real >= 0 && n_real <= E && always >= 0, "moe_route: %d experts of %d, %d always on", n_real, E, always);
+    return route_launch(logits, sel_bias, T, E, k, 3, 0, scale, E, always, RouteGroups{groups, keep, n_real}, ids, wts, stream);
 }
 
 extern "C" int tsb_moe_route(const float* logits, const float* sel_bias, int T, int E, int k, int mode, int normalize,
@@ -154,6 +228,7 @@ extern "C" int tsb_moe_route(const float* logits, const float* sel_bias, int T, 
 // ---------------------------------------------------------------------------------------------
 // Sorting the (token, slot) pairs by expert for the grouped GEMM, without a host read-back:
 //   order[i]  the pair at sorted place i       pos[p]  the sorted place of pair p
+// Pairs with a negative id have no place: their pos is -1, and as many places at the end have order -1.
 //   tiles     {expert or -1, first place, end place} for pieces of at most bn places of one expert; a fixed number of
 //             entries (ceil(P / bn) + E), the surplus marked -1
 // Pairs of one expert come in no particular order (every row's product is its own).  Up to SORT_ONE_CTA pairs one CTA does
@@ -163,7 +238,7 @@ extern "C" int tsb_moe_route(const float* logits, const float* sel_bias, int T, 
 #define SORT_ONE_CTA 4096
 
 struct SortArgs {
-    const int* ids;          // [P], each in [0, E)
+    const int* ids;          // [P], each in [0, E), or negative: no place
     int* order; int* pos; int* tiles;
     int* counts;             // [chunks, E] scratch (null for the one-CTA form)
     int P, E, bn, n_tiles;
@@ -206,10 +281,21 @@ __device__ __forceinline__ int count_up(int* cnt, int e, bool on) {
     return base + __popc(same & ((1u << lane) - 1u));
 }
 
-// thread e holds expert e's pair count: offsets (returned) and the tile list
+// pair p takes the next place of its expert (every thread of the warp calls)
+__device__ __forceinline__ void place_pair(const SortArgs& a, int* cnt, int p) {
+    const int e = p < a.P ? a.ids[p] : -1;
+    const int i = count_up(cnt, e, e >= 0);
+    if (e >= 0) a.order[i] = p;
+    if (p < a.P) a.pos[p] = e >= 0 ? i : -1;
+}
+
+// thread e holds expert e's pair count: offsets (returned), the tile list, and the places that no pair takes
 __device__ __forceinline__ int sort_tiles(const SortArgs& a, int count, int* sh) {
     const int e = threadIdx.x;
     const int start = scan1024(count, sh);
+    const int taken = sh[31];
+    for (int i = taken + e; i < a.P; i += SORT_CHUNK) a.order[i] = -1;
+    __syncthreads();
     const int nt = (count + a.bn - 1) / a.bn;
     const int first = scan1024(nt, sh);
     if (e < a.E)
@@ -233,7 +319,8 @@ __global__ void __launch_bounds__(SORT_CHUNK) moe_sort_one_kernel(SortArgs a) {
     __syncthreads();
     for (int p0 = 0; p0 < a.P; p0 += SORT_CHUNK) {
         const int p = p0 + threadIdx.x;
-        count_up(cnt, p < a.P ? a.ids[p] : 0, p < a.P);
+        const int e = p < a.P ? a.ids[p] : -1;
+        count_up(cnt, e, e >= 0);
     }
     __syncthreads();
     const int start = sort_tiles(a, threadIdx.x < a.E ? cnt[threadIdx.x] : 0, sh);
@@ -242,11 +329,7 @@ __global__ void __launch_bounds__(SORT_CHUNK) moe_sort_one_kernel(SortArgs a) {
     __syncthreads();
     for (int p0 = 0; p0 < a.P; p0 += SORT_CHUNK) {
         const int p = p0 + threadIdx.x;
-        const int i = count_up(cnt, p < a.P ? a.ids[p] : 0, p < a.P);
-        if (p < a.P) {
-            a.order[i] = p;
-            a.pos[p] = i;
-        }
+        place_pair(a, cnt, p);
     }
 }
 
@@ -256,8 +339,8 @@ __global__ void __launch_bounds__(SORT_CHUNK) moe_sort_count_kernel(SortArgs a) 
     pdl_trigger();
     cnt[threadIdx.x] = 0;
     __syncthreads();
-    const int p = blockIdx.x * SORT_CHUNK + threadIdx.x;
-    count_up(cnt, p < a.P ? a.ids[p] : 0, p < a.P);
+    const int p = blockIdx.x * SORT_CHUNK + threadIdx.x, e = p < a.P ? a.ids[p] : -1;
+    count_up(cnt, e, e >= 0);
     __syncthreads();
     if (threadIdx.x < a.E) a.counts[(long)blockIdx.x * a.E + threadIdx.x] = cnt[threadIdx.x];
 }
@@ -286,11 +369,7 @@ __global__ void __launch_bounds__(SORT_CHUNK) moe_sort_scatter_kernel(SortArgs a
     if (threadIdx.x < a.E) cnt[threadIdx.x] = a.counts[(long)blockIdx.x * a.E + threadIdx.x];
     __syncthreads();
     const int p = blockIdx.x * SORT_CHUNK + threadIdx.x;
-    const int i = count_up(cnt, p < a.P ? a.ids[p] : 0, p < a.P);
-    if (p < a.P) {
-        a.order[i] = p;
-        a.pos[p] = i;
-    }
+    place_pair(a, cnt, p);
 }
 
 extern "C" int tsb_moe_sort(const int* ids, int P, int E, int bn, int* order, int* pos, int* tiles, int n_tiles, int* counts, void* stream) {
@@ -312,13 +391,14 @@ extern "C" int tsb_moe_sort(const int* ids, int P, int E, int bn, int* order, in
     return TSB_OK;
 }
 
-// out[i] = x[order[i] / div] (bf16 rows of K, a multiple of 8): the activation rows in sorted order, one warp per row.
+// out[i] = x[order[i] / div] (bf16 rows of K, a multiple of 8): the activation rows in sorted order, one warp per row.  Rows with
+// a negative order are left alone.
 __global__ void __launch_bounds__(256) gather_bf16_rows_kernel(const bf16* __restrict__ x, const int* __restrict__ order, int P, int div,
                                                                int K, bf16* __restrict__ out) {
     pdl_wait();
     pdl_trigger();
     const int i = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (i >= P) return;
+    if (i >= P || order[i] < 0) return;
     const uint4* s = reinterpret_cast<const uint4*>(x + (long)(order[i] / div) * K);
     uint4* d = reinterpret_cast<uint4*>(out + (long)i * K);
     for (int c = lane; c < K / 8; c += 32) d[c] = s[c];

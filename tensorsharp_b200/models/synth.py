@@ -649,3 +649,114 @@ def write_sogulix(folder: str, config: Optional[dict] = None, *, seed=0, device=
     with open(os.path.join(folder, CONFIG_NAME), "w", encoding="utf-8") as f:
         json.dump(cfg, f, indent=1)
     write_safetensors(os.path.join(folder, WEIGHTS_NAME), t)
+
+
+def kegetar_config(*, layers="papa", mlps="dmdm", width=128, heads=4, kv_heads=2, dim=32, vdim=48, window=24, keep_first=3, rot_dims=None,
+                   rot_base=10000.0, yarn=(8.0, 256, 32.0, 1.0), linear_heads=3, linear_dim=32, linear_vdim=48, tau=16.0, decay_rank=8,
+                   own_heads=4, own_kv_heads=1, own_dim=32, own_window=20, ff=64, expert_ff=32, limit=1.5, experts=6, identity=2, top=3,
+                   groups=(4, 3), shared_ff=40, shared_limit=1.0, buckets=251, muls=(31, 17), vocab=512, residual_mult=0.5, eps=1e-6,
+                   weights_of=None, scale=None) -> dict:
+    """A config.json of the Kegetar architecture: ``layers`` has a ``p`` (parallel) or an ``a`` (attention) per layer, ``mlps`` a ``d``
+    (dense), an ``m`` (mixture of experts) or a ``-``; ``weights_of``: layer -> the layer whose weights it uses.  The rank of the
+    decay map is read off the tensors; the configuration names it for the writer."""
+    def spec(i):
+        if layers[i] == "p":
+            mixer = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale if scale is not None else dim ** -0.5,
+                              "mask": {"size": window, "keep_first": keep_first},
+                              "rot": {"dims": rot_dims if rot_dims is not None else dim, "base": rot_base,
+                                      "scaling": dict(zip(("factor", "original", "fast", "slow"), yarn))}},
+                     "right": {"heads": linear_heads, "dim": linear_dim, "vdim": linear_vdim, "tau": tau, "decay_rank": decay_rank}}
+        else:
+            mixer = {"heads": own_heads, "kv_heads": own_kv_heads, "dim": own_dim, "vdim": own_dim, "mask": {"size": own_window},
+                     "scale": scale if scale is not None else own_dim ** -0.5}
+        mlp = {"d": {"kind": "dense", "ff": ff}, "-": None,
+               "m": {"kind": "moe", "expert": {"ff": expert_ff, "limit": limit}, "shared": {"ff": shared_ff, "limit": shared_limit},
+                     "router": {"experts": experts, "identity": identity, "top": top, "groups": {"count": groups[0], "keep": groups[1]}}}}[mlps[i]]
+        s = {"type": "parallel" if layers[i] == "p" else "attention", "mixer": mixer, "mlp": mlp}
+        if weights_of and i in weights_of:
+            s["weights_of"] = weights_of[i]
+        return s
+    return {"architecture": "Kegetar", "vocab": vocab, "width": width, "norm": {"eps": eps}, "residual_mult": residual_mult,
+            "embedding": {"bigram": {"buckets": buckets, "mul_prev": muls[0], "mul_cur": muls[1]}}, "layers": [spec(i) for i in range(len(layers))]}
+
+
+def write_kegetar(folder: str, config: Optional[dict] = None, *, seed=0, device=None, gain=1.0, **sizes) -> None:
+    """A model folder with random bf16 weights for ``config`` (default: :func:`kegetar_config` of ``sizes``): matrices
+    N(0, gain / fan-in), norm weights around their neutral value, biases and choice corrections small, decays spread from
+    channels that forget at once to channels that hardly forget."""
+    import json
+    import os
+
+    from ..gguf.folder import CONFIG_NAME, WEIGHTS_NAME, write_safetensors
+    cfg = config if config is not None else kegetar_config(**sizes)
+    dev = torch.device(device or ("cuda" if torch.cuda.is_available() else "cpu"))
+    gen = torch.Generator(device=dev)
+    gen.manual_seed(seed)
+    t = {}
+
+    def mat(name, rows, cols, std=None):
+        w = torch.randn((rows, cols), generator=gen, device=dev) * (std if std is not None else math.sqrt(gain / cols))
+        t[name] = w.to(torch.bfloat16).cpu()
+
+    def vec(name, n, mean, std):
+        t[name] = (mean + std * torch.randn(n, generator=gen, device=dev)).to(torch.bfloat16).cpu()
+
+    def expert(p, ff):
+        mat(p + "gate", ff, D)
+        mat(p + "up", ff, D)
+        mat(p + "down", D, ff)
+
+    D = cfg["width"]
+    mat("embed", cfg["vocab"], D, 1.0)
+    mat("bigram", cfg["embedding"]["bigram"]["buckets"] + 1, D, 0.5)
+    for i, s in enumerate(cfg["layers"]):
+        if s.get("weights_of") is not None:
+            continue
+        p, m, f = f"l{i}.", s["mixer"], s["mlp"]
+        q = p + "mix."
+        vec(p + "norm1", D, 0.0, 0.15)
+        if s["type"] == "parallel":
+            a, g = m["left"], m["right"]
+            mat(q + "left.q", a["heads"] * a["dim"], D)
+            mat(q + "left.k", a["kv_heads"] * a["dim"], D)
+            mat(q + "left.v", a["kv_heads"] * a["vdim"], D)
+            vec(q + "left.q.norm", a["dim"], 1.2, 0.2)
+            vec(q + "left.k.norm", a["dim"], 1.2, 0.2)
+            mat(q + "left.g", a["heads"] * a["vdim"], D)
+            mat(q + "left.o", D, a["heads"] * a["vdim"])
+            n, e, r = g["heads"] * g["dim"], g["heads"] * g["vdim"], g["decay_rank"]
+            for x, rows in (("q", n), ("k", n), ("v", e), ("g", e)):
+                mat(q + "right." + x, rows, D)
+            mat(q + "right.o", D, e)
+            vec(q + "right.norm", g["vdim"], 1.0, 0.15)
+            mat(q + "right.a1", r, D)
+            mat(q + "right.a2", n, r)
+            vec(q + "right.a2.b", n, 1.0, 3.0)
+            vec(q + "left.out", D, 1.0, 0.15)
+            vec(q + "right.out", D, 1.0, 0.15)
+        else:
+            n, k = m["heads"] * m["dim"], m["kv_heads"] * m["dim"]
+            for x, rows in (("q", n), ("k", k)):
+                mat(q + x, rows, D)
+                vec(q + x + ".b", rows, 0.0, 0.2)
+                vec(q + x + ".norm", rows, 1.2, 0.2)
+            mat(q + "o", D, n)
+        if f is not None:
+            vec(p + "norm2", D, 0.0, 0.15)
+            if f["kind"] == "dense":
+                expert(p + "mlp.", f["ff"])
+                for x, rows in (("gate", f["ff"]), ("up", f["ff"]), ("down", D)):
+                    vec(f"{p}mlp.{x}.b", rows, 0.0, 0.2)
+            else:
+                n = f["router"]["experts"] + f["router"]["identity"]
+                for e in range(f["router"]["experts"]):
+                    expert(f"{p}mlp.e{e}.", f["expert"]["ff"])
+                mat(p + "mlp.router", n, D)
+                vec(p + "mlp.correction", n, -0.1, 0.1)
+                expert(p + "mlp.shared.", f["shared"]["ff"])
+    vec("final.norm", D, 0.0, 0.15)
+    mat("head", cfg["vocab"], D)
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, CONFIG_NAME), "w", encoding="utf-8") as f:
+        json.dump(cfg, f, indent=1)
+    write_safetensors(os.path.join(folder, WEIGHTS_NAME), t)

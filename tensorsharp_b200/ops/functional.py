@@ -13,6 +13,7 @@ Data conventions
 """
 from __future__ import annotations
 
+import math
 import os
 from dataclasses import dataclass, field
 from typing import Optional, Tuple
@@ -51,6 +52,9 @@ class RopeSpec:
     corr_lo: float = 0.0
     corr_hi: float = 0.0
     freq_factors: Optional[torch.Tensor] = None
+    # frequency of every pair (float64, on the compute device) in place of the base and scaling above; cos and sin are
+    # multiplied by attn_factor
+    freq: Optional[torch.Tensor] = None
 
 
 @dataclass
@@ -188,6 +192,46 @@ def parallel_seam(h: torch.Tensor, eps: float, n: int, *, y=(None, None), scale=
         elif i < outputs:
             out[i] = res[i]
     return h, out[0], out[1]
+
+
+def post_norm_seam(h: torch.Tensor, eps: float, n: int, *, y=None, z: Optional[torch.Tensor] = None, branch=(None, None), mix: float = 1.0,
+                   post: Optional[torch.Tensor] = None, pre: Optional[torch.Tensor] = None, dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """The seam of a decoder that normalises its sublayers' outputs, one kernel on CUDA: ``h`` (f32 ``[T, D]``, in place) gains
+    the RMS norm of ``y`` (a tensor or :class:`MoeParts`) with the weight ``post``; with a second branch ``z`` it is the norm of
+    ``mix`` times the sum of both branches' own norms (weights ``branch``).  Returns what the next product reads: ``h`` itself,
+    or its RMS norm with the weight ``pre``.  Statistics run over the first ``n`` columns, the rest is padding."""
+    parts = y if isinstance(y, MoeParts) else None
+    if h.is_cuda:
+        return _k().post_norm(h, eps, n, y=parts.y if parts else y, z=z, ids=parts.ids if parts else None, pos=parts.pos if parts else None,
+                              wts=parts.w if parts else None, parts=parts.k if parts else 1, branch=branch, mix=mix, post=post, pre=pre,
+                              out_dtype=dtype or torch.bfloat16)
+
+    def rms(x):
+        return x * torch.rsqrt((x * x).sum(-1, keepdim=True) / n + eps)
+    if y is not None:
+        x = parts.sum(h) if parts else y.float()
+        if z is not None:
+            x = mix * (rms(x) * branch[0] + rms(z.float()) * branch[1])
+        h.add_(rms(x) * post)
+    return rms(h) * pre if pre is not None else h.clone()
+
+
+def embed_pairs(tok: QuantWeight, pair: QuantWeight, batch: Batch, prev: torch.Tensor, *, mul_prev: int, mul_cur: int,
+                dtype: Optional[torch.dtype] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Token embedding plus that of the pair (previous token, token): row (previous * mul_prev + token * mul_cur) mod buckets of
+    ``pair`` [buckets + 1, D], the last row for a sequence's first token.  ``prev`` (int32 per slot, negative: none) is the token
+    ahead of each sequence's new ones and is advanced.  Returns (f32 [T, D], the same as the next product reads it)."""
+    if batch.tokens.is_cuda:
+        return _k().pair_embed(tok, pair, batch.tokens, batch.cu_q, batch.seq_slots, prev, mul_prev=mul_prev, mul_cur=mul_cur,
+                               out_dtype=dtype or torch.bfloat16)
+    ids, buckets = batch.tokens.long(), pair.rows - 1
+    before = torch.cat([ids[:1], ids[:-1]])
+    for b, slot in enumerate(batch.seq_slots.tolist()):
+        before[batch.h_cu_q[b]] = prev[slot]
+        prev[slot] = ids[batch.h_cu_q[b + 1] - 1]
+    rows = torch.where(before < 0, torch.full_like(ids, buckets), (before * mul_prev + ids * mul_cur) % buckets)
+    h = tok.dequantize()[ids] + pair.dequantize()[rows]
+    return h, h.clone()
 
 
 def as_act(x, w: Optional[QuantWeight] = None) -> Act:
@@ -400,7 +444,8 @@ def qkv_rope_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, *, Hq: int
             key = ("rope", id(rope))
             table = batch.cache.get(key)
             if table is None:
-                table = kk.rope_table(batch.positions, rp, rope.freq_factors)
+                table = (kk.rotary_table(batch.positions, rope.freq, rope.attn_factor) if rope.freq is not None else
+                         kk.rope_table(batch.positions, rp, rope.freq_factors))
                 batch.cache[key] = table
         f32 = k_cache.dtype == torch.float32
         q_out = torch.empty((T, Hq, Dh), dtype=torch.float32 if f32 else torch.bfloat16, device=q.device)
@@ -435,9 +480,13 @@ def qkv_rope_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, *, Hq: int
     if v_norm:
         vf = ref.rmsnorm(vf, None, eps)
     if rope is not None and rope.rot_dim > 0:
-        cos, sin = ref.rope_cos_sin(batch.positions, rope.rot_dim, rope.theta_base, rope.freq_scale,
-                                    rope.ext_factor, rope.attn_factor, rope.corr_lo, rope.corr_hi,
-                                    rope.freq_factors)
+        if rope.freq is not None:
+            ang = batch.positions.double().unsqueeze(1) * rope.freq
+            cos, sin = (ang.cos() * rope.attn_factor).float(), (ang.sin() * rope.attn_factor).float()
+        else:
+            cos, sin = ref.rope_cos_sin(batch.positions, rope.rot_dim, rope.theta_base, rope.freq_scale,
+                                        rope.ext_factor, rope.attn_factor, rope.corr_lo, rope.corr_hi,
+                                        rope.freq_factors)
         qf = ref.apply_rope(qf, cos, sin, rope.rot_dim, rope.mode)
         kf = ref.apply_rope(kf, cos, sin, rope.rot_dim, rope.mode)
     if write_kv:
@@ -518,17 +567,21 @@ def decode_splits(batch: Batch, Hkv: int, window: int) -> int:
 
 def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch: Batch, *, scale: float,
               Hq: int, Hkv: int, Dh: int, window: int = 0, sinks: Optional[torch.Tensor] = None,
-              softcap: float = 0.0, as_act: bool = False, Dv: Optional[int] = None, gate: Optional[torch.Tensor] = None):
+              softcap: float = 0.0, as_act: bool = False, Dv: Optional[int] = None, gate: Optional[torch.Tensor] = None, keep_first: int = 0,
+              slopes: Optional[torch.Tensor] = None, own_values: bool = False):
     """Causal attention of the packed queries against the paged cache -> [T, Hq * Dh].  ``as_act`` returns an
     ``Act``; on the CUDA decode path it already carries the int8 form written by the combine kernel, so
     the quantised projection that follows needs no quantise launch.  ``Dv``: value head size where it differs from
     ``Dh`` (the result is then [T, Hq * Dv]); ``gate`` [T, Hq] (a view, last dim dense): head h's output is
-    multiplied by sigmoid(gate[:, h]); float32 caches run in 32 bits."""
+    multiplied by sigmoid(gate[:, h]), with a gate [T, Hq * Dv] every column by its own; float32 caches run in 32 bits.
+    ``keep_first``: with a window, so many positions at the start stay visible; ``slopes`` [Hq]: slopes[h] times the distance
+    is taken off the score; ``own_values``: a row of ``k_cache`` (see :func:`joint_norm_cache`) is key and value at once."""
     T = q.shape[0]
     Dv = Dv or Dh
-    if q.is_cuda and (Dv != Dh or gate is not None or k_cache.dtype == torch.float32):
+    if q.is_cuda and (Dv != Dh or gate is not None or k_cache.dtype == torch.float32 or keep_first or slopes is not None or own_values):
         return _gated_attention(q, k_cache, v_cache, batch, scale=scale, Hq=Hq, Hkv=Hkv, Dh=Dh, Dv=Dv, window=window,
-                                sinks=sinks, softcap=softcap, gate=gate)
+                                sinks=sinks, softcap=softcap, gate=gate, keep_first=keep_first, slopes=slopes,
+                                kv_scale=Hkv * Dh if own_values else 0)
     if as_act:
         if q.is_cuda and batch.is_decode and Dh % 32 == 0:
             sp = decode_splits(batch, Hkv, window)
@@ -560,28 +613,37 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, bat
         L = batch.h_kv_lens[b]
         pages = batch.block_table[b, :(L + ps - 1) // ps].long()
         idx = (pages.unsqueeze(1) * ps + torch.arange(ps)).reshape(-1)[:L]
-        kb, vb = kv_gather(k_cache, idx), kv_gather(v_cache, idx)
+        if own_values:
+            rows = k_cache[idx].view(L, -1)
+            if window:
+                rows = rows.clone()
+                rows[:max(0, L - (q1 - q0) - window + 1)] = 0              # out of every query's sight; may be stale in a ring
+            vb = rows[:, :Hkv * Dh].view(L, Hkv, Dh)
+            kb = vb * rows[:, Hkv * Dh].view(L, 1, 1)
+        else:
+            kb, vb = kv_gather(k_cache, idx), kv_gather(v_cache, idx)
         outs.append(ref.attention(q[q0:q1], kb, vb, batch.positions[q0:q1], scale=scale, window=window, sinks=sinks,
-                                  softcap=softcap))
+                                  softcap=softcap, keep_first=keep_first, slopes=slopes))
     out = torch.cat(outs, 0)
     if gate is not None:
-        out = out * torch.sigmoid(gate.float()).unsqueeze(-1)
+        out = out * torch.sigmoid(gate.float()).view(T, Hq, -1)
     return out.reshape(T, Hq * Dv)
 
 
-def _gated_attention(q, k_cache, v_cache, batch: Batch, *, scale, Hq, Hkv, Dh, Dv, window, sinks, softcap, gate) -> torch.Tensor:
+def _gated_attention(q, k_cache, v_cache, batch: Batch, *, scale, Hq, Hkv, Dh, Dv, window, sinks, softcap, gate, keep_first=0, slopes=None,
+                     kv_scale=0) -> torch.Tensor:
     """The CUDA side of :func:`attention` for the forms beyond one head size and bf16: keys and values of different
-    sizes, a sigmoid gate per head, 32-bit caches."""
+    sizes, sigmoid gates, kept first positions, distance biases, rows that are key and value at once, 32-bit caches."""
     kk = _k()
     T = q.shape[0]
     if is_fp8(k_cache):
         raise ValueError("8-bit pages have no gated attention")
     kw = dict(scale=scale, Hq=Hq, Hkv=Hkv, Dh=Dh, Dv=Dv, page_size=batch.page_size, sinks=sinks, softcap=softcap, window=window,
-              gate=gate)
+              gate=gate, keep_first=keep_first, slopes=slopes, kv_scale=kv_scale)
     if k_cache.dtype == torch.float32:
         return kk.attn_f32(q, k_cache, v_cache, batch.block_table, batch.kv_lens, batch.cu_q, **kw).view(T, Hq * Dv)
     if batch.is_decode:
-        sp = decode_splits(batch, Hkv, window)
+        sp = decode_splits(batch, Hkv, window + keep_first if window else 0)
         out = kk.attn_decode(q, k_cache, v_cache, batch.block_table, batch.kv_lens, splits=sp,
                              split_len=decode_split_len(batch, sp, window), **kw)
     else:
@@ -622,6 +684,44 @@ class LatentSpec:
 def rotary_freqs(dims: int, base: float, device) -> torch.Tensor:
     """base^(-2 i / dims) of every pair, float64."""
     return torch.tensor([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64, device=device)
+
+
+def yarn_freqs(dims: int, base: float, scaling: Optional[dict], device) -> Tuple[torch.Tensor, float]:
+    """Frequencies of :func:`rotary_freqs` with YaRN scaling {factor, original, fast, slow} (None: as they are), and the factor
+    on cos and sin: pairs that turn more than ``fast`` times over the original context keep their frequency, those that turn
+    less than ``slow`` times have it divided by ``factor``, with a linear ramp over the pair's number in between."""
+    f = rotary_freqs(dims, base, device)
+    if not scaling:
+        return f, 1.0
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+
+    def pair(turns: float) -> float:                  # twice the number of the pair that turns so often, as a real number
+        return dims * math.log(original / (2 * math.pi * turns)) / (2 * math.log(float(base)))
+    lo, hi = max(math.floor(pair(float(scaling["fast"]))), 0), min(math.ceil(pair(float(scaling["slow"]))), dims - 1)
+    i = torch.arange(dims // 2, dtype=torch.float64, device=device)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return f / factor * ramp + f * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
+def alibi_slopes(heads: int, device) -> torch.Tensor:
+    """Geometric slopes 2^(-8 (h + 1) / heads) of a distance bias."""
+    return torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], dtype=torch.float32, device=device)
+
+
+def joint_norm_cache(y: torch.Tensor, w: torch.Tensor, cache: torch.Tensor, batch: Batch, *, nq: int, nk: int, q_n: int, k_n: int, eps: float) -> torch.Tensor:
+    """Query and key norms over whole projections for attention whose values are the keys ahead of their norm.  Rows of ``y``:
+    [q (nq) | k (nk)], padded heads.  A cached row holds k as it is and then 1 / rms(k); the keys' norm weight is part of ``w``
+    (the query weight times that of the query head's key head), so q / rms(q) * w against k times the row's factor is the
+    score.  ``q_n``, ``k_n``: sizes without padding.  Returns the queries [T, nq]."""
+    if y.is_cuda:
+        return _k().joint_norm(y, w, cache, batch.slots, nq=nq, nk=nk, q_n=q_n, k_n=k_n, eps=eps)
+    y = y.float()
+    q, k = y[:, :nq], y[:, nq:nq + nk]
+    row = torch.zeros((y.shape[0], nk + 8))
+    row[:, :nk] = k
+    row[:, nk] = torch.rsqrt((k * k).sum(-1) / k_n + eps)
+    kv_scatter(cache, batch.slots, row.unsqueeze(1))
+    return q * torch.rsqrt((q * q).sum(-1, keepdim=True) / q_n + eps) * w
 
 
 def rotary_table(batch: Batch, s: LatentSpec) -> torch.Tensor:
@@ -797,17 +897,45 @@ def route_softmax_renorm(logits: torch.Tensor, E: int, k: int, scale: float, n_a
     return ids.to(torch.int32), w
 
 
+def route_softmax_groups(logits: torch.Tensor, correction: Optional[torch.Tensor], k: int, *, groups: int, keep: int, n_real: int,
+                         n_always: int = 0):
+    """Softmax over all logits; the ``k`` largest of softmax + ``correction`` among the ``keep`` best of ``groups`` equal groups of
+    neighbours (a group is as good as its best entry); the weights are the softmax values, not renormalised.  Entries from
+    ``n_real`` on are identity experts: their id is -1.  The ids 0 .. n_always - 1 (slices of a shared expert) come first on every
+    token with weight 1, the routed experts are numbered from ``n_always`` on.  -> (ids int32, weights f32), [T, n_always + k]."""
+    if logits.is_cuda:
+        return _k().moe_route_grouped(logits, k, correction=correction, groups=groups, keep=keep, n_real=n_real, n_always=n_always)
+    s = torch.softmax(logits.float(), -1)
+    choice = s + correction if correction is not None else s
+    T, E = s.shape
+    by_group = choice.view(T, groups, E // groups)
+    best = torch.topk(by_group.max(-1).values, keep, dim=-1).indices
+    shut = torch.ones((T, groups, 1), dtype=torch.bool).scatter_(1, best.unsqueeze(-1), False)
+    ids = torch.topk(by_group.masked_fill(shut, float("-inf")).view(T, E), k, dim=-1).indices
+    w = s.gather(-1, ids)
+    ids = torch.where(ids < n_real, ids + n_always, torch.full_like(ids, -1))
+    return (torch.cat([torch.arange(n_always).expand(T, n_always), ids], 1).to(torch.int32),
+            torch.cat([torch.ones((T, n_always)), w], 1))
+
+
 @dataclass
 class MoeParts:
     """The experts' output rows before they are summed per token: token t's result is the sum over j < k of
-    ``w[t * k + j] * y[pos[t * k + j]]`` (``w`` None: rows are weighted already; ``pos`` None: row t * k + j)."""
+    ``w[t * k + j] * y[pos[t * k + j]]`` (``w`` None: rows are weighted already; ``pos`` None: row t * k + j).  Where
+    ``ids[t * k + j]`` is negative (an identity expert) the layer's input stands in place of the row."""
     y: torch.Tensor
     k: int
     pos: Optional[torch.Tensor] = None
     w: Optional[torch.Tensor] = None
+    ids: Optional[torch.Tensor] = None
 
-    def sum(self) -> torch.Tensor:
+    def sum(self, x: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``x`` [T, D]: the layer's input (with ``ids``)."""
         y = self.y.float()
+        if self.ids is not None:
+            ids = self.ids.view(-1, self.k)
+            own = (self.w.view(-1, self.k) * (ids < 0)).sum(1, keepdim=True)
+            return own * x + y
         if self.pos is not None:
             y = y[self.pos.long()]
         if self.w is not None:
@@ -815,36 +943,51 @@ class MoeParts:
         return y.view(-1, self.k, y.shape[-1]).sum(1)
 
 
-def moe_expert_parts(a: Act, ids: torch.Tensor, weights: torch.Tensor, gate_up: QuantWeight, down: QuantWeight, *, act: str) -> MoeParts:
-    """:func:`moe_experts` without its last step, for a consumer that sums the rows itself (``residual_layernorm``):
-    every expert is local, there are no biases, and ``act`` is gated."""
+def moe_expert_parts(a: Act, ids: torch.Tensor, weights: torch.Tensor, gate_up: QuantWeight, down: QuantWeight, *, act: str,
+                     clamp: Optional[Tuple[float, float, int]] = None, identity: bool = False) -> MoeParts:
+    """:func:`moe_experts` without its last step, for a consumer that sums the rows itself (``residual_layernorm``,
+    ``post_norm_seam``): every expert is local, there are no biases, and ``act`` is gated.  ``clamp`` (limit, limit of the first
+    experts, how many): the clamp of "swiglu_oai"; ids below that number are on every token and come first in ``ids``'
+    rows.  ``identity``: negative ids stand for the layer's input itself."""
     T, k = ids.shape
     if ids.device.type != "cuda":
-        return MoeParts(moe_experts(a, ids, weights, gate_up, down, act=act), 1)
+        if clamp is None:
+            return MoeParts(moe_experts(a, ids, weights, gate_up, down, act=act), 1)
+        y = torch.zeros((T, down.N))
+        half = gate_up.N // 2
+        for e in range(gate_up.experts):
+            tok, slot = (ids == e).nonzero(as_tuple=True)
+            if tok.numel():
+                u = linear(Act(a.b[tok]), gate_up.expert(e))
+                u = ref.glu(act, u[:, :half], u[:, half:], clamp[1] if e < clamp[2] else clamp[0])
+                y.index_add_(0, tok, linear(Act(u), down.expert(e)) * weights[tok, slot].unsqueeze(1))
+        return MoeParts(y, k, None, weights, ids) if identity else MoeParts(y, 1)
     kk = _k()
+    flat_ids = ids if identity else None
+    row_clamp = (clamp[0], clamp[1], T * clamp[2]) if clamp else None          # sorted by expert, the first experts' rows come first
     P, E, F_out, D = T * k, gate_up.experts, gate_up.N // 2, down.N
     wts = weights.reshape(-1)
     if a.b.dtype == torch.float32:
         bn = 64
         order, tiles, pos = kk.moe_sort(ids, E, bn)
         y1 = kk.gemm_f32(gate_up, a.b, tiles=tiles, rows=order, row_div=k)
-        h = kk.glu_f32(y1[:, :F_out], y1[:, F_out:], act)
-        return MoeParts(kk.gemm_f32(down, h, tiles=tiles), k, pos, wts)
+        h = kk.glu_f32(y1[:, :F_out], y1[:, F_out:], act, row_clamp)
+        return MoeParts(kk.gemm_f32(down, h, tiles=tiles), k, pos, wts, flat_ids)
     if P <= 4 * GEMV_MAX_M:
         flat = ids.reshape(-1)
         gu = torch.empty((P, F_out), dtype=torch.bfloat16, device=ids.device)
-        kk.gemv(gate_up, xb=a.b, M=1, ids=flat, x_div=k, act=act, out=gu)
+        kk.gemv(gate_up, xb=a.b, M=1, ids=flat, x_div=k, act=act, out=gu, clamp=clamp)
         y = torch.empty((P, D), dtype=torch.float32, device=ids.device)
         kk.gemv(down, xb=gu, M=1, ids=flat, x_div=1, out=y)
-        return MoeParts(y, k, None, wts)
+        return MoeParts(y, k, None, wts, flat_ids)
     avg = max(1, P // E)
     bn = 32 if avg <= 32 else 64 if avg <= 64 else 128 if avg <= 128 else 256
     order, tiles, pos = kk.moe_sort(ids, E, bn)
     xs = kk.gather_bf16_rows(a.b, order, k)
     y1 = kk.gemm_bf16_grouped(_dequant_scratch(gate_up), E, xs, tiles, bn, out_dtype=torch.bfloat16, zero=False)
-    h, _, _ = kk.glu(y1, y1[:, F_out:], act, F_out, gate_up.N, gate_up.N, P)
+    h, _, _ = kk.glu(y1, y1[:, F_out:], act, F_out, gate_up.N, gate_up.N, P, clamp=row_clamp)
     y2 = kk.gemm_bf16_grouped(_dequant_scratch(down), E, h, tiles, bn, out_dtype=torch.bfloat16, zero=False)
-    return MoeParts(y2, k, pos, wts)
+    return MoeParts(y2, k, pos, wts, flat_ids)
 
 
 def moe_experts(a: Act, ids: torch.Tensor, weights: torch.Tensor, gate_up: QuantWeight, down: QuantWeight, *,
@@ -1101,6 +1244,56 @@ def general_delta(y: torch.Tensor, w2: QuantWeight, w0: torch.Tensor, ab: torch.
         o[q0:q1] = ref.general_delta(r[q0:q1], k[q0:q1], v[q0:q1], decay[q0:q1], a[q0:q1], state[slots[b]])
     o = o * torch.rsqrt((o * o).sum(-1, keepdim=True) / n + eps)
     return o.reshape(T, HD) * norm_w * torch.sigmoid(y[:, 4 * HD:5 * HD])
+
+
+@dataclass
+class GatedLinearSpec:
+    """Sizes of a gated linear attention mixer (``D``, ``E``: padded key and value head sizes)."""
+    H: int
+    dim: int
+    vdim: int
+    tau: float
+
+    def __post_init__(self):
+        self.D = (self.dim + 31) // 32 * 32
+        pad = 16 if self.vdim <= 128 else 32
+        self.E = (self.vdim + pad - 1) // pad * pad
+        self.q_scale = self.dim ** -0.5
+
+
+GATED_LINEAR_CHUNK_MIN = 12          # tokens of the longest portion from which the chunk kernel is used
+
+
+def gated_linear_segments(batch: Batch, s: GatedLinearSpec) -> int:
+    """Pieces in which the chunk kernel takes the batch's sequences: about two CTAs per SM, no fewer than 64 tokens each."""
+    ctas = batch.B * s.H * (2 if s.E > 128 else 1)
+    return max(1, min(round(2 * 148 / ctas), batch.max_q_len // 64))
+
+
+def gated_linear(y: torch.Tensor, s: GatedLinearSpec, cols: Tuple[int, ...], w2: QuantWeight, zb: torch.Tensor, norm_w: torch.Tensor,
+                 state: torch.Tensor, batch: Batch, *, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """Gated linear attention with a decay per key channel over the packed tokens -> normed and gated output [T, H * E].  Columns
+    ``cols`` of ``y``: queries, keys (H * D each), values, gate (H * E each), low rank part of the decay; ``w2`` [H * D, rank up to
+    8], ``zb``: its second map and offset.  ``state`` f32 [slots, H, values, keys].  Heads are padded with zeros."""
+    if y.is_cuda:
+        kk = _k()
+        if y.dtype != torch.bfloat16 or batch.max_q_len < GATED_LINEAR_CHUNK_MIN:
+            return kk.gla_step(y, s, cols, _weight_matrix(w2), zb, norm_w, state, batch.cu_q, batch.seq_slots, eps=eps, out_dtype=dtype)
+        z = linear(Act(y[:, cols[4]:cols[4] + w2.K]), w2, out_dtype=torch.float32)
+        return kk.gla_prompt(y, s, cols, z, zb, norm_w, state, batch.cu_q, batch.seq_slots, eps=eps, max_q=batch.max_q_len,
+                             segs=gated_linear_segments(batch, s))
+    T, y = y.shape[0], y.float()
+    H, D, E = s.H, s.D, s.E
+    q, k = (y[:, c:c + H * D].view(T, H, D) for c in cols[:2])
+    v = y[:, cols[2]:cols[2] + H * E].view(T, H, E)
+    z = y[:, cols[4]:cols[4] + w2.K] @ w2.dequantize().t() + zb
+    decay = torch.exp(torch.nn.functional.logsigmoid(z) / s.tau).view(T, H, D)
+    o, slots = torch.empty((T, H, E)), batch.seq_slots.tolist()
+    for b in range(batch.B):
+        q0, q1 = batch.h_cu_q[b], batch.h_cu_q[b + 1]
+        o[q0:q1] = ref.gated_linear(q[q0:q1] * s.q_scale, k[q0:q1], v[q0:q1], decay[q0:q1], state[slots[b]])
+    o = o * torch.rsqrt((o * o).sum(-1, keepdim=True) / s.vdim + eps) * norm_w
+    return o.reshape(T, H * E) * torch.nn.functional.silu(y[:, cols[3]:cols[3] + H * E])
 
 
 def _weight_matrix(w: QuantWeight) -> torch.Tensor:

@@ -81,7 +81,8 @@ class AttnArgs(C.Structure):
                 ("max_pages", C.c_int), ("splits", C.c_int), ("q_pos0", _vp), ("lse_out", _vp),
                 ("out_q", _vp), ("out_ds", _vp), ("ticket", _vp), ("split_len", C.c_int),
                 ("gate", _vp), ("gate_tok", C.c_long), ("gate_f32", C.c_int), ("Dv", C.c_int),
-                ("k_ld", C.c_long), ("v_ld", C.c_long)]
+                ("k_ld", C.c_long), ("v_ld", C.c_long), ("keep_first", C.c_int), ("slopes", _vp), ("gate_cols", C.c_int),
+                ("kv_scale", C.c_int)]
 
 
 _configured = False
@@ -122,13 +123,14 @@ def quantize_q8(x: torch.Tensor):
 
 def gemv(w: QuantWeight, *, xq=None, xds=None, xb=None, M: int, out_dtype=torch.float32, bias=None, residual=None,
          act=None, ids=None, row_scale=None, x_div: int = 1, out: Optional[torch.Tensor] = None,
-         push: Optional[int] = None) -> Optional[torch.Tensor]:
+         push: Optional[int] = None, clamp=None) -> Optional[torch.Tensor]:
     """Small-batch matvec over quantised weights.  With ``ids`` ([P] int32) each problem p
     uses expert ids[p], activation row p // x_div and output row p.  ``push`` (device address of a
     tensor-parallel exchange descriptor) sends the f32 result to every rank's mailbox instead of
-    ``out``."""
+    ``out``.  ``clamp`` (limit, limit of the first experts, how many): the clamp of "swiglu_oai" (default 7)."""
     a = ACT[act]
     glu = 1 <= a <= 4
+    lim, lim_first, n_first = clamp or (7.0, 7.0, 0)
     n_out = w.N // 2 if glu else w.N
     problems = int(ids.numel()) if ids is not None else 1
     rows = problems if ids is not None else M
@@ -136,11 +138,12 @@ def gemv(w: QuantWeight, *, xq=None, xds=None, xb=None, M: int, out_dtype=torch.
     if out is None and push is None:
         out = torch.empty((rows, n_out), dtype=out_dtype, device=dev)
     ps = _planes(w)
-    native.check(_lib().tsb_gemv_push(ps[0], ps[1], ps[2], ps[3], C.c_int(int(w.ggml_type)), C.c_int(w.N), C.c_int(w.K),
-                                      _p(xq), _p(xds), _p(xb), _p(out), _p(bias), _p(residual), _p(ids), _p(row_scale),
-                                      C.c_int(M), C.c_int(problems), C.c_int(x_div),
-                                      C.c_int(1 if (out is None or out.dtype == torch.float32) else 0), C.c_int(a),
-                                      C.c_void_p(push) if push else None, _stream()), "gemv")
+    native.check(_lib().tsb_gemv_clamped(ps[0], ps[1], ps[2], ps[3], C.c_int(int(w.ggml_type)), C.c_int(w.N), C.c_int(w.K),
+                                         _p(xq), _p(xds), _p(xb), _p(out), _p(bias), _p(residual), _p(ids), _p(row_scale),
+                                         C.c_int(M), C.c_int(problems), C.c_int(x_div),
+                                         C.c_int(1 if (out is None or out.dtype == torch.float32) else 0), C.c_int(a),
+                                         C.c_void_p(push) if push else None, C.c_float(lim), C.c_float(lim_first), C.c_int(n_first),
+                                         _stream()), "gemv")
     _count(1)
     return out
 
@@ -181,12 +184,26 @@ def moe_route(logits: torch.Tensor, k: int, *, mode: int = 0, sel_bias=None, nor
     return ids, w
 
 
+def moe_route_grouped(logits: torch.Tensor, k: int, *, correction, groups: int, keep: int, n_real: int, n_always: int = 0, scale: float = 1.0):
+    """Router with groups of neighbours and identity experts (functional.py: route_softmax_groups): f32 logits [T, E] ->
+    (ids int32, weights f32), both [T, n_always + k]."""
+    assert logits.is_cuda and logits.dtype == torch.float32 and logits.is_contiguous()
+    T, E = logits.shape
+    ids = torch.empty((T, n_always + k), dtype=torch.int32, device=logits.device)
+    w = torch.empty((T, n_always + k), dtype=torch.float32, device=logits.device)
+    native.check(_lib().tsb_moe_route_grouped(_p(logits), _p(correction), C.c_int(T), C.c_int(E), C.c_int(n_real), C.c_int(k), C.c_int(groups),
+                                              C.c_int(keep), C.c_float(scale), C.c_int(n_always), _p(ids), _p(w), _stream()), "moe_route")
+    _count(1)
+    return ids, w
+
+
 def moe_sort(ids: torch.Tensor, E: int, bn: int):
-    """Sort the (token, slot) pairs of ``ids`` (int32, every value in [0, E)) by expert on the device.  Returns ``order``
-    (the pair at each sorted place), ``tiles`` int32 [ceil(P / bn) + E, 3] (expert or -1, first, end place; at most bn
-    places each) and ``pos`` (the sorted place of each pair)."""
+    """Sort the (token, slot) pairs of ``ids`` (int32, every value in [0, E) or negative) by expert on the device.  Returns
+    ``order`` (the pair at each sorted place; -1 at the end, for the pairs with a negative id), ``tiles`` int32
+    [ceil(P / bn) + E, 3] (expert or -1, first, end place; at most bn places each) and ``pos`` (the sorted place of each pair, -1
+    for a negative id)."""
     assert ids.dtype == torch.int32 and ids.is_contiguous()
-    check_index("moe_sort", "expert id", ids, E)
+    check_index("moe_sort", "expert id", ids, E, low=-1)
     P, dev = ids.numel(), ids.device
     n_tiles = (P + bn - 1) // bn + E
     order, pos = torch.empty(P, dtype=torch.int32, device=dev), torch.empty(P, dtype=torch.int32, device=dev)
@@ -199,7 +216,7 @@ def moe_sort(ids: torch.Tensor, E: int, bn: int):
 
 
 def gather_bf16_rows(x: torch.Tensor, order: torch.Tensor, div: int) -> torch.Tensor:
-    """x[order // div] for bf16 rows."""
+    """x[order // div] for bf16 rows (what stands in rows with a negative order is undefined)."""
     assert x.dtype == torch.bfloat16 and x.is_contiguous() and order.dtype == torch.int32
     out = torch.empty((order.numel(), x.shape[1]), dtype=torch.bfloat16, device=x.device)
     native.check(_lib().tsb_gather_bf16_rows(_p(x), _p(order), C.c_int(order.numel()), C.c_int(div), C.c_int(x.shape[1]), _p(out), _stream()),
@@ -394,8 +411,10 @@ def rope_table(pos: torch.Tensor, rope: RopeParams, freq_factors=None) -> torch.
 
 
 def glu(gate: torch.Tensor, up: Optional[torch.Tensor], act: str, F: int, g_stride: int, u_stride: int, rows: int,
-        want_bf16=True, want_q8=False):
+        want_bf16=True, want_q8=False, clamp=None):
+    """``clamp`` (limit, limit of the first rows, how many): the clamp of "swiglu_oai" (default 7)."""
     dev = gate.device
+    lim, lim_first, rows_first = clamp or (7.0, 7.0, 0)
     out = torch.empty((rows, F), dtype=torch.bfloat16, device=dev) if want_bf16 else None
     yq = yds = None
     if want_q8:
@@ -403,7 +422,7 @@ def glu(gate: torch.Tensor, up: Optional[torch.Tensor], act: str, F: int, g_stri
         yds = torch.empty((rows, F // 32, 2), dtype=torch.float32, device=dev)
     native.check(_lib().tsb_glu(_p(gate), _p(up), C.c_int(gate.dtype == torch.float32), C.c_long(g_stride),
                                 C.c_long(u_stride), C.c_long(rows), C.c_int(F), C.c_int(ACT[act]), _p(out), _p(yq),
-                                _p(yds), _stream()), "glu")
+                                _p(yds), C.c_float(lim), C.c_float(lim_first), C.c_long(rows_first), _stream()), "glu")
     _count(1)
     return out, yq, yds
 
@@ -444,7 +463,7 @@ def decode_advance(sampled, batch) -> None:
 
 
 def _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, cu_q, sinks, scale, softcap, window, Hq, Hkv, Dh,
-               page_size, B, Dv=None, gate=None):
+               page_size, B, Dv=None, gate=None, keep_first=0, slopes=None, kv_scale=0):
     check_index("attention", "block-table page", block_table, k_cache.shape[0] // page_size)
     check_index("attention", "cache length", kv_lens, block_table.shape[1] * page_size + 1)
     a = AttnArgs()
@@ -455,27 +474,35 @@ def _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, cu_q, sinks, scal
     a.max_pages = block_table.shape[1]
     a.splits = 1
     a.Dv = Dv or Dh
+    assert slopes is None or (slopes.dtype == torch.float32 and slopes.is_contiguous() and slopes.numel() == Hq)
+    a.keep_first, a.slopes, a.kv_scale = int(keep_first) if window else 0, _p(slopes), int(kv_scale)
+    if kv_scale:                          # rows that are key and value at once, with the factor of the key behind them
+        assert k_cache.dim() == 3 and k_cache.stride(2) == 1 and k_cache.shape[-1] >= kv_scale + 1 and kv_scale >= Hkv * Dh
+        a.k_ld = a.v_ld = k_cache.stride(0)
+        k_cache = v_cache = None
     # a slot's rows may be a slice of a wider row (no gaps between the heads)
     for c, heads, d, ld in ((k_cache, Hkv, Dh, "k_ld"), (v_cache, Hkv, Dv or Dh, "v_ld")):
-        if c.dim() == 3 and c.stride(0) != heads * d:
+        if c is not None and c.dim() == 3 and c.stride(0) != heads * d:
             assert c.stride(2) == 1 and (heads == 1 or c.stride(1) == d)
             setattr(a, ld, c.stride(0))
     if gate is not None:
-        assert gate.shape == (q.shape[0], Hq) and gate.stride(1) == 1
+        assert gate.stride(1) == 1 and gate.shape[0] == q.shape[0] and gate.shape[1] in (Hq, Hq * a.Dv)
+        a.gate_cols = int(gate.shape[1] != Hq)
         a.gate, a.gate_tok, a.gate_f32 = gate.data_ptr(), gate.stride(0), int(gate.dtype == torch.float32)
     return a
 
 
 def attn_decode(q, k_cache, v_cache, block_table, kv_lens, *, scale, Hq, Hkv, Dh, page_size, splits, sinks=None,
-                softcap=0.0, window=0, out=None, want_q8=False, split_len=0, Dv=None, gate=None):
+                softcap=0.0, window=0, out=None, want_q8=False, split_len=0, Dv=None, gate=None, **forms):
     """q [B, Hq, Dh] bf16; one query per sequence against the paged cache.  ``want_q8`` also returns the
-    output as int8 groups of 32 with (scale, sum) written by the combine kernel: (out, q, ds)."""
+    output as int8 groups of 32 with (scale, sum) written by the combine kernel: (out, q, ds).  ``forms``: keep_first,
+    slopes, kv_scale (see AttnArgs)."""
     B = q.shape[0]
     Dv = Dv or Dh
     if out is None:
         out = torch.empty((B, Hq, Dv), dtype=q.dtype, device=q.device)
     a = _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, None, sinks, scale, softcap, window, Hq, Hkv, Dh,
-                   page_size, B, Dv, gate)
+                   page_size, B, Dv, gate, **forms)
     a.splits = splits
     a.split_len = split_len
     part_o = torch.empty((B, Hq, splits, Dv), dtype=torch.float32, device=q.device)
@@ -528,7 +555,7 @@ def kv_load_fp8(k_cache: torch.Tensor, v_cache: torch.Tensor, idx: torch.Tensor)
 
 
 def attn_prefill(q, k_cache, v_cache, block_table, kv_lens, cu_q, max_q_len, *, scale, Hq, Hkv, Dh, page_size,
-                 sinks=None, softcap=0.0, window=0, out=None, q_pos0=None, lse_out=None, Dv=None, gate=None):
+                 sinks=None, softcap=0.0, window=0, out=None, q_pos0=None, lse_out=None, Dv=None, gate=None, **forms):
     """q [T, Hq, Dh] bf16 packed over sequences (cu_q [B+1]).  ``q_pos0`` [B] int32 overrides the cache
     position of each sequence's first query (default kv_len - q_len); ``lse_out`` [T, Hq] f32 receives the
     log-sum-exp of the scores, for merging partial results over KV shards."""
@@ -536,7 +563,7 @@ def attn_prefill(q, k_cache, v_cache, block_table, kv_lens, cu_q, max_q_len, *, 
     if out is None:
         out = torch.empty((q.shape[0], Hq, Dv or Dh), dtype=q.dtype, device=q.device)
     a = _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, cu_q, sinks, scale, softcap, window, Hq, Hkv, Dh,
-                   page_size, B, Dv, gate)
+                   page_size, B, Dv, gate, **forms)
     a.q_pos0 = q_pos0.data_ptr() if q_pos0 is not None else None
     a.lse_out = lse_out.data_ptr() if lse_out is not None else None
     native.check(_lib().tsb_attn_prefill(C.byref(a), C.c_int(max_q_len), _stream()), "attn_prefill")
@@ -545,12 +572,12 @@ def attn_prefill(q, k_cache, v_cache, block_table, kv_lens, cu_q, max_q_len, *, 
 
 
 def attn_f32(q, k_cache, v_cache, block_table, kv_lens, cu_q, *, scale, Hq, Hkv, Dh, page_size, Dv=None, sinks=None, softcap=0.0,
-             window=0, gate=None):
+             window=0, gate=None, **forms):
     """Attention in 32 bits over a float32 cache, prompts and decode alike: q [T, Hq, Dh] -> [T, Hq, Dv]."""
     assert q.dtype == k_cache.dtype == v_cache.dtype == torch.float32 and (gate is None or gate.dtype == torch.float32)
     out = torch.empty((q.shape[0], Hq, Dv or Dh), dtype=torch.float32, device=q.device)
     a = _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, cu_q, sinks, scale, softcap, window, Hq, Hkv, Dh, page_size,
-                   kv_lens.shape[0], Dv, gate)
+                   kv_lens.shape[0], Dv, gate, **forms)
     native.check(_lib().tsb_attn_f32(C.byref(a), C.c_int(q.shape[0]), _stream()), "attn_f32")
     _count(1)
     return out
@@ -635,6 +662,123 @@ def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
     return out
 
 
+class PostNormArgs(C.Structure):
+    _fields_ = [("h", _vp), ("y", _vp), ("z", _vp), ("ids", _vp), ("pos", _vp), ("wts", _vp), ("b1", _vp), ("b2", _vp), ("post", _vp),
+                ("pre", _vp), ("out", _vp), ("rows", C.c_long), ("D", C.c_int), ("n", C.c_int), ("parts", C.c_int), ("y_f32", C.c_int),
+                ("out_f32", C.c_int), ("eps", C.c_float), ("mix", C.c_float)]
+
+
+def post_norm(h: torch.Tensor, eps: float, n: int, *, y=None, z=None, ids=None, pos=None, wts=None, parts: int = 1, branch=(None, None),
+              mix: float = 1.0, post=None, pre=None, out_dtype=torch.bfloat16) -> torch.Tensor:
+    """The seam of csrc/post_norm.cu: h (f32 [T, D], in place) gains the norm of the sublayer's output; returns h, or its norm
+    with the weight ``pre``, in ``out_dtype``."""
+    assert h.dtype == torch.float32 and h.is_contiguous()
+    T, D = h.shape
+    a = PostNormArgs()
+    a.h, a.rows, a.D, a.n, a.parts, a.eps, a.mix = _p(h), T, D, n, parts, eps, mix
+    if y is not None:
+        assert y.is_contiguous() and y.shape[-1] == D and y.dtype in (torch.float32, torch.bfloat16)
+        assert (y.shape[0] == T * parts or pos is not None) and (pos is None or (pos.dtype == torch.int32 and pos.numel() == T * parts))
+        assert z is None or (z.shape == y.shape == h.shape and z.dtype == y.dtype and z.is_contiguous())
+        assert wts is None or (wts.dtype == torch.float32 and wts.is_contiguous() and wts.numel() == T * parts)
+        assert ids is None or (ids.dtype == torch.int32 and ids.is_contiguous() and ids.numel() == T * parts)
+        check_index("post_norm", "part row", pos, y.shape[0], low=-1)
+        a.y, a.z, a.ids, a.pos, a.wts, a.y_f32 = _p(y), _p(z), _p(ids), _p(pos), _p(wts), int(y.dtype == torch.float32)
+        a.b1, a.b2, a.post = _p(branch[0]), _p(branch[1]), _p(post)
+    out = torch.empty((T, D), dtype=out_dtype, device=h.device)
+    a.pre, a.out, a.out_f32 = _p(pre), _p(out), int(out_dtype == torch.float32)
+    native.check(_lib().tsb_post_norm(C.byref(a), _stream()), "post_norm")
+    _count(1)
+    return out
+
+
+def pair_embed(tok: QuantWeight, pair: QuantWeight, ids, cu_q, seq_slots, prev, *, mul_prev: int, mul_cur: int, out_dtype):
+    """Token rows plus bigram rows: (f32 [T, D], the same in ``out_dtype``); ``prev`` int32 per slot is read and advanced."""
+    T, D, dev = ids.numel(), tok.K, ids.device
+    check_index("pair_embed", "state slot", seq_slots, prev.shape[0])
+    check_index("pair_embed", "row offset", cu_q, T + 1)
+    check_index("pair_embed", "token", ids, tok.rows)
+    assert ids.dtype == cu_q.dtype == prev.dtype == torch.int32 and seq_slots.dtype == torch.int64 and prev.is_contiguous()
+    assert tok.ggml_type == pair.ggml_type and pair.K == D
+    h, out = torch.empty((T, D), dtype=torch.float32, device=dev), torch.empty((T, D), dtype=out_dtype, device=dev)
+    native.check(_lib().tsb_pair_embed(_p(tok.planes[0]), _p(pair.planes[0]), C.c_int(int(tok.ggml_type)), C.c_int(tok.rows), C.c_int(D), _p(ids),
+                                       _p(cu_q), _p(seq_slots), _p(prev), _p(h), _p(out), C.c_int(out_dtype == torch.float32), C.c_int(T),
+                                       C.c_int(cu_q.numel() - 1), C.c_long(pair.rows - 1), C.c_long(mul_prev), C.c_long(mul_cur), _stream()), "pair_embed")
+    _count(1)
+    return h, out
+
+
+class JointNormArgs(C.Structure):
+    _fields_ = [("y", _vp), ("y_s", C.c_long), ("y_f32", C.c_int), ("w", _vp), ("slot", _vp), ("q", _vp), ("cache", _vp), ("ld", C.c_long),
+                ("T", C.c_int), ("nq", C.c_int), ("nk", C.c_int), ("q_n", C.c_int), ("k_n", C.c_int), ("out_f32", C.c_int), ("eps", C.c_float)]
+
+
+def joint_norm(y: torch.Tensor, w: torch.Tensor, cache: torch.Tensor, slots: torch.Tensor, *, nq: int, nk: int, q_n: int, k_n: int, eps: float) -> torch.Tensor:
+    """Rows [q (nq) | k (nk)]: q over its root mean square times ``w`` -> [T, nq]; k and 1 / its root mean square to the cache rows."""
+    T = y.shape[0]
+    check_index("joint_norm", "cache slot", slots, cache.shape[0])
+    assert y.stride(1) == 1 and y.shape[1] >= nq + nk and cache.is_contiguous() and cache.shape[-1] == nk + 8 and w.numel() == nq
+    a = JointNormArgs()
+    q = torch.empty((T, nq), dtype=cache.dtype, device=y.device)
+    a.y, a.y_s, a.y_f32, a.w, a.slot, a.q, a.cache, a.ld = _p(y), y.stride(0), int(y.dtype == torch.float32), _p(w), _p(slots), _p(q), _p(cache), nk + 8
+    a.T, a.nq, a.nk, a.q_n, a.k_n, a.out_f32, a.eps = T, nq, nk, q_n, k_n, int(cache.dtype == torch.float32), eps
+    native.check(_lib().tsb_joint_norm(C.byref(a), _stream()), "joint_norm")
+    _count(1)
+    return q
+
+
+class GlaArgs(C.Structure):
+    _fields_ = [("y", _vp), ("y_s", C.c_long), ("y_f32", C.c_int), ("q", C.c_long), ("k", C.c_long), ("v", C.c_long), ("g", C.c_long), ("t", C.c_long),
+                ("z", _vp), ("z_s", C.c_long), ("w2", _vp), ("w2_f32", C.c_int), ("zb", _vp), ("norm_w", _vp), ("state", _vp), ("state_s", C.c_long),
+                ("cu_q", _vp), ("seq_slots", _vp), ("seg", _vp), ("seg_w", _vp), ("core", _vp), ("out", _vp), ("out_s", C.c_long),
+                ("out_f32", C.c_int), ("T", C.c_int), ("B", C.c_int), ("H", C.c_int), ("D", C.c_int), ("E", C.c_int), ("e_n", C.c_int),
+                ("rank", C.c_int), ("segs", C.c_int), ("seg_len", C.c_int), ("eps", C.c_float), ("q_scale", C.c_float), ("inv_tau", C.c_float)]
+
+
+def _gla_args(y, s, cols, zb, norm_w, state, cu_q, seq_slots, eps: float, out_dtype):
+    T = y.shape[0]
+    check_index("gated_linear", "state slot", seq_slots, state.shape[0])
+    check_index("gated_linear", "row offset", cu_q, T + 1)
+    assert y.stride(1) == 1 and state.dtype == torch.float32 and state.shape[1:] == (s.H, s.E, s.D) and seq_slots.dtype == torch.int64
+    assert state.stride(1) == s.E * s.D and state.stride(2) == s.D and state.stride(3) == 1
+    a = GlaArgs()
+    a.y, a.y_s, a.y_f32 = _p(y), y.stride(0), int(y.dtype == torch.float32)
+    a.q, a.k, a.v, a.g, a.t = cols
+    a.zb, a.norm_w, a.state, a.state_s, a.cu_q, a.seq_slots = _p(zb), _p(norm_w), _p(state), state.stride(0), _p(cu_q), _p(seq_slots)
+    out = torch.empty((T, s.H * s.E), dtype=out_dtype, device=y.device)
+    a.out, a.out_s, a.out_f32 = _p(out), s.H * s.E, int(out_dtype == torch.float32)
+    a.T, a.B, a.H, a.D, a.E, a.e_n, a.eps, a.q_scale, a.inv_tau = T, cu_q.numel() - 1, s.H, s.D, s.E, s.vdim, eps, s.q_scale, 1.0 / s.tau
+    return a, out
+
+
+def gla_step(y, s, cols, w2: torch.Tensor, zb, norm_w, state, cu_q, seq_slots, *, eps: float, out_dtype) -> torch.Tensor:
+    """Gated linear attention token by token (csrc/gated_linear.cu), decay map, norm and gate included."""
+    a, out = _gla_args(y, s, cols, zb, norm_w, state, cu_q, seq_slots, eps, out_dtype)
+    assert w2.is_contiguous() and w2.shape[0] == s.H * s.D and y.shape[1] >= cols[4] + w2.shape[1]
+    a.w2, a.w2_f32, a.rank = _p(w2), int(w2.dtype == torch.float32), w2.shape[1]
+    native.check(_lib().tsb_gla_step(C.byref(a), _stream()), "gla_step")
+    _count(1)
+    return out
+
+
+def gla_prompt(y, s, cols, z: torch.Tensor, zb, norm_w, state, cu_q, seq_slots, *, eps: float, max_q: int, segs: int) -> torch.Tensor:
+    """The same for prompts of bf16 models, 16 tokens at a time on the tensor cores, in ``segs`` segments per sequence (the
+    longest has ``max_q`` tokens); ``z`` f32 [T, H * D]: the decay's projection."""
+    assert y.dtype == torch.bfloat16 and z.dtype == torch.float32 and z.shape == (y.shape[0], s.H * s.D) and z.stride(1) == 1
+    a, out = _gla_args(y, s, cols, zb, norm_w, state, cu_q, seq_slots, eps, torch.bfloat16)
+    seg_len = (-(-max_q // segs) + 15) // 16 * 16
+    segs = -(-max_q // seg_len)
+    f32 = dict(dtype=torch.float32, device=y.device)
+    if segs > 1:
+        seg, seg_w = torch.empty((a.B, segs, s.H, s.E, s.D), **f32), torch.empty((a.B, segs, s.H, s.D), **f32)
+        a.seg, a.seg_w = _p(seg), _p(seg_w)
+    core = torch.empty((y.shape[0], s.H, s.E), **f32) if s.E > 128 else None
+    a.z, a.z_s, a.core, a.segs, a.seg_len = _p(z), z.stride(0), _p(core), segs, seg_len
+    native.check(_lib().tsb_gla_prompt(C.byref(a), C.c_int(max_q), _stream()), "gla_prompt")
+    _count(1 + 2 * (segs > 1) + (core is not None))
+    return out
+
+
 class LatentArgs(C.Structure):
     _fields_ = [("y", _vp), ("y_s", C.c_long), ("y_f32", C.c_int), ("qn", _vp), ("kn", _vp), ("cs", _vp), ("slots", _vp), ("cache", _vp),
                 ("cq", _vp), ("f32", C.c_int), ("T", C.c_int), ("qr", C.c_int), ("qp", C.c_int), ("R", C.c_int), ("rot", C.c_int),
@@ -646,11 +790,12 @@ class LatentArgs(C.Structure):
                 ("Ro", C.c_int)]
 
 
-def rotary_table(pos: torch.Tensor, freq: torch.Tensor) -> torch.Tensor:
-    """(cos, sin) of pos * freq: float32 [T, pairs, 2]; ``freq`` float64 on the device."""
+def rotary_table(pos: torch.Tensor, freq: torch.Tensor, gain: float = 1.0) -> torch.Tensor:
+    """(cos, sin) of pos * freq, times ``gain``: float32 [T, pairs, 2]; ``freq`` float64 on the device."""
     assert pos.dtype == torch.int32 and freq.dtype == torch.float64
     out = torch.empty((pos.numel(), freq.numel(), 2), dtype=torch.float32, device=pos.device)
-    native.check(_lib().tsb_rotary_table(_p(pos), _p(freq), _p(out), C.c_int(pos.numel()), C.c_int(freq.numel()), _stream()), "rotary_table")
+    native.check(_lib().tsb_rotary_table(_p(pos), _p(freq), _p(out), C.c_int(pos.numel()), C.c_int(freq.numel()),
+                                         C.c_float(gain), _stream()), "rotary_table")
     _count(1)
     return out
 
@@ -832,13 +977,15 @@ def gemm_f32(w: QuantWeight, x: torch.Tensor, *, bias=None, tiles=None, rows=Non
     return out
 
 
-def glu_f32(gate: torch.Tensor, up: Optional[torch.Tensor], act: str) -> torch.Tensor:
-    """Gated activation of two float32 [T, F] views in 32 bits."""
+def glu_f32(gate: torch.Tensor, up: Optional[torch.Tensor], act: str, clamp=None) -> torch.Tensor:
+    """Gated activation of two float32 [T, F] views in 32 bits (``clamp`` as for :func:`glu`)."""
+    lim, lim_first, rows_first = clamp or (7.0, 7.0, 0)
     T, F = gate.shape
     assert gate.dtype == torch.float32 and gate.stride(1) == 1 and (up is None or (up.dtype == torch.float32 and up.stride(1) == 1))
     out = torch.empty((T, F), dtype=torch.float32, device=gate.device)
     native.check(_lib().tsb_glu_f32(_p(gate), _p(up), C.c_long(gate.stride(0)), C.c_long(up.stride(0) if up is not None else 0), C.c_long(T),
-                                    C.c_int(F), C.c_int(ACT[act]), _p(out), _stream()), "glu_f32")
+                                    C.c_int(F), C.c_int(ACT[act]), _p(out), C.c_float(lim), C.c_float(lim_first), C.c_long(rows_first),
+                                    _stream()), "glu_f32")
     _count(1)
     return out
 

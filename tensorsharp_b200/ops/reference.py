@@ -78,7 +78,7 @@ def apply_rope(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, rot_dim: i
     return torch.cat([out, xp], -1)
 
 
-def glu(act: str, g: torch.Tensor, u: Optional[torch.Tensor]) -> torch.Tensor:
+def glu(act: str, g: torch.Tensor, u: Optional[torch.Tensor], clamp: float = 7.0) -> torch.Tensor:
     g = g.float()
     u = u.float() if u is not None else None
     if act == "swiglu":
@@ -88,8 +88,8 @@ def glu(act: str, g: torch.Tensor, u: Optional[torch.Tensor]) -> torch.Tensor:
     if act == "geglu_erf":
         return torch.nn.functional.gelu(g) * u
     if act == "swiglu_oai":
-        x = g.clamp(max=7.0)
-        y = u.clamp(-7.0, 7.0)
+        x = g.clamp(max=clamp)
+        y = u.clamp(-clamp, clamp)
         return x * torch.sigmoid(1.702 * x) * (y + 1.0)
     if act == "relu2":
         return torch.relu(g) ** 2
@@ -101,9 +101,11 @@ def glu(act: str, g: torch.Tensor, u: Optional[torch.Tensor]) -> torch.Tensor:
 
 
 def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_pos: torch.Tensor, *, scale: float,
-              window: int = 0, sinks: Optional[torch.Tensor] = None, softcap: float = 0.0) -> torch.Tensor:
+              window: int = 0, sinks: Optional[torch.Tensor] = None, softcap: float = 0.0, keep_first: int = 0,
+              slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Naive attention for one sequence.  q [Tq, Hq, Dh]; k, v [Tk, Hkv, Dh] hold cache
-    positions 0..Tk-1; q_pos [Tq] are the queries' positions.  Returns [Tq, Hq, Dh] f32."""
+    positions 0..Tk-1; q_pos [Tq] are the queries' positions.  ``keep_first`` positions stay visible outside the window;
+    ``slopes`` [Hq] times the distance is taken off the scores.  Returns [Tq, Hq, Dh] f32."""
     Tq, Hq, Dh = q.shape
     Tk, Hkv, _ = k.shape
     g = Hq // Hkv
@@ -115,9 +117,11 @@ def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_pos: torch.Te
         s = softcap * torch.tanh(s / softcap)
     j = torch.arange(Tk, device=q.device).view(1, 1, Tk)
     p = q_pos.view(1, Tq, 1)
+    if slopes is not None:
+        s = s - slopes.float().view(Hq, 1, 1) * (p - j)
     ok = j <= p
     if window and window > 0:
-        ok = ok & (j > p - window)
+        ok = ok & ((j > p - window) | (j < keep_first))
     s = s.masked_fill(~ok, float("-inf"))
     if sinks is not None:
         s = torch.cat([s, sinks.float().view(Hq, 1, 1).expand(Hq, Tq, 1)], -1)
@@ -143,6 +147,16 @@ def general_delta(r, k, v, decay, a, state: torch.Tensor) -> torch.Tensor:
         read = torch.einsum("hvk,hk->hv", state, u[t])
         state.mul_(decay[t].unsqueeze(1)).sub_(read.unsqueeze(2) * au[t].unsqueeze(1)).add_(v[t].unsqueeze(2) * k[t].unsqueeze(1))
         out[t] = torch.einsum("hvk,hk->hv", state, r[t])
+    return out
+
+
+def gated_linear(q, k, v, decay, state: torch.Tensor) -> torch.Tensor:
+    """Gated linear attention of one sequence: q, k, decay [T, H, D], v [T, H, E]; ``state`` [H, E, D] is advanced in place.
+    Per token: S <- S diag(decay) + v k^T;  o = S q."""
+    out = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        state.mul_(decay[t].unsqueeze(1)).add_(v[t].unsqueeze(2) * k[t].unsqueeze(1))
+        out[t] = torch.einsum("hvk,hk->hv", state, q[t])
     return out
 
 
