@@ -617,7 +617,7 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, bat
             rows = k_cache[idx].view(L, -1)
             if window:
                 rows = rows.clone()
-                rows[:max(0, L - (q1 - q0) - window + 1)] = 0              # out of every query's sight; may be stale in a ring
+                rows[keep_first:max(keep_first, L - (q1 - q0) - window + 1)] = 0       # out of every query's sight; may be stale in a ring
             vb = rows[:, :Hkv * Dh].view(L, Hkv, Dh)
             kb = vb * rows[:, Hkv * Dh].view(L, 1, 1)
         else:
