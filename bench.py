@@ -57,7 +57,7 @@ def parse_args():
     ap.add_argument("--trace", default=None, metavar="FILE",
                     help="after the timed runs, record three more graph replays with the CUDA activity tracer, write the "
                          "kernel events of the middle one to FILE (JSON) and print its per-kernel table to stderr")
-    ap.add_argument("--design", default=None, choices=["fobolorn", "sogulix"],
+    ap.add_argument("--design", default=None, choices=["fobolorn", "sogulix", "kegetar"],
                     help="measure this design at several sizes beside the closest other model at equal size (one JSON line per "
                          "size and model) instead of the headline workload")
     ap.add_argument("--design-size", default=None, help="with --design: only this size")
@@ -499,6 +499,10 @@ def run_reference(args) -> dict:
 # sizes, beside gpt-oss heads of the larger size.
 # Sogulix beside dense Qwen3.5 (the other hybrid of a delta rule and attention): as many heads of the same size in the
 # recurrent layers, one attention layer in four; "looped" runs its first four layers twice, beside as many layers as it runs.
+# Kegetar beside Qwen3.5 (linear and ordinary attention, experts with a shared one): every other layer of Kegetar is parallel, and
+# half of Qwen3.5's layers are recurrent with as many heads of the same size; "dense" without experts, with 16 query heads per KV
+# head; "uneven" with windows that bite, kept first tokens, smaller heads in the linear half, and identity experts (of 40 entries
+# a token takes four, Qwen3.5 four of 32 experts).
 _Q35 = dict(n_experts=0, interval=4, vocab=32000, context=16384)
 DESIGNS = {
     "fobolorn": ("gpt-oss", {
@@ -520,13 +524,30 @@ DESIGNS = {
                         delta_heads=24, delta_dim=64, decay_rank=48, ff=4096, vocab=32000),
                    dict(n_layers=12, hidden=1536, n_heads=12, n_kv_heads=4, head_dim=64, rope_dims=32, hk=24, hv=24, dk=64, dv=64, ffn=4096, **_Q35)),
     }),
+    "kegetar": ("qwen3.5", {
+        "2048x8": (dict(layers="pa" * 4, mlps="m" * 8, width=2048, heads=16, kv_heads=4, dim=128, vdim=128, window=1 << 20, keep_first=0, linear_heads=16,
+                        linear_dim=128, linear_vdim=128, decay_rank=64, own_heads=16, own_kv_heads=4, own_dim=128, own_window=1 << 20, expert_ff=1024,
+                        experts=32, identity=0, top=4, groups=(4, 3), shared_ff=1024, shared_limit=1.5, vocab=32000),
+                   dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, rope_dims=64, hk=16, hv=16, dk=128, dv=128, interval=2,
+                        n_experts=32, top_k=4, expert_ffn=1024, shared_ffn=1024, vocab=32000, context=16384)),
+        "dense": (dict(layers="pa" * 2, mlps="d" * 4, width=4096, heads=32, kv_heads=8, dim=128, vdim=128, window=1 << 20, keep_first=0, linear_heads=32,
+                       linear_dim=128, linear_vdim=128, decay_rank=64, own_heads=32, own_kv_heads=2, own_dim=128, own_window=1 << 20, ff=12288,
+                       vocab=32000),
+                  dict(n_layers=4, hidden=4096, n_heads=32, n_kv_heads=8, head_dim=128, rope_dims=64, hk=32, hv=32, dk=128, dv=128, ffn=12288,
+                       **{**_Q35, "interval": 2})),
+        "uneven": (dict(layers="pa" * 4, mlps="m" * 8, width=2048, heads=16, kv_heads=4, dim=96, vdim=128, window=1024, keep_first=64, linear_heads=32,
+                        linear_dim=64, linear_vdim=64, decay_rank=32, own_heads=16, own_kv_heads=1, own_dim=128, own_window=512, expert_ff=1024,
+                        experts=32, identity=8, top=4, groups=(4, 3), shared_ff=1024, shared_limit=3.0, vocab=32000),
+                   dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, rope_dims=64, hk=32, hv=32, dk=64, dv=64, interval=2,
+                        n_experts=32, top_k=4, expert_ffn=1024, shared_ffn=1024, vocab=32000, context=16384)),
+    }),
 }
 
 
 def write_design(name: str, path: str, sizes: dict) -> str:
     """The synthetic model ``name`` of these sizes at ``path`` (a folder, or a GGUF file of that stem); returns where it is."""
     from tensorsharp_b200.models import synth
-    if name in ("fobolorn", "sogulix"):
+    if name in ("fobolorn", "sogulix", "kegetar"):
         getattr(synth, f"write_{name}")(path, seed=0, **sizes)
         return path
     path += ".gguf"
