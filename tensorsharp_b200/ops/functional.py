@@ -1265,9 +1265,10 @@ GATED_LINEAR_CHUNK_MIN = 12          # tokens of the longest portion from which 
 
 
 def gated_linear_segments(batch: Batch, s: GatedLinearSpec) -> int:
-    """Pieces in which the chunk kernel takes the batch's sequences: about two CTAs per SM, no fewer than 64 tokens each."""
-    ctas = batch.B * s.H * (2 if s.E > 128 else 1)
-    return max(1, min(round(2 * 148 / ctas), batch.max_q_len // 64))
+    """Pieces in which the chunk kernel takes the batch's sequences: about sixteen warps per SM (one per 16 value columns), no
+    fewer than 64 tokens each."""
+    warps = batch.B * s.H * s.E // 16
+    return max(1, min(round(16 * 148 / warps), batch.max_q_len // 64))
 
 
 def gated_linear(y: torch.Tensor, s: GatedLinearSpec, cols: Tuple[int, ...], w2: QuantWeight, zb: torch.Tensor, norm_w: torch.Tensor,
