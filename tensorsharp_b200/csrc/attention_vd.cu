@@ -10,7 +10,7 @@
 //
 // These kernels also know a window with kept first positions (two ranges of key tiles), a distance bias per head, a gate per
 // output column, and caches whose rows are key and value at once (AttnArgs::kv_scale): one tile is then staged and read both
-// ways, and the scores get the factor of their key.
+// ways, and the scores get the factor of their key.  They are instances of their own (FORMS), which leaves the others as they are.
 #include "attn_args.cuh"
 #include "attn_mma.cuh"
 #include "common.cuh"
@@ -101,7 +101,7 @@ __device__ __forceinline__ void vd_qk(float (&s)[KT / 8][4], const bf16* q16, in
 // ------------------------------------------------------------------------------------------
 // Prefill: grid (query tiles, Hq, B), 128 threads.
 // ------------------------------------------------------------------------------------------
-template <int DV>
+template <int DV, bool FORMS>
 __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
     constexpr int BM = 64, BN = 64;
     pdl_wait();
@@ -125,10 +125,10 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
     const int j_hi = min(pos0 + m0 + rows, kvlen);
     const int t_lo = j_lo / BN, t_hi = (j_hi + BN - 1) / BN;
     // tiles in order: those of the kept first positions that lie ahead of the window, then the window's
-    const int n_first = a.keep_first > 0 ? min(t_lo, (a.keep_first + BN - 1) / BN) : 0, n_tiles = n_first + t_hi - t_lo;
-    const bool one_row = a.kv_scale != 0;
+    const int n_first = FORMS && a.keep_first > 0 ? min(t_lo, (a.keep_first + BN - 1) / BN) : 0, n_tiles = n_first + t_hi - t_lo;
+    const bool one_row = FORMS && a.kv_scale != 0;
     float* sF = reinterpret_cast<float*>(sV);                          // 2 stages of key factors, in place of the value tiles
-    const float slope = a.slopes ? a.slopes[h] : 0.f;
+    const float slope = FORMS && a.slopes ? a.slopes[h] : 0.f;
 
     for (int i = threadIdx.x; i < BM * ck; i += 128) {
         const int r = i / ck, c = i % ck;
@@ -198,7 +198,7 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
                 for (int e = 0; e < 4; ++e) s[nt][e] = a.softcap * tanhf(s[nt][e] * inv_cap);
             f = 1.f;
         }
-        if (a.slopes != nullptr) {
+        if (FORMS && a.slopes != nullptr) {
             const int d0 = t * BN + (lane & 3) * 2 - qpos_a;                        // key minus query
 #pragma unroll
             for (int nt = 0; nt < BN / 8; ++nt)
@@ -215,7 +215,7 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
                 for (int e = 0; e < 4; ++e) {
                     const int j = t * BN + nt * 8 + (lane & 3) * 2 + (e & 1);
                     const int qp = (e < 2) ? qpos_a : qpos_b;
-                    const bool ok = j <= qp && j < kvlen && (a.window <= 0 || j > qp - a.window || j < a.keep_first);
+                    const bool ok = j <= qp && j < kvlen && (a.window <= 0 || j > qp - a.window || (FORMS && j < a.keep_first));
                     s[nt][e] = ok ? s[nt][e] : -INFINITY;
                 }
         }
@@ -238,7 +238,7 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
         inv[r] = ll > 0.f ? oc / ll : 0.f;
         const int row = r_lo + 8 * r;
         if (row < rows) {
-            if (!a.gate_cols) inv[r] *= attn_gate(a, q0 + m0 + row, h);
+            if (!FORMS || !a.gate_cols) inv[r] *= attn_gate(a, q0 + m0 + row, h);
             if (a.lse_out != nullptr && (lane & 3) == 0)
                 a.lse_out[(long)(q0 + m0 + row) * a.Hq + h] = lrow[r] > 0.f ? mrow[r] + __logf(lrow[r]) : -INFINITY;
         }
@@ -246,7 +246,7 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i) {
         const int d = i * 8 + (lane & 3) * 2;
-        if (a.gate_cols) {
+        if (FORMS && a.gate_cols) {
             const long t = q0 + m0 + r_lo;
             if (r_lo < rows) { o[i][0] *= attn_gate(a, t, h, d); o[i][1] *= attn_gate(a, t, h, d + 1); }
             if (r_lo + 8 < rows) { o[i][2] *= attn_gate(a, t + 8, h, d); o[i][3] *= attn_gate(a, t + 8, h, d + 1); }
@@ -262,7 +262,7 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
 // Decode: grid (splits, Hkv * chunks, B), 128 threads; a CTA serves up to 16 query heads of one KV head.  Each warp walks
 // its own 32-key pieces of the split.
 // ------------------------------------------------------------------------------------------
-template <int DV>
+template <int DV, bool FORMS>
 __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chunks) {
     constexpr int KT = 32, cv = DV / 8;
     pdl_wait();
@@ -271,7 +271,7 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
     const int dk = a.Dh, ldk = dk + 8, ldv = DV + 8, ck = dk / 8;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     bf16* sQ = reinterpret_cast<bf16*>(smem_raw);                       // [16][ldk]
-    bf16* sK = sQ + 16 * ldk + warp * KT * (a.kv_scale ? ldk : ldk + ldv);                 // this warp's K tile
+    bf16* sK = sQ + 16 * ldk + warp * KT * (FORMS && a.kv_scale ? ldk : ldk + ldv);                 // this warp's K tile
     bf16* sV = sK + KT * ldk;                                           // and V tile
     const int split = blockIdx.x, hk = blockIdx.y / chunks, b = blockIdx.z;
     const int group = a.Hq / a.Hkv, first = (blockIdx.y % chunks) * 16;
@@ -285,13 +285,13 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
     }
     // the visible positions, numbered without a gap: the kept first ones ahead of the window, then the window
     const int len = a.kv_lens[b];
-    const int lo = (a.window > 0 && len > a.window) ? len - a.window : 0, nf = min(a.keep_first, lo), gap = lo - nf;
+    const int lo = (a.window > 0 && len > a.window) ? len - a.window : 0, nf = FORMS ? min(a.keep_first, lo) : 0, gap = lo - nf;
     const int span = len - gap;
     const int per = a.split_len > 0 ? a.split_len : ((((span + a.splits - 1) / a.splits) + 31) & ~31);
     const int s0 = split * per, s1 = min(span, s0 + per);
-    const bool one_row = a.kv_scale != 0;
+    const bool one_row = FORMS && a.kv_scale != 0;
     float slope[2] = {0.f, 0.f};
-    if (a.slopes != nullptr) {
+    if (FORMS && a.slopes != nullptr) {
 #pragma unroll
         for (int r = 0; r < 2; ++r)
             if ((lane >> 2) + 8 * r < G) slope[r] = a.slopes[h0 + (lane >> 2) + 8 * r];
@@ -344,7 +344,7 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
                 for (int e = 0; e < 4; ++e) s[nt][e] = a.softcap * tanhf(s[nt][e] * a.scale / a.softcap);
             f = 1.f;
         }
-        if (a.slopes != nullptr) {
+        if (FORMS && a.slopes != nullptr) {
 #pragma unroll
             for (int nt = 0; nt < KT / 8; ++nt)
 #pragma unroll
@@ -403,26 +403,32 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
     }
 }
 
-template <int DV>
-static int launch_vd(const AttnArgs& a, int max_q, cudaStream_t s) {
+template <int DV, bool FORMS>
+static int launch_vd_form(const AttnArgs& a, int max_q, cudaStream_t s) {
     const int ldk = a.Dh + 8, ldv = DV + 8;
     static bool configured = false;
     if (!configured) {
-        TSB_CHECK_CUDA(cudaFuncSetAttribute(attn_prefill_vd_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-        TSB_CHECK_CUDA(cudaFuncSetAttribute(attn_decode_vd_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        TSB_CHECK_CUDA(cudaFuncSetAttribute(attn_prefill_vd_kernel<DV, FORMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        TSB_CHECK_CUDA(cudaFuncSetAttribute(attn_decode_vd_kernel<DV, FORMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
         configured = true;
     }
     if (max_q > 0) {
         const size_t smem = (size_t)(64 * ldk + 2 * 64 * (a.kv_scale ? ldk + 2 : ldk + ldv)) * sizeof(bf16);       // (a factor per row: two elements)
-        TSB_CHECK_CUDA(tsb_launch(attn_prefill_vd_kernel<DV>, dim3((max_q + 63) / 64, a.Hq, a.B), dim3(128), smem, s, a));
+        TSB_CHECK_CUDA(tsb_launch(attn_prefill_vd_kernel<DV, FORMS>, dim3((max_q + 63) / 64, a.Hq, a.B), dim3(128), smem, s, a));
     } else {
         const int chunks = (a.Hq / a.Hkv + 15) / 16;
         const size_t stage = (size_t)(16 * ldk + 4 * 32 * (a.kv_scale ? ldk : ldk + ldv)) * sizeof(bf16), merge = (size_t)(128 + 4 * 16 * DV) * sizeof(float);
-        TSB_CHECK_CUDA(tsb_launch(attn_decode_vd_kernel<DV>, dim3(a.splits, a.Hkv * chunks, a.B), dim3(128), stage > merge ? stage : merge, s,
+        TSB_CHECK_CUDA(tsb_launch(attn_decode_vd_kernel<DV, FORMS>, dim3(a.splits, a.Hkv * chunks, a.B), dim3(128), stage > merge ? stage : merge, s,
                                   a, chunks));
     }
     TSB_CHECK_LAUNCH();
     return TSB_OK;
+}
+
+template <int DV>
+static int launch_vd(const AttnArgs& a, int max_q, cudaStream_t s) {
+    const bool forms = a.keep_first > 0 || a.slopes != nullptr || a.gate_cols || a.kv_scale;
+    return forms ? launch_vd_form<DV, true>(a, max_q, s) : launch_vd_form<DV, false>(a, max_q, s);
 }
 
 static int dispatch_vd(const AttnArgs& in, int max_q, cudaStream_t s) {
