@@ -125,7 +125,7 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
     const int j_hi = min(pos0 + m0 + rows, kvlen);
     const int t_lo = j_lo / BN, t_hi = (j_hi + BN - 1) / BN;
     // tiles in order: those of the kept first positions that lie ahead of the window, then the window's
-    const int n_first = FORMS && a.keep_first > 0 ? min(t_lo, (a.keep_first + BN - 1) / BN) : 0, n_tiles = n_first + t_hi - t_lo;
+    const int n_first = FORMS && a.keep_first > 0 ? min(t_lo, (a.keep_first + BN - 1) / BN) : 0;
     const bool one_row = FORMS && a.kv_scale != 0;
     float* sF = reinterpret_cast<float*>(sV);                          // 2 stages of key factors, in place of the value tiles
     const float slope = FORMS && a.slopes ? a.slopes[h] : 0.f;
@@ -162,8 +162,7 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
             for (int c = 0; c < cv; c += 2) *reinterpret_cast<uint4*>(pv + (c + half) * 8) = make_uint4(0, 0, 0, 0);
         }
     };
-    auto tile = [&](int u) { return u < n_first ? u : t_lo + u - n_first; };
-    load_kv(tile(0), 0);
+    load_kv(n_first > 0 ? 0 : t_lo, 0);
     cp_async_commit();
 
     float o[DV / 8][4];
@@ -174,9 +173,9 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
     const int qpos_a = pos0 + m0 + r_lo, qpos_b = qpos_a + 8;
     const int q_first = pos0 + m0 + warp * 16;
 
-    for (int u = 0; u < n_tiles; ++u) {
-        const int stage = u & 1, t = tile(u);
-        if (u + 1 < n_tiles) load_kv(tile(u + 1), stage ^ 1);
+    for (int t = n_first > 0 ? 0 : t_lo, flip = 0; t < t_hi; t = FORMS && t + 1 == n_first ? t_lo : t + 1, flip ^= 1) {
+        const int stage = FORMS ? flip : (t - t_lo) & 1, next = FORMS && t + 1 == n_first ? t_lo : t + 1;
+        if (next < t_hi) load_kv(next, stage ^ 1);
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
