@@ -527,7 +527,7 @@ DESIGNS = {
     "kegetar": ("qwen3.5", {
         "2048x8": (dict(layers="pa" * 4, mlps="m" * 8, width=2048, heads=16, kv_heads=4, dim=128, vdim=128, window=1 << 20, keep_first=0, linear_heads=16,
                         linear_dim=128, linear_vdim=128, decay_rank=64, own_heads=16, own_kv_heads=4, own_dim=128, own_window=1 << 20, expert_ff=1024,
-                        experts=32, identity=0, top=4, groups=(4, 3), shared_ff=1024, shared_limit=1.5, vocab=32000),
+                        experts=32, identity=0, top=4, groups=(8, 6), shared_ff=1024, vocab=32000),
                    dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, rope_dims=64, hk=16, hv=16, dk=128, dv=128, interval=2,
                         n_experts=32, top_k=4, expert_ffn=1024, shared_ffn=1024, vocab=32000, context=16384)),
         "dense": (dict(layers="pa" * 2, mlps="d" * 4, width=4096, heads=32, kv_heads=8, dim=128, vdim=128, window=1 << 20, keep_first=0, linear_heads=32,
@@ -537,7 +537,7 @@ DESIGNS = {
                        **{**_Q35, "interval": 2})),
         "uneven": (dict(layers="pa" * 4, mlps="m" * 8, width=2048, heads=16, kv_heads=4, dim=96, vdim=128, window=1024, keep_first=64, linear_heads=32,
                         linear_dim=64, linear_vdim=64, decay_rank=32, own_heads=16, own_kv_heads=1, own_dim=128, own_window=512, expert_ff=1024,
-                        experts=32, identity=8, top=4, groups=(4, 3), shared_ff=1024, shared_limit=3.0, vocab=32000),
+                        experts=32, identity=8, top=4, groups=(8, 6), shared_ff=1024, vocab=32000),
                    dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, rope_dims=64, hk=32, hv=32, dk=64, dv=64, interval=2,
                         n_experts=32, top_k=4, expert_ffn=1024, shared_ffn=1024, vocab=32000, context=16384)),
     }),

@@ -652,9 +652,9 @@ def write_sogulix(folder: str, config: Optional[dict] = None, *, seed=0, device=
 
 
 def kegetar_config(*, layers="papa", mlps="dmdm", width=128, heads=4, kv_heads=2, dim=32, vdim=48, window=24, keep_first=3, rot_dims=None,
-                   rot_base=10000.0, yarn=(8.0, 256, 32.0, 1.0), linear_heads=3, linear_dim=32, linear_vdim=48, tau=16.0, decay_rank=8,
-                   own_heads=4, own_kv_heads=1, own_dim=32, own_window=20, ff=64, expert_ff=32, limit=1.5, experts=6, identity=2, top=3,
-                   groups=(4, 3), shared_ff=40, shared_limit=1.0, buckets=251, muls=(31, 17), vocab=512, residual_mult=0.5, eps=1e-6,
+                   rot_base=10000.0, yarn=(6.0, 300, 24.0, 1.5), linear_heads=3, linear_dim=32, linear_vdim=48, tau=12.0, decay_rank=8,
+                   own_heads=4, own_kv_heads=1, own_dim=32, own_window=20, ff=64, expert_ff=32, limit=1.2, experts=6, identity=2, top=3,
+                   groups=(4, 2), shared_ff=40, shared_limit=0.9, buckets=251, muls=(37, 11), vocab=512, residual_mult=0.7, eps=1e-5,
                    weights_of=None, scale=None) -> dict:
     """A config.json of the Kegetar architecture: ``layers`` has a ``p`` (parallel) or an ``a`` (attention) per layer, ``mlps`` a ``d``
     (dense), an ``m`` (mixture of experts) or a ``-``; ``weights_of``: layer -> the layer whose weights it uses.  The rank of the
