@@ -10,7 +10,9 @@
 //
 // These kernels also know a window with kept first positions (two ranges of key tiles), a distance bias per head, a gate per
 // output column, and caches whose rows are key and value at once (AttnArgs::kv_scale): one tile is then staged and read both
-// ways, and the scores get the factor of their key.  They are instances of their own (FORMS), which leaves the others as they are.
+// ways, and the scores get the factor of their key.  They are instances of their own (FORM 1), which leaves the others as they are.
+// Further instances (FORM 2) know all of that, a distance bias r1 ln(1 + r2 d), and weights sigmoid(score + bias) in place of the
+// softmax: those need no running maximum and no sum.  In prompts the bias of a tile's 127 distances is found once, by one thread each.
 #include "attn_args.cuh"
 #include "attn_mma.cuh"
 #include "common.cuh"
@@ -58,6 +60,24 @@ __device__ __forceinline__ void vd_softmax(float (&s)[KT / 8][4], float (&o)[NO]
     }
 }
 
+constexpr float VD_LOG2E = 1.4426950408889634f;
+__device__ __forceinline__ float vd_ex2(float x) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+__device__ __forceinline__ float vd_rcp(float x) {
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+// The score x (unscaled product) with soft cap c (0: none): c tanh(f x / c) = c - 2 c / (1 + e^(2 f x / c)), to an absolute error of a
+// few 1e-7 c.  `two`: 2 f log2(e) / c.
+__device__ __forceinline__ float vd_cap(float x, float f, float c, float two) {
+    return c > 0.f ? fmaf(-2.f * c, vd_rcp(1.f + vd_ex2(x * two)), c) : x * f;
+}
+__device__ __forceinline__ float vd_sigmoid(float x) { return vd_rcp(1.f + vd_ex2(-VD_LOG2E * x)); }
+
 template <int KT, int DV>
 __device__ __forceinline__ void vd_pv(const float (&s)[KT / 8][4], float (&o)[DV / 8][4], const bf16* tV, int ldv, int lane) {
 #pragma unroll
@@ -101,9 +121,11 @@ __device__ __forceinline__ void vd_qk(float (&s)[KT / 8][4], const bf16* q16, in
 // ------------------------------------------------------------------------------------------
 // Prefill: grid (query tiles, Hq, B), 128 threads.
 // ------------------------------------------------------------------------------------------
-template <int DV, bool FORMS>
+template <int DV, int FORM>
 __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
     constexpr int BM = 64, BN = 64;
+    constexpr bool FORMS = FORM > 0, EXT = FORM == 2;
+    __shared__ float s_dist[EXT ? 128 : 1];          // what is added to the score, per distance of a tile (query row - key column + 63)
     pdl_wait();
     pdl_trigger();
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -129,6 +151,9 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
     const bool one_row = FORMS && a.kv_scale != 0;
     float* sF = reinterpret_cast<float*>(sV);                          // 2 stages of key factors, in place of the value tiles
     const float slope = FORMS && a.slopes ? a.slopes[h] : 0.f;
+    const bool sig = EXT && a.sig_bias != nullptr;
+    const float pb = sig ? a.sig_bias[h] : 0.f, r1 = EXT && a.log_r1 ? a.log_r1[h] : 0.f, r2 = EXT && a.log_r1 ? a.log_r2[h] : 0.f;
+    const float cap2 = EXT && a.softcap > 0.f ? 2.f * VD_LOG2E * a.scale / a.softcap : 0.f;
 
     for (int i = threadIdx.x; i < BM * ck; i += 128) {
         const int r = i / ck, c = i % ck;
@@ -177,6 +202,7 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
         const int stage = FORMS ? flip : (t - t_lo) & 1, next = FORMS && t + 1 == n_first ? t_lo : t + 1;
         if (next < t_hi) load_kv(next, stage ^ 1);
         cp_async_commit();
+        if (EXT) s_dist[threadIdx.x] = pb - r1 * log1pf(r2 * (float)max(0, pos0 + m0 - t * BN + (int)threadIdx.x - 63));
         cp_async_wait<1>();
         __syncthreads();
         float s[BN / 8][4];
@@ -189,7 +215,14 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
             }
         }
         float f = a.scale;
-        if (a.softcap > 0.f) {
+        if (EXT) {
+            const float* dist = s_dist + r_lo - (lane & 3) * 2 + 63;
+#pragma unroll
+            for (int nt = 0; nt < BN / 8; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[nt][e] = vd_cap(s[nt][e], a.scale, a.softcap, cap2) + dist[(e < 2 ? 0 : 8) - nt * 8 - (e & 1)];
+            f = 1.f;
+        } else if (a.softcap > 0.f) {
             const float inv_cap = a.scale / a.softcap;
 #pragma unroll
             for (int nt = 0; nt < BN / 8; ++nt)
@@ -218,7 +251,14 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
                     s[nt][e] = ok ? s[nt][e] : -INFINITY;
                 }
         }
-        vd_softmax<BN, DV / 8>(s, o, mrow, lrow, f);
+        if (sig) {
+#pragma unroll
+            for (int nt = 0; nt < BN / 8; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[nt][e] = vd_sigmoid(s[nt][e]);             // -inf: 0
+        } else {
+            vd_softmax<BN, DV / 8>(s, o, mrow, lrow, f);
+        }
         vd_pv<BN, DV>(s, o, one_row ? sK + stage * BN * ldk : sV + stage * BN * ldv, ldv, lane);      // one row: ldk = ldv
         __syncthreads();
     }
@@ -234,7 +274,7 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
             oc = (mm == -INFINITY) ? 0.f : __expf(mm - mn);
             ll = ll * oc + __expf(sk - mn);
         }
-        inv[r] = ll > 0.f ? oc / ll : 0.f;
+        inv[r] = sig ? 1.f : ll > 0.f ? oc / ll : 0.f;
         const int row = r_lo + 8 * r;
         if (row < rows) {
             if (!FORMS || !a.gate_cols) inv[r] *= attn_gate(a, q0 + m0 + row, h);
@@ -261,9 +301,10 @@ __global__ void __launch_bounds__(128) attn_prefill_vd_kernel(AttnArgs a) {
 // Decode: grid (splits, Hkv * chunks, B), 128 threads; a CTA serves up to 16 query heads of one KV head.  Each warp walks
 // its own 32-key pieces of the split.
 // ------------------------------------------------------------------------------------------
-template <int DV, bool FORMS>
+template <int DV, int FORM>
 __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chunks) {
     constexpr int KT = 32, cv = DV / 8;
+    constexpr bool FORMS = FORM > 0, EXT = FORM == 2;
     pdl_wait();
     pdl_trigger();
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -294,6 +335,19 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
 #pragma unroll
         for (int r = 0; r < 2; ++r)
             if ((lane >> 2) + 8 * r < G) slope[r] = a.slopes[h0 + (lane >> 2) + 8 * r];
+    }
+    const bool sig = EXT && a.sig_bias != nullptr;
+    const float cap2 = EXT && a.softcap > 0.f ? 2.f * VD_LOG2E * a.scale / a.softcap : 0.f;
+    float pb[2] = {0.f, 0.f}, r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};
+    if (EXT) {
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int row = (lane >> 2) + 8 * r;
+            if (row < G) {
+                if (sig) pb[r] = a.sig_bias[h0 + row];
+                if (a.log_r1 != nullptr) { r1[r] = a.log_r1[h0 + row]; r2[r] = a.log_r2[h0 + row]; }
+            }
+        }
     }
     __syncthreads();
 
@@ -336,7 +390,17 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
             }
         }
         float f = a.scale;
-        if (a.softcap > 0.f) {
+        if (EXT) {
+#pragma unroll
+            for (int nt = 0; nt < KT / 8; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int i = base + nt * 8 + (lane & 3) * 2 + (e & 1), r = e >> 1;
+                    const float d = (float)max(0, len - 1 - (i < nf ? i : i + gap));
+                    s[nt][e] = vd_cap(s[nt][e], a.scale, a.softcap, cap2) + (pb[r] - r1[r] * __logf(fmaf(r2[r], d, 1.f)));
+                }
+            f = 1.f;
+        } else if (a.softcap > 0.f) {
 #pragma unroll
             for (int nt = 0; nt < KT / 8; ++nt)
 #pragma unroll
@@ -358,7 +422,14 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
 #pragma unroll
             for (int e = 0; e < 4; ++e)
                 if (base + nt * 8 + (lane & 3) * 2 + (e & 1) >= s1) s[nt][e] = -INFINITY;
-        vd_softmax<KT, DV / 8>(s, o, mrow, lrow, f);
+        if (sig) {
+#pragma unroll
+            for (int nt = 0; nt < KT / 8; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[nt][e] = vd_sigmoid(s[nt][e]);
+        } else {
+            vd_softmax<KT, DV / 8>(s, o, mrow, lrow, f);
+        }
         vd_pv<KT, DV>(s, o, one_row ? sK : sV, ldv, lane);
         __syncwarp();
     }
@@ -366,6 +437,7 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
     for (int r = 0; r < 2; ++r) {
         lrow[r] += __shfl_xor_sync(0xffffffffu, lrow[r], 1);
         lrow[r] += __shfl_xor_sync(0xffffffffu, lrow[r], 2);
+        if (sig) mrow[r] = 0.f;                                         // partial sums are added as they are
     }
     __syncthreads();
     float* red_m = reinterpret_cast<float*>(smem_raw);                  // [4][16]
@@ -402,7 +474,7 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
     }
 }
 
-template <int DV, bool FORMS>
+template <int DV, int FORMS>
 static int launch_vd_form(const AttnArgs& a, int max_q, cudaStream_t s) {
     const int ldk = a.Dh + 8, ldv = DV + 8;
     static bool configured = false;
@@ -426,8 +498,9 @@ static int launch_vd_form(const AttnArgs& a, int max_q, cudaStream_t s) {
 
 template <int DV>
 static int launch_vd(const AttnArgs& a, int max_q, cudaStream_t s) {
+    if (a.log_r1 != nullptr || a.sig_bias != nullptr) return launch_vd_form<DV, 2>(a, max_q, s);
     const bool forms = a.keep_first > 0 || a.slopes != nullptr || a.gate_cols || a.kv_scale;
-    return forms ? launch_vd_form<DV, true>(a, max_q, s) : launch_vd_form<DV, false>(a, max_q, s);
+    return forms ? launch_vd_form<DV, 1>(a, max_q, s) : launch_vd_form<DV, 0>(a, max_q, s);
 }
 
 static int dispatch_vd(const AttnArgs& in, int max_q, cudaStream_t s) {
@@ -437,6 +510,8 @@ static int dispatch_vd(const AttnArgs& in, int max_q, cudaStream_t s) {
     if (a.v_ld == 0) a.v_ld = (long)a.Hkv * a.Dv;
     TSB_CHECK_ARG(a.kv_scale == 0 || (a.Dv == a.Dh && a.kv_scale % 2 == 0), "attention: rows of %d / %d elements are not key and value at once", a.Dh, a.Dv);
     TSB_CHECK_ARG(a.keep_first >= 0 && (a.keep_first == 0 || a.window > 0), "attention: kept first positions without a window");
+    TSB_CHECK_ARG(a.sig_bias == nullptr || (a.sinks == nullptr && a.lse_out == nullptr), "attention: sigmoid weights have no sink and no log-sum-exp");
+    TSB_CHECK_ARG((a.log_r1 == nullptr) == (a.log_r2 == nullptr), "attention: a logarithmic distance bias has two numbers per head");
     TSB_CHECK_ARG(a.split_len == 0 || a.window <= 0, "attention: fixed splits with a window");
     TSB_CHECK_ARG(a.k_ld % 8 == 0 && a.v_ld % 8 == 0, "attention: cache rows of %ld / %ld elements are not 16-byte aligned", a.k_ld, a.v_ld);
     if (a.Dh <= 0 || a.Dh > 256 || a.Dh % 16 || a.Dv <= 0 || a.Dv > 256 || a.Dv % 16) {

@@ -45,12 +45,15 @@ struct AttnArgs {
     int gate_cols;            // 1: the gate has a value per output column, gate[t * gate_tok + h * Dv + d]
     int kv_scale;             // != 0: a row of k_cache is key and value at once (Dv = Dh; v_cache is not read), and the score of a
                               // key is multiplied by the f32 number that starts at element kv_scale of its row
+    const float* log_r1;      // [Hq] or null: log_r1[h] ln(1 + log_r2[h] (query position - key position)) is taken off the score
+    const float* log_r2;
+    const float* sig_bias;    // [Hq] or null: no softmax; a visible key's weight is sigmoid(score + sig_bias[h])
 };
 
 // Whether only the kernels for head sizes of their own know a form that these arguments ask for.
 static inline bool attn_needs_vd(const AttnArgs& a) {
     return (a.Dv != 0 && a.Dv != a.Dh) || a.k_ld != 0 || a.v_ld != 0 || a.keep_first > 0 || a.slopes != nullptr || a.gate_cols || a.kv_scale ||
-           (a.Dh != 64 && a.Dh != 128 && a.Dh != 256 && a.Dh != 512);
+           a.log_r1 != nullptr || a.sig_bias != nullptr || (a.Dh != 64 && a.Dh != 128 && a.Dh != 256 && a.Dh != 512);
 }
 
 #ifdef __CUDACC__

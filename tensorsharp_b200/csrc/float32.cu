@@ -116,8 +116,9 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnArgs a) {
     // the visible positions, numbered without a gap: the kept first ones ahead of the window, then the window
     const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0, nf = min(a.keep_first, lo), gap = lo - nf, last = pos - gap;
     const float slope = a.slopes ? a.slopes[h] : 0.f;
-    const bool one_row = a.kv_scale != 0;
-    float m = -INFINITY, l = 0.f, acc[NJ];
+    const bool one_row = a.kv_scale != 0, sig = a.sig_bias != nullptr;
+    const float pb = sig ? a.sig_bias[h] : 0.f, r1 = a.log_r1 ? a.log_r1[h] : 0.f, r2 = a.log_r1 ? a.log_r2[h] : 0.f;
+    float m = sig ? 0.f : -INFINITY, l = 0.f, acc[NJ];
 #pragma unroll
     for (int j = 0; j < NJ; ++j) acc[j] = 0.f;
     for (int base = warp * 32; base <= last; base += 128) {
@@ -133,10 +134,11 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnArgs a) {
             s *= a.scale;
             if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
             s = fmaf(slope, (float)(j - pos), s);
+            if (a.log_r1 != nullptr) s -= r1 * log1pf(r2 * (float)(pos - j));
         }
-        const float mx = fmaxf(m, warp_max(s));
-        const float corr = m == -INFINITY ? 0.f : expf(m - mx);
-        const float p = ok ? expf(s - mx) : 0.f;
+        const float mx = sig ? 0.f : fmaxf(m, warp_max(s));
+        const float corr = m == -INFINITY ? 0.f : sig ? 1.f : expf(m - mx);
+        const float p = !ok ? 0.f : sig ? 1.f / (1.f + expf(-(s + pb))) : expf(s - mx);
         l = l * corr + warp_sum(p);
         m = mx;
 #pragma unroll
@@ -167,6 +169,7 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnArgs a) {
         c[w] = sml[w][0] == -INFINITY ? 0.f : expf(sml[w][0] - mm);
         ll += sml[w][1] * c[w];
     }
+    if (sig) ll = 1.f;                           // weights that are not normalised
     float g = 1.f;
     const float* gate = reinterpret_cast<const float*>(a.gate);
     if (gate != nullptr && !a.gate_cols) g = 1.f / (1.f + expf(-gate[(long)t * a.gate_tok + h]));
@@ -186,6 +189,8 @@ extern "C" int tsb_attn_f32(const AttnArgs* args, int T, void* stream) {
     TSB_CHECK_ARG(a.Hkv > 0 && a.Hq % a.Hkv == 0 && a.cu_q != nullptr, "attn_f32: Hq=%d Hkv=%d", a.Hq, a.Hkv);
     TSB_CHECK_ARG(a.Dh > 0 && a.Dh <= 1024 && a.Dv > 0 && a.Dv <= ATTN_F32_MAX_DV, "attn_f32: head sizes %d / %d", a.Dh, a.Dv);
     TSB_CHECK_ARG(a.kv_scale == 0 || a.Dv == a.Dh, "attn_f32: rows of %d / %d elements are not key and value at once", a.Dh, a.Dv);
+    TSB_CHECK_ARG(a.sig_bias == nullptr || a.sinks == nullptr, "attn_f32: sigmoid weights have no sink");
+    TSB_CHECK_ARG((a.log_r1 == nullptr) == (a.log_r2 == nullptr), "attn_f32: a logarithmic distance bias has two numbers per head");
     TSB_CHECK_ARG(a.gate != nullptr || !a.gate_cols, "attn_f32: no gate given");
     TSB_CHECK_ARG(a.gate == nullptr || a.gate_f32, "attn_f32: the gate must be float32");
     if (T == 0) return TSB_OK;

@@ -5,7 +5,7 @@ from .base import ModelBase, ModelConfig, supported_architectures  # noqa: F401
 
 def _load_all():
     import importlib
-    for m in ("qwen3", "gptoss", "qwen35", "gemma", "nemotron", "mistral3", "fobolorn", "sogulix", "kegetar"):
+    for m in ("qwen3", "gptoss", "qwen35", "gemma", "nemotron", "mistral3", "fobolorn", "sogulix", "kegetar", "lisorax"):
         try:
             importlib.import_module(f"{__name__}.{m}")
         except ModuleNotFoundError as exc:

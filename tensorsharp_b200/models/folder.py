@@ -69,6 +69,27 @@ class FolderModel(ModelBase):
         w = w if t == GGMLType.BF16 else w.float()
         return QuantWeight.from_raw(w.contiguous().view(-1).view(torch.uint8), t, tuple(w.shape), self.device, name)
 
+    def _heads(self, name: str, H: int, d: int, dp: int) -> torch.Tensor:
+        """[H * d, width] -> [H * dp, D], every head padded with zero rows."""
+        w = self._mat(name, cols=self.cfg.hidden)
+        if w.shape[0] != H * d:
+            raise ValueError(f"{self.path}: tensor {name!r} has {w.shape[0]} rows, {H} heads of {d} need {H * d}")
+        return TF.pad(w.view(H, d, -1), (0, 0, 0, dp - d)).reshape(H * dp, -1)
+
+    def _head_vec(self, name: str, H: int, d: int, dp: int) -> torch.Tensor:
+        return TF.pad(self._host(name).float().view(H, d), (0, dp - d)).reshape(-1)
+
+    def _out(self, name: str, H: int, d: int, dp: int):
+        """Output projection [D, H * d] with the heads' columns padded."""
+        D = self.cfg.hidden
+        return self._qw(TF.pad(self._mat(name, rows=D).view(D, H, d), (0, dp - d)).reshape(D, H * dp), name)
+
+    @staticmethod
+    def _rows(w: QuantWeight, first: int, end: int) -> QuantWeight:
+        """Rows [first, end) of a float matrix, on the same memory."""
+        per = w.planes[0].numel() // w.rows
+        return QuantWeight(w.ggml_type, end - first, w.K, [w.planes[0][first * per:end * per]], 1, w.name)
+
     # ------------------------------------------------------------------ execution
     @property
     def bf16(self) -> bool:

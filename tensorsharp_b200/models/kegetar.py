@@ -106,21 +106,6 @@ class KegetarModel(FolderModel):
         w = (self._host(name).float() + 1.0) * self.residual_mult
         return TF.pad(w, (0, self.cfg.hidden - w.shape[0])).to(self.device).contiguous()
 
-    def _heads(self, name: str, H: int, d: int, dp: int) -> torch.Tensor:
-        """[H * d, width] -> [H * dp, D], every head padded with zero rows."""
-        w = self._mat(name, cols=self.cfg.hidden)
-        if w.shape[0] != H * d:
-            raise ValueError(f"{self.path}: tensor {name!r} has {w.shape[0]} rows, {H} heads of {d} need {H * d}")
-        return TF.pad(w.view(H, d, -1), (0, 0, 0, dp - d)).reshape(H * dp, -1)
-
-    def _head_vec(self, name: str, H: int, d: int, dp: int) -> torch.Tensor:
-        return TF.pad(self._host(name).float().view(H, d), (0, dp - d)).reshape(-1)
-
-    def _out(self, name: str, H: int, d: int, dp: int):
-        """Output projection [D, H * d] with the heads' columns padded."""
-        D = self.cfg.hidden
-        return self._qw(TF.pad(self._mat(name, rows=D).view(D, H, d), (0, dp - d)).reshape(D, H * dp), name)
-
     def _attn_spec(self, p: str, m: dict, vdim: int) -> AttnSpec:
         mask = m.get("mask") or {}
         s = AttnSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), vdim, float(m["scale"]), int(mask.get("size", 0)), int(mask.get("keep_first", 0)))

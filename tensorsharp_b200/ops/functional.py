@@ -216,6 +216,67 @@ def post_norm_seam(h: torch.Tensor, eps: float, n: int, *, y=None, z: Optional[t
     return rms(h) * pre if pre is not None else h.clone()
 
 
+def conv_seam(h: torch.Tensor, eps: float, n: int, *, w: torch.Tensor, y: Optional[torch.Tensor] = None, parts: Optional["MoeParts"] = None,
+              taps: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None, batch: Optional[Batch] = None, plain: bool = True,
+              dtype: Optional[torch.dtype] = None):
+    """The seam of a decoder whose sublayers read one norm, one of them through a convolution over time; one kernel on CUDA.  ``h``
+    (f32 ``[T, D]``) plus the sublayers' outputs ``y`` and the sum of ``parts``; v, the RMS norm of that with the weight ``w``; and
+    v + conv(v), a causal convolution per channel with ``taps`` [K, D] (the last row is the current token's).  ``state`` (f32
+    ``[slots, K - 1, D]``, oldest first) holds each sequence's last values of v between calls.  The norm runs over the first ``n``
+    columns, the rest is padding.  Returns (new h, v or None without ``plain``, v + conv(v) or None without ``taps``)."""
+    if h.is_cuda:
+        return _k().conv_seam(h, eps, n, w=w, y=y, parts=parts, taps=taps, state=state, batch=batch, plain=plain, out_dtype=dtype or torch.bfloat16)
+    if y is not None:
+        h = h + y.float()
+    if parts is not None:
+        h = h + parts.sum()
+    v = h * torch.rsqrt((h * h).sum(-1, keepdim=True) / n + eps) * w
+    c = None
+    if taps is not None:
+        c = v + _conv_over_time(v, taps, None, state, batch)
+    return h, v if plain else None, c
+
+
+CONV_MAX_TAPS = 8          # of the convolutions over time below and of conv_seam
+
+
+def _conv_over_time(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, batch: Batch) -> torch.Tensor:
+    """CPU: causal convolution per channel over the packed rows, ``w`` [K, C]; ``state`` [slots, K - 1, C] is advanced."""
+    outs = []
+    for b, slot in enumerate(batch.seq_slots.tolist()):
+        o, tail = ref.causal_conv1d(x[batch.h_cu_q[b]:batch.h_cu_q[b + 1]], w.t(), bias, state[slot], act_silu=False)
+        state[slot] = tail
+        outs.append(o)
+    return torch.cat(outs, 0)
+
+
+def short_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, batch: Batch, *, block: int = 0,
+               dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """Causal convolution over time on every channel of a projection, no activation: ``x`` [T, C] (a view, rows may be strided),
+    ``w`` [K, C] (the last row is the current token's); ``state`` f32 [slots, K - 1, C] holds each sequence's last inputs, oldest
+    first.  Returns [T, C], or with ``block`` the columns in blocks of that size one below the other, [C / block * T, block]."""
+    T, C = x.shape
+    if x.is_cuda:
+        return _k().short_conv(x, w, bias, state, batch, block=block, out_dtype=dtype or torch.float32)
+    o = _conv_over_time(x, w, bias, state, batch)
+    return o.view(T, C // block, block).transpose(0, 1).reshape(-1, block) if block else o
+
+
+def conv_qkv_cache(y: torch.Tensor, w: torch.Tensor, state: torch.Tensor, batch: Batch, *, nq: int, dtype: torch.dtype,
+                   k_cache: Optional[torch.Tensor] = None, v_cache: Optional[torch.Tensor] = None, q_temp: Optional[Tuple[float, float]] = None) -> torch.Tensor:
+    """:func:`short_conv` on projection rows [q (nq) | k | v]: k and v go to the paged caches at ``batch.slots`` (without caches the
+    rows are queries only), q times the position's temperature (coef, every) is returned, [T, nq] in ``dtype``, the caches' type."""
+    if y.is_cuda:
+        return _k().conv_qkv(y, w, state, batch, nq=nq, dtype=dtype, k_cache=k_cache, v_cache=v_cache, q_temp=q_temp)
+    o = _conv_over_time(y, w, None, state, batch)
+    if k_cache is not None:
+        nk = k_cache.shape[1] * k_cache.shape[2]
+        kv_scatter(k_cache, batch.slots, o[:, nq:nq + nk].unflatten(1, tuple(k_cache.shape[1:])))
+        kv_scatter(v_cache, batch.slots, o[:, nq + nk:].unflatten(1, tuple(v_cache.shape[1:])))
+    q = o[:, :nq]
+    return q * ref.query_temperature(batch.positions, *q_temp).unsqueeze(1) if q_temp is not None else q
+
+
 def embed_pairs(tok: QuantWeight, pair: QuantWeight, batch: Batch, prev: torch.Tensor, *, mul_prev: int, mul_cur: int,
                 dtype: Optional[torch.dtype] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """Token embedding plus that of the pair (previous token, token): row (previous * mul_prev + token * mul_cur) mod buckets of
@@ -568,20 +629,24 @@ def decode_splits(batch: Batch, Hkv: int, window: int) -> int:
 def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch: Batch, *, scale: float,
               Hq: int, Hkv: int, Dh: int, window: int = 0, sinks: Optional[torch.Tensor] = None,
               softcap: float = 0.0, as_act: bool = False, Dv: Optional[int] = None, gate: Optional[torch.Tensor] = None, keep_first: int = 0,
-              slopes: Optional[torch.Tensor] = None, own_values: bool = False):
+              slopes: Optional[torch.Tensor] = None, own_values: bool = False, log_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None,
+              sigmoid_bias: Optional[torch.Tensor] = None):
     """Causal attention of the packed queries against the paged cache -> [T, Hq * Dh].  ``as_act`` returns an
     ``Act``; on the CUDA decode path it already carries the int8 form written by the combine kernel, so
     the quantised projection that follows needs no quantise launch.  ``Dv``: value head size where it differs from
     ``Dh`` (the result is then [T, Hq * Dv]); ``gate`` [T, Hq] (a view, last dim dense): head h's output is
     multiplied by sigmoid(gate[:, h]), with a gate [T, Hq * Dv] every column by its own; float32 caches run in 32 bits.
     ``keep_first``: with a window, so many positions at the start stay visible; ``slopes`` [Hq]: slopes[h] times the distance
-    is taken off the score; ``own_values``: a row of ``k_cache`` (see :func:`joint_norm_cache`) is key and value at once."""
+    is taken off the score; ``own_values``: a row of ``k_cache`` (see :func:`joint_norm_cache`) is key and value at once;
+    ``log_bias`` (r1, r2) [Hq] each: r1[h] ln(1 + r2[h] distance) is taken off the score (after the soft cap);
+    ``sigmoid_bias`` [Hq]: no softmax, a visible key has the weight sigmoid(score + sigmoid_bias[h])."""
     T = q.shape[0]
     Dv = Dv or Dh
-    if q.is_cuda and (Dv != Dh or gate is not None or k_cache.dtype == torch.float32 or keep_first or slopes is not None or own_values):
+    if q.is_cuda and (Dv != Dh or gate is not None or k_cache.dtype == torch.float32 or keep_first or slopes is not None or own_values
+                      or log_bias is not None or sigmoid_bias is not None):
         return _gated_attention(q, k_cache, v_cache, batch, scale=scale, Hq=Hq, Hkv=Hkv, Dh=Dh, Dv=Dv, window=window,
                                 sinks=sinks, softcap=softcap, gate=gate, keep_first=keep_first, slopes=slopes,
-                                kv_scale=Hkv * Dh if own_values else 0)
+                                kv_scale=Hkv * Dh if own_values else 0, log_bias=log_bias, sigmoid_bias=sigmoid_bias)
     if as_act:
         if q.is_cuda and batch.is_decode and Dh % 32 == 0:
             sp = decode_splits(batch, Hkv, window)
@@ -623,7 +688,7 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, bat
         else:
             kb, vb = kv_gather(k_cache, idx), kv_gather(v_cache, idx)
         outs.append(ref.attention(q[q0:q1], kb, vb, batch.positions[q0:q1], scale=scale, window=window, sinks=sinks,
-                                  softcap=softcap, keep_first=keep_first, slopes=slopes))
+                                  softcap=softcap, keep_first=keep_first, slopes=slopes, log_bias=log_bias, sigmoid_bias=sigmoid_bias))
     out = torch.cat(outs, 0)
     if gate is not None:
         out = out * torch.sigmoid(gate.float()).view(T, Hq, -1)
@@ -631,15 +696,15 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, bat
 
 
 def _gated_attention(q, k_cache, v_cache, batch: Batch, *, scale, Hq, Hkv, Dh, Dv, window, sinks, softcap, gate, keep_first=0, slopes=None,
-                     kv_scale=0) -> torch.Tensor:
+                     kv_scale=0, log_bias=None, sigmoid_bias=None) -> torch.Tensor:
     """The CUDA side of :func:`attention` for the forms beyond one head size and bf16: keys and values of different
-    sizes, sigmoid gates, kept first positions, distance biases, rows that are key and value at once, 32-bit caches."""
+    sizes, sigmoid gates, kept first positions, distance biases, sigmoid weights, rows that are key and value at once, 32-bit caches."""
     kk = _k()
     T = q.shape[0]
     if is_fp8(k_cache):
         raise ValueError("8-bit pages have no gated attention")
     kw = dict(scale=scale, Hq=Hq, Hkv=Hkv, Dh=Dh, Dv=Dv, page_size=batch.page_size, sinks=sinks, softcap=softcap, window=window,
-              gate=gate, keep_first=keep_first, slopes=slopes, kv_scale=kv_scale)
+              gate=gate, keep_first=keep_first, slopes=slopes, kv_scale=kv_scale, log_bias=log_bias, sigmoid_bias=sigmoid_bias)
     if k_cache.dtype == torch.float32:
         return kk.attn_f32(q, k_cache, v_cache, batch.block_table, batch.kv_lens, batch.cu_q, **kw).view(T, Hq * Dv)
     if batch.is_decode:
@@ -860,7 +925,7 @@ MOE_TILE_MAX_PAIRS = int(os.environ.get("TSB_MOE_TILE_MAX_PAIRS", "1024"))
 def route_topk_softmax(logits: torch.Tensor, k: int):
     """Top-k on the router logits, then softmax over the selected k (GPT-OSS, Qwen3.5 decode;
     GptOssModel.cs:814-865).  Equivalent to softmax over all -> top-k -> renormalise."""
-    if logits.is_cuda and logits.dtype == torch.float32 and logits.shape[-1] <= 1024 and k <= 16:
+    if logits.is_cuda and logits.dtype == torch.float32 and logits.shape[-1] <= 1024 and k <= 32:
         return _k().moe_route(logits.contiguous(), k, mode=0)
     vals, ids = torch.topk(logits.float(), k, dim=-1)
     return ids.to(torch.int32), torch.softmax(vals, -1)
@@ -1295,6 +1360,117 @@ def gated_linear(y: torch.Tensor, s: GatedLinearSpec, cols: Tuple[int, ...], w2:
         o[q0:q1] = ref.gated_linear(q[q0:q1] * s.q_scale, k[q0:q1], v[q0:q1], decay[q0:q1], state[slots[b]])
     o = o * torch.rsqrt((o * o).sum(-1, keepdim=True) / s.vdim + eps) * norm_w
     return o.reshape(T, H * E) * torch.nn.functional.silu(y[:, cols[3]:cols[3] + H * E])
+
+
+@dataclass
+class RglruSpec:
+    """Sizes of a recurrent block with real-gated linear recurrent units: ``blocks`` of ``size`` channels, padded to ``block``."""
+    width: int
+    blocks: int
+
+    def __post_init__(self):
+        self.size = self.width // self.blocks
+        self.block = (self.size + 7) // 8 * 8
+        self.W = self.blocks * self.block
+
+
+def rglru_segments(batch: Batch, s: RglruSpec) -> int:
+    """Pieces in which the scan takes the batch's sequences: about 2048 threads per SM, no fewer than 32 tokens each."""
+    return max(1, min(round(2048 * 148 / (batch.B * s.W)), batch.max_q_len // 32, 128))
+
+
+def rglru(y: torch.Tensor, s: RglruSpec, conv_w: torch.Tensor, conv_b: torch.Tensor, gates: QuantWeight, gate_b: torch.Tensor, rate: torch.Tensor,
+          conv_state: torch.Tensor, state: torch.Tensor, batch: Batch, *, dtype: torch.dtype) -> torch.Tensor:
+    """Recurrent block with real-gated linear recurrent units over the packed tokens -> [T, W].  Rows of ``y``: [output branch (W) |
+    input branch (W)]; u = the short convolution of the input branch (``conv_w`` [K, W], ``conv_b``); gates r and i per block:
+    sigmoid(``gates`` u + ``gate_b``), ``gates`` a stack of [2 block, block] (r's rows, then i's), ``gate_b`` [2, W]; ``rate`` [W] <= 0
+    per channel.  log a = rate r; S <- a S + sqrt(1 - a^2) i u; the result is S gelu(output branch).  ``state`` f32 [slots, W]."""
+    W, T = s.W, batch.T
+    x = y[:, W:2 * W]
+    if y.is_cuda:
+        kk = _k()
+        if T <= GEMV_MAX_M:
+            u = kk.short_conv(x, conv_w, conv_b, conv_state, batch, out_dtype=torch.float32)
+            return kk.rglru_step(y, u, s, _weight_matrix(gates), gate_b, rate, state, batch, out_dtype=dtype)
+        f32 = y.dtype == torch.float32 and dtype == torch.float32
+        u = kk.short_conv(x, conv_w, conv_b, conv_state, batch, block=s.block, out_dtype=dtype)
+        tiles = block_tiles(batch, s.blocks, 64 if f32 else 256)
+        z = (kk.gemm_f32(gates, u, tiles=tiles) if f32 else
+             kk.gemm_bf16_grouped(_dequant_scratch(gates), s.blocks, u, tiles, 256, out_dtype=torch.float32, zero=False))
+        return kk.rglru_scan(y, u, z, s, gate_b, rate, state, batch, out_dtype=dtype, segs=rglru_segments(batch, s))
+    y = y.float()
+    u = _conv_over_time(y[:, W:2 * W], conv_w, conv_b, conv_state, batch)
+    z = torch.einsum("tbi,boi->tbo", u.view(T, s.blocks, s.block), gates.dequantize().view(s.blocks, 2 * s.block, s.block))
+    r, i = (torch.sigmoid(z[..., p * s.block:(p + 1) * s.block].reshape(T, W) + gate_b[p]) for p in (0, 1))
+    out = torch.empty((T, W))
+    for b, slot in enumerate(batch.seq_slots.tolist()):
+        q0, q1 = batch.h_cu_q[b], batch.h_cu_q[b + 1]
+        out[q0:q1] = ref.real_gated_recurrence(u[q0:q1], r[q0:q1], i[q0:q1], rate, state[slot])
+    return out * torch.nn.functional.gelu(y[:, :W], approximate="tanh")
+
+
+def block_tiles(batch: Batch, blocks: int, bn: int) -> torch.Tensor:
+    """Work list of a grouped product over ``blocks`` matrices, each with the T rows of the batch (rows block after block): int32
+    [n, 3] (matrix, first row, end row), at most ``bn`` rows each; memoised per step."""
+    key = ("block_tiles", blocks, bn)
+    t = batch.cache.get(key)
+    if t is None:
+        T = batch.T
+        rows = [(b, b * T + r, b * T + min(r + bn, T)) for b in range(blocks) for r in range(0, T, bn)]
+        t = batch.cache[key] = torch.tensor(rows, dtype=torch.int32).to(batch.tokens.device)
+    return t
+
+
+@dataclass
+class MlstmSpec:
+    """Sizes of an mLSTM mixer (``D``, ``E``: padded key and value head sizes); ``cap`` bounds the gates' logarithms."""
+    H: int
+    dim: int
+    vdim: int
+    cap: float
+
+    def __post_init__(self):
+        self.D = (self.dim + 31) // 32 * 32
+        pad = 16 if self.vdim <= 128 else 32
+        self.E = (self.vdim + pad - 1) // pad * pad
+        self.q_scale = self.dim ** -0.5
+
+
+MLSTM_CHUNK_MIN = 16          # tokens of the longest portion from which the chunk kernel is used
+
+
+def mlstm_segments(batch: Batch, s: MlstmSpec) -> int:
+    """Pieces in which the chunk kernel takes the batch's sequences: about eight warps per SM (one per 16 value columns), no
+    fewer than 128 tokens each."""
+    warps = batch.B * s.H * s.E // 16
+    return max(1, min(round(8 * 148 / warps), batch.max_q_len // 128))
+
+
+def mlstm(y: torch.Tensor, s: MlstmSpec, cols: Tuple[int, int, int, int], z: torch.Tensor, zb: torch.Tensor, norm_w: torch.Tensor, S: torch.Tensor,
+          n: torch.Tensor, m: torch.Tensor, batch: Batch, *, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """Matrix memory with exponential gates over the packed tokens -> normed and gated output [T, H * E].  Columns ``cols`` of ``y``:
+    queries, keys (H * D each), values, output gate (H * E each); ``z`` [T, 2 H] f32 and ``zb``: the input and forget gates'
+    projections and offsets, i = cap tanh(z / cap), f = log sigmoid(cap tanh(z / cap)).  The heads' outputs are divided by their
+    root mean square, times ``norm_w`` [H * E], times sigmoid of the output gate.  State, f32 with a row per slot: ``S`` [slots, H,
+    values, keys], ``n`` [slots, H, keys], ``m`` [slots, H].  Heads are padded with zeros."""
+    if y.is_cuda:
+        kk = _k()
+        kw = dict(eps=eps, out_dtype=dtype)
+        if y.dtype != torch.bfloat16 or batch.max_q_len < MLSTM_CHUNK_MIN:
+            return kk.mlstm_step(y, s, cols, z, zb, norm_w, S, n, m, batch, **kw)
+        return kk.mlstm_prompt(y, s, cols, z, zb, norm_w, S, n, m, batch, segs=mlstm_segments(batch, s), **kw)
+    T, y = y.shape[0], y.float()
+    H, D, E = s.H, s.D, s.E
+    q, k = (y[:, c:c + H * D].view(T, H, D) for c in cols[:2])
+    v = y[:, cols[2]:cols[2] + H * E].view(T, H, E)
+    z = s.cap * torch.tanh((z.float() + zb) / s.cap)
+    i, f = z[:, :H], torch.nn.functional.logsigmoid(z[:, H:])
+    o = torch.empty((T, H, E))
+    for b, slot in enumerate(batch.seq_slots.tolist()):
+        a = slice(batch.h_cu_q[b], batch.h_cu_q[b + 1])
+        o[a] = ref.mlstm(q[a] * s.q_scale, k[a], v[a], i[a], f[a], S[slot], n[slot], m[slot])
+    o = o * torch.rsqrt((o * o).sum(-1, keepdim=True) / s.vdim + eps)
+    return o.reshape(T, H * E) * norm_w * torch.sigmoid(y[:, cols[3]:cols[3] + H * E])
 
 
 def _weight_matrix(w: QuantWeight) -> torch.Tensor:

@@ -82,7 +82,7 @@ class AttnArgs(C.Structure):
                 ("out_q", _vp), ("out_ds", _vp), ("ticket", _vp), ("split_len", C.c_int),
                 ("gate", _vp), ("gate_tok", C.c_long), ("gate_f32", C.c_int), ("Dv", C.c_int),
                 ("k_ld", C.c_long), ("v_ld", C.c_long), ("keep_first", C.c_int), ("slopes", _vp), ("gate_cols", C.c_int),
-                ("kv_scale", C.c_int)]
+                ("kv_scale", C.c_int), ("log_r1", _vp), ("log_r2", _vp), ("sig_bias", _vp)]
 
 
 _configured = False
@@ -463,7 +463,7 @@ def decode_advance(sampled, batch) -> None:
 
 
 def _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, cu_q, sinks, scale, softcap, window, Hq, Hkv, Dh,
-               page_size, B, Dv=None, gate=None, keep_first=0, slopes=None, kv_scale=0):
+               page_size, B, Dv=None, gate=None, keep_first=0, slopes=None, kv_scale=0, log_bias=None, sigmoid_bias=None):
     check_index("attention", "block-table page", block_table, k_cache.shape[0] // page_size)
     check_index("attention", "cache length", kv_lens, block_table.shape[1] * page_size + 1)
     a = AttnArgs()
@@ -476,6 +476,11 @@ def _attn_args(q, k_cache, v_cache, out, block_table, kv_lens, cu_q, sinks, scal
     a.Dv = Dv or Dh
     assert slopes is None or (slopes.dtype == torch.float32 and slopes.is_contiguous() and slopes.numel() == Hq)
     a.keep_first, a.slopes, a.kv_scale = int(keep_first) if window else 0, _p(slopes), int(kv_scale)
+    for t in (*(log_bias or ()), sigmoid_bias):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == Hq)
+    if log_bias is not None:
+        a.log_r1, a.log_r2 = _p(log_bias[0]), _p(log_bias[1])
+    a.sig_bias = _p(sigmoid_bias)
     if kv_scale:                          # rows that are key and value at once, with the factor of the key behind them
         assert k_cache.dim() == 3 and k_cache.stride(2) == 1 and k_cache.shape[-1] >= kv_scale + 1 and kv_scale >= Hkv * Dh
         a.k_ld = a.v_ld = k_cache.stride(0)
@@ -496,7 +501,7 @@ def attn_decode(q, k_cache, v_cache, block_table, kv_lens, *, scale, Hq, Hkv, Dh
                 softcap=0.0, window=0, out=None, want_q8=False, split_len=0, Dv=None, gate=None, **forms):
     """q [B, Hq, Dh] bf16; one query per sequence against the paged cache.  ``want_q8`` also returns the
     output as int8 groups of 32 with (scale, sum) written by the combine kernel: (out, q, ds).  ``forms``: keep_first,
-    slopes, kv_scale (see AttnArgs)."""
+    slopes, kv_scale, log_bias, sigmoid_bias (see AttnArgs)."""
     B = q.shape[0]
     Dv = Dv or Dh
     if out is None:
@@ -776,6 +781,210 @@ def gla_prompt(y, s, cols, z: torch.Tensor, zb, norm_w, state, cu_q, seq_slots, 
     a.z, a.z_s, a.core, a.segs, a.seg_len = _p(z), z.stride(0), _p(core), segs, seg_len
     native.check(_lib().tsb_gla_prompt(C.byref(a), C.c_int(max_q), _stream()), "gla_prompt")
     _count(1 + 2 * (segs > 1) + (core is not None))
+    return out
+
+
+class ConvSeamArgs(C.Structure):
+    _fields_ = [("h", _vp), ("h_out", _vp), ("y", _vp), ("p", _vp), ("pos", _vp), ("wts", _vp), ("w", _vp), ("taps", _vp), ("state", _vp),
+                ("cu_q", _vp), ("seq_slots", _vp), ("out", _vp), ("conv", _vp), ("rows", C.c_long), ("state_s", C.c_long),
+                ("D", C.c_int), ("n", C.c_int), ("B", C.c_int), ("K", C.c_int), ("parts", C.c_int), ("y_f32", C.c_int), ("p_f32", C.c_int),
+                ("out_f32", C.c_int), ("span", C.c_int), ("eps", C.c_float)]
+
+
+def _carried(what: str, state: torch.Tensor, rest: tuple, cu_q, seq_slots, T: int) -> int:
+    """Checks a per-slot f32 state of rows ``rest`` (a view whose slots are strided, dense inside) and returns the slot stride."""
+    check_index(what, "state slot", seq_slots, state.shape[0])
+    check_index(what, "row offset", cu_q, T + 1)
+    assert state.dtype == torch.float32 and tuple(state.shape[1:]) == tuple(rest) and seq_slots.dtype == torch.int64 and cu_q.dtype == torch.int32
+    want = 1
+    for d in range(state.dim() - 1, 0, -1):
+        assert state.shape[d] <= 1 or state.stride(d) == want
+        want *= state.shape[d]
+    return state.stride(0)
+
+
+def conv_seam(h: torch.Tensor, eps: float, n: int, *, w, y=None, parts=None, taps=None, state=None, batch=None, plain: bool = True,
+              out_dtype=torch.bfloat16):
+    """The seam of csrc/conv_seam.cu: (new residual, ``h`` itself when there is nothing to add; norm or None; norm plus its
+    convolution over time, or None)."""
+    assert h.dtype == torch.float32 and h.is_contiguous() and w.numel() == h.shape[1]
+    T, D = h.shape
+    a = ConvSeamArgs()
+    a.h, a.w, a.rows, a.D, a.n, a.eps, a.out_f32 = _p(h), _p(w), T, D, n, eps, int(out_dtype == torch.float32)
+    res = h
+    if y is not None or parts is not None:
+        res = torch.empty_like(h)
+        a.h_out = _p(res)
+    if y is not None:
+        assert y.shape == h.shape and y.is_contiguous() and y.dtype in (torch.float32, torch.bfloat16)
+        a.y, a.y_f32 = _p(y), int(y.dtype == torch.float32)
+    if parts is not None:
+        k, p = parts.k, parts.y
+        assert p.is_contiguous() and p.shape[1] == D and p.dtype in (torch.float32, torch.bfloat16) and parts.ids is None
+        assert (p.shape[0] == T * k or parts.pos is not None) and (parts.pos is None or (parts.pos.dtype == torch.int32 and parts.pos.numel() == T * k))
+        assert parts.w is None or (parts.w.dtype == torch.float32 and parts.w.is_contiguous() and parts.w.numel() == T * k)
+        check_index("conv_seam", "part row", parts.pos, p.shape[0], low=-1)
+        a.p, a.p_f32, a.pos, a.wts, a.parts = _p(p), int(p.dtype == torch.float32), _p(parts.pos), _p(parts.w), k
+    out = conv = None
+    if plain:
+        out = torch.empty((T, D), dtype=out_dtype, device=h.device)
+        a.out = _p(out)
+    if taps is not None:
+        conv = torch.empty((T, D), dtype=out_dtype, device=h.device)
+        K = taps.shape[0]
+        assert taps.dtype == torch.float32 and taps.is_contiguous() and taps.shape[1] == D
+        a.state_s = _carried("conv_seam", state, (K - 1, D), batch.cu_q, batch.seq_slots, T)
+        a.conv, a.taps, a.K, a.state, a.cu_q, a.seq_slots, a.B = _p(conv), _p(taps), K, _p(state), _p(batch.cu_q), _p(batch.seq_slots), batch.B
+    native.check(_lib().tsb_conv_seam(C.byref(a), _stream()), "conv_seam")
+    _count(1)
+    return res, out, conv
+
+
+class ShortConvArgs(C.Structure):
+    _fields_ = [("x", _vp), ("x_s", C.c_long), ("x_f32", C.c_int), ("w", _vp), ("bias", _vp), ("state", _vp), ("state_s", C.c_long),
+                ("cu_q", _vp), ("seq_slots", _vp), ("out", _vp), ("out_s", C.c_long), ("out_f32", C.c_int), ("block", C.c_int),
+                ("pos", _vp), ("slot", _vp), ("k_cache", _vp), ("v_cache", _vp), ("nq", C.c_int), ("nk", C.c_int), ("qt_coef", C.c_float),
+                ("qt_every", C.c_float), ("T", C.c_int), ("C", C.c_int), ("K", C.c_int), ("B", C.c_int), ("span", C.c_int)]
+
+
+def _short_conv_args(x, w, bias, state, batch) -> ShortConvArgs:
+    T, Cc = x.shape
+    K = w.shape[0]
+    assert x.stride(1) == 1 and x.dtype in (torch.float32, torch.bfloat16) and w.dtype == torch.float32 and w.is_contiguous() and w.shape[1] == Cc
+    assert x.data_ptr() % (16 if x.dtype == torch.float32 else 8) == 0
+    a = ShortConvArgs()
+    a.state_s = _carried("short_conv", state, (K - 1, Cc), batch.cu_q, batch.seq_slots, T)
+    a.x, a.x_s, a.x_f32, a.w, a.bias, a.state = _p(x), x.stride(0), int(x.dtype == torch.float32), _p(w), _p(bias), _p(state)
+    a.cu_q, a.seq_slots, a.T, a.C, a.K, a.B = _p(batch.cu_q), _p(batch.seq_slots), T, Cc, K, batch.B
+    return a
+
+
+def short_conv(x, w, bias, state, batch, *, block: int = 0, out_dtype=torch.float32) -> torch.Tensor:
+    """Causal convolution per channel (csrc/short_conv.cu) -> [T, C], or [C / block * T, block]."""
+    T, Cc = x.shape
+    a = _short_conv_args(x, w, bias, state, batch)
+    out = torch.empty((Cc // block * T, block) if block else (T, Cc), dtype=out_dtype, device=x.device)
+    a.out, a.out_s, a.out_f32, a.block = _p(out), Cc, int(out_dtype == torch.float32), block
+    native.check(_lib().tsb_short_conv(C.byref(a), _stream()), "short_conv")
+    _count(1)
+    return out
+
+
+def conv_qkv(y, w, state, batch, *, nq: int, dtype, k_cache=None, v_cache=None, q_temp=None) -> torch.Tensor:
+    """The same on projection rows [q | k | v] of attention: keys and values to their cache slots, returns the queries [T, nq]."""
+    T, Cc = y.shape
+    a = _short_conv_args(y, w, None, state, batch)
+    if k_cache is not None:
+        check_index("short_conv", "cache slot", batch.slots, k_cache.shape[0])
+        a.nk = k_cache.shape[1] * k_cache.shape[2]
+        assert k_cache.dtype == dtype and k_cache.is_contiguous() and v_cache.is_contiguous() and v_cache.dtype == dtype and nq + a.nk + v_cache.shape[1] * v_cache.shape[2] == Cc
+        a.k_cache, a.v_cache = _p(k_cache), _p(v_cache)
+    else:
+        assert nq == Cc
+    q = torch.empty((y.shape[0], nq), dtype=dtype, device=y.device)
+    assert dtype in (torch.float32, torch.bfloat16) and batch.positions.dtype == torch.int32 and batch.slots.dtype == torch.int64
+    a.out, a.out_s, a.out_f32, a.nq, a.pos, a.slot = _p(q), nq, int(dtype == torch.float32), nq, _p(batch.positions), _p(batch.slots)
+    a.qt_coef, a.qt_every = q_temp or (0.0, 0.0)
+    native.check(_lib().tsb_short_conv(C.byref(a), _stream()), "short_conv")
+    _count(1)
+    return q
+
+
+class RglruArgs(C.Structure):
+    _fields_ = [("y", _vp), ("y_s", C.c_long), ("y_f32", C.c_int), ("u", _vp), ("u_f32", C.c_int), ("w", _vp), ("w_f32", C.c_int), ("z", _vp),
+                ("gate_b", _vp), ("rate", _vp), ("state", _vp), ("state_s", C.c_long), ("cu_q", _vp), ("seq_slots", _vp), ("seg_a", _vp),
+                ("seg_s", _vp), ("out", _vp), ("out_f32", C.c_int), ("T", C.c_int), ("B", C.c_int), ("W", C.c_int), ("block", C.c_int),
+                ("segs", C.c_int), ("seg_len", C.c_int)]
+
+
+def _rglru_args(y, u, s, gate_b, rate, state, batch, out_dtype):
+    T = y.shape[0]
+    assert y.stride(1) == 1 and y.shape[1] >= s.W and u.is_contiguous() and u.numel() == T * s.W and gate_b.shape == (2, s.W) and gate_b.is_contiguous()
+    a = RglruArgs()
+    a.state_s = _carried("rglru", state, (s.W,), batch.cu_q, batch.seq_slots, T)
+    a.y, a.y_s, a.y_f32, a.u, a.u_f32 = _p(y), y.stride(0), int(y.dtype == torch.float32), _p(u), int(u.dtype == torch.float32)
+    a.gate_b, a.rate, a.state, a.cu_q, a.seq_slots = _p(gate_b), _p(rate), _p(state), _p(batch.cu_q), _p(batch.seq_slots)
+    out = torch.empty((T, s.W), dtype=out_dtype, device=y.device)
+    a.out, a.out_f32, a.T, a.B, a.W, a.block = _p(out), int(out_dtype == torch.float32), T, batch.B, s.W, s.block
+    return a, out
+
+
+def rglru_step(y, u, s, w: torch.Tensor, gate_b, rate, state, batch, *, out_dtype) -> torch.Tensor:
+    """Real-gated linear recurrent units token by token (csrc/rglru.cu), gates and output branch included; ``u`` f32 [T, W]."""
+    a, out = _rglru_args(y, u, s, gate_b, rate, state, batch, out_dtype)
+    assert u.dtype == torch.float32 and w.is_contiguous() and w.numel() == 2 * s.W * s.block
+    a.w, a.w_f32 = _p(w), int(w.dtype == torch.float32)
+    native.check(_lib().tsb_rglru_step(C.byref(a), _stream()), "rglru_step")
+    _count(1)
+    return out
+
+
+def rglru_scan(y, u, z, s, gate_b, rate, state, batch, *, out_dtype, segs: int) -> torch.Tensor:
+    """The same for prompts, from the gates' products ``z`` f32 [blocks * T, 2 block], in ``segs`` segments per sequence."""
+    a, out = _rglru_args(y, u, s, gate_b, rate, state, batch, out_dtype)
+    assert z.dtype == torch.float32 and z.is_contiguous() and z.shape == (s.blocks * y.shape[0], 2 * s.block)
+    max_q = batch.max_q_len
+    a.seg_len = -(-max_q // segs)
+    a.segs = -(-max_q // a.seg_len)
+    a.z = _p(z)
+    if a.segs > 1:
+        seg = torch.empty((2, a.B, a.segs, s.W), dtype=torch.float32, device=y.device)
+        a.seg_a, a.seg_s = _p(seg[0]), _p(seg[1])
+    native.check(_lib().tsb_rglru_scan(C.byref(a), C.c_int(max_q), _stream()), "rglru_scan")
+    _count(1 + (a.segs > 1))
+    return out
+
+
+class MlstmArgs(C.Structure):
+    _fields_ = [("y", _vp), ("y_s", C.c_long), ("y_f32", C.c_int), ("q", C.c_long), ("k", C.c_long), ("v", C.c_long), ("g", C.c_long),
+                ("z", _vp), ("z_s", C.c_long), ("zb", _vp), ("norm_w", _vp), ("S", _vp), ("n", _vp), ("m", _vp), ("state_s", C.c_long),
+                ("cu_q", _vp), ("seq_slots", _vp), ("fim", _vp), ("m0", _vp), ("seg", _vp), ("seg_n", _vp), ("seg_w", _vp), ("core", _vp),
+                ("out", _vp), ("out_s", C.c_long), ("out_f32", C.c_int), ("T", C.c_int), ("B", C.c_int), ("H", C.c_int), ("D", C.c_int),
+                ("E", C.c_int), ("e_n", C.c_int), ("segs", C.c_int), ("seg_len", C.c_int), ("eps", C.c_float), ("q_scale", C.c_float),
+                ("cap", C.c_float)]
+
+
+def _mlstm_args(y, s, cols, z, zb, norm_w, S, n, m, batch, eps: float, out_dtype):
+    T = y.shape[0]
+    assert y.stride(1) == 1 and z.dtype == torch.float32 and z.shape == (T, 2 * s.H) and z.stride(1) == 1 and zb.numel() == 2 * s.H
+    assert norm_w.numel() == s.H * s.E and S.stride(0) == n.stride(0) == m.stride(0)
+    a = MlstmArgs()
+    for t, rest in ((S, (s.H, s.E, s.D)), (n, (s.H, s.D)), (m, (s.H,))):
+        a.state_s = _carried("mlstm", t, rest, batch.cu_q, batch.seq_slots, T)
+    a.y, a.y_s, a.y_f32 = _p(y), y.stride(0), int(y.dtype == torch.float32)
+    a.q, a.k, a.v, a.g = cols
+    a.z, a.z_s, a.zb, a.norm_w, a.S, a.n, a.m = _p(z), z.stride(0), _p(zb), _p(norm_w), _p(S), _p(n), _p(m)
+    a.cu_q, a.seq_slots = _p(batch.cu_q), _p(batch.seq_slots)
+    out = torch.empty((T, s.H * s.E), dtype=out_dtype, device=y.device)
+    a.out, a.out_s, a.out_f32 = _p(out), s.H * s.E, int(out_dtype == torch.float32)
+    a.T, a.B, a.H, a.D, a.E, a.e_n, a.eps, a.q_scale, a.cap = T, batch.B, s.H, s.D, s.E, s.vdim, eps, s.q_scale, s.cap
+    return a, out
+
+
+def mlstm_step(y, s, cols, z, zb, norm_w, S, n, m, batch, *, eps: float, out_dtype) -> torch.Tensor:
+    """mLSTM token by token (csrc/mlstm.cu), gates, norm and output gate included."""
+    a, out = _mlstm_args(y, s, cols, z, zb, norm_w, S, n, m, batch, eps, out_dtype)
+    native.check(_lib().tsb_mlstm_step(C.byref(a), _stream()), "mlstm_step")
+    _count(1)
+    return out
+
+
+def mlstm_prompt(y, s, cols, z, zb, norm_w, S, n, m, batch, *, eps: float, out_dtype, segs: int) -> torch.Tensor:
+    """The same for prompts of bf16 models, 64 tokens at a time on the tensor cores, in ``segs`` segments per sequence."""
+    assert y.dtype == out_dtype == torch.bfloat16
+    a, out = _mlstm_args(y, s, cols, z, zb, norm_w, S, n, m, batch, eps, out_dtype)
+    max_q, T = batch.max_q_len, y.shape[0]
+    a.seg_len = (-(-max_q // segs) + 63) // 64 * 64
+    a.segs = segs = -(-max_q // a.seg_len)
+    f32 = dict(dtype=torch.float32, device=y.device)
+    fim, m0, seg_n = torch.empty((3, s.H, T), **f32), torch.empty((a.B, s.H), **f32), torch.empty((a.B, segs, s.H, s.D), **f32)
+    seg = seg_w = None
+    if segs > 1:
+        seg, seg_w = torch.empty((a.B, segs, s.H, s.E, s.D), **f32), torch.empty((a.B, segs, s.H), **f32)
+    core = torch.empty((T, s.H, s.E), **f32) if s.E > 128 else None
+    a.fim, a.m0, a.seg_n, a.seg, a.seg_w, a.core = _p(fim), _p(m0), _p(seg_n), _p(seg), _p(seg_w), _p(core)
+    native.check(_lib().tsb_mlstm_prompt(C.byref(a), C.c_int(max_q), _stream()), "mlstm_prompt")
+    _count(2 + 2 * (segs > 1) + (core is not None))
     return out
 
 

@@ -102,10 +102,11 @@ def glu(act: str, g: torch.Tensor, u: Optional[torch.Tensor], clamp: float = 7.0
 
 def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_pos: torch.Tensor, *, scale: float,
               window: int = 0, sinks: Optional[torch.Tensor] = None, softcap: float = 0.0, keep_first: int = 0,
-              slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+              slopes: Optional[torch.Tensor] = None, log_bias=None, sigmoid_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Naive attention for one sequence.  q [Tq, Hq, Dh]; k, v [Tk, Hkv, Dh] hold cache
     positions 0..Tk-1; q_pos [Tq] are the queries' positions.  ``keep_first`` positions stay visible outside the window;
-    ``slopes`` [Hq] times the distance is taken off the scores.  Returns [Tq, Hq, Dh] f32."""
+    ``slopes`` [Hq] times the distance is taken off the scores, ``log_bias`` (r1, r2) [Hq] takes off r1 ln(1 + r2 distance).
+    With ``sigmoid_bias`` [Hq] the weights are sigmoid(score + bias) as they are.  Returns [Tq, Hq, Dh] f32."""
     Tq, Hq, Dh = q.shape
     Tk, Hkv, _ = k.shape
     g = Hq // Hkv
@@ -119,10 +120,15 @@ def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_pos: torch.Te
     p = q_pos.view(1, Tq, 1)
     if slopes is not None:
         s = s - slopes.float().view(Hq, 1, 1) * (p - j)
+    if log_bias is not None:
+        r1, r2 = (r.float().view(Hq, 1, 1) for r in log_bias)
+        s = s - r1 * torch.log1p(r2 * (p - j).clamp(min=0))
     ok = j <= p
     if window and window > 0:
         ok = ok & ((j > p - window) | (j < keep_first))
     s = s.masked_fill(~ok, float("-inf"))
+    if sigmoid_bias is not None:
+        return torch.matmul(torch.sigmoid(s + sigmoid_bias.float().view(Hq, 1, 1)), vf).permute(1, 0, 2).contiguous()
     if sinks is not None:
         s = torch.cat([s, sinks.float().view(Hq, 1, 1).expand(Hq, Tq, 1)], -1)
         pr = torch.softmax(s, -1)[..., :Tk]
@@ -157,6 +163,35 @@ def gated_linear(q, k, v, decay, state: torch.Tensor) -> torch.Tensor:
     for t in range(q.shape[0]):
         state.mul_(decay[t].unsqueeze(1)).add_(v[t].unsqueeze(2) * k[t].unsqueeze(1))
         out[t] = torch.einsum("hvk,hk->hv", state, q[t])
+    return out
+
+
+def real_gated_recurrence(u, r, i, rate, state: torch.Tensor) -> torch.Tensor:
+    """Real-gated linear recurrent unit of one sequence: u and the gates r, i [T, W], ``rate`` [W] (<= 0); ``state`` [W] is advanced in
+    place.  Per token: log a = rate r;  S <- a S + sqrt(1 - a^2) i u.  Returns S after every token."""
+    la = rate * r
+    x = torch.sqrt(-torch.expm1(2.0 * la)) * i * u
+    a = torch.exp(la)
+    out = torch.empty_like(u)
+    for t in range(u.shape[0]):
+        state.mul_(a[t]).add_(x[t])
+        out[t] = state
+    return out
+
+
+def mlstm(q, k, v, i, f, S: torch.Tensor, n: torch.Tensor, m: torch.Tensor) -> torch.Tensor:
+    """Matrix memory with exponential gates of one sequence: q, k [T, H, D], v [T, H, E], log gates i, f [T, H]; S [H, E, D], its
+    normaliser n [H, D] and the stabiliser m [H] are advanced in place.  Per token, with m' = max(f + m, i): S and n are scaled by
+    e^(f + m - m') and gain e^(i - m') v k^T and e^(i - m') k;  o = S q / (max(|n . q|, e^-m') + 1e-6)."""
+    out = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        m1 = torch.maximum(f[t] + m, i[t])
+        a, b = torch.exp(f[t] + m - m1), torch.exp(i[t] - m1)
+        m.copy_(m1)
+        S.mul_(a.view(-1, 1, 1)).add_((b.unsqueeze(1) * v[t]).unsqueeze(2) * k[t].unsqueeze(1))
+        n.mul_(a.unsqueeze(1)).add_(b.unsqueeze(1) * k[t])
+        den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m1)) + 1e-6
+        out[t] = torch.einsum("hvk,hk->hv", S, q[t]) / den.unsqueeze(1)
     return out
 
 

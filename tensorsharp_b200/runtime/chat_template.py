@@ -350,7 +350,7 @@ def render_hardcoded(messages, add_generation_prompt=True, architecture=None, to
         return render_qwen35(messages, add_generation_prompt, enable_thinking, tools)
     if a == "mistral3":
         return render_mistral3(messages, add_generation_prompt)
-    if a in ("fobolorn", "sogulix", "kegetar"):          # no roles and no special tokens: the turns one after the other
+    if a in ("fobolorn", "sogulix", "kegetar", "lisorax"):          # no roles and no special tokens: the turns one after the other
         return " ".join(m.content for m in messages if m.content)
     return render_qwen3(messages, add_generation_prompt, tools, enable_thinking)
 
