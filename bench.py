@@ -57,7 +57,7 @@ def parse_args():
     ap.add_argument("--trace", default=None, metavar="FILE",
                     help="after the timed runs, record three more graph replays with the CUDA activity tracer, write the "
                          "kernel events of the middle one to FILE (JSON) and print its per-kernel table to stderr")
-    ap.add_argument("--design", default=None, choices=["fobolorn", "sogulix", "kegetar"],
+    ap.add_argument("--design", default=None, choices=["fobolorn", "sogulix", "kegetar", "lisorax"],
                     help="measure this design at several sizes beside the closest other model at equal size (one JSON line per "
                          "size and model) instead of the headline workload")
     ap.add_argument("--design-size", default=None, help="with --design: only this size")
@@ -503,6 +503,9 @@ def run_reference(args) -> dict:
 # half of Qwen3.5's layers are recurrent with as many heads of the same size; "dense" without experts, with 16 query heads per KV
 # head; "uneven" with windows that bite, kept first tokens, smaller heads in the linear half, and identity experts (of 40 entries
 # a token takes four, Qwen3.5 four of 32 experts).
+# Lisorax beside Qwen3.5 (recurrent and ordinary attention layers, experts with a shared one): three of four layers are recurrent in both,
+# with as many mLSTM as delta-rule heads of the same size; Qwen3.5 routes to as many experts less one and runs the shared one.
+# "narrow" has two of four layers recurrent, attention heads of 96 / 128, and layers that read another layer's cache.
 _Q35 = dict(n_experts=0, interval=4, vocab=32000, context=16384)
 DESIGNS = {
     "fobolorn": ("gpt-oss", {
@@ -541,13 +544,28 @@ DESIGNS = {
                    dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, rope_dims=64, hk=32, hv=32, dk=64, dv=64, interval=2,
                         n_experts=32, top_k=4, expert_ffn=1024, shared_ffn=1024, vocab=32000, context=16384)),
     }),
+    "lisorax": ("qwen3.5", {
+        "2048x8": (dict(layers="rmra" * 2, mlps="m" * 8, width=2048, heads=16, kv_heads=4, dim=128, vdim=128, conv=4, q_temp=(0.1, 4096), softcap=50.0,
+                        blocks=16, rec_conv=4, mem_heads=16, mem_dim=128, mem_vdim=128, canon=4, experts=32, top=4, expert_ff=1024, vocab=32000),
+                   dict(n_layers=8, hidden=2048, n_heads=16, n_kv_heads=4, head_dim=128, rope_dims=64, hk=16, hv=16, dk=128, dv=128, interval=4,
+                        n_experts=32, top_k=3, expert_ffn=1024, shared_ffn=1024, vocab=32000, context=16384)),
+        "4096x4": (dict(layers="rmra", mlps="m" * 4, width=4096, heads=32, kv_heads=8, dim=128, vdim=128, conv=4, q_temp=(0.1, 4096), softcap=50.0,
+                        blocks=16, rec_conv=4, mem_heads=32, mem_dim=128, mem_vdim=128, canon=4, experts=16, top=2, expert_ff=2048, vocab=32000),
+                   dict(n_layers=4, hidden=4096, n_heads=32, n_kv_heads=8, head_dim=128, rope_dims=64, hk=32, hv=32, dk=128, dv=128, interval=4,
+                        n_experts=16, top_k=1, expert_ffn=2048, shared_ffn=2048, vocab=32000, context=16384)),
+        "narrow": (dict(layers="mara" * 2, mlps="m" * 8, width=1536, heads=16, kv_heads=4, dim=96, vdim=128, conv=3, q_temp=(0.1, 4096), softcap=30.0,
+                        kv_from={3: 1, 7: 5}, rec_width=2048, blocks=8, rec_conv=4, mem_heads=24, mem_dim=64, mem_vdim=64, canon=3, experts=32, top=4,
+                        expert_ff=768, vocab=32000),
+                   dict(n_layers=8, hidden=1536, n_heads=16, n_kv_heads=4, head_dim=128, rope_dims=64, hk=24, hv=24, dk=64, dv=64, interval=2,
+                        n_experts=32, top_k=3, expert_ffn=768, shared_ffn=768, vocab=32000, context=16384)),
+    }),
 }
 
 
 def write_design(name: str, path: str, sizes: dict) -> str:
     """The synthetic model ``name`` of these sizes at ``path`` (a folder, or a GGUF file of that stem); returns where it is."""
     from tensorsharp_b200.models import synth
-    if name in ("fobolorn", "sogulix", "kegetar"):
+    if name in ("fobolorn", "sogulix", "kegetar", "lisorax"):
         getattr(synth, f"write_{name}")(path, seed=0, **sizes)
         return path
     path += ".gguf"

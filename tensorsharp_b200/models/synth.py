@@ -760,3 +760,99 @@ def write_kegetar(folder: str, config: Optional[dict] = None, *, seed=0, device=
     with open(os.path.join(folder, CONFIG_NAME), "w", encoding="utf-8") as f:
         json.dump(cfg, f, indent=1)
     write_safetensors(os.path.join(folder, WEIGHTS_NAME), t)
+
+
+def lisorax_config(*, layers="rama", mlps="mmmm", width=128, heads=4, kv_heads=2, dim=32, vdim=48, conv=4, q_temp=(0.4, 50), softcap=20.0, scale=None,
+                   kv_from=None, rec_width=None, blocks=4, rec_conv=3, mem_heads=3, mem_dim=32, mem_vdim=48, gate_cap=10.0, canon=3, experts=6, top=2,
+                   expert_ff=32, embed_scale=0.7, vocab=512, eps=1e-5) -> dict:
+    """A config.json of the Lisorax architecture: ``layers`` has an ``a`` (attention), an ``r`` (rglru) or an ``m`` (mlstm) per layer,
+    ``mlps`` an ``m`` (mixture of experts) or a ``-``; ``kv_from``: attention layer -> the layer whose keys and values it reads."""
+    def spec(i):
+        if layers[i] == "a":
+            mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv, "softcap": softcap,
+                     "scale": scale if scale is not None else dim ** -0.5}
+            if q_temp:
+                mixer["q_temp"] = {"coef": q_temp[0], "every": q_temp[1]}
+            if (kv_from or {}).get(i) is not None:
+                mixer["kv_from"] = kv_from[i]
+        elif layers[i] == "r":
+            mixer = {"width": rec_width or width, "blocks": blocks, "conv": rec_conv}
+        else:
+            mixer = {"heads": mem_heads, "dim": mem_dim, "vdim": mem_vdim, "gate_cap": gate_cap}
+        mlp = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}} if mlps[i] == "m" else None
+        return {"type": {"a": "attention", "r": "rglru", "m": "mlstm"}[layers[i]], "mixer": mixer, "mlp": mlp}
+    return {"architecture": "Lisorax", "vocab": vocab, "width": width, "norm": {"eps": eps}, "canon": {"taps": canon},
+            "embedding": {"scale": embed_scale}, "layers": [spec(i) for i in range(len(layers))]}
+
+
+def write_lisorax(folder: str, config: Optional[dict] = None, *, seed=0, device=None, gain=1.0, **sizes) -> None:
+    """A model folder with random bf16 weights for ``config`` (default: :func:`lisorax_config` of ``sizes``): matrices
+    N(0, gain / fan-in), norm weights around 1, convolutions of order 1, gates from forgetting at once to hardly at all, distance
+    biases from next to none to strong ones, key weights that leave a few keys to matter."""
+    import json
+    import os
+
+    from ..gguf.folder import CONFIG_NAME, WEIGHTS_NAME, write_safetensors
+    cfg = config if config is not None else lisorax_config(**sizes)
+    dev = torch.device(device or ("cuda" if torch.cuda.is_available() else "cpu"))
+    gen = torch.Generator(device=dev)
+    gen.manual_seed(seed)
+    t = {}
+
+    def rand(name, shape, std, mean=0.0):
+        t[name] = (mean + std * torch.randn(shape, generator=gen, device=dev)).to(torch.bfloat16).cpu()
+
+    def mat(name, rows, cols, std=None):
+        rand(name, (rows, cols), std if std is not None else math.sqrt(gain / cols))
+
+    def spread(name, n, lo, hi):
+        t[name] = (lo + (hi - lo) * torch.rand(n, generator=gen, device=dev)).to(torch.bfloat16).cpu()
+
+    D = cfg["width"]
+    mat("embed", cfg["vocab"], D, 1.0)
+    for i, s in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", s["mixer"], s["mlp"]
+        q = p + "mix."
+        rand(p + "norm1", (D,), 0.15, 1.0)
+        mat(p + "canon1", D, cfg["canon"]["taps"], 0.3)
+        if s["type"] == "attention":
+            H, G = m["heads"], m["kv_heads"]
+            for x, rows in (("q", H * m["dim"]),) + ((("k", G * m["dim"]), ("v", G * m["vdim"])) if m.get("kv_from") is None else ()):
+                mat(q + x, rows, D)
+                mat(f"{q}{x}.conv", rows, m["conv"], m["conv"] ** -0.5)
+            spread(q + "r1", H, 0.05, 1.5)
+            spread(q + "r2", H, 0.02, 0.5)
+            spread(q + "pb", H, -3.0, -1.0)
+            mat(q + "o", D, H * m["vdim"])
+        elif s["type"] == "rglru":
+            W, B = m["width"], m["blocks"]
+            for x in ("y", "x"):
+                mat(q + x, W, D)
+                rand(f"{q}{x}.b", (W,), 0.1)
+            mat(q + "conv", W, m["conv"], m["conv"] ** -0.5)
+            rand(q + "conv.b", (W,), 0.1)
+            for x, spread_b in (("ra", 3.0), ("ri", 1.0)):
+                rand(q + x, (B, W // B, W // B), math.sqrt(B / W))
+                rand(f"{q}{x}.b", (B, W // B), spread_b)
+            spread(q + "lam", W, -5.0, 2.0)
+            mat(q + "o", D, W)
+        else:
+            H = m["heads"]
+            for x, rows in (("q", H * m["dim"]), ("k", H * m["dim"]), ("v", H * m["vdim"]), ("g", H * m["vdim"]), ("i", H), ("f", H)):
+                mat(q + x, rows, D)
+            rand(q + "i.b", (H,), 1.5)
+            spread(q + "f.b", H, -1.0, 8.0)
+            rand(q + "norm", (H * m["vdim"],), 0.15, 1.0)
+            mat(q + "o", D, H * m["vdim"])
+        if f is not None:
+            for e in range(f["router"]["experts"]):
+                for x in ("gate", "up"):
+                    mat(f"{p}mlp.e{e}.{x}", f["expert"]["ff"], D)
+                mat(f"{p}mlp.e{e}.down", D, f["expert"]["ff"])
+            mat(p + "mlp.router", f["router"]["experts"], D)
+            rand(p + "mlp.router.b", (f["router"]["experts"],), 0.5)
+    rand("final.norm", (D,), 0.15, 1.0)
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, CONFIG_NAME), "w", encoding="utf-8") as f:
+        json.dump(cfg, f, indent=1)
+    write_safetensors(os.path.join(folder, WEIGHTS_NAME), t)
