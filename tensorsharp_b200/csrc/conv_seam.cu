@@ -1,14 +1,18 @@
 // The seam of a decoder whose sublayers run side by side on one norm of the residual stream, one of them behind a causal
-// convolution over time, in one kernel:
+// convolution over time:
 //
 //   x    = h + y + sum over the parts of w_j p_j      (residual stream, f32; p: the rows a mixture of experts leaves per token)
 //   v    = rmsnorm(x) * w                             -> out
 //   c_t  = v_t + sum_j taps[j] v_(t - K + 1 + j)      -> conv (per channel; zeros ahead of a sequence's start)
 //
 // A sequence's last K - 1 values of v are carried in `state` (f32, [K - 1][D] per slot, oldest first).  The new residual goes to
-// a buffer of its own (h_out), so a block may compute rows ahead of its own ones again.  A block takes up to `span` >= K - 1
-// consecutive rows of one sequence and holds the last K - 1 of v in registers; the first block of a sequence is the only one
-// that reads the slot's old values, and it writes the new ones.
+// a buffer of its own (h_out).
+//
+//   few rows    conv_seam_kernel<CONV>: everything in one kernel.  A block takes up to `span` >= K - 1 consecutive rows of one
+//               sequence, computes the K - 1 rows ahead of them again and holds the last K - 1 of v in registers
+//   many rows   a block per row for the sum and the norm, which leaves the row's 1 / rms; then seam_conv_kernel, a thread per four
+//               channels and run of tokens, makes v again from that and convolves
+// Either way the first block or run of a sequence is the only one that reads the slot's old values, and it writes the new ones.
 // Rows are padded with zeros to a multiple of 8 columns; the mean of squares runs over the first n.
 #include "common.cuh"
 
@@ -26,6 +30,7 @@ struct ConvSeamArgs {
     const long* seq_slots;    // [B]
     void* out;                // [rows, D] or null
     void* conv;               // [rows, D] or null
+    float* rs;                // [rows]: 1 / rms of every row, where the convolution is a kernel of its own
     long rows, state_s;
     int D, n, B, K, parts, y_f32, p_f32, out_f32, span;
     float eps;
@@ -59,7 +64,8 @@ __device__ __forceinline__ void cs_fma(float4& x, float4 w, float4 t) {
 
 // v of one row; `store`: the new residual is written.  `red`: 64 floats, whose halves consecutive calls use in turn.
 template <int V>
-__device__ __forceinline__ void cs_row(const ConvSeamArgs& a, long row, float4 (&v)[V], const float4& w0, float* red, int& flip, bool store) {
+__device__ __forceinline__ void cs_row(const ConvSeamArgs& a, long row, float4 (&v)[V], const float4& w0, float* red, int& flip, bool store,
+                                       float* rms = nullptr) {
     const int nvec = a.D >> 2, nt = blockDim.x;
 #pragma unroll
     for (int j = 0; j < V; ++j) {
@@ -111,6 +117,7 @@ __device__ __forceinline__ void cs_row(const ConvSeamArgs& a, long row, float4 (
         q = warp_sum(lane < nw ? half[lane] : 0.f);
     }
     const float rs = 1.f / sqrtf(q / (float)a.n + a.eps);
+    if (rms != nullptr && threadIdx.x == 0) *rms = rs;
 #pragma unroll
     for (int j = 0; j < V; ++j) {
         const int i = threadIdx.x + j * nt;
@@ -135,7 +142,7 @@ __global__ void __launch_bounds__(V == 1 ? 1024 : 512) conv_seam_kernel(ConvSeam
         pdl_wait();
         pdl_trigger();
         const long row = blockIdx.x;
-        cs_row<V>(a, row, v, w0, red, flip, a.h_out != nullptr);
+        cs_row<V>(a, row, v, w0, red, flip, a.h_out != nullptr, a.rs != nullptr ? a.rs + row : nullptr);
 #pragma unroll
         for (int j = 0; j < V; ++j) {
             const int i = threadIdx.x + j * nt;
@@ -233,6 +240,63 @@ __global__ void __launch_bounds__(V == 1 ? 1024 : 512) conv_seam_kernel(ConvSeam
     }
 }
 
+// Grid (runs of `span` tokens, pieces of 512 channels), 128 threads.
+template <int H>
+__global__ void __launch_bounds__(128) seam_conv_kernel(ConvSeamArgs a) {
+    constexpr int U = 4;                                       // rows loaded together
+    pdl_wait();
+    pdl_trigger();
+    const int i = blockIdx.y * 128 + threadIdx.x;
+    int b = 0;
+    long before = 0;
+    for (;; ++b) {
+        if (b == a.B) return;
+        const long n = a.cu_q[b + 1] - a.cu_q[b], runs = (n + a.span - 1) / a.span;
+        if ((long)blockIdx.x < before + runs) break;
+        before += runs;
+    }
+    if (4 * i >= a.D) return;
+    const long first = a.cu_q[b], end = a.cu_q[b + 1], r0 = first + ((long)blockIdx.x - before) * a.span, r1 = min(end, r0 + a.span);
+    const float* x = a.h_out != nullptr ? a.h_out : a.h;
+    float* st = a.state + a.seq_slots[b] * a.state_s;
+    const float4 w = cs_ld4(a.w, i);
+    auto norm = [&](float4 t, float rs) { return make_float4(t.x * rs * w.x, t.y * rs * w.y, t.z * rs * w.z, t.w * rs * w.w); };
+    float4 tap[H + 1], hist[H > 0 ? H : 1];
+#pragma unroll
+    for (int k = 0; k <= H; ++k) tap[k] = cs_ld4(a.taps + (long)k * a.D, i);
+#pragma unroll
+    for (int k = 0; k < H; ++k) hist[k] = r0 == first ? cs_ld4(st + (long)k * a.D, i) : norm(cs_ld4(x + (r0 - H + k) * a.D, i), a.rs[r0 - H + k]);
+    for (long row = r0; row < r1; row += U) {
+        float4 t[U];
+        float rs[U];
+#pragma unroll
+        for (int q = 0; q < U; ++q)
+            if (row + q < r1) {
+                t[q] = cs_ld4(x + (row + q) * a.D, i);
+                rs[q] = a.rs[row + q];
+            }
+#pragma unroll
+        for (int q = 0; q < U; ++q) {
+            if (row + q >= r1) break;
+            const float4 v = norm(t[q], rs[q]);
+            float4 c = v;
+#pragma unroll
+            for (int k = 0; k < H; ++k) cs_fma(c, tap[k], hist[k]);
+            cs_fma(c, tap[H], v);
+#pragma unroll
+            for (int k = 0; k + 1 < H; ++k) hist[k] = hist[k + 1];
+            if (H > 0) hist[H - 1] = v;
+            cs_st4(a.conv, row + q, a.D, i, a.out_f32, c);
+        }
+    }
+    if (H == 0 || r0 != first) return;
+#pragma unroll
+    for (int k = 0; k < H; ++k) {
+        const float4 v = r1 < end ? norm(cs_ld4(x + (end - H + k) * a.D, i), a.rs[end - H + k]) : hist[k];
+        reinterpret_cast<float4*>(st + (long)k * a.D)[i] = v;
+    }
+}
+
 template <int V>
 static int launch_conv_seam(const ConvSeamArgs& a, dim3 grid, dim3 block, cudaStream_t s) {
     if (a.taps == nullptr) {
@@ -247,25 +311,8 @@ static int launch_conv_seam(const ConvSeamArgs& a, dim3 grid, dim3 block, cudaSt
     return TSB_OK;
 }
 
-extern "C" int tsb_conv_seam(const ConvSeamArgs* args, void* stream) {
-    ConvSeamArgs a = *args;
-    TSB_CHECK_ARG(a.D > 0 && a.D % 8 == 0 && a.n > 0 && a.n <= a.D && a.state_s % 4 == 0, "conv_seam: bad shape D=%d n=%d", a.D, a.n);
-    TSB_CHECK_ARG((a.y == nullptr && a.p == nullptr) == (a.h_out == nullptr) && a.h_out != a.h, "conv_seam: the new residual has a buffer of its own");
-    TSB_CHECK_ARG(a.p == nullptr || a.parts > 0, "conv_seam: %d parts", a.parts);
-    TSB_CHECK_ARG(a.taps == nullptr || (a.K >= 1 && a.K <= 8 && a.conv && a.cu_q && a.seq_slots && a.B > 0 && (a.K == 1 || a.state)),
-                  "conv_seam: %d taps (1 to 8), or no state or output for them", a.K);
-    if (a.rows == 0) return TSB_OK;
-    cudaStream_t s = (cudaStream_t)stream;
+static int conv_seam_rows(const ConvSeamArgs& a, unsigned blocks, cudaStream_t s) {
     const int nvec = a.D / 4;
-    unsigned blocks = (unsigned)a.rows;
-    a.span = 1;
-    if (a.taps != nullptr && a.rows > a.B) {
-        // few rows: short runs, for latency; many: up to 16 in a row per block, since each block computes K - 1 rows again
-        const long per = a.rows / 592;
-        a.span = per < 4 ? 4 : per > 16 ? 16 : (int)per;
-        if (a.span < a.K - 1) a.span = a.K - 1;
-        blocks = (unsigned)(a.rows / a.span + a.B);
-    }
     const dim3 grid(blocks);
     int rc;
     if (nvec <= 256 || (a.rows < 296 && nvec <= 1024)) {
@@ -279,4 +326,37 @@ extern "C" int tsb_conv_seam(const ConvSeamArgs* args, void* stream) {
     if (rc != TSB_OK) return rc;
     TSB_CHECK_LAUNCH();
     return TSB_OK;
+}
+
+extern "C" int tsb_conv_seam(const ConvSeamArgs* args, void* stream) {
+    ConvSeamArgs a = *args;
+    TSB_CHECK_ARG(a.D > 0 && a.D % 8 == 0 && a.n > 0 && a.n <= a.D && a.state_s % 4 == 0, "conv_seam: bad shape D=%d n=%d", a.D, a.n);
+    TSB_CHECK_ARG((a.y == nullptr && a.p == nullptr) == (a.h_out == nullptr) && a.h_out != a.h, "conv_seam: the new residual has a buffer of its own");
+    TSB_CHECK_ARG(a.p == nullptr || a.parts > 0, "conv_seam: %d parts", a.parts);
+    TSB_CHECK_ARG(a.taps == nullptr || (a.K >= 1 && a.K <= 8 && a.conv && a.cu_q && a.seq_slots && a.B > 0 && (a.K == 1 || a.state)),
+                  "conv_seam: %d taps (1 to 8), or no state or output for them", a.K);
+    if (a.rows == 0) return TSB_OK;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int nvec = a.D / 4;
+    if (a.taps != nullptr && a.rs != nullptr) {
+        // many rows: the sum and the norm without the convolution first
+        const float* taps = a.taps;
+        a.taps = nullptr;
+        const int rc = conv_seam_rows(a, (unsigned)a.rows, s);
+        if (rc != TSB_OK) return rc;
+        a.taps = taps;
+        const long per = a.rows * nvec / (148 * 1024);                 // enough threads first, then longer runs
+        a.span = per < 4 ? 4 : per > 32 ? 32 : (int)per;
+        if (a.span < a.K - 1) a.span = a.K - 1;
+        const dim3 grid((unsigned)(a.rows / a.span + a.B), (nvec + 127) / 128);
+        switch (a.K - 1) {
+#define X(H) case H: TSB_CHECK_CUDA(tsb_launch(seam_conv_kernel<H>, grid, dim3(128), 0, s, a)); break;
+            X(0) X(1) X(2) X(3) X(4) X(5) X(6) X(7)
+#undef X
+        }
+        TSB_CHECK_LAUNCH();
+        return TSB_OK;
+    }
+    a.span = a.rows == a.B ? 1 : a.K - 1 > 4 ? a.K - 1 : 4;
+    return conv_seam_rows(a, (unsigned)(a.taps == nullptr || a.rows == a.B ? a.rows : a.rows / a.span + a.B), s);
 }

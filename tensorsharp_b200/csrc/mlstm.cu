@@ -59,9 +59,9 @@ __device__ __forceinline__ float ml_exp(float x) {             // x <= 0 up to r
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x * ML_LOG2E));
     return r;
 }
-__device__ __forceinline__ void ml_gates(const MlstmArgs& p, long t, int h, float& i, float& f) {
-    i = p.cap * tanhf((p.z[t * p.z_s + h] + p.zb[h]) / p.cap);
-    const float u = p.cap * tanhf((p.z[t * p.z_s + p.H + h] + p.zb[p.H + h]) / p.cap);
+__device__ __forceinline__ void ml_gates(const MlstmArgs& p, float zi, float zf, int h, float& i, float& f) {
+    i = p.cap * tanhf((zi + p.zb[h]) / p.cap);
+    const float u = p.cap * tanhf((zf + p.zb[p.H + h]) / p.cap);
     f = fminf(u, 0.f) - log1pf(expf(-fabsf(u)));
 }
 __device__ __forceinline__ float ml_sum8(float v) {
@@ -109,7 +109,7 @@ __global__ void __launch_bounds__(KPL <= 16 ? 1024 : 512) mlstm_step_kernel(Mlst
         if (tid < mine) sv[tid] = ml_ld(p.y, row + p.v + (long)h * p.E + c0 + tid, p.y_f32);
         const float gate = on && l8 == 0 ? ml_ld(p.y, row + p.g + (long)h * p.E + col, p.y_f32) : 0.f;
         float gi, gf;
-        ml_gates(p, t, h, gi, gf);
+        ml_gates(p, p.z[t * p.z_s + h], p.z[t * p.z_s + p.H + h], h, gi, gf);
         const float m1 = fmaxf(gf + m, gi), wa = expf(gf + m - m1), wb = expf(gi - m1);
         m = m1;
         __syncthreads();
@@ -190,14 +190,25 @@ __global__ void __launch_bounds__(1024) mlstm_gates_kernel(MlstmArgs p) {
     float* I = F + (long)p.H * p.T;
     float* M = I + (long)p.H * p.T;
     float F0 = 0.f, I0 = -INFINITY;
-#pragma unroll 4
-    for (int t = lo; t < hi; ++t) {
-        float i, f;
-        ml_gates(p, q0 + t, h, i, f);
-        F[t] = f;
-        I[t] = i;
-        F0 += f;
-        I0 = fmaxf(f + I0, i);
+    constexpr int U = 8;                                           // tokens loaded together
+    for (int t0 = lo; t0 < hi; t0 += U) {
+        float zi[U], zf[U];
+#pragma unroll
+        for (int x = 0; x < U; ++x) {
+            const float* z = p.z + (long)(q0 + min(t0 + x, hi - 1)) * p.z_s + h;
+            zi[x] = z[0];
+            zf[x] = z[p.H];
+        }
+#pragma unroll
+        for (int x = 0; x < U; ++x) {
+            if (t0 + x >= hi) break;
+            float i, f;
+            ml_gates(p, zi[x], zf[x], h, i, f);
+            F[t0 + x] = f;
+            I[t0 + x] = i;
+            F0 += f;
+            I0 = fmaxf(f + I0, i);
+        }
     }
     // inclusive scan over the warp, then over the warps: (a, then b) = (Fa + Fb, max(Fb + Ia, Ib))
 #pragma unroll

@@ -69,17 +69,21 @@ __device__ __forceinline__ float rg_dot8(uint4 w, const float* x, float z) {
     return z;
 }
 constexpr int RG_CH = 2;                    // channels per warp
+constexpr int RG_SEQ = 8;                   // sequences per CTA
 }  // namespace
 
-// Grid (blocks * slices of 16 channels, B), 256 threads; per channel, half a warp has the row of Wr and the other half that of Wi.
+// Grid (blocks * slices of 16 channels, groups of RG_SEQ sequences), 256 threads; per channel, half a warp has the row of Wr and the
+// other half that of Wi.  A group's rows follow one another; lane i holds the state of the group's sequence i.
 __global__ void __launch_bounds__(256) rglru_step_kernel(RglruArgs a) {
-    extern __shared__ __align__(16) float su[];             // [block]
-    const int slices = (a.block + 8 * RG_CH - 1) / (8 * RG_CH), blk = blockIdx.x / slices, b = blockIdx.y;
+    extern __shared__ __align__(16) float su[];             // [2][block]
+    const int slices = (a.block + 8 * RG_CH - 1) / (8 * RG_CH), blk = blockIdx.x / slices, b0 = blockIdx.y * RG_SEQ, b1 = min(a.B, b0 + RG_SEQ);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = lane >> 4, l16 = lane & 15;
     const int c0 = (blockIdx.x % slices) * 8 * RG_CH + warp * RG_CH, bs = a.block;
     // weights, state and metadata are not written by the kernel launched directly before
-    const int q0 = a.cu_q[b], n = a.cu_q[b + 1] - q0;
-    float* st = a.state + a.seq_slots[b] * a.state_s + (long)blk * bs;
+    const int q0 = a.cu_q[b0], q1 = a.cu_q[b1];
+    const bool mine = b0 + lane < b1;
+    const int ends = mine ? a.cu_q[b0 + lane + 1] : q1;
+    float* st = a.state + (mine ? a.seq_slots[b0 + lane] : 0) * a.state_s + (long)blk * bs;
     float s[RG_CH], bias[RG_CH], rate[RG_CH];
     uint4 w0[RG_CH];
     long row[RG_CH];
@@ -88,7 +92,7 @@ __global__ void __launch_bounds__(256) rglru_step_kernel(RglruArgs a) {
         const int c = c0 + j;
         const bool on = c < bs;
         row[j] = ((long)blk * 2 * bs + (long)half * bs + (on ? c : 0)) * bs;
-        s[j] = on ? st[c] : 0.f;
+        s[j] = on && mine ? st[c] : 0.f;
         bias[j] = on ? a.gate_b[(long)half * a.W + blk * bs + c] : 0.f;
         rate[j] = on ? a.rate[blk * bs + c] : 0.f;
         w0[j] = make_uint4(0u, 0u, 0u, 0u);
@@ -96,34 +100,48 @@ __global__ void __launch_bounds__(256) rglru_step_kernel(RglruArgs a) {
     }
     pdl_wait();
     pdl_trigger();
-    for (int t = q0; t < q0 + n; ++t) {
-        const float* u = reinterpret_cast<const float*>(a.u) + (long)t * a.W + (long)blk * bs;
-        for (int i = threadIdx.x; i < bs; i += 256) su[i] = u[i];
-        __syncthreads();
+    const float* u = reinterpret_cast<const float*>(a.u) + (long)blk * bs;
+    const int yc = blk * bs + c0 + (lane & 1);              // lanes 0 and 1: the output branch of the warp's channels
+    auto branch = [&](int t) { return lane < RG_CH && c0 + lane < bs ? rg_ld(a.y, (long)t * a.y_s + yc, a.y_f32) : 0.f; };
+    int seq = 0;
+    float y = q0 < q1 ? branch(q0) : 0.f;
+    if (q0 < q1)
+        for (int i = threadIdx.x; i < bs; i += 256) su[i] = u[(long)q0 * a.W + i];
+    for (int t = q0; t < q1; ++t) {
+        float* cur = su + ((t - q0) & 1) * bs;
+        __syncthreads();                                    // this row is here, and everybody is done with the one before
+        float y_next = 0.f;
+        if (t + 1 < q1) {
+            float* nxt = su + ((t + 1 - q0) & 1) * bs;
+            for (int i = threadIdx.x; i < bs; i += 256) nxt[i] = u[(long)(t + 1) * a.W + i];
+            y_next = branch(t + 1);
+        }
+        while (__shfl_sync(0xffffffffu, ends, seq) <= t) ++seq;      // (sequences without a token are passed over)
+        float res = 0.f;
 #pragma unroll
         for (int j = 0; j < RG_CH; ++j) {
             float z = 0.f;
             if (!a.w_f32) {
-                if (8 * l16 < bs) z = rg_dot8(w0[j], su + 8 * l16, z);
+                if (8 * l16 < bs) z = rg_dot8(w0[j], cur + 8 * l16, z);
                 for (int i = 8 * l16 + 128; i < bs; i += 128)
-                    z = rg_dot8(*reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.w) + row[j] + i), su + i, z);
+                    z = rg_dot8(*reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.w) + row[j] + i), cur + i, z);
             } else {
-                for (int i = l16; i < bs; i += 16) z = fmaf(reinterpret_cast<const float*>(a.w)[row[j] + i], su[i], z);
+                for (int i = l16; i < bs; i += 16) z = fmaf(reinterpret_cast<const float*>(a.w)[row[j] + i], cur[i], z);
             }
 #pragma unroll
             for (int o = 8; o > 0; o >>= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
-            const float gate = rg_sigmoid(z + bias[j]), other = __shfl_xor_sync(0xffffffffu, gate, 16);
-            if (lane == 0 && c0 + j < bs) {
-                float decay, mul;
-                rg_decay(rate[j] * gate, decay, mul);
-                s[j] = fmaf(decay, s[j], mul * other * su[c0 + j]);
-                const long c = (long)blk * bs + c0 + j;
-                rg_st(a, (long)t * a.W + c, s[j] * rg_gelu(rg_ld(a.y, (long)t * a.y_s + c, a.y_f32)));
-            }
+            const float gate = rg_sigmoid(z + bias[j]);
+            const float r = __shfl_sync(0xffffffffu, gate, 0), i = __shfl_sync(0xffffffffu, gate, 16);
+            float decay, mul;
+            rg_decay(rate[j] * r, decay, mul);
+            const float S = fmaf(decay, __shfl_sync(0xffffffffu, s[j], seq), mul * i * (c0 + j < bs ? cur[c0 + j] : 0.f));
+            if (lane == seq) s[j] = S;
+            if (lane == j) res = S;
         }
-        __syncthreads();
+        if (lane < RG_CH && c0 + lane < bs) rg_st(a, (long)t * a.W + yc, res * rg_gelu(y));
+        y = y_next;
     }
-    if (lane == 0 && n > 0) {
+    if (mine && q0 < q1) {
 #pragma unroll
         for (int j = 0; j < RG_CH; ++j)
             if (c0 + j < bs) st[c0 + j] = s[j];
@@ -158,19 +176,26 @@ __global__ void __launch_bounds__(128) rglru_scan_kernel(RglruArgs a) {
             for (int j = 1; j <= sgm; ++j) S = fmaf(rg_ex2(a.seg_a[seg + (long)j * a.W] * RG_LOG2E), S, a.seg_s[seg + (long)j * a.W]);
         }
     }
-#pragma unroll 4
-    for (int t = 0; t < n; ++t) {
-        const float r = rg_sigmoid(z[(long)t * 2 * a.block] + br), i = rg_sigmoid(z[(long)t * 2 * a.block + a.block] + bi);
-        const float u = rg_ld(a.u, u0 + (long)t * a.block, a.u_f32);
-        const float la = rate * r;
-        float decay, mul;
-        rg_decay(la, decay, mul);
-        S = fmaf(decay, S, mul * i * u);
-        if (OUT) {
-            const long row = q0 + from + t;
-            rg_st(a, row * a.W + c, S * rg_gelu(rg_ld(a.y, row * a.y_s + c, a.y_f32)));
-        } else {
-            sum += la;
+    constexpr int U = 8;                                           // tokens loaded together
+    for (int t0 = 0; t0 < n; t0 += U) {
+        float zr[U], zi[U], u[U], y[U];
+#pragma unroll
+        for (int x = 0; x < U; ++x) {
+            const long t = min(t0 + x, n - 1);
+            zr[x] = z[t * 2 * a.block];
+            zi[x] = z[t * 2 * a.block + a.block];
+            u[x] = rg_ld(a.u, u0 + t * a.block, a.u_f32);
+            y[x] = OUT ? rg_ld(a.y, (q0 + from + t) * a.y_s + c, a.y_f32) : 0.f;
+        }
+#pragma unroll
+        for (int x = 0; x < U; ++x) {
+            if (t0 + x >= n) break;
+            const float la = rate * rg_sigmoid(zr[x] + br);
+            float decay, mul;
+            rg_decay(la, decay, mul);
+            S = fmaf(decay, S, mul * rg_sigmoid(zi[x] + bi) * u[x]);
+            if (OUT) rg_st(a, (q0 + from + t0 + x) * (long)a.W + c, S * rg_gelu(y[x]));
+            else sum += la;
         }
     }
     if (!OUT) {
@@ -190,10 +215,11 @@ extern "C" int tsb_rglru_step(const RglruArgs* args, void* stream) {
     const RglruArgs& a = *args;
     const int rc = rglru_check(a, "rglru_step");
     if (rc != TSB_OK) return rc;
-    TSB_CHECK_ARG(a.u_f32 && a.block <= 8192, "rglru_step: blocks of %d channels (limit 8192), f32 inputs", a.block);
+    TSB_CHECK_ARG(a.u_f32 && a.block <= 4096, "rglru_step: blocks of %d channels (limit 4096), f32 inputs", a.block);
     if (a.B == 0 || a.T == 0) return TSB_OK;
     const int slices = (a.block + 8 * RG_CH - 1) / (8 * RG_CH);
-    TSB_CHECK_CUDA(tsb_launch(rglru_step_kernel, dim3(a.W / a.block * slices, a.B), dim3(256), a.block * sizeof(float), (cudaStream_t)stream, a));
+    TSB_CHECK_CUDA(tsb_launch(rglru_step_kernel, dim3(a.W / a.block * slices, (a.B + RG_SEQ - 1) / RG_SEQ), dim3(256), 2 * a.block * sizeof(float),
+                              (cudaStream_t)stream, a));
     TSB_CHECK_LAUNCH();
     return TSB_OK;
 }

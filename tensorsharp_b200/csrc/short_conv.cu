@@ -103,21 +103,34 @@ __global__ void __launch_bounds__(128) short_conv_kernel(ShortConvArgs a) {
 #pragma unroll
         for (int k = 0; k < H; ++k) hist[k] = sc_ld4(a.x, (r0 - H + k) * a.x_s + c, a.x_f32);
     }
-#pragma unroll 4
-    for (long row = r0; row < r1; ++row) {
-        const float4 u = sc_ld4(a.x, row * a.x_s + c, a.x_f32);
-        float4 o = bias;
+    constexpr int U = 4;                                       // rows loaded together
+    for (long row = r0; row < r1; row += U) {
+        float4 x[U];
+        long to[U];
+        float f[U];
 #pragma unroll
-        for (int k = 0; k < H; ++k) sc_fma(o, w[k], hist[k]);
-        sc_fma(o, w[H], u);
+        for (int q = 0; q < U; ++q)
+            if (row + q < r1) {
+                x[q] = sc_ld4(a.x, (row + q) * a.x_s + c, a.x_f32);
+                to[q] = QKV && index != nullptr ? index[row + q] : row + q;
+                f[q] = QKV && coef != 0.f ? (float)a.pos[row + q] : 0.f;
+            }
 #pragma unroll
-        for (int k = 0; k + 1 < H; ++k) hist[k] = hist[k + 1];
-        if (H > 0) hist[H - 1] = u;
-        if (QKV && coef != 0.f) {
-            const float f = 1.f + coef * logf(floorf(((float)a.pos[row] + 1.f) / a.qt_every) + 1.f);
-            o = make_float4(o.x * f, o.y * f, o.z * f, o.w * f);
+        for (int q = 0; q < U; ++q) {
+            if (row + q >= r1) break;
+            float4 o = bias;
+#pragma unroll
+            for (int k = 0; k < H; ++k) sc_fma(o, w[k], hist[k]);
+            sc_fma(o, w[H], x[q]);
+#pragma unroll
+            for (int k = 0; k + 1 < H; ++k) hist[k] = hist[k + 1];
+            if (H > 0) hist[H - 1] = x[q];
+            if (QKV && coef != 0.f) {
+                const float m = 1.f + coef * logf(floorf((f[q] + 1.f) / a.qt_every) + 1.f);
+                o = make_float4(o.x * m, o.y * m, o.z * m, o.w * m);
+            }
+            sc_st4(dst, at + to[q] * step, a.out_f32, o);
         }
-        sc_st4(dst, at + (QKV && index != nullptr ? index[row] : row) * step, a.out_f32, o);
     }
     if (H == 0 || r0 != first) return;
     if (r1 < end) {

@@ -219,7 +219,7 @@ def post_norm_seam(h: torch.Tensor, eps: float, n: int, *, y=None, z: Optional[t
 def conv_seam(h: torch.Tensor, eps: float, n: int, *, w: torch.Tensor, y: Optional[torch.Tensor] = None, parts: Optional["MoeParts"] = None,
               taps: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None, batch: Optional[Batch] = None, plain: bool = True,
               dtype: Optional[torch.dtype] = None):
-    """The seam of a decoder whose sublayers read one norm, one of them through a convolution over time; one kernel on CUDA.  ``h``
+    """The seam of a decoder whose sublayers read one norm, one of them through a convolution over time.  ``h``
     (f32 ``[T, D]``) plus the sublayers' outputs ``y`` and the sum of ``parts``; v, the RMS norm of that with the weight ``w``; and
     v + conv(v), a causal convolution per channel with ``taps`` [K, D] (the last row is the current token's).  ``state`` (f32
     ``[slots, K - 1, D]``, oldest first) holds each sequence's last values of v between calls.  The norm runs over the first ``n``
@@ -1375,8 +1375,8 @@ class RglruSpec:
 
 
 def rglru_segments(batch: Batch, s: RglruSpec) -> int:
-    """Pieces in which the scan takes the batch's sequences: about 2048 threads per SM, no fewer than 32 tokens each."""
-    return max(1, min(round(2048 * 148 / (batch.B * s.W)), batch.max_q_len // 32, 128))
+    """Pieces in which the scan takes the batch's sequences: about 1024 threads per SM, no fewer than 32 tokens each."""
+    return max(1, min(round(1024 * 148 / (batch.B * s.W)), batch.max_q_len // 32, 128))
 
 
 def rglru(y: torch.Tensor, s: RglruSpec, conv_w: torch.Tensor, conv_b: torch.Tensor, gates: QuantWeight, gate_b: torch.Tensor, rate: torch.Tensor,

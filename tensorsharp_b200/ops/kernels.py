@@ -784,9 +784,12 @@ def gla_prompt(y, s, cols, z: torch.Tensor, zb, norm_w, state, cu_q, seq_slots, 
     return out
 
 
+SEAM_FUSED_ROWS = 64          # rows up to which the seam and its convolution are one kernel
+
+
 class ConvSeamArgs(C.Structure):
     _fields_ = [("h", _vp), ("h_out", _vp), ("y", _vp), ("p", _vp), ("pos", _vp), ("wts", _vp), ("w", _vp), ("taps", _vp), ("state", _vp),
-                ("cu_q", _vp), ("seq_slots", _vp), ("out", _vp), ("conv", _vp), ("rows", C.c_long), ("state_s", C.c_long),
+                ("cu_q", _vp), ("seq_slots", _vp), ("out", _vp), ("conv", _vp), ("rs", _vp), ("rows", C.c_long), ("state_s", C.c_long),
                 ("D", C.c_int), ("n", C.c_int), ("B", C.c_int), ("K", C.c_int), ("parts", C.c_int), ("y_f32", C.c_int), ("p_f32", C.c_int),
                 ("out_f32", C.c_int), ("span", C.c_int), ("eps", C.c_float)]
 
@@ -835,8 +838,11 @@ def conv_seam(h: torch.Tensor, eps: float, n: int, *, w, y=None, parts=None, tap
         assert taps.dtype == torch.float32 and taps.is_contiguous() and taps.shape[1] == D
         a.state_s = _carried("conv_seam", state, (K - 1, D), batch.cu_q, batch.seq_slots, T)
         a.conv, a.taps, a.K, a.state, a.cu_q, a.seq_slots, a.B = _p(conv), _p(taps), K, _p(state), _p(batch.cu_q), _p(batch.seq_slots), batch.B
+        if T > SEAM_FUSED_ROWS:
+            rs = torch.empty(T, dtype=torch.float32, device=h.device)
+            a.rs = _p(rs)
     native.check(_lib().tsb_conv_seam(C.byref(a), _stream()), "conv_seam")
-    _count(1)
+    _count(2 if a.rs else 1)
     return res, out, conv
 
 
