@@ -803,7 +803,7 @@ def _carried(what: str, state: torch.Tensor, rest: tuple, cu_q, seq_slots, T: in
     for d in range(state.dim() - 1, 0, -1):
         assert state.shape[d] <= 1 or state.stride(d) == want
         want *= state.shape[d]
-    return state.stride(0)
+    return state.stride(0) if state.shape[0] > 1 else 0          # (torch may give a dimension of one slot any stride)
 
 
 def conv_seam(h: torch.Tensor, eps: float, n: int, *, w, y=None, parts=None, taps=None, state=None, batch=None, plain: bool = True,
@@ -953,10 +953,11 @@ class MlstmArgs(C.Structure):
 def _mlstm_args(y, s, cols, z, zb, norm_w, S, n, m, batch, eps: float, out_dtype):
     T = y.shape[0]
     assert y.stride(1) == 1 and z.dtype == torch.float32 and z.shape == (T, 2 * s.H) and z.stride(1) == 1 and zb.numel() == 2 * s.H
-    assert norm_w.numel() == s.H * s.E and S.stride(0) == n.stride(0) == m.stride(0)
+    assert norm_w.numel() == s.H * s.E
     a = MlstmArgs()
-    for t, rest in ((S, (s.H, s.E, s.D)), (n, (s.H, s.D)), (m, (s.H,))):
-        a.state_s = _carried("mlstm", t, rest, batch.cu_q, batch.seq_slots, T)
+    strides = {_carried("mlstm", t, rest, batch.cu_q, batch.seq_slots, T) for t, rest in ((S, (s.H, s.E, s.D)), (n, (s.H, s.D)), (m, (s.H,)))}
+    assert len(strides) == 1                              # all three are parts of one row per slot
+    a.state_s = strides.pop()
     a.y, a.y_s, a.y_f32 = _p(y), y.stride(0), int(y.dtype == torch.float32)
     a.q, a.k, a.v, a.g = cols
     a.z, a.z_s, a.zb, a.norm_w, a.S, a.n, a.m = _p(z), z.stride(0), _p(zb), _p(norm_w), _p(S), _p(n), _p(m)

@@ -701,8 +701,20 @@ def test_a_large_decode_batch(models, place):
     for i in torch.randperm(19, generator=torch.Generator().manual_seed(0)).tolist():
         eng.step([(i, ids[i][:-3], [])])
     rows = [eng.step([(i, [ids[i][len(ids[i]) - 3 + t]], [0]) for i in range(19)]) for t in range(3)]
-    for i in range(19):
-        agree(torch.stack([r[i] for r in rows]), oracle("plain", cfg, w, ids[i])[-3:], place)
+    agree(torch.cat([torch.stack([r[i] for r in rows]) for i in range(19)]), torch.cat([oracle("plain", cfg, w, ids[i])[-3:] for i in range(19)]), place)
+
+
+@pytest.mark.parametrize("place", PLACES)
+def test_a_pool_of_one_slot(models, place):
+    """The single-sequence interface, prompt and steps, twice on the same slot."""
+    folder, cfg, w = models("unequal")
+    m = load(folder, place, max_seqs=1)
+    poison(m)
+    ids = tokens(50, cfg["vocab"], 11)
+    m.forward(ids[:7])
+    m.reset_kv_cache()
+    got = [m.forward(ids[:30])] + [m.forward([t]) for t in ids[30:]]
+    agree(torch.stack(got), oracle("unequal", cfg, w, ids)[29:], place)
 
 
 @pytest.mark.parametrize("place", PLACES)
