@@ -190,7 +190,8 @@ __global__ void __launch_bounds__(1024) mlstm_gates_kernel(MlstmArgs p) {
     float* I = F + (long)p.H * p.T;
     float* M = I + (long)p.H * p.T;
     float F0 = 0.f, I0 = -INFINITY;
-    constexpr int U = 8;                                           // tokens loaded together
+    constexpr int U = 8;                                           // tokens loaded together; a run of so many stays in registers
+    float fr[U], ir[U];
     for (int t0 = lo; t0 < hi; t0 += U) {
         float zi[U], zf[U];
 #pragma unroll
@@ -204,8 +205,8 @@ __global__ void __launch_bounds__(1024) mlstm_gates_kernel(MlstmArgs p) {
             if (t0 + x >= hi) break;
             float i, f;
             ml_gates(p, zi[x], zf[x], h, i, f);
-            F[t0 + x] = f;
-            I[t0 + x] = i;
+            F[t0 + x] = fr[x] = f;
+            I[t0 + x] = ir[x] = i;
             F0 += f;
             I0 = fmaxf(f + I0, i);
         }
@@ -223,9 +224,12 @@ __global__ void __launch_bounds__(1024) mlstm_gates_kernel(MlstmArgs p) {
     for (int w = 0; w < warp; ++w) m = fmaxf(sf[w] + m, si[w]);
     const float pf = __shfl_up_sync(0xffffffffu, F0, 1), pi = __shfl_up_sync(0xffffffffu, I0, 1);
     if (lane > 0) m = fmaxf(pf + m, pi);
-    for (int t = lo; t < hi; ++t) {
-        m = fmaxf(F[t] + m, I[t]);
-        M[t] = m;
+    if (run <= U) {
+#pragma unroll
+        for (int x = 0; x < U; ++x)
+            if (lo + x < hi) M[lo + x] = m = fmaxf(fr[x] + m, ir[x]);
+    } else {
+        for (int t = lo; t < hi; ++t) M[t] = m = fmaxf(F[t] + m, I[t]);
     }
     __syncthreads();                                               // everybody has read the slot's m
     if (lo < hi && hi == n) p.m[slot + h] = m;

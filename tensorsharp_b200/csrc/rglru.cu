@@ -7,8 +7,8 @@
 //
 //   few tokens   rglru_step_kernel: gates, recurrence and output branch in one kernel, token by token
 //   prompts      the gates' products run as one grouped matrix product (a group per block), then a scan.  A prompt is cut into
-//                segments so that all SMs work: rglru_scan_kernel<false> finds every segment's decay and what it adds to an empty
-//                state, rglru_scan_kernel<true> folds those of the segments ahead and gives the outputs
+//                segments so that all SMs work: rglru_scan_kernel without OUT finds every segment's decay and what it adds to an empty
+//                state, the one with OUT folds those of the segments ahead and gives the outputs
 #include "common.cuh"
 
 struct RglruArgs {
@@ -37,7 +37,11 @@ __device__ __forceinline__ float rg_ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
     return r;
 }
-__device__ __forceinline__ float rg_sigmoid(float x) { return __fdividef(1.f, 1.f + rg_ex2(-RG_LOG2E * x)); }
+__device__ __forceinline__ float rg_sigmoid(float x) {
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + rg_ex2(-RG_LOG2E * x)));
+    return r;
+}
 // gelu with the tanh form: 0.5 (1 + tanh(c)) = sigmoid(2 c)
 __device__ __forceinline__ float rg_gelu(float x) { return x * rg_sigmoid(1.5957691216057308f * x * fmaf(0.044715f * x, x, 1.f)); }
 // a = e^la and sqrt(1 - a^2) for la <= 0.  Near a = 1 the difference would lose what matters: -expm1(t), t = 2 la, by its Taylor series
@@ -52,7 +56,7 @@ __device__ __forceinline__ void rg_decay(float la, float& a, float& mul) {
     p = fmaf(p, t, 1.f / 6.f);
     p = fmaf(p, t, 0.5f);
     p = fmaf(p, t, 1.f);
-    mul = sqrtf(t > -0.25f ? -t * p : fmaf(-a, a, 1.f));
+    asm("sqrt.approx.f32 %0, %1;" : "=f"(mul) : "f"(t > -0.25f ? -t * p : fmaf(-a, a, 1.f)));
 }
 __device__ __forceinline__ void rg_st(const RglruArgs& a, long at, float v) {
     if (a.out_f32) reinterpret_cast<float*>(a.out)[at] = v;
@@ -72,84 +76,111 @@ constexpr int RG_CH = 2;                    // channels per warp
 constexpr int RG_SEQ = 8;                   // sequences per CTA
 }  // namespace
 
-// Grid (blocks * slices of 16 channels, groups of RG_SEQ sequences), 256 threads; per channel, half a warp has the row of Wr and the
-// other half that of Wi.  A group's rows follow one another; lane i holds the state of the group's sequence i.
+// Grid (blocks * slices of 16 channels, groups of RG_SEQ sequences), 256 threads.  A group's rows follow one another and are taken
+// RG_SEQ at a time.  A warp has two channels; half of it has their rows of Wr and the other half those of Wi.  Of the sixteen sums
+// (channel, row) of a half, lane 8 * channel + row ends up with one, so gates, decays and the output branch are found for all of
+// them at once.  The same lane holds the state of the group's sequence `row`.
 __global__ void __launch_bounds__(256) rglru_step_kernel(RglruArgs a) {
-    extern __shared__ __align__(16) float su[];             // [2][block]
+    constexpr int R = RG_SEQ;
+    static_assert(R == 8 && RG_CH == 2, "a half warp's lanes are (channel, row)");
+    extern __shared__ __align__(16) float su[];             // [R][block]
     const int slices = (a.block + 8 * RG_CH - 1) / (8 * RG_CH), blk = blockIdx.x / slices, b0 = blockIdx.y * RG_SEQ, b1 = min(a.B, b0 + RG_SEQ);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = lane >> 4, l16 = lane & 15;
-    const int c0 = (blockIdx.x % slices) * 8 * RG_CH + warp * RG_CH, bs = a.block;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = lane >> 4, l16 = lane & 15, ch = l16 & 8, rr = l16 & 7;
+    const int c0 = (blockIdx.x % slices) * 8 * RG_CH + warp * RG_CH, bs = a.block, c = c0 + (ch >> 3);
     // weights, state and metadata are not written by the kernel launched directly before
     const int q0 = a.cu_q[b0], q1 = a.cu_q[b1];
-    const bool mine = b0 + lane < b1;
-    const int ends = mine ? a.cu_q[b0 + lane + 1] : q1;
-    float* st = a.state + (mine ? a.seq_slots[b0 + lane] : 0) * a.state_s + (long)blk * bs;
-    float s[RG_CH], bias[RG_CH], rate[RG_CH];
+    const bool on = c < bs, mine = on && b0 + rr < b1;
+    int ends[R];                                            // ends of the group's sequences
+#pragma unroll
+    for (int i = 0; i < R; ++i) ends[i] = a.cu_q[min(b0 + i + 1, b1)];
+    float* st = a.state + (mine ? a.seq_slots[b0 + rr] : 0) * a.state_s + (long)blk * bs;
+    float S = mine ? st[c] : 0.f;
+    const float bias = on ? a.gate_b[(long)half * a.W + blk * bs + c] : 0.f, rate = on ? a.rate[blk * bs + c] : 0.f;
     uint4 w0[RG_CH];
     long row[RG_CH];
 #pragma unroll
     for (int j = 0; j < RG_CH; ++j) {
-        const int c = c0 + j;
-        const bool on = c < bs;
-        row[j] = ((long)blk * 2 * bs + (long)half * bs + (on ? c : 0)) * bs;
-        s[j] = on && mine ? st[c] : 0.f;
-        bias[j] = on ? a.gate_b[(long)half * a.W + blk * bs + c] : 0.f;
-        rate[j] = on ? a.rate[blk * bs + c] : 0.f;
+        row[j] = ((long)blk * 2 * bs + (long)half * bs + (c0 + j < bs ? c0 + j : 0)) * bs;
         w0[j] = make_uint4(0u, 0u, 0u, 0u);
         if (!a.w_f32 && 8 * l16 < bs) w0[j] = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.w) + row[j] + 8 * l16);
     }
     pdl_wait();
     pdl_trigger();
     const float* u = reinterpret_cast<const float*>(a.u) + (long)blk * bs;
-    const int yc = blk * bs + c0 + (lane & 1);              // lanes 0 and 1: the output branch of the warp's channels
-    auto branch = [&](int t) { return lane < RG_CH && c0 + lane < bs ? rg_ld(a.y, (long)t * a.y_s + yc, a.y_f32) : 0.f; };
-    int seq = 0;
-    float y = q0 < q1 ? branch(q0) : 0.f;
-    if (q0 < q1)
-        for (int i = threadIdx.x; i < bs; i += 256) su[i] = u[(long)q0 * a.W + i];
-    for (int t = q0; t < q1; ++t) {
-        float* cur = su + ((t - q0) & 1) * bs;
-        __syncthreads();                                    // this row is here, and everybody is done with the one before
-        float y_next = 0.f;
-        if (t + 1 < q1) {
-            float* nxt = su + ((t + 1 - q0) & 1) * bs;
-            for (int i = threadIdx.x; i < bs; i += 256) nxt[i] = u[(long)(t + 1) * a.W + i];
-            y_next = branch(t + 1);
+    for (int t0 = q0; t0 < q1; t0 += R) {
+        const int rows = min(R, q1 - t0);
+        if (t0 > q0) __syncthreads();                       // everybody is done with the rows before
+        for (int i = threadIdx.x; i < R * (bs / 4); i += 256) {
+            const int r = i / (bs / 4), e = (i % (bs / 4)) * 4;
+            *reinterpret_cast<float4*>(su + r * bs + e) =
+                r < rows ? *reinterpret_cast<const float4*>(u + (long)(t0 + r) * a.W + e) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
-        while (__shfl_sync(0xffffffffu, ends, seq) <= t) ++seq;      // (sequences without a token are passed over)
-        float res = 0.f;
+        const bool live = on && rr < rows, writes = live && half == 0;
+        const float y = writes ? rg_ld(a.y, (long)(t0 + rr) * a.y_s + blk * bs + c, a.y_f32) : 0.f;
+        float z[RG_CH * R];
 #pragma unroll
-        for (int j = 0; j < RG_CH; ++j) {
-            float z = 0.f;
-            if (!a.w_f32) {
-                if (8 * l16 < bs) z = rg_dot8(w0[j], cur + 8 * l16, z);
-                for (int i = 8 * l16 + 128; i < bs; i += 128)
-                    z = rg_dot8(*reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.w) + row[j] + i), cur + i, z);
-            } else {
-                for (int i = l16; i < bs; i += 16) z = fmaf(reinterpret_cast<const float*>(a.w)[row[j] + i], cur[i], z);
+        for (int i = 0; i < RG_CH * R; ++i) z[i] = 0.f;
+        __syncthreads();
+        if (!a.w_f32) {
+            for (int i = 8 * l16; i < bs; i += 128) {
+                uint4 w[RG_CH];
+#pragma unroll
+                for (int j = 0; j < RG_CH; ++j) w[j] = i < 128 ? w0[j] : *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.w) + row[j] + i);
+#pragma unroll
+                for (int r = 0; r < R; ++r)
+                    if (r < rows) {
+                        z[r] = rg_dot8(w[0], su + r * bs + i, z[r]);
+                        z[R + r] = rg_dot8(w[1], su + r * bs + i, z[R + r]);
+                    }
             }
+        } else {
+            const float* w = reinterpret_cast<const float*>(a.w);
+            for (int i = l16; i < bs; i += 16)
 #pragma unroll
-            for (int o = 8; o > 0; o >>= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
-            const float gate = rg_sigmoid(z + bias[j]);
-            const float r = __shfl_sync(0xffffffffu, gate, 0), i = __shfl_sync(0xffffffffu, gate, 16);
-            float decay, mul;
-            rg_decay(rate[j] * r, decay, mul);
-            const float S = fmaf(decay, __shfl_sync(0xffffffffu, s[j], seq), mul * i * (c0 + j < bs ? cur[c0 + j] : 0.f));
-            if (lane == seq) s[j] = S;
-            if (lane == j) res = S;
+                for (int r = 0; r < R; ++r) {
+                    z[r] = fmaf(w[row[0] + i], su[r * bs + i], z[r]);
+                    z[R + r] = fmaf(w[row[1] + i], su[r * bs + i], z[R + r]);
+                }
         }
-        if (lane < RG_CH && c0 + lane < bs) rg_st(a, (long)t * a.W + yc, res * rg_gelu(y));
-        y = y_next;
-    }
-    if (mine && q0 < q1) {
+        // sums over the half: in every step a lane keeps one half of its numbers and hands the other to its partner
 #pragma unroll
-        for (int j = 0; j < RG_CH; ++j)
-            if (c0 + j < bs) st[c0 + j] = s[j];
+        for (int n = 8; n > 0; n >>= 1)
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+                if (i < n) {
+                    const bool up = l16 & n;
+                    const float give = up ? z[i] : z[i + n];
+                    z[i] = (up ? z[i + n] : z[i]) + __shfl_xor_sync(0xffffffffu, give, n);
+                }
+        const float gate = rg_sigmoid(z[0] + bias), other = __shfl_xor_sync(0xffffffffu, gate, 16);
+        float decay, mul;
+        rg_decay(rate * (half ? other : gate), decay, mul);
+        const float add = live ? mul * (half ? gate : other) * su[rr * bs + c] : 0.f;
+        int seq = 0;                                        // the row's sequence
+#pragma unroll
+        for (int i = 0; i < R; ++i) seq += ends[i] <= t0 + rr;
+        const int first = __shfl_sync(0xffffffffu, seq, 0);
+        float res = 0.f;
+        if (__all_sync(0xffffffffu, rr >= rows || seq == first + rr)) {      // one token of each sequence
+            res = fmaf(decay, __shfl_sync(0xffffffffu, S, ch | (seq & 7)), add);
+            const float mine_now = __shfl_sync(0xffffffffu, res, ch | ((rr - first) & 7));
+            if (rr >= first && rr - first < rows) S = mine_now;
+        } else {
+            for (int r = 0; r < rows; ++r) {
+                const int sq = __shfl_sync(0xffffffffu, seq, r);
+                const float d = __shfl_sync(0xffffffffu, decay, ch | r), x = __shfl_sync(0xffffffffu, add, ch | r);
+                if (rr == sq) S = fmaf(d, S, x);
+                const float now = __shfl_sync(0xffffffffu, S, ch | sq);
+                if (rr == r) res = now;
+            }
+        }
+        if (writes) rg_st(a, (long)(t0 + rr) * a.W + blk * bs + c, res * rg_gelu(y));
     }
+    if (mine && half == 0 && q0 < q1) st[c] = S;
 }
 
 // Grid (channels / 128, segments, B), a thread per channel.
-template <bool OUT>
+template <bool OUT, bool F32>
 __global__ void __launch_bounds__(128) rglru_scan_kernel(RglruArgs a) {
     pdl_wait();
     pdl_trigger();
@@ -184,8 +215,8 @@ __global__ void __launch_bounds__(128) rglru_scan_kernel(RglruArgs a) {
             const long t = min(t0 + x, n - 1);
             zr[x] = z[t * 2 * a.block];
             zi[x] = z[t * 2 * a.block + a.block];
-            u[x] = rg_ld(a.u, u0 + t * a.block, a.u_f32);
-            y[x] = OUT ? rg_ld(a.y, (q0 + from + t) * a.y_s + c, a.y_f32) : 0.f;
+            u[x] = rg_ld(a.u, u0 + t * a.block, F32);
+            y[x] = OUT ? rg_ld(a.y, (q0 + from + t) * a.y_s + c, F32) : 0.f;
         }
 #pragma unroll
         for (int x = 0; x < U; ++x) {
@@ -194,8 +225,9 @@ __global__ void __launch_bounds__(128) rglru_scan_kernel(RglruArgs a) {
             float decay, mul;
             rg_decay(la, decay, mul);
             S = fmaf(decay, S, mul * rg_sigmoid(zi[x] + bi) * u[x]);
-            if (OUT) rg_st(a, (q0 + from + t0 + x) * (long)a.W + c, S * rg_gelu(y[x]));
-            else sum += la;
+            if (!OUT) sum += la;
+            else if (F32) reinterpret_cast<float*>(a.out)[(q0 + from + t0 + x) * (long)a.W + c] = S * rg_gelu(y[x]);
+            else reinterpret_cast<bf16*>(a.out)[(q0 + from + t0 + x) * (long)a.W + c] = f2bf(S * rg_gelu(y[x]));
         }
     }
     if (!OUT) {
@@ -215,10 +247,11 @@ extern "C" int tsb_rglru_step(const RglruArgs* args, void* stream) {
     const RglruArgs& a = *args;
     const int rc = rglru_check(a, "rglru_step");
     if (rc != TSB_OK) return rc;
-    TSB_CHECK_ARG(a.u_f32 && a.block <= 4096, "rglru_step: blocks of %d channels (limit 4096), f32 inputs", a.block);
+    TSB_CHECK_ARG(a.u_f32 && a.block <= 7168, "rglru_step: blocks of %d channels (limit 7168), f32 inputs", a.block);
     if (a.B == 0 || a.T == 0) return TSB_OK;
     const int slices = (a.block + 8 * RG_CH - 1) / (8 * RG_CH);
-    TSB_CHECK_CUDA(tsb_launch(rglru_step_kernel, dim3(a.W / a.block * slices, (a.B + RG_SEQ - 1) / RG_SEQ), dim3(256), 2 * a.block * sizeof(float),
+    if (a.block > 1536) TSB_CHECK_CUDA(cudaFuncSetAttribute(rglru_step_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, RG_SEQ * a.block * (int)sizeof(float)));
+    TSB_CHECK_CUDA(tsb_launch(rglru_step_kernel, dim3(a.W / a.block * slices, (a.B + RG_SEQ - 1) / RG_SEQ), dim3(256), RG_SEQ * a.block * sizeof(float),
                               (cudaStream_t)stream, a));
     TSB_CHECK_LAUNCH();
     return TSB_OK;
@@ -231,11 +264,16 @@ extern "C" int tsb_rglru_scan(const RglruArgs* args, int max_q, void* stream) {
     if (rc != TSB_OK) return rc;
     TSB_CHECK_ARG(a.segs > 0 && a.segs <= 65535 && a.seg_len > 0 && (long)a.segs * a.seg_len >= max_q && (a.segs == 1 || (a.seg_a && a.seg_s)),
                   "rglru_scan: %d segments of %d tokens for %d", a.segs, a.seg_len, max_q);
+    TSB_CHECK_ARG(a.u_f32 == a.y_f32 && a.u_f32 == a.out_f32, "rglru_scan: inputs and results of one type");
     if (a.B == 0 || a.T == 0) return TSB_OK;
     cudaStream_t s = (cudaStream_t)stream;
     const unsigned gx = (a.W + 127) / 128;
-    if (a.segs > 1) TSB_CHECK_CUDA(tsb_launch(rglru_scan_kernel<false>, dim3(gx, a.segs - 1, a.B), dim3(128), 0, s, a));
-    TSB_CHECK_CUDA(tsb_launch(rglru_scan_kernel<true>, dim3(gx, a.segs, a.B), dim3(128), 0, s, a));
+    if (a.segs > 1) {
+        if (a.u_f32) TSB_CHECK_CUDA(tsb_launch(rglru_scan_kernel<false, true>, dim3(gx, a.segs - 1, a.B), dim3(128), 0, s, a));
+        else TSB_CHECK_CUDA(tsb_launch(rglru_scan_kernel<false, false>, dim3(gx, a.segs - 1, a.B), dim3(128), 0, s, a));
+    }
+    if (a.u_f32) TSB_CHECK_CUDA(tsb_launch(rglru_scan_kernel<true, true>, dim3(gx, a.segs, a.B), dim3(128), 0, s, a));
+    else TSB_CHECK_CUDA(tsb_launch(rglru_scan_kernel<true, false>, dim3(gx, a.segs, a.B), dim3(128), 0, s, a));
     TSB_CHECK_LAUNCH();
     return TSB_OK;
 }

@@ -28,12 +28,25 @@ struct ShortConvArgs {
 };
 
 namespace {
-__device__ __forceinline__ float4 sc_ld4(const void* p, long at, int f32) {
-    if (f32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + at);
-    const uint2 r = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(p) + at);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const bf162*>(&r.x));
-    const float2 b = __bfloat1622float2(*reinterpret_cast<const bf162*>(&r.y));
-    return make_float4(a.x, a.y, b.x, b.y);
+// four values as they are stored
+template <bool F32> struct Raw4 {
+    uint2 r;
+    __device__ __forceinline__ void load(const void* p, long at) { r = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(p) + at); }
+    __device__ __forceinline__ float4 get() const {
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const bf162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const bf162*>(&r.y));
+        return make_float4(a.x, a.y, b.x, b.y);
+    }
+};
+template <> struct Raw4<true> {
+    float4 r;
+    __device__ __forceinline__ void load(const void* p, long at) { r = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + at); }
+    __device__ __forceinline__ float4 get() const { return r; }
+};
+template <bool F32>
+__device__ __forceinline__ float4 sc_ld4(const void* p, long at) {
+    Raw4<F32> x;
+    x.load(p, at);
+    return x.get();
 }
 __device__ __forceinline__ void sc_st4(void* p, long at, int f32, float4 o) {
     if (f32) {
@@ -51,7 +64,7 @@ __device__ __forceinline__ void sc_fma(float4& x, float4 w, float4 t) {
 }  // namespace
 
 // Grid (runs, pieces of 512 channels), 128 threads.
-template <int H, bool QKV>
+template <int H, bool QKV, bool F32>
 __global__ void __launch_bounds__(128) short_conv_kernel(ShortConvArgs a) {
     const int c = (blockIdx.y * 128 + threadIdx.x) * 4;
     int b = 0;
@@ -101,41 +114,40 @@ __global__ void __launch_bounds__(128) short_conv_kernel(ShortConvArgs a) {
     pdl_trigger();
     if (r0 != first) {
 #pragma unroll
-        for (int k = 0; k < H; ++k) hist[k] = sc_ld4(a.x, (r0 - H + k) * a.x_s + c, a.x_f32);
+        for (int k = 0; k < H; ++k) hist[k] = sc_ld4<F32>(a.x, (r0 - H + k) * a.x_s + c);
     }
-    constexpr int U = 4;                                       // rows loaded together
+    constexpr int U = F32 ? 4 : 8;                             // rows loaded together
     for (long row = r0; row < r1; row += U) {
-        float4 x[U];
-        long to[U];
-        float f[U];
+        Raw4<F32> x[U];
+        int at_pos[U];                                         // slot or position, whichever these channels need
 #pragma unroll
-        for (int q = 0; q < U; ++q)
-            if (row + q < r1) {
-                x[q] = sc_ld4(a.x, (row + q) * a.x_s + c, a.x_f32);
-                to[q] = QKV && index != nullptr ? index[row + q] : row + q;
-                f[q] = QKV && coef != 0.f ? (float)a.pos[row + q] : 0.f;
-            }
+        for (int q = 0; q < U; ++q) {
+            const long t = min(row + q, r1 - 1);
+            x[q].load(a.x, t * a.x_s + c);
+            if (QKV) at_pos[q] = index != nullptr ? (int)index[t] : coef != 0.f ? a.pos[t] : 0;
+        }
 #pragma unroll
         for (int q = 0; q < U; ++q) {
             if (row + q >= r1) break;
+            const float4 u = x[q].get();
             float4 o = bias;
 #pragma unroll
             for (int k = 0; k < H; ++k) sc_fma(o, w[k], hist[k]);
-            sc_fma(o, w[H], x[q]);
+            sc_fma(o, w[H], u);
 #pragma unroll
             for (int k = 0; k + 1 < H; ++k) hist[k] = hist[k + 1];
-            if (H > 0) hist[H - 1] = x[q];
+            if (H > 0) hist[H - 1] = u;
             if (QKV && coef != 0.f) {
-                const float m = 1.f + coef * logf(floorf((f[q] + 1.f) / a.qt_every) + 1.f);
+                const float m = 1.f + coef * logf(floorf(((float)at_pos[q] + 1.f) / a.qt_every) + 1.f);
                 o = make_float4(o.x * m, o.y * m, o.z * m, o.w * m);
             }
-            sc_st4(dst, at + to[q] * step, a.out_f32, o);
+            sc_st4(dst, at + (QKV && index != nullptr ? (long)at_pos[q] : row + q) * step, a.out_f32, o);
         }
     }
     if (H == 0 || r0 != first) return;
     if (r1 < end) {
 #pragma unroll
-        for (int k = 0; k < H; ++k) *reinterpret_cast<float4*>(st + (long)k * a.C) = sc_ld4(a.x, (end - H + k) * a.x_s + c, a.x_f32);
+        for (int k = 0; k < H; ++k) *reinterpret_cast<float4*>(st + (long)k * a.C) = sc_ld4<F32>(a.x, (end - H + k) * a.x_s + c);
     } else {
 #pragma unroll
         for (int k = 0; k < H; ++k) *reinterpret_cast<float4*>(st + (long)k * a.C) = hist[k];
@@ -156,20 +168,22 @@ extern "C" int tsb_short_conv(const ShortConvArgs* args, void* stream) {
     a.span = 1;
     if (a.T > a.B) {
         const long per = (long)a.T * (a.C / 4) / (148 * 1024);         // enough threads first, then longer runs
-        a.span = per < 4 ? 4 : per > 32 ? 32 : (int)per;
+        a.span = per < 4 ? 4 : per > 32 ? 32 : per < 8 ? (int)per : (int)per & ~7;
         if (a.span < a.K - 1) a.span = a.K - 1;
         runs = (unsigned)(a.T / a.span + a.B);
     }
     const dim3 grid(runs, (a.C / 4 + 127) / 128), block(128);
     cudaStream_t s = (cudaStream_t)stream;
     switch (a.K - 1) {
-#define X(H)                                                                                          \
-    case H:                                                                                           \
-        if (qkv) TSB_CHECK_CUDA(tsb_launch(short_conv_kernel<H, true>, grid, block, 0, s, a));        \
-        else TSB_CHECK_CUDA(tsb_launch(short_conv_kernel<H, false>, grid, block, 0, s, a));           \
+#define GO(H, Q) (a.x_f32 ? tsb_launch(short_conv_kernel<H, Q, true>, grid, block, 0, s, a) : tsb_launch(short_conv_kernel<H, Q, false>, grid, block, 0, s, a))
+#define X(H)                                             \
+    case H:                                              \
+        if (qkv) TSB_CHECK_CUDA(GO(H, true));            \
+        else TSB_CHECK_CUDA(GO(H, false));               \
         break;
         X(0) X(1) X(2) X(3) X(4) X(5) X(6) X(7)
 #undef X
+#undef GO
     }
     TSB_CHECK_LAUNCH();
     return TSB_OK;

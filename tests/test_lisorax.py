@@ -360,7 +360,7 @@ def test_what_a_key_weighs():
     assert torch.allclose(O.key_weights(q, k, 0.5, None, none, r2, pb)[30].sum() - before, O.sigmoid(torch.tensor(3.0)).double() - O.sigmoid(pb))
 
 
-UNITS = [(40, 5, 2), (24, 1, 4), (96, 3, 1), (408, 3, 8), (512, 4, 3), (200, 25, 4), (640, 2, 4)]
+UNITS = [(40, 5, 2), (24, 1, 4), (96, 3, 1), (408, 3, 8), (512, 4, 3), (200, 25, 4), (640, 2, 4), (1600, 1, 2)]
 
 
 @pytest.mark.parametrize("place", PLACES)
