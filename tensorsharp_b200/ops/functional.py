@@ -1374,6 +1374,9 @@ class RglruSpec:
         self.W = self.blocks * self.block
 
 
+RGLRU_SCAN_MIN = 5          # tokens of the longest portion from which batches of more than GEMV_MAX_M rows take the scan
+
+
 def rglru_segments(batch: Batch, s: RglruSpec) -> int:
     """Pieces in which the scan takes the batch's sequences: about 1024 threads per SM, no fewer than 32 tokens each."""
     return max(1, min(round(1024 * 148 / (batch.B * s.W)), batch.max_q_len // 32, 128))
@@ -1389,7 +1392,7 @@ def rglru(y: torch.Tensor, s: RglruSpec, conv_w: torch.Tensor, conv_b: torch.Ten
     x = y[:, W:2 * W]
     if y.is_cuda:
         kk = _k()
-        if T <= GEMV_MAX_M:
+        if T <= GEMV_MAX_M or batch.max_q_len < RGLRU_SCAN_MIN:
             u = kk.short_conv(x, conv_w, conv_b, conv_state, batch, out_dtype=torch.float32)
             return kk.rglru_step(y, u, s, _weight_matrix(gates), gate_b, rate, state, batch, out_dtype=dtype)
         f32 = y.dtype == torch.float32 and dtype == torch.float32

@@ -690,6 +690,24 @@ def test_alone_and_in_a_batch(models, place):
     assert e.median() < (0.02 if place == "bf16" else 1e-5) and (e > (0.07 if place == "bf16" else 5e-5)).sum() <= (3 if place == "bf16" else 0)
 
 
+@pytest.mark.parametrize("place", PLACES)
+@pytest.mark.parametrize("portion", [4, 5, 7])
+def test_many_short_portions(models, place, portion):
+    """More rows than the small-batch paths take, in portions shorter than the prompt kernels take."""
+    folder, cfg, w = models("plain")
+    m = load(folder, place, max_seqs=6)
+    poison(m)
+    ids = [tokens(21 + i, cfg["vocab"], i) for i in range(6)]
+    eng, got = StepEngine(m, 6), [[] for _ in ids]
+    for at in range(0, 27, portion):
+        part = [(i, t[at:at + portion]) for i, t in enumerate(ids) if at < len(t)]
+        out, row = eng.step([(i, t, list(range(len(t)))) for i, t in part]), 0
+        for i, t in part:
+            got[i].append(out[row:row + len(t)])
+            row += len(t)
+    agree(torch.cat([torch.cat(g) for g in got]), torch.cat([oracle("plain", cfg, w, t) for t in ids]), place)
+
+
 @gpu
 @pytest.mark.parametrize("place", ["f32", "bf16"])
 def test_a_large_decode_batch(models, place):
@@ -701,6 +719,7 @@ def test_a_large_decode_batch(models, place):
     for i in torch.randperm(19, generator=torch.Generator().manual_seed(0)).tolist():
         eng.step([(i, ids[i][:-3], [])])
     rows = [eng.step([(i, [ids[i][len(ids[i]) - 3 + t]], [0]) for i in range(19)]) for t in range(3)]
+    assert eng.stepper.replays == 3
     agree(torch.cat([torch.stack([r[i] for r in rows]) for i in range(19)]), torch.cat([oracle("plain", cfg, w, ids[i])[-3:] for i in range(19)]), place)
 
 
