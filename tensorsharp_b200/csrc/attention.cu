@@ -299,8 +299,7 @@ __global__ void attn_combine_kernel(AttnArgs a) {
     const float sink = a.sinks ? a.sinks[h] : -INFINITY;
     const float mm = fmaxf(sink, warp_max(fmaxf(ml0.x, ml1.x)));
     const float c0 = (ml0.x == -INFINITY) ? 0.f : __expf(ml0.x - mm), c1 = (ml1.x == -INFINITY) ? 0.f : __expf(ml1.x - mm);
-    float ll = warp_sum(ml0.y * c0 + ml1.y * c1) + (a.sinks ? __expf(sink - mm) : 0.f);
-    if (a.sig_bias != nullptr) ll = 1.f;             // weights that are not normalised
+    const float ll = warp_sum(ml0.y * c0 + ml1.y * c1) + (a.sinks ? __expf(sink - mm) : 0.f);
     float o = 0.f;
     const int dd = d < a.Dh ? d : 0;
     for (int s0 = 0; s0 < a.splits; s0 += 32) {

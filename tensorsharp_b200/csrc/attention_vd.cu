@@ -470,7 +470,8 @@ __global__ void __launch_bounds__(128) attn_decode_vd_kernel(AttnArgs a, int chu
         }
         const long pi = ((long)b * a.Hq + h0 + g) * a.splits + split;
         a.part_o[pi * DV + d] = ov;
-        if (d == 0) { a.part_ml[pi * 2] = mm; a.part_ml[pi * 2 + 1] = ll; }
+        // sigmoid weights: maxima 0 and a sum of 1 over all splits, so that the merge adds the parts as they are
+        if (d == 0) { a.part_ml[pi * 2] = mm; a.part_ml[pi * 2 + 1] = !sig ? ll : split == 0 ? 1.f : 0.f; }
     }
 }
 
